@@ -436,6 +436,85 @@ int b200_residual_add(const void* x, const void* residual, void* out, int64_t co
 int b200_swiglu_pair(const void* gate, int64_t gate_stride, const void* up, int64_t up_stride, void* out, int32_t rows,
                      int32_t width, b200_stream_t stream);
 
+/* ------------------------------------------------------------------------------------------------------------------
+ * Mixers and residual streams of hybrid stacks (no counterpart in the reference).  `f32` selects fp32 activations and
+ * weights instead of bf16 ("E" below); recurrent states, residual streams, norms, gates, scores and softmax are fp32
+ * either way.  Packed batches: cu_* are int32 [batch + 1] row offsets, slots int32 [batch] the cache slot of each
+ * sequence, start int32 [batch] the position of its first packed token (0 = the sequence begins: states start from
+ * zero).  Decode forms: row b = slot b; pos int64 [batch] is the position of the new token; active int64 [batch] or
+ * NULL: a slot with 0 leaves caches and states untouched.  Feature sizes are padded by the caller with zero weights;
+ * "true" sizes are what norms divide by.
+ *
+ * b200_hyper_connect: S residual streams (fp32 [rows, S, width]) between two sublayers:
+ *     x_t <- sum_s mix[s,t] x_s + out[t] * y;   h = (sum_s in[s] x_s) / sqrt(mean(.^2) + eps) * gain
+ *   weights = [mix S*S | out S | in S | gain] fp32.  ids != NULL: the streams are first set to table[ids[row]] (y NULL).
+ *   y == NULL, ids == NULL: streams are only read. */
+int b200_hyper_connect(const void* ids, int32_t ids_are_int64, const void* table, float* streams, const void* y,
+                       const float* weights, void* h, int32_t rows, int32_t num_streams,
+                       int32_t width, int32_t true_width, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);
+/* b200_swiglu for fp32 activations. */
+int b200_swiglu_f32(const float* gate_up, int64_t row_stride, float* out, int32_t rows, int32_t intermediate,
+                    b200_stream_t stream);
+
+/* minGRU: zxg = rows of [z | x | g] projections, each `width` wide; bias fp32 [2*width] (z, x); state fp32 [slots, width];
+ *   z = sigmoid(z + zb), u = x + xb, c = u >= 0 ? u + 1/2 : sigmoid(u), S <- (1-z) S + z c, out = S * silu(g).
+ * Prefill cuts sequences into `chunks` chunks of `chunk` tokens; workspace of b200_mingru_workspace_bytes(). */
+int64_t b200_mingru_workspace_bytes(int32_t batch, int32_t chunks, int32_t width);
+int b200_mingru_prefill(const void* zxg, int64_t stride, const float* bias, float* state, const int32_t* cu_seqlens,
+                        const int32_t* slots, const int32_t* start, void* workspace, void* out, int32_t batch, int32_t chunk,
+                        int32_t chunks, int32_t width, int32_t f32, b200_stream_t stream);
+int b200_mingru_decode(const void* zxg, int64_t stride, const float* bias, float* state, const int64_t* pos,
+                       const int64_t* active, void* out, int32_t batch, int32_t width, int32_t f32, int32_t overlap,
+                       b200_stream_t stream);
+
+/* HGRN2: qfv = rows of [q heads*dim | f heads*dim | v heads*vdim]; lower, bias fp32 [heads*dim]; norm fp32 [vdim];
+ * state fp32 [slots, heads, dim, vdim];  f = l + (1-l) sigmoid(f + bias), S <- diag(f) S + (1-f) v^T, o = S^T silu(q),
+ * out = o / sqrt(mean(o^2) + eps) * norm per head.  o_scratch: fp32 [tokens, heads*vdim]. */
+int b200_hgrn2_prefill(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
+                       const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start, float* o_scratch, void* out,
+                       int32_t batch, int32_t tokens, int32_t heads, int32_t dim, int32_t vdim, int32_t true_vdim, float eps,
+                       int32_t f32, b200_stream_t stream);
+int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
+                      const int64_t* pos, const int64_t* active, void* out, int32_t batch, int32_t heads, int32_t dim,
+                      int32_t vdim, int32_t true_vdim, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);
+
+/* Latent attention.  Cache rows are [latent rank | rotated key part rot] in pages of 16 tokens; rank, dim, vdim, rot and
+ * q_rank padded to multiples of 64.  angles: fp32 (cos, sin) pairs [positions, rot_pairs], amplitude included.
+ * b200_latent_prep: fused rows [query latent | kv latent | rotated part] -> cq = rms(query latent) * q_weight, and, when
+ *   cache is given, the cache row of position pos[row] of slot[row] (NULL: slot = row).
+ * b200_rope_interleaved: rotates pairs (x[offset+2i], x[offset+2i+1]) of every head in place.
+ * b200_latent_gather: packed cache rows of positions k_pos0[s] + (0 .. cu_k[s+1]-cu_k[s]-1).
+ * b200_latent_prefill(_simple): q [tokens, heads, dim+rot] (rotated) against kv [keys, heads*dim | heads*vdim] and the
+ *   rotated parts of ctx [keys, rank+rot]; query i of sequence s sits at position q_pos0[s] + i and sees positions
+ *   (p - window, p].  _simple: any shape, bf16 or fp32; the other: bf16, tcgen05, dim + rot <= 256, vdim <= 256.
+ * b200_latent_absorb: q' = [W_uk^T q_unrotated | rotated part], w_uk [heads, dim, rank].
+ * b200_latent_decode(_simple): q' against the paged rows, the visible range split in `splits` runs of pages: ml fp32
+ *   [batch, heads, splits, 2] (maximum, sum), o fp32 [batch, heads, splits, rank] unnormalised.
+ * b200_latent_value: merges the splits and applies w_uv [heads, vdim, rank]. */
+int b200_latent_prep(const void* fused, int64_t stride, const float* q_weight, const float* kv_weight, const void* pos,
+                     int32_t pos_is_int64, const int32_t* slot, const int64_t* active, const int32_t* block_table,
+                     int64_t table_stride, const float* angles, void* cache, void* cq, int32_t rows, int32_t q_rank,
+                     int32_t true_q_rank, int32_t rank, int32_t true_rank, int32_t rot, int32_t rot_pairs, float eps,
+                     int32_t f32, int32_t overlap, b200_stream_t stream);
+int b200_rope_interleaved(void* x, int64_t row_stride, int32_t head_stride, int32_t offset, int32_t heads, int32_t pairs,
+                          const int32_t* pos, const float* angles, int32_t rows, int32_t f32, b200_stream_t stream);
+int b200_latent_gather(const void* cache, void* out, const int32_t* block_table, int64_t table_stride, const int32_t* slots,
+                       const int32_t* cu_k, const int32_t* k_pos0, int32_t batch, int32_t max_keys, int32_t row_bytes,
+                       b200_stream_t stream);
+int b200_latent_prefill_simple(const void* q, const void* kv, const void* ctx, void* out, const int32_t* cu_q,
+                               const int32_t* cu_k, const int32_t* q_pos0, const int32_t* k_pos0, int32_t batch, int32_t max_q,
+                               int32_t heads, int32_t dim, int32_t rot, int32_t vdim, int32_t rank, int32_t window, float scale,
+                               int32_t f32, b200_stream_t stream);
+int b200_latent_absorb(const void* q, const void* w_uk, const int64_t* pos, const float* angles, void* out, int32_t batch,
+                       int32_t heads, int32_t dim, int32_t rot, int32_t rot_pairs, int32_t rank, int32_t f32, int32_t overlap,
+                       b200_stream_t stream);
+int b200_latent_decode_simple(const void* q, const void* cache, const int32_t* block_table, int64_t table_stride,
+                              const int64_t* pos, const int64_t* active, float* ml, float* o, int32_t batch, int32_t heads,
+                              int32_t rank, int32_t rot, int32_t window, int32_t splits, float scale, int32_t f32,
+                              int32_t overlap, b200_stream_t stream);
+int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* out, int32_t batch, int32_t heads, int32_t rank,
+                      int32_t vdim, int32_t splits, int32_t f32, int32_t overlap, b200_stream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

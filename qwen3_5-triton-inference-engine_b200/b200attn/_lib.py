@@ -63,8 +63,23 @@ SIGNATURES: dict[str, list] = {
     "b200_swiglu_pair": [P, I64, P, I64, P, I32, I32, P],
     "b200_gdn_chunked_prefill_fused": [P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I32, I32,
                                        P, P, I64, I64, I32, I32, I32, P],
+    "b200_hyper_connect": [P, I32, P, P, P, P, P, I32, I32, I32, I32, c_float, I32, I32, P],
+    "b200_swiglu_f32": [P, I64, P, I32, I32, P],
+    "b200_mingru_prefill": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, P],
+    "b200_mingru_decode": [P, I64, P, P, P, P, P, I32, I32, I32, I32, P],
+    "b200_hgrn2_prefill": [P, I64, P, P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, P],
+    "b200_hgrn2_decode": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, c_float, I32, I32, P],
+    "b200_latent_prep": [P, I64, P, P, P, I32, P, P, P, I64, P, P, P, I32, I32, I32, I32, I32, I32, I32, c_float, I32, I32,
+                         P],
+    "b200_rope_interleaved": [P, I64, I32, I32, I32, I32, P, P, I32, I32, P],
+    "b200_latent_gather": [P, P, P, I64, P, P, P, I32, I32, I32, P],
+    "b200_latent_prefill_simple": [P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, c_float, I32, P],
+    "b200_latent_absorb": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, P],
+    "b200_latent_decode_simple": [P, P, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, P],
+    "b200_latent_value": [P, P, P, P, I32, I32, I32, I32, I32, I32, I32, P],
 }
 OTHER = {
+    "b200_mingru_workspace_bytes": ([I32, I32, I32], c_int64),
     "b200_last_error": ([], c_char_p),
     "b200_abi_version": ([], c_int),
     "b200_wait_timed_out": ([], c_int),
@@ -80,18 +95,20 @@ class B200Error(RuntimeError):
     pass
 
 
-def load() -> ctypes.CDLL:
-    """Load the library once; raises if it has not been built (python build.py)."""
+def load(path: Path | None = None) -> ctypes.CDLL:
+    """Load the library once; raises if it has not been built (python build.py).  path: the library of one part, which
+    carries a subset of the symbols (build.py `ensure`), for a process that needs no more."""
     global _lib
     if _lib is None:
-        if not LIB_PATH.exists():
-            raise B200Error(f"{LIB_PATH} not found: build it with `python {PKG_DIR / 'build.py'}`; there is no fallback path")
-        lib = ctypes.CDLL(str(LIB_PATH))
-        for name, argtypes in SIGNATURES.items():
-            fn = getattr(lib, name)
-            fn.argtypes = argtypes
-            fn.restype = c_int
-        for name, (argtypes, restype) in OTHER.items():
+        path = LIB_PATH if path is None else Path(path)
+        if not path.exists():
+            raise B200Error(f"{path} not found: build it with `python {PKG_DIR / 'build.py'}`; there is no fallback path")
+        lib = ctypes.CDLL(str(path))
+        partial = path != LIB_PATH
+        table = {name: (argtypes, c_int) for name, argtypes in SIGNATURES.items()} | OTHER
+        for name, (argtypes, restype) in table.items():
+            if partial and not hasattr(lib, name):
+                continue                        # calling it raises AttributeError
             fn = getattr(lib, name)
             fn.argtypes = argtypes
             fn.restype = restype

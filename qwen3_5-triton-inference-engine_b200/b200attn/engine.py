@@ -16,6 +16,7 @@ import numpy as np
 import torch
 
 from . import glue, glue_ops, ops
+from .slots import SlotEngine
 
 
 def _raw(op):
@@ -84,50 +85,28 @@ def random_weights(cfg: ModelConfig, seed: int, device, std: float = 0.02) -> di
     return {"embed": rnd(cfg.vocab, cfg.hidden), "norm": rnd(cfg.hidden), "layers": layers}
 
 
-class Engine:
-    """One replica: weights, caches and the two entry points `prefill` and `step`."""
+class Engine(SlotEngine):
+    """One replica of the Qwen3.5 architecture: weights, caches and the two entry points `prefill` and `step`."""
 
     def __init__(self, cfg: ModelConfig, weights: dict, batch: int, max_context: int, device, page_seed: int = 0,
                  fused_glue: bool = True, on_demand_pages: bool = False, num_pages: int | None = None):
         """fused_glue: run the row-wise operators of a decode step (residual + RMSNorm, SwiGLU, conv + q/k norms +
         gates, gated RMSNorm) as this package's single-launch kernels; False keeps them as eager PyTorch (glue.py).
-        on_demand_pages: KV pages come from a shared pool of `num_pages` (default: enough for every slot at
-        `max_context`) as sequences grow (`serving.PageAllocator`), the `batch` sequences are independent SLOTS that
-        `prefill_slots` fills one group at a time, and `set_active` masks the idle ones - what `ContinuousBatcher`
-        drives.  Without it every slot owns its pages from the start, as the reference reserves them
-        (engine/cache.py:154-159)."""
-        self.cfg, self.w, self.batch, self.device = cfg, weights, batch, torch.device(device)
+        Slots, pages and the page table: `SlotEngine`."""
+        super().__init__(batch, max_context, device, page_seed, on_demand_pages, num_pages)
+        self.cfg, self.w = cfg, weights
         self.fused_glue = fused_glue
-        pages_per_seq = (max_context + ops.PAGE_SIZE - 1) // ops.PAGE_SIZE
-        self.pages = None
-        self.active = None
-        if on_demand_pages:
-            from .serving import PageAllocator
-            num_pages = batch * pages_per_seq + 1 if num_pages is None else num_pages
-            self.pages = PageAllocator(num_pages, batch, pages_per_seq, device=self.device)
-            self.block_table = self.pages.block_table
-            self.active = torch.ones(batch, dtype=torch.int64, device=self.device)   # 1 = the slot decodes
-        else:
-            num_pages = batch * pages_per_seq
-            perm = torch.randperm(num_pages, generator=torch.Generator().manual_seed(page_seed))
-            self.block_table = perm.view(batch, pages_per_seq).to(torch.int32).to(self.device)
-        self.max_context = pages_per_seq * ops.PAGE_SIZE
-        self.pos = torch.zeros(batch, dtype=torch.int64, device=self.device)
         self.kv, self.conv_state, self.rec_state = {}, {}, {}
         for i in range(cfg.num_layers):
             if cfg.is_attention(i):
-                self.kv[i] = ops.allocate_paged_kv_cache(num_pages, cfg.num_kv_heads, cfg.head_dim, device=self.device)
+                self.kv[i] = ops.allocate_paged_kv_cache(self.num_pages, cfg.num_kv_heads, cfg.head_dim, device=self.device)
             else:
                 self.conv_state[i] = torch.zeros(batch, 4, 3 * cfg.gdn_width, dtype=torch.bfloat16, device=self.device)
                 self.rec_state[i] = torch.zeros(batch, cfg.gdn_heads, cfg.gdn_dim, cfg.gdn_dim, dtype=torch.float32,
                                                 device=self.device)
         self.workspace = ops.fused_decode_workspace(self.device)
-        self.argmax_ws = ops.argmax_workspace(self.device)
         r = cfg.rotary_dim
         self.inv_freq = (1.0 / (cfg.rope_theta ** (torch.arange(0, r, 2, dtype=torch.float32) / r))).to(self.device)
-        self.tok = torch.zeros(batch, dtype=torch.int64, device=self.device)   # input of the next step
-        self.graph = None
-        self._warmed = False     # an eager decode step has run (first-call set-up of the kernels is done)
 
     # ------------------------------------------------------------------------------------------------ shared pieces
     def _streams_weight(self, weight, swiglu: bool = False) -> bool:
@@ -176,38 +155,12 @@ class Engine:
         return glue.lm_head_argmax(self._norm(x, self.w["norm"]), self.w["embed"], last_only=False)
 
     # ------------------------------------------------------------------------------------------------------ prefill
-    @torch.no_grad()
-    def prefill(self, prompts: list[list[int]]) -> torch.Tensor:
-        """Packed varlen prefill of `batch` prompts (engine/runner.py:212-405 with a PackedBatch); fills every cache,
-        sets pos, returns the first generated token of each sequence (int64 [B]) and leaves it in `self.tok`."""
-        assert len(prompts) == self.batch
-        if self.pages is not None:
-            for slot, prompt in enumerate(prompts):
-                self.pages.release(slot)
-                self.pages.ensure(slot, len(prompt) + 1)
-        return self._prefill(prompts, None)
-
-    @torch.no_grad()
-    def prefill_slots(self, slots: list[int], prompts: list[list[int]]) -> torch.Tensor:
-        """Packed prefill of `prompts` into the given slots only (their pages must already be there: the caller is the
-        batcher, which calls `pages.ensure` first); the other slots keep their state.  Returns the first generated
-        token of each prompt (int64 [len(slots)]) and leaves them in `self.tok[slots]`."""
-        assert self.pages is not None, "slot-wise prefill needs on_demand_pages=True"
-        assert len(slots) == len(prompts) and len(set(slots)) == len(slots)
-        assert all(0 <= s < self.batch for s in slots)
-        return self._prefill(prompts, torch.tensor(slots, dtype=torch.int64, device=self.device))
-
-    def set_active(self, mask) -> None:
-        """Which slots decode (host list of bools).  An idle slot still rides along in the step's launches - the batch
-        dimension of a captured graph is fixed - but its position is forced back to zero after every step and its page
-        table row points at the spare page, so nothing it writes is ever read."""
-        assert self.active is not None and len(mask) == self.batch
-        self.active.copy_(torch.tensor([1 if m else 0 for m in mask], dtype=torch.int64), non_blocking=True)
-
     def _prefill(self, prompts: list[list[int]], slots) -> torch.Tensor:
         cfg = self.cfg
         assert all(0 < len(p) <= self.max_context for p in prompts)
         lengths = [len(p) for p in prompts]
+        if slots is not None:
+            slots = torch.tensor(slots, dtype=torch.int64, device=self.device)
         table = self.block_table if slots is None else self.block_table.index_select(0, slots)
 
         def put(dst, src):          # write a per-sequence result into all slots, or into the chosen ones
@@ -412,32 +365,3 @@ class Engine:
         if self.active is not None:
             self.pos.mul_(self.active)       # idle slots stay at position 0 (and on the spare page)
         return nxt
-
-    def capture(self) -> None:
-        """Capture one decode step (read self.tok, write the next ids back into self.tok) into a CUDA graph.
-        At least one eager `step()` must have run before: the first call of several kernels does per-device set-up
-        (shared-memory limits, symbol addresses, workspaces) that must not happen under stream capture."""
-        assert self._warmed, "run one eager step() before capture(): first calls do set-up that cannot be captured"
-        side = torch.cuda.Stream(device=self.device)
-        side.wait_stream(torch.cuda.current_stream(self.device))
-        graph = torch.cuda.CUDAGraph()
-        with torch.cuda.stream(side):
-            with torch.cuda.graph(graph, stream=side):
-                self._advance()
-        torch.cuda.current_stream(self.device).wait_stream(side)
-        self.graph = graph
-
-    def step(self) -> torch.Tensor:
-        """Advance every sequence by one token; returns the device tensor holding the new ids (valid until the next
-        step)."""
-        if self.graph is not None:
-            self.graph.replay()
-        else:
-            self._advance()
-            self._warmed = True
-        return self.tok
-
-    def _advance(self) -> None:
-        nxt = self._decode(self.tok)
-        if nxt.data_ptr() != self.tok.data_ptr():        # a step that did not write the ids in place
-            self.tok.copy_(nxt)

@@ -1,0 +1,206 @@
+"""Torch-facing wrappers of the kernels of hybrid stacks (include/b200_attn.h, last section): hyper-connected residual
+streams, minGRU, HGRN2 and latent attention.  The element type of activations and weights (bf16 or fp32) is taken from
+the tensors; shapes follow the padded layout the weight loader makes (`hybrid.py`)."""
+from __future__ import annotations
+
+import torch
+
+from . import _lib
+from .ops import PAGE_SIZE, _ptr, _require_cuda, _stream
+
+LATENT_MAX_SPLITS = 64
+
+
+def _f32(t) -> int:
+    assert t.dtype in (torch.bfloat16, torch.float32)
+    return int(t.dtype == torch.float32)
+
+
+def hyper_connect(streams, weights, true_width: int, eps: float, dtype, y=None, ids=None, table=None, overlap: int = 0):
+    """One step between two sublayers (b200_hyper_connect): mixes `y` into `streams` [rows, S, width] (in place), or sets
+    them from `table[ids]`; returns the next sublayer's normed input [rows, width]."""
+    assert streams.dtype == weights.dtype == torch.float32 and streams.is_contiguous() and weights.is_contiguous()
+    rows, s, width = streams.shape
+    assert weights.numel() == s * s + 2 * s + 1
+    h = torch.empty((rows, width), dtype=dtype, device=streams.device)
+    if y is not None:
+        assert y.shape == (rows, width) and y.is_contiguous() and y.dtype == dtype
+    if ids is not None:
+        assert ids.numel() == rows and ids.is_contiguous() and ids.dtype in (torch.int32, torch.int64)
+        assert table.dtype == dtype and table.shape[1] == width and table.is_contiguous()
+    _require_cuda(streams, weights)
+    _lib.call("b200_hyper_connect", _ptr(ids), int(ids is not None and ids.dtype == torch.int64), _ptr(table), _ptr(streams),
+              _ptr(y), _ptr(weights), _ptr(h), rows, s, width, true_width, float(eps), _f32(h), int(overlap),
+              _stream())
+    return h
+
+
+def swiglu_f32(gate_up, intermediate: int):
+    assert gate_up.dtype == torch.float32 and gate_up.stride(1) == 1 and gate_up.shape[1] >= 2 * intermediate
+    _require_cuda(gate_up)
+    out = torch.empty((gate_up.shape[0], intermediate), dtype=torch.float32, device=gate_up.device)
+    _lib.call("b200_swiglu_f32", _ptr(gate_up), gate_up.stride(0), _ptr(out), gate_up.shape[0], intermediate, _stream())
+    return out
+
+
+# ------------------------------------------------------------------------------------------------------------- minGRU
+def mingru_chunking(max_len: int) -> tuple[int, int]:
+    """(chunk length, chunks of the longest sequence): at least 64 tokens a chunk, at most 64 chunks."""
+    chunk = max(64, -(-max_len // 64))
+    return chunk, -(-max_len // chunk)
+
+
+def mingru_prefill(zxg, bias, state, batch):
+    """zxg [tokens, 3*width] projections of a packed batch (`batch`: PackedBatch); state [slots, width] fp32, in place."""
+    width = state.shape[1]
+    assert zxg.shape[1] == 3 * width and zxg.stride(1) == 1 and bias.numel() == 2 * width
+    assert state.dtype == bias.dtype == torch.float32 and state.is_contiguous() and bias.is_contiguous()
+    _require_cuda(zxg, bias, state)
+    chunk, chunks = mingru_chunking(batch.max_len)
+    n = batch.count
+    ws = torch.empty(_lib.load().b200_mingru_workspace_bytes(n, chunks, width), dtype=torch.uint8, device=zxg.device)
+    out = torch.empty((zxg.shape[0], width), dtype=zxg.dtype, device=zxg.device)
+    _lib.call("b200_mingru_prefill", _ptr(zxg), zxg.stride(0), _ptr(bias), _ptr(state), _ptr(batch.cu), _ptr(batch.slots),
+              _ptr(batch.start), _ptr(ws), _ptr(out), n, chunk, chunks, width, _f32(zxg), _stream())
+    return out
+
+
+def mingru_decode(zxg, bias, state, pos, active, overlap: int = 0):
+    rows, width = state.shape
+    assert zxg.shape == (rows, 3 * width) and zxg.stride(1) == 1 and pos.dtype == torch.int64
+    _require_cuda(zxg, bias, state, pos)
+    out = torch.empty((rows, width), dtype=zxg.dtype, device=zxg.device)
+    _lib.call("b200_mingru_decode", _ptr(zxg), zxg.stride(0), _ptr(bias), _ptr(state), _ptr(pos), _ptr(active), _ptr(out), rows,
+              width, _f32(zxg), int(overlap), _stream())
+    return out
+
+
+# -------------------------------------------------------------------------------------------------------------- HGRN2
+def _check_hgrn2(qfv, lower, bias, norm, state):
+    _, heads, dim, vdim = state.shape
+    assert qfv.shape[1] == 2 * heads * dim + heads * vdim and qfv.stride(1) == 1
+    assert lower.numel() == bias.numel() == heads * dim and norm.numel() == vdim
+    for t in (lower, bias, norm, state):
+        assert t.dtype == torch.float32 and t.is_contiguous()
+    _require_cuda(qfv, lower, bias, norm, state)
+    return heads, dim, vdim
+
+
+def hgrn2_prefill(qfv, lower, bias, norm, state, batch, true_vdim: int, eps: float):
+    """qfv [tokens, 2*heads*dim + heads*vdim]; state [slots, heads, dim, vdim] fp32, in place."""
+    heads, dim, vdim = _check_hgrn2(qfv, lower, bias, norm, state)
+    tokens = qfv.shape[0]
+    scratch = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=qfv.device)
+    out = torch.empty((tokens, heads * vdim), dtype=qfv.dtype, device=qfv.device)
+    _lib.call("b200_hgrn2_prefill", _ptr(qfv), qfv.stride(0), _ptr(lower), _ptr(bias), _ptr(norm), _ptr(state), _ptr(batch.cu),
+              _ptr(batch.slots), _ptr(batch.start), _ptr(scratch), _ptr(out), batch.count, tokens, heads, dim, vdim, true_vdim,
+              float(eps), _f32(qfv), _stream())
+    return out
+
+
+def hgrn2_decode(qfv, lower, bias, norm, state, pos, active, true_vdim: int, eps: float, overlap: int = 0):
+    heads, dim, vdim = _check_hgrn2(qfv, lower, bias, norm, state)
+    rows = state.shape[0]
+    assert qfv.shape[0] == rows
+    out = torch.empty((rows, heads * vdim), dtype=qfv.dtype, device=qfv.device)
+    _lib.call("b200_hgrn2_decode", _ptr(qfv), qfv.stride(0), _ptr(lower), _ptr(bias), _ptr(norm), _ptr(state), _ptr(pos),
+              _ptr(active), _ptr(out), rows, heads, dim, vdim, true_vdim, float(eps), _f32(qfv), int(overlap), _stream())
+    return out
+
+
+# --------------------------------------------------------------------------------------------------- latent attention
+def allocate_latent_cache(num_pages: int, row: int, dtype, *, device="cuda"):
+    """Zero-filled pages of [latent | rotated key part] rows (the padding columns stay zero)."""
+    return torch.zeros((num_pages, PAGE_SIZE, row), dtype=dtype, device=device)
+
+
+def latent_prep(fused, q_weight, kv_weight, pos, slot, active, block_table, angles, cache, true_q_rank: int, rank: int,
+                true_rank: int, eps: float, overlap: int = 0):
+    """Query-latent norm, and (cache given) latent norm + key rotation + paged write.  Returns cq [rows, q_rank]."""
+    q_rank, rows = q_weight.numel(), fused.shape[0]
+    rot = 0
+    if cache is not None:
+        rot = cache.shape[2] - rank
+        assert fused.shape[1] == q_rank + rank + rot and kv_weight.numel() == rank and cache.dtype == fused.dtype
+    assert fused.stride(1) == 1 and angles.dtype == torch.float32 and angles.is_contiguous()
+    assert pos.dtype in (torch.int32, torch.int64)
+    _require_cuda(fused, q_weight, pos, block_table, angles)
+    cq = torch.empty((rows, q_rank), dtype=fused.dtype, device=fused.device)
+    _lib.call("b200_latent_prep", _ptr(fused), fused.stride(0), _ptr(q_weight), _ptr(kv_weight), _ptr(pos),
+              int(pos.dtype == torch.int64), _ptr(slot), _ptr(active), _ptr(block_table), block_table.stride(0), _ptr(angles),
+              _ptr(cache), _ptr(cq), rows, q_rank, true_q_rank, rank, true_rank, rot,
+              angles.shape[1] if cache is not None else 0, float(eps), _f32(fused), int(overlap), _stream())
+    return cq
+
+
+def rope_interleaved(x, offset: int, pos, angles) -> None:
+    """Rotates pairs (offset + 2i, offset + 2i + 1) of x [rows, heads, D] in place; pos int32 [rows]."""
+    assert x.ndim == 3 and x.is_contiguous() and pos.dtype == torch.int32 and angles.is_contiguous()
+    _require_cuda(x, pos, angles)
+    _lib.call("b200_rope_interleaved", _ptr(x), x.stride(0), x.stride(1), offset, x.shape[1], angles.shape[1], _ptr(pos),
+              _ptr(angles), x.shape[0], _f32(x), _stream())
+
+
+def latent_gather(cache, block_table, slots, cu_k, k_pos0, keys: int, max_keys: int):
+    """Cache rows of a run of positions per sequence, packed: [keys, row]."""
+    out = torch.empty((keys, cache.shape[2]), dtype=cache.dtype, device=cache.device)
+    _require_cuda(cache, block_table, slots, cu_k, k_pos0)
+    _lib.call("b200_latent_gather", _ptr(cache), _ptr(out), _ptr(block_table), block_table.stride(0), _ptr(slots), _ptr(cu_k),
+              _ptr(k_pos0), slots.numel(), max_keys, cache.shape[2] * cache.element_size(), _stream())
+    return out
+
+
+def latent_prefill(q, kv, ctx, cu_q, cu_k, q_pos0, k_pos0, max_q: int, vdim: int, rank: int, window: int, scale: float):
+    """Windowed causal attention of packed queries q [tokens, heads, dim + rot] over expanded keys and values
+    kv [keys, heads*dim | heads*vdim] and the shared rotated parts in ctx [keys, rank + rot] -> [tokens, heads*vdim]."""
+    tokens, heads, width = q.shape
+    rot = ctx.shape[1] - rank
+    dim = width - rot
+    assert kv.shape == (ctx.shape[0], heads * (dim + vdim)) and q.is_contiguous() and kv.is_contiguous() and ctx.is_contiguous()
+    _require_cuda(q, kv, ctx)
+    out = torch.empty((tokens, heads * vdim), dtype=q.dtype, device=q.device)
+    _lib.call("b200_latent_prefill_simple", _ptr(q), _ptr(kv), _ptr(ctx), _ptr(out), _ptr(cu_q), _ptr(cu_k), _ptr(q_pos0),
+              _ptr(k_pos0), cu_q.numel() - 1, max_q, heads, dim, rot, vdim, rank, min(window, 1 << 30), float(scale), _f32(q),
+              _stream())
+    return out
+
+
+def latent_absorb(q, w_uk, pos, angles, overlap: int = 0):
+    """q [B, heads, dim + rot], w_uk [heads, dim, rank] -> [B, heads, rank + rot] with the rotated part rotated."""
+    batch, heads, width = q.shape
+    _, dim, rank = w_uk.shape
+    rot = width - dim
+    assert q.is_contiguous() and w_uk.is_contiguous() and w_uk.shape[0] == heads and pos.dtype == torch.int64
+    _require_cuda(q, w_uk, pos, angles)
+    out = torch.empty((batch, heads, rank + rot), dtype=q.dtype, device=q.device)
+    _lib.call("b200_latent_absorb", _ptr(q), _ptr(w_uk), _ptr(pos), _ptr(angles), _ptr(out), batch, heads, dim, rot,
+              angles.shape[1], rank, _f32(q), int(overlap), _stream())
+    return out
+
+
+def latent_decode_workspace(batch: int, heads: int, rank: int, splits: int, device) -> tuple[torch.Tensor, torch.Tensor]:
+    return (torch.empty((batch, heads, splits, 2), dtype=torch.float32, device=device),
+            torch.empty((batch, heads, splits, rank), dtype=torch.float32, device=device))
+
+
+def latent_decode(q, cache, block_table, pos, active, workspace, window: int, scale: float, overlap: int = 0) -> None:
+    """Decode attention of q [B, heads, rank + rot] over the paged rows; leaves the split results in `workspace`."""
+    ml, o = workspace
+    batch, heads, splits, rank = o.shape
+    assert q.shape == (batch, heads, cache.shape[2]) and q.is_contiguous() and pos.dtype == torch.int64
+    _require_cuda(q, cache, block_table, pos, ml, o)
+    _lib.call("b200_latent_decode_simple", _ptr(q), _ptr(cache), _ptr(block_table), block_table.stride(0), _ptr(pos),
+              _ptr(active), _ptr(ml), _ptr(o), batch, heads, rank, cache.shape[2] - rank, min(window, 1 << 30), splits,
+              float(scale), _f32(q), int(overlap), _stream())
+
+
+def latent_value(workspace, w_uv, dtype, overlap: int = 0):
+    """Merges the splits and applies w_uv [heads, vdim, rank] -> [B, heads*vdim]."""
+    ml, o = workspace
+    batch, heads, splits, rank = o.shape
+    vdim = w_uv.shape[1]
+    assert w_uv.shape == (heads, vdim, rank) and w_uv.is_contiguous() and w_uv.dtype == dtype
+    out = torch.empty((batch, heads * vdim), dtype=dtype, device=o.device)
+    _lib.call("b200_latent_value", _ptr(ml), _ptr(o), _ptr(w_uv), _ptr(out), batch, heads, rank, vdim, splits, _f32(w_uv),
+              int(overlap), _stream())
+    return out

@@ -3,6 +3,7 @@
     python build.py            # incremental: recompiles sources newer than their object
     python build.py --force
     python build.py --verbose  # adds -Xptxas -v (registers / spills / shared memory per kernel)
+    python build.py --part hybrid   # only what that model family needs, as libb200hybrid.so
 
 nvcc cross-compiles, so this runs on a machine without a GPU.
 """
@@ -20,6 +21,13 @@ CSRC = HERE / "csrc"
 INCLUDE = HERE.parent / "include"
 OBJ = HERE / "build"
 LIB = HERE / "libb200attn.so"
+
+# Sources one model family needs, linked into a library of their own (b200attn/_lib.py loads it when the whole library
+# has not been built): what a first run on a machine without built files compiles.
+PARTS = {
+    "hybrid": (HERE / "libb200hybrid.so", ["paged_kv", "tensor_maps", "layer_glue", "skinny_gemm", "streams", "linear_rnn",
+                                           "latent"]),
+}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -39,8 +47,23 @@ def _newest_header() -> float:
     return max(h.stat().st_mtime for h in headers)
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    sources = sorted(CSRC.glob("*.cu"))
+def ensure(part: str) -> Path:
+    """The library a process that only needs `part` loads: the whole one when it is built and newer than the part's
+    sources, else the part's own, (re)built if necessary."""
+    lib, names = PARTS[part]
+    newest = max([_newest_header()] + [(CSRC / f"{n}.cu").stat().st_mtime for n in names])
+    if LIB.exists() and LIB.stat().st_mtime >= newest:
+        return LIB
+    return build(part=part)
+
+
+def build(force: bool = False, verbose: bool = False, part: str | None = None) -> Path:
+    out = LIB
+    if part is None:
+        sources = sorted(CSRC.glob("*.cu"))
+    else:
+        out, names = PARTS[part]
+        sources = [CSRC / f"{n}.cu" for n in names]
     if not sources:
         raise RuntimeError(f"no CUDA sources under {CSRC}")
     OBJ.mkdir(exist_ok=True)
@@ -67,19 +90,20 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     if failed:
         raise RuntimeError("nvcc failed (see stderr)")
     objs = [str(OBJ / (s.stem + ".o")) for s in sources]
-    if jobs or not LIB.exists():
-        link = [_nvcc(), "-shared", "-o", str(LIB), *objs, "-gencode", "arch=compute_100a,code=sm_100a",
+    if jobs or not out.exists() or out.stat().st_mtime < max(Path(o).stat().st_mtime for o in objs):
+        link = [_nvcc(), "-shared", "-o", str(out), *objs, "-gencode", "arch=compute_100a,code=sm_100a",
                 "-Xcompiler", "-fPIC", "-lcudart"]
         res = subprocess.run(link, capture_output=True, text=True)
         if res.returncode != 0:
             sys.stderr.write(res.stdout + res.stderr)
             raise RuntimeError("link failed")
-    return LIB
+    return out
 
 
 if __name__ == "__main__":
     ap = argparse.ArgumentParser()
     ap.add_argument("--force", action="store_true")
     ap.add_argument("--verbose", action="store_true")
+    ap.add_argument("--part", choices=sorted(PARTS))
     a = ap.parse_args()
-    print(build(force=a.force, verbose=a.verbose))
+    print(build(force=a.force, verbose=a.verbose, part=a.part))

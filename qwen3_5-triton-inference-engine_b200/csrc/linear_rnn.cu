@@ -1,0 +1,590 @@
+// Recurrent mixers whose gates read only the current token, over packed batches (prefill) and one token per slot
+// (decode).  States are fp32 and live in per-slot caches; a sequence whose first token sits at position 0 starts from
+// zero whatever the slot held before.
+//
+//   minGRU (element-wise):  z = sigmoid(z' + zb), u = x' + xb, c = u >= 0 ? u + 1/2 : sigmoid(u)
+//                           S_t = (1 - z) S_(t-1) + z c,   out = S_t * silu(g)
+//     Prefill cuts every sequence into chunks: pass 1 reduces a chunk to (product of 1 - z, state it leaves from zero),
+//     pass 2 folds the chunks in front of its own and replays its chunk.  HBM bound; both passes stream 16-byte rows.
+//   Forget-gated outer-product recurrence (HGRN2 form):  f = l + (1 - l) sigmoid(f' + fb), q = silu(q')
+//                           S_t = diag(f) S_(t-1) + (1 - f) v^T,   o = S_t^T q,   out = rms(o) * w per head
+//     Prefill is token-serial in fp32 (no cumulative products of gates, so nothing can under- or overflow): a warp owns
+//     COLS state columns, a lane dim/32 rows of each as packed fp32 pairs (fma.rn.f32x2); 16 tokens of gates are staged
+//     in shared memory at a time, the next 16 are loaded while they are worked on.
+#include "b200_attn.h"
+#include "elem.cuh"
+
+namespace b200 {
+
+// ------------------------------------------------------------------------------------------------------------ minGRU
+struct MinGruParams {
+  const void* zxg;          // [rows, stride] E: [z | x | g], each `width` wide
+  int64_t stride;
+  const float* bias;        // [z bias | x bias] 2 * width
+  float* state;             // [slots, width]
+  const int32_t* cu;        // [n + 1] packed rows of the sequences
+  const int32_t* slots;     // [n]
+  const int32_t* start;     // [n] position of each sequence's first packed token
+  float2* chunk_ab;         // [n, chunks, width] workspace of pass 1
+  void* out;                // [rows, width] E
+  int width, chunk, chunks;
+};
+
+template <typename E>
+__device__ __forceinline__ void mingru_gate(float z_raw, float u, float zb, float xb, float& keep, float& add) {
+  const float z = sigmoid_f<E>(z_raw + zb);
+  u += xb;
+  const float cand = u >= 0.f ? u + 0.5f : sigmoid_f<E>(u);
+  keep = 1.0f - z;
+  add = z * cand;
+}
+
+// grid (width / (128 * 2), chunks, sequences); thread = 2 channels
+template <typename E, bool REPLAY>
+__global__ void __launch_bounds__(128) mingru_scan_kernel(const __grid_constant__ MinGruParams p) {
+  const int seq = blockIdx.z, chunk = blockIdx.y;
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 2;
+  const int row0 = p.cu[seq], len = p.cu[seq + 1] - row0;
+  const int t0 = chunk * p.chunk, t1 = min(t0 + p.chunk, len);
+  if (t0 >= len || c >= p.width) return;
+  if (!REPLAY && t1 == len) return;  // nobody folds the last chunk
+  const float2 zb = *reinterpret_cast<const float2*>(p.bias + c), xb = *reinterpret_cast<const float2*>(p.bias + p.width + c);
+  float s0 = 0.f, s1 = 0.f, a0 = 1.f, a1 = 1.f;
+  float* state = p.state + static_cast<int64_t>(p.slots[seq]) * p.width + c;
+  const int64_t ab_base = static_cast<int64_t>(seq) * p.chunks * p.width + c;
+  if (REPLAY) {
+    if (p.start[seq] > 0) {
+      // (unchanged during this launch: the commit kernel behind it writes the slot)
+      const float2 s = *reinterpret_cast<const float2*>(state);
+      s0 = s.x;
+      s1 = s.y;
+    }
+#pragma unroll 4
+    for (int i = 0; i < chunk; ++i) {
+      const float4 ab = *reinterpret_cast<const float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(i) * p.width);
+      s0 = fmaf(ab.x, s0, ab.y);
+      s1 = fmaf(ab.z, s1, ab.w);
+    }
+  }
+  const E* base = static_cast<const E*>(p.zxg) + static_cast<int64_t>(row0) * p.stride + c;
+  auto two = [](const E* q) {
+    if constexpr (sizeof(E) == 2) {
+      const uint32_t v = *reinterpret_cast<const uint32_t*>(q);
+      return make_float2(bf16_lo(v), bf16_hi(v));
+    } else {
+      return *reinterpret_cast<const float2*>(q);
+    }
+  };
+  constexpr int U = 8;  // rows in flight
+  for (int t = t0; t < t1; t += U) {
+    float2 z[U], x[U], g[U];
+#pragma unroll
+    for (int i = 0; i < U; ++i)
+      if (t + i < t1) {
+        const E* r = base + static_cast<int64_t>(t + i) * p.stride;
+        z[i] = two(r);
+        x[i] = two(r + p.width);
+        if (REPLAY) g[i] = two(r + 2 * p.width);
+      }
+#pragma unroll
+    for (int i = 0; i < U; ++i)
+      if (t + i < t1) {
+        float k0, k1, b0, b1;
+        mingru_gate<E>(z[i].x, x[i].x, zb.x, xb.x, k0, b0);
+        mingru_gate<E>(z[i].y, x[i].y, zb.y, xb.y, k1, b1);
+        s0 = fmaf(k0, s0, b0);
+        s1 = fmaf(k1, s1, b1);
+        if (REPLAY) {
+          E* o = static_cast<E*>(p.out) + static_cast<int64_t>(row0 + t + i) * p.width + c;
+          const float o0 = s0 * silu_f<E>(g[i].x), o1 = s1 * silu_f<E>(g[i].y);
+          if constexpr (sizeof(E) == 2) *reinterpret_cast<uint32_t*>(o) = pack_bf16(o0, o1);
+          else *reinterpret_cast<float2*>(o) = make_float2(o0, o1);
+        } else {
+          a0 *= k0;
+          a1 *= k1;
+        }
+      }
+  }
+  if (!REPLAY) *reinterpret_cast<float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(chunk) * p.width) = make_float4(a0, s0, a1, s1);
+  else if (t1 == len) {
+    // final state into the workspace's last chunk slot; a copy kernel behind this one moves it to the slot, so that no
+    // chunk of this launch can see it
+    *reinterpret_cast<float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(p.chunks - 1) * p.width) = make_float4(s0, 0.f, s1, 0.f);
+  }
+}
+
+__global__ void __launch_bounds__(256) mingru_commit_kernel(const __grid_constant__ MinGruParams p) {
+  const int seq = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
+  if (c >= p.width || p.cu[seq + 1] == p.cu[seq]) return;
+  p.state[static_cast<int64_t>(p.slots[seq]) * p.width + c] =
+      p.chunk_ab[(static_cast<int64_t>(seq) * p.chunks + p.chunks - 1) * p.width + c].x;
+}
+
+// one token per slot; thread = 4 channels
+template <typename E>
+__global__ void __launch_bounds__(128) mingru_decode_kernel(const E* zxg, int64_t stride, const float* bias, float* state,
+                                                            const int64_t* pos, const int64_t* active, E* out, int width,
+                                                            int overlap) {
+  const int b = blockIdx.y, c = (blockIdx.x * 128 + threadIdx.x) * 4;
+  if (overlap & OVERLAP_TRIGGER) pdl_trigger();
+  pdl_wait();
+  if (c >= width) return;
+  const bool on = !active || active[b] != 0;
+  const bool fresh = pos[b] == 0;
+  const E* r = zxg + b * stride + c;
+  const float4 z = load4(r), x = load4(r + width), g = load4(r + 2 * width);
+  const float4 zb = load4(bias + c), xb = load4(bias + width + c);
+  float* st = state + static_cast<int64_t>(b) * width + c;
+  float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : load4(st);
+  float k, a;
+  mingru_gate<E>(z.x, x.x, zb.x, xb.x, k, a), s.x = fmaf(k, s.x, a);
+  mingru_gate<E>(z.y, x.y, zb.y, xb.y, k, a), s.y = fmaf(k, s.y, a);
+  mingru_gate<E>(z.z, x.z, zb.z, xb.z, k, a), s.z = fmaf(k, s.z, a);
+  mingru_gate<E>(z.w, x.w, zb.w, xb.w, k, a), s.w = fmaf(k, s.w, a);
+  if (on) store4(st, s);
+  store4(out + static_cast<int64_t>(b) * width + c,
+         make_float4(s.x * silu_f<E>(g.x), s.y * silu_f<E>(g.y), s.z * silu_f<E>(g.z), s.w * silu_f<E>(g.w)));
+}
+
+// ------------------------------------------------------------------------------------------------------------- HGRN2
+// packed fp32 pairs
+struct F2 {
+  uint64_t v;
+};
+__device__ __forceinline__ F2 f2(float lo, float hi) {
+  F2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 unf2(F2 a) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a.v));
+  return r;
+}
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+  F2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+  return r;
+}
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+  F2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return r;
+}
+
+struct OuterRnnParams {
+  const void* qfv;         // [rows, stride] E: [q heads*dim | f heads*dim | v heads*vdim]
+  int64_t stride;
+  const float* lower;      // [heads*dim]
+  const float* bias;       // [heads*dim]
+  float* state;            // [slots, heads, dim, vdim]
+  const int32_t* cu;
+  const int32_t* slots;
+  const int32_t* start;
+  float* o;                // [rows, heads*vdim] fp32, before the head norm
+  int heads, dim, vdim;    // padded sizes: dim a multiple of 32, vdim a multiple of 16
+};
+
+constexpr int OR_TB = 16;        // tokens staged at a time
+constexpr int OR_WARPS = 4;
+constexpr int OR_THREADS = OR_WARPS * 32;
+
+// RP = row pairs per lane (dim = 64 * RP, or dim = 32 with RP = 1 and the second row of a pair absent -> dim is padded
+// to a multiple of 64 by the caller of this template), COLS = columns per warp.
+// grid (vdim / (4 * COLS), heads, sequences)
+template <typename E, int RP, int COLS>
+__global__ void __launch_bounds__(OR_THREADS) outer_rnn_prefill_kernel(const __grid_constant__ OuterRnnParams p) {
+  constexpr int DIM = 64 * RP;                       // rows incl. padding
+  constexpr int CT = OR_WARPS * COLS;                // columns of the CTA
+  constexpr int CPT = (DIM + OR_THREADS - 1) / OR_THREADS;  // gate channels per thread
+  extern __shared__ __align__(16) float or_smem[];
+  float* fs = or_smem;                               // [2][TB][DIM]
+  float* qs = fs + 2 * OR_TB * DIM;                  // [2][TB][DIM]
+  float* vs = qs + 2 * OR_TB * DIM;                  // [2][TB][CT][2]  every v twice: a ready-made pair
+  float* os = vs + 2 * OR_TB * CT * 2;               // [TB][CT]
+  const int seq = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * CT;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int row0 = p.cu[seq], len = p.cu[seq + 1] - row0;
+  if (len <= 0) return;
+  const int hd = p.heads * p.dim;
+  const E* base = static_cast<const E*>(p.qfv) + static_cast<int64_t>(row0) * p.stride;
+  float low[CPT], fb[CPT];
+#pragma unroll
+  for (int i = 0; i < CPT; ++i) {
+    const int ch = tid + i * OR_THREADS;
+    low[i] = ch < p.dim ? p.lower[head * p.dim + ch] : 0.f;
+    fb[i] = ch < p.dim ? p.bias[head * p.dim + ch] : 0.f;
+  }
+  // the raw rows of the next block travel in registers
+  float rq[CPT][OR_TB], rf[CPT][OR_TB], rv[(OR_TB * CT + OR_THREADS - 1) / OR_THREADS];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+      const int ch = tid + i * OR_THREADS;
+      if (ch < p.dim) {
+#pragma unroll
+        for (int t = 0; t < OR_TB; ++t)
+          if (t0 + t < len) {
+            const E* r = base + static_cast<int64_t>(t0 + t) * p.stride + head * p.dim + ch;
+            rq[i][t] = load1(r);
+            rf[i][t] = load1(r + hd);
+          }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < (OR_TB * CT + OR_THREADS - 1) / OR_THREADS; ++i) {
+      const int e = tid + i * OR_THREADS, t = e / CT, c = e % CT;
+      rv[i] = 0.f;
+      if (e < OR_TB * CT && t0 + t < len && col0 + c < p.vdim)
+        rv[i] = load1(base + static_cast<int64_t>(t0 + t) * p.stride + 2 * hd + head * p.vdim + col0 + c);
+    }
+  };
+  auto stage = [&](int t0, int buf) {
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+      const int ch = tid + i * OR_THREADS;
+      if (ch < DIM) {
+#pragma unroll
+        for (int t = 0; t < OR_TB; ++t) {
+          float q = 0.f, f = 1.f;                    // padding rows and tokens: keep the state, read nothing
+          if (ch < p.dim && t0 + t < len) {
+            q = silu_f<E>(rq[i][t]);
+            f = low[i] + (1.0f - low[i]) * sigmoid_f<E>(rf[i][t] + fb[i]);
+          }
+          fs[(buf * OR_TB + t) * DIM + ch] = f;
+          qs[(buf * OR_TB + t) * DIM + ch] = q;
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < (OR_TB * CT + OR_THREADS - 1) / OR_THREADS; ++i) {
+      const int e = tid + i * OR_THREADS;
+      if (e < OR_TB * CT) *reinterpret_cast<float2*>(vs + (buf * OR_TB * CT + e) * 2) = make_float2(rv[i], rv[i]);
+    }
+  };
+  // state: rows lane * 2 * RP + 2 * i (+1), columns col0 + warp * COLS + c
+  F2 S[RP][COLS];
+  float* st = p.state + (static_cast<int64_t>(p.slots[seq]) * p.heads + head) * p.dim * p.vdim;
+  const bool carry = p.start[seq] > 0;
+  const int my_col = col0 + warp * COLS;
+#pragma unroll
+  for (int i = 0; i < RP; ++i)
+#pragma unroll
+    for (int c = 0; c < COLS; ++c) {
+      const int r = lane * 2 * RP + 2 * i;
+      float lo = 0.f, hi = 0.f;
+      if (carry && my_col + c < p.vdim) {
+        if (r < p.dim) lo = st[static_cast<int64_t>(r) * p.vdim + my_col + c];
+        if (r + 1 < p.dim) hi = st[static_cast<int64_t>(r + 1) * p.vdim + my_col + c];
+      }
+      S[i][c] = f2(lo, hi);
+    }
+  fetch(0);
+  stage(0, 0);
+  __syncthreads();
+  const int blocks = (len + OR_TB - 1) / OR_TB;
+  for (int blk = 0; blk < blocks; ++blk) {
+    const int t0 = blk * OR_TB, buf = blk & 1;
+    if (blk + 1 < blocks) fetch(t0 + OR_TB);
+    const int n = min(OR_TB, len - t0);
+    const float* fsb = fs + buf * OR_TB * DIM + lane * 2 * RP;
+    const float* qsb = qs + buf * OR_TB * DIM + lane * 2 * RP;
+    const float* vsb = vs + (buf * OR_TB * CT + warp * COLS) * 2;
+#pragma unroll 2
+    for (int t = 0; t < n; ++t) {
+      F2 f[RP], q[RP], k[RP], v[COLS];
+#pragma unroll
+      for (int i = 0; i < RP; ++i) {
+        const float2 a = *reinterpret_cast<const float2*>(fsb + t * DIM + 2 * i);
+        const float2 b = *reinterpret_cast<const float2*>(qsb + t * DIM + 2 * i);
+        f[i] = f2(a.x, a.y);
+        q[i] = f2(b.x, b.y);
+        k[i] = f2(1.0f - a.x, 1.0f - a.y);
+      }
+#pragma unroll
+      for (int c = 0; c < COLS; c += 2) {
+        const float4 w = *reinterpret_cast<const float4*>(vsb + (t * CT + c) * 2);
+        v[c] = f2(w.x, w.y);
+        v[c + 1] = f2(w.z, w.w);
+      }
+      float o[COLS];
+#pragma unroll
+      for (int c = 0; c < COLS; ++c) {
+        F2 acc = f2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < RP; ++i) {
+          S[i][c] = fma2(f[i], S[i][c], mul2(k[i], v[c]));
+          acc = fma2(q[i], S[i][c], acc);
+        }
+        const float2 a = unf2(acc);
+        o[c] = a.x + a.y;
+      }
+      // sum over the 32 lanes, halving the number of columns a lane carries at each step
+#pragma unroll
+      for (int half = COLS / 2, bit = 16; half >= 1; half >>= 1, bit >>= 1) {
+        const bool upper = (lane & bit) != 0;
+#pragma unroll
+        for (int c = 0; c < half; ++c) {
+          const float give = upper ? o[c] : o[c + half];
+          const float keep = upper ? o[c + half] : o[c];
+          o[c] = keep + __shfl_xor_sync(0xffffffffu, give, bit);
+        }
+      }
+      constexpr int LOGC = COLS == 8 ? 3 : COLS == 4 ? 2 : 1;
+#pragma unroll
+      for (int bit = 16 >> LOGC; bit >= 1; bit >>= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], bit);
+      // lane's column: its top LOGC bits select it, most significant first
+      if ((lane & ((32 >> LOGC) - 1)) == 0) os[t * CT + warp * COLS + (lane >> (5 - LOGC))] = o[0];
+    }
+    if (blk + 1 < blocks) stage(t0 + OR_TB, buf ^ 1);
+    __syncthreads();
+    for (int e = tid; e < n * CT; e += OR_THREADS) {
+      const int t = e / CT, c = e % CT;
+      if (col0 + c < p.vdim) p.o[static_cast<int64_t>(row0 + t0 + t) * p.heads * p.vdim + head * p.vdim + col0 + c] = os[e];
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < RP; ++i)
+#pragma unroll
+    for (int c = 0; c < COLS; ++c) {
+      const int r = lane * 2 * RP + 2 * i;
+      const float2 a = unf2(S[i][c]);
+      if (my_col + c < p.vdim) {
+        if (r < p.dim) st[static_cast<int64_t>(r) * p.vdim + my_col + c] = a.x;
+        if (r + 1 < p.dim) st[static_cast<int64_t>(r + 1) * p.vdim + my_col + c] = a.y;
+      }
+    }
+}
+
+// out[r, :] = o[r, :] / sqrt(mean(o^2) + eps) * w for rows (token, head); one warp per row
+template <typename E>
+__global__ void __launch_bounds__(256) head_rms_kernel(const float* o, const float* w, E* out, int64_t rows, int vdim,
+                                                       int true_vdim, float eps) {
+  const int64_t r = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (r >= rows) return;
+  const float* x = o + r * vdim;
+  float sq = 0.f;
+  for (int c = lane * 4; c < vdim; c += 128) {
+    const float4 a = load4(x + c);
+    sq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+  }
+  const float scale = 1.0f / sqrtf(warp_sum(sq) / static_cast<float>(true_vdim) + eps);
+  for (int c = lane * 4; c < vdim; c += 128) {
+    const float4 a = load4(x + c), g = load4(w + c);
+    store4(out + r * vdim + c, make_float4(a.x * scale * g.x, a.y * scale * g.y, a.z * scale * g.z, a.w * scale * g.w));
+  }
+}
+
+// One token per slot, one CTA per (head, slot): state in, state out, head norm inside.  A warp walks rows, its lanes
+// cover the columns four at a time (several rows at once when vdim < 128).
+constexpr int OD_WARPS = 8;
+constexpr int OD_MAX_VDIM = 512;
+template <typename E>
+__global__ void __launch_bounds__(OD_WARPS * 32)
+outer_rnn_decode_kernel(const E* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
+                        const int64_t* pos, const int64_t* active, E* out, int heads, int dim, int vdim, int true_vdim,
+                        float eps, int lanes_per_row, int overlap) {
+  extern __shared__ __align__(16) float od_smem[];
+  float* fs = od_smem;            // [dim]
+  float* qs = fs + dim;           // [dim]
+  float* vv = qs + dim;           // [vdim]
+  float* part = vv + vdim;        // [OD_WARPS][vdim]
+  __shared__ float red[32];
+  const int head = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (overlap & OVERLAP_TRIGGER) pdl_trigger();
+  pdl_wait();
+  const bool on = !active || active[b] != 0;
+  const bool fresh = pos[b] == 0;
+  const E* row = qfv + b * stride;
+  const int hd = heads * dim;
+  for (int i = tid; i < dim; i += OD_WARPS * 32) {
+    const int ch = head * dim + i;
+    const float l = lower[ch];
+    qs[i] = silu_f<E>(load1(row + ch));
+    fs[i] = l + (1.0f - l) * sigmoid_f<E>(load1(row + hd + ch) + bias[ch]);
+  }
+  for (int i = tid; i < vdim; i += OD_WARPS * 32) vv[i] = load1(row + 2 * hd + head * vdim + i);
+  __syncthreads();
+  float* st = state + (static_cast<int64_t>(b) * heads + head) * dim * vdim;
+  const int rows_at_once = 32 / lanes_per_row, sub = lane / lanes_per_row, cl = (lane % lanes_per_row) * 4;
+  for (int c0 = 0; c0 < vdim; c0 += 128) {
+    const int c = c0 + cl;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < vdim) {
+      const float4 v = load4(vv + c);
+      constexpr int U = 8;
+      const int step = OD_WARPS * rows_at_once;
+      for (int r0 = warp * rows_at_once + sub; r0 < dim; r0 += step * U) {
+        float4 s[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int r = r0 + u * step;
+          s[u] = (r < dim && !fresh) ? load4(st + static_cast<int64_t>(r) * vdim + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int r = r0 + u * step;
+          if (r < dim) {
+            const float f = fs[r], k = 1.0f - f, q = qs[r];
+            s[u].x = fmaf(f, s[u].x, k * v.x), s[u].y = fmaf(f, s[u].y, k * v.y);
+            s[u].z = fmaf(f, s[u].z, k * v.z), s[u].w = fmaf(f, s[u].w, k * v.w);
+            if (on) store4(st + static_cast<int64_t>(r) * vdim + c, s[u]);
+            o.x = fmaf(q, s[u].x, o.x), o.y = fmaf(q, s[u].y, o.y);
+            o.z = fmaf(q, s[u].z, o.z), o.w = fmaf(q, s[u].w, o.w);
+          }
+        }
+      }
+    }
+    for (int bit = lanes_per_row; bit < 32; bit <<= 1) {
+      o.x += __shfl_xor_sync(0xffffffffu, o.x, bit), o.y += __shfl_xor_sync(0xffffffffu, o.y, bit);
+      o.z += __shfl_xor_sync(0xffffffffu, o.z, bit), o.w += __shfl_xor_sync(0xffffffffu, o.w, bit);
+    }
+    if (sub == 0 && c < vdim) store4(part + warp * vdim + c, o);
+  }
+  __syncthreads();
+  float sum[OD_MAX_VDIM / (OD_WARPS * 32)], sq[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < OD_MAX_VDIM / (OD_WARPS * 32); ++i) {
+    const int c = tid + i * OD_WARPS * 32;
+    sum[i] = 0.f;
+    if (c < vdim)
+#pragma unroll
+      for (int w = 0; w < OD_WARPS; ++w) sum[i] += part[w * vdim + c];
+    sq[0] += sum[i] * sum[i];
+  }
+  block_sum<1>(sq, red);
+  const float scale = 1.0f / sqrtf(sq[0] / static_cast<float>(true_vdim) + eps);
+#pragma unroll
+  for (int i = 0; i < OD_MAX_VDIM / (OD_WARPS * 32); ++i) {
+    const int c = tid + i * OD_WARPS * 32;
+    if (c < vdim) store1(out + (static_cast<int64_t>(b) * heads + head) * vdim + c, sum[i] * scale * norm[c]);
+  }
+}
+
+template <typename E, int RP, int COLS>
+static int launch_outer_cols(const OuterRnnParams& p, int n, cudaStream_t st) {
+  constexpr int DIM = 64 * RP, CT = OR_WARPS * COLS;
+  constexpr int smem = (4 * OR_TB * DIM + 2 * OR_TB * CT * 2 + OR_TB * CT) * 4;
+  static_assert(smem <= 200 * 1024, "staging must fit");
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (smem > 48 * 1024 && dev >= 0 && dev < 64 && !configured[dev]) {
+    if (cudaFuncSetAttribute(outer_rnn_prefill_kernel<E, RP, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      return fail(ERR_RUNTIME, "hgrn2_prefill: cannot raise dynamic shared memory to %d", smem);
+    configured[dev] = true;
+  }
+  outer_rnn_prefill_kernel<E, RP, COLS><<<dim3((p.vdim + CT - 1) / CT, p.heads, n), OR_THREADS, smem, st>>>(p);
+  return check_launch("hgrn2_prefill");
+}
+
+template <typename E, int RP>
+static int launch_outer(const OuterRnnParams& p, int n, cudaStream_t st) {
+  // wide columns share the gates of a token among more state; narrow ones give more CTAs when there are few heads
+  const int64_t wide = static_cast<int64_t>((p.vdim + 31) / 32) * p.heads * n;
+  if (RP <= 2 && wide >= 2 * sm_count()) return launch_outer_cols<E, RP, 8>(p, n, st);
+  return launch_outer_cols<E, RP, 4>(p, n, st);
+}
+
+template <typename E>
+static int launch_outer_rows(const OuterRnnParams& p, int n, cudaStream_t st) {
+  if (p.dim <= 64) return launch_outer<E, 1>(p, n, st);
+  if (p.dim <= 128) return launch_outer<E, 2>(p, n, st);
+  return launch_outer<E, 4>(p, n, st);
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" int64_t b200_mingru_workspace_bytes(int32_t batch, int32_t chunks, int32_t width) {
+  return static_cast<int64_t>(batch) * chunks * width * 8;
+}
+
+extern "C" int b200_mingru_prefill(const void* zxg, int64_t stride, const float* bias, float* state, const int32_t* cu_seqlens,
+                                   const int32_t* slots, const int32_t* start, void* workspace, void* out, int32_t batch,
+                                   int32_t chunk, int32_t chunks, int32_t width, int32_t f32, b200_stream_t stream) {
+  if (batch <= 0 || chunks <= 0) return OK;
+  B200_REQUIRE(width > 0 && width % 4 == 0 && stride % 4 == 0 && chunk > 0 && batch <= 65535 && chunks <= 65535,
+               "mingru_prefill: width and stride must be multiples of 4, at most 65535 sequences and chunks");
+  B200_REQUIRE(aligned16(zxg) && aligned16(bias) && aligned16(state) && aligned16(workspace) && aligned16(out),
+               "mingru_prefill: tensors must be 16-byte aligned");
+  MinGruParams p = {zxg, stride, bias, state, cu_seqlens, slots, start, static_cast<float2*>(workspace), out, width, chunk, chunks};
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((width / 2 + 127) / 128, chunks, batch);
+  if (f32) {
+    if (chunks > 1) mingru_scan_kernel<float, false><<<grid, 128, 0, st>>>(p);
+    mingru_scan_kernel<float, true><<<grid, 128, 0, st>>>(p);
+  } else {
+    if (chunks > 1) mingru_scan_kernel<__nv_bfloat16, false><<<grid, 128, 0, st>>>(p);
+    mingru_scan_kernel<__nv_bfloat16, true><<<grid, 128, 0, st>>>(p);
+  }
+  mingru_commit_kernel<<<dim3((width + 255) / 256, batch), 256, 0, st>>>(p);
+  return check_launch("mingru_prefill");
+}
+
+extern "C" int b200_mingru_decode(const void* zxg, int64_t stride, const float* bias, float* state, const int64_t* pos,
+                                  const int64_t* active, void* out, int32_t batch, int32_t width, int32_t f32,
+                                  int32_t overlap, b200_stream_t stream) {
+  if (batch <= 0) return OK;
+  B200_REQUIRE(width > 0 && width % 4 == 0 && stride % 4 == 0 && batch <= 65535,
+               "mingru_decode: width and stride must be multiples of 4, at most 65535 slots");
+  B200_REQUIRE(aligned16(zxg) && aligned16(bias) && aligned16(state) && aligned16(out), "mingru_decode: unaligned tensor");
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((width / 4 + 127) / 128, batch);
+  const bool early = (overlap & OVERLAP_START) != 0;
+  const cudaError_t e =
+      f32 ? launch_pdl(early, mingru_decode_kernel<float>, grid, dim3(128), 0, st, static_cast<const float*>(zxg), stride, bias,
+                       state, pos, active, static_cast<float*>(out), width, overlap)
+          : launch_pdl(early, mingru_decode_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, static_cast<const __nv_bfloat16*>(zxg),
+                       stride, bias, state, pos, active, static_cast<__nv_bfloat16*>(out), width, overlap);
+  if (e != cudaSuccess) return fail(ERR_LAUNCH, "mingru_decode: %s", cudaGetErrorString(e));
+  return check_launch("mingru_decode");
+}
+
+extern "C" int b200_hgrn2_prefill(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm,
+                                  float* state, const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start,
+                                  float* o_scratch, void* out, int32_t batch, int32_t tokens, int32_t heads, int32_t dim,
+                                  int32_t vdim, int32_t true_vdim, float eps, int32_t f32, b200_stream_t stream) {
+  if (batch <= 0 || tokens <= 0) return OK;
+  B200_REQUIRE(dim > 0 && dim <= 256 && vdim > 0 && vdim % 4 == 0 && vdim <= OD_MAX_VDIM && true_vdim <= vdim,
+               "hgrn2_prefill: dim at most 256, vdim a multiple of 4 and at most %d (got %d, %d)", OD_MAX_VDIM, dim, vdim);
+  B200_REQUIRE(heads > 0 && heads <= 65535 && batch <= 65535, "hgrn2_prefill: at most 65535 heads and sequences");
+  B200_REQUIRE(aligned16(o_scratch) && aligned16(out) && aligned16(norm), "hgrn2_prefill: unaligned tensor");
+  OuterRnnParams p = {qfv, stride, lower, bias, state, cu_seqlens, slots, start, o_scratch, heads, dim, vdim};
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const int rc = f32 ? launch_outer_rows<float>(p, batch, st) : launch_outer_rows<__nv_bfloat16>(p, batch, st);
+  if (rc != OK) return rc;
+  const int64_t rows = static_cast<int64_t>(tokens) * heads;
+  const unsigned grid = static_cast<unsigned>((rows + 7) / 8);
+  if (f32) head_rms_kernel<float><<<grid, 256, 0, st>>>(o_scratch, norm, static_cast<float*>(out), rows, vdim, true_vdim, eps);
+  else head_rms_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(o_scratch, norm, static_cast<__nv_bfloat16*>(out), rows, vdim, true_vdim, eps);
+  return check_launch("hgrn2_prefill (norm)");
+}
+
+extern "C" int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm,
+                                 float* state, const int64_t* pos, const int64_t* active, void* out, int32_t batch,
+                                 int32_t heads, int32_t dim, int32_t vdim, int32_t true_vdim, float eps, int32_t f32,
+                                 int32_t overlap, b200_stream_t stream) {
+  if (batch <= 0) return OK;
+  B200_REQUIRE(dim > 0 && dim <= 1024 && vdim > 0 && vdim % 4 == 0 && vdim <= OD_MAX_VDIM && true_vdim <= vdim,
+               "hgrn2_decode: dim at most 1024, vdim a multiple of 4 and at most %d (got %d, %d)", OD_MAX_VDIM, dim, vdim);
+  B200_REQUIRE(heads > 0 && batch <= 65535 && aligned16(state), "hgrn2_decode: unaligned state or too many slots");
+  int lanes = 1;
+  while (lanes < 32 && lanes * 4 < vdim) lanes <<= 1;
+  const int smem = (2 * dim + vdim + OD_WARPS * vdim) * 4 + 16;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const bool early = (overlap & OVERLAP_START) != 0;
+  const dim3 grid(heads, batch);
+  const cudaError_t e =
+      f32 ? launch_pdl(early, outer_rnn_decode_kernel<float>, grid, dim3(OD_WARPS * 32), smem, st, static_cast<const float*>(qfv),
+                       stride, lower, bias, norm, state, pos, active, static_cast<float*>(out), heads, dim, vdim, true_vdim,
+                       eps, lanes, overlap)
+          : launch_pdl(early, outer_rnn_decode_kernel<__nv_bfloat16>, grid, dim3(OD_WARPS * 32), smem, st,
+                       static_cast<const __nv_bfloat16*>(qfv), stride, lower, bias, norm, state, pos, active,
+                       static_cast<__nv_bfloat16*>(out), heads, dim, vdim, true_vdim, eps, lanes, overlap);
+  if (e != cudaSuccess) return fail(ERR_LAUNCH, "hgrn2_decode: %s", cudaGetErrorString(e));
+  return check_launch("hgrn2_decode");
+}

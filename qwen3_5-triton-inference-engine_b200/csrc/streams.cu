@@ -1,0 +1,169 @@
+// Hyper-connected residual streams: the step between two sublayers of a stack that keeps S copies of the residual, one
+// launch for what would be a mix of the streams, the weighted return of the sublayer's output, the read-out of the next
+// sublayer's input and its RMS norm with a single gain:
+//     x_t <- sum_s mix[s, t] x_s + out[t] * y        (all streams from the old ones)
+//     h   = (sum_s in[s] x_s) / sqrt(mean(.^2) + eps) * gain
+// Streams live in fp32 [rows, S, width]; y and h are bf16 or fp32 activations.  Without y the streams come from the
+// embedding table (every stream equal to the token's row), or are only read.
+// HBM / latency bound: one CTA per row, a thread owns 4 columns of every stream per step, all loads before the
+// reduction.  Width is padded to a multiple of 4 with zero columns; the mean runs over the true width.
+#include "b200_attn.h"
+#include "elem.cuh"
+
+namespace b200 {
+
+constexpr int HC_MAX_WIDTH = 8192;
+constexpr int HC_MAX_STREAMS = 16;
+
+struct HyperParams {
+  const void* ids;        // embedding form: token ids of the rows
+  int ids_are_int64;
+  const void* table;      // [vocab, width] E
+  float* streams;         // [rows, S, width]
+  const void* y;          // [rows, width] E or NULL
+  const float* weights;   // [mix S*S | out S | in S | gain]
+  void* h;                // [rows, width] E
+  int s, width, true_width, overlap;
+  float eps;
+};
+
+// V: float4 groups a thread may own
+template <typename E, int MAXS, int V>
+__global__ void __launch_bounds__(512) hyper_connect_kernel(const __grid_constant__ HyperParams p) {
+  __shared__ float wt[HC_MAX_STREAMS * HC_MAX_STREAMS + 2 * HC_MAX_STREAMS + 1];
+  __shared__ float red[32];
+  const int row = blockIdx.x, tid = threadIdx.x, s = p.s, width = p.width;
+  for (int i = tid; i < s * s + 2 * s + 1; i += blockDim.x) wt[i] = p.weights[i];
+  if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
+  pdl_wait();
+  __syncthreads();
+  const float *mix = wt, *out = wt + s * s, *in = out + s;
+  float* x = p.streams + static_cast<int64_t>(row) * s * width;
+  float4 u[V];
+  float sq[1] = {0.f};
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int c = (tid + v * blockDim.x) * 4;
+    u[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c >= width) continue;
+    if (p.ids) {
+      const int64_t id = p.ids_are_int64 ? static_cast<const int64_t*>(p.ids)[row]
+                                         : static_cast<int64_t>(static_cast<const int32_t*>(p.ids)[row]);
+      const float4 e = load4(static_cast<const E*>(p.table) + id * width + c);
+      float total = 0.f;
+#pragma unroll
+      for (int i = 0; i < MAXS; ++i)
+        if (i < s) {
+          store4(x + i * width + c, e);
+          total += in[i];
+        }
+      u[v] = make_float4(total * e.x, total * e.y, total * e.z, total * e.w);
+    } else {
+      float4 old[MAXS];
+#pragma unroll
+      for (int i = 0; i < MAXS; ++i)
+        if (i < s) old[i] = load4(x + i * width + c);
+      if (p.y) {
+        const float4 y = load4(static_cast<const E*>(p.y) + static_cast<int64_t>(row) * width + c);
+#pragma unroll
+        for (int t = 0; t < MAXS; ++t)
+          if (t < s) {
+            const float o = out[t];
+            float4 a = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+#pragma unroll
+            for (int i = 0; i < MAXS; ++i)
+              if (i < s) {
+                const float m = mix[i * s + t];
+                a.x = fmaf(m, old[i].x, a.x), a.y = fmaf(m, old[i].y, a.y);
+                a.z = fmaf(m, old[i].z, a.z), a.w = fmaf(m, old[i].w, a.w);
+              }
+            store4(x + t * width + c, a);
+            const float n = in[t];
+            u[v].x = fmaf(n, a.x, u[v].x), u[v].y = fmaf(n, a.y, u[v].y);
+            u[v].z = fmaf(n, a.z, u[v].z), u[v].w = fmaf(n, a.w, u[v].w);
+          }
+      } else {
+#pragma unroll
+        for (int i = 0; i < MAXS; ++i)
+          if (i < s) {
+            const float n = in[i];
+            u[v].x = fmaf(n, old[i].x, u[v].x), u[v].y = fmaf(n, old[i].y, u[v].y);
+            u[v].z = fmaf(n, old[i].z, u[v].z), u[v].w = fmaf(n, old[i].w, u[v].w);
+          }
+      }
+    }
+    sq[0] += u[v].x * u[v].x + u[v].y * u[v].y + u[v].z * u[v].z + u[v].w * u[v].w;
+  }
+  block_sum<1>(sq, red);
+  const float scale = wt[s * s + 2 * s] / sqrtf(sq[0] / static_cast<float>(p.true_width) + p.eps);
+  E* h = static_cast<E*>(p.h) + static_cast<int64_t>(row) * width;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int c = (tid + v * blockDim.x) * 4;
+    if (c < width) store4(h + c, make_float4(u[v].x * scale, u[v].y * scale, u[v].z * scale, u[v].w * scale));
+  }
+}
+
+template <typename E, int MAXS>
+static cudaError_t launch_hyper(const HyperParams& p, int rows, cudaStream_t st) {
+  const int quads = p.width / 4;
+  const bool early = (p.overlap & OVERLAP_START) != 0;
+  int threads = (quads + 31) / 32 * 32;
+  if (threads <= 512) return launch_pdl(early, hyper_connect_kernel<E, MAXS, 1>, dim3(rows), dim3(threads), 0, st, p);
+  threads = ((quads + 3) / 4 + 31) / 32 * 32;
+  return launch_pdl(early, hyper_connect_kernel<E, MAXS, 4>, dim3(rows), dim3(threads), 0, st, p);
+}
+
+template <typename E>
+static cudaError_t launch_hyper_e(const HyperParams& p, int rows, cudaStream_t st) {
+  if (p.s == 1) return launch_hyper<E, 1>(p, rows, st);
+  if (p.s == 2) return launch_hyper<E, 2>(p, rows, st);
+  if (p.s <= 4) return launch_hyper<E, 4>(p, rows, st);
+  return launch_hyper<E, HC_MAX_STREAMS>(p, rows, st);
+}
+
+// out[r, c] = silu(gate_up[r, c]) * gate_up[r, width + c] for fp32 activations (the bf16 form is b200_swiglu)
+__global__ void __launch_bounds__(256) swiglu_f32_kernel(const float* gate_up, int64_t stride, float* out, int width) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= width) return;
+  const float* row = gate_up + blockIdx.y * stride;
+  const float4 g = load4(row + c), u = load4(row + width + c);
+  store4(out + static_cast<int64_t>(blockIdx.y) * width + c,
+         make_float4(silu_f<float>(g.x) * u.x, silu_f<float>(g.y) * u.y, silu_f<float>(g.z) * u.z, silu_f<float>(g.w) * u.w));
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" int b200_hyper_connect(const void* ids, int32_t ids_are_int64, const void* table, float* streams, const void* y,
+                                  const float* weights, void* h, int32_t rows, int32_t num_streams, int32_t width, int32_t true_width, float eps, int32_t f32,
+                                  int32_t overlap, b200_stream_t stream) {
+  if (rows <= 0) return OK;
+  B200_REQUIRE(num_streams >= 1 && num_streams <= HC_MAX_STREAMS, "hyper_connect: 1 to %d streams (got %d)",
+               HC_MAX_STREAMS, num_streams);
+  B200_REQUIRE(width > 0 && width % 4 == 0 && width <= HC_MAX_WIDTH && true_width > 0 && true_width <= width,
+               "hyper_connect: width must be a multiple of 4, at most %d, and cover the true width (got %d, %d)",
+               HC_MAX_WIDTH, width, true_width);
+  B200_REQUIRE(streams && weights && h && aligned16(streams) && aligned16(h) && (!y || aligned16(y)),
+               "hyper_connect: NULL or unaligned tensor");
+  B200_REQUIRE(!ids || (table && aligned16(table) && !y), "hyper_connect: the embedding form takes a table, no y");
+  HyperParams p = {ids, ids_are_int64, table, streams, y, weights, h, num_streams, width, true_width, overlap, eps};
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const cudaError_t e = f32 ? launch_hyper_e<float>(p, rows, st) : launch_hyper_e<__nv_bfloat16>(p, rows, st);
+  if (e != cudaSuccess) return fail(ERR_LAUNCH, "hyper_connect: %s", cudaGetErrorString(e));
+  return check_launch("hyper_connect");
+}
+
+extern "C" int b200_swiglu_f32(const float* gate_up, int64_t row_stride, float* out, int32_t rows, int32_t intermediate,
+                               b200_stream_t stream) {
+  if (rows <= 0) return OK;
+  B200_REQUIRE(intermediate > 0 && intermediate % 4 == 0 && row_stride % 4 == 0 && aligned16(gate_up) && aligned16(out),
+               "swiglu_f32: width and stride must be multiples of 4, tensors 16-byte aligned");
+  for (int r0 = 0; r0 < rows; r0 += 65535) {
+    const int n = rows - r0 < 65535 ? rows - r0 : 65535;
+    swiglu_f32_kernel<<<dim3((intermediate / 4 + 255) / 256, n), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
+        gate_up + r0 * row_stride, row_stride, out + static_cast<int64_t>(r0) * intermediate, intermediate);
+  }
+  return check_launch("swiglu_f32");
+}
