@@ -505,6 +505,10 @@ int b200_latent_prefill_simple(const void* q, const void* kv, const void* ctx, v
                                const int32_t* cu_k, const int32_t* q_pos0, const int32_t* k_pos0, int32_t batch, int32_t max_q,
                                int32_t heads, int32_t dim, int32_t rot, int32_t vdim, int32_t rank, int32_t window, float scale,
                                int32_t f32, b200_stream_t stream);
+int b200_latent_prefill(const void* q, const void* kv, const void* ctx, void* out, const int32_t* cu_q, const int32_t* cu_k,
+                        const int32_t* q_pos0, const int32_t* k_pos0, int32_t batch, int32_t max_q, int32_t tokens,
+                        int32_t keys, int32_t heads, int32_t dim, int32_t true_dim, int32_t rot, int32_t true_rot,
+                        int32_t vdim, int32_t rank, int32_t window, float scale, b200_stream_t stream);
 int b200_latent_absorb(const void* q, const void* w_uk, const int64_t* pos, const float* angles, void* out, int32_t batch,
                        int32_t heads, int32_t dim, int32_t rot, int32_t rot_pairs, int32_t rank, int32_t f32, int32_t overlap,
                        b200_stream_t stream);
@@ -512,6 +516,10 @@ int b200_latent_decode_simple(const void* q, const void* cache, const int32_t* b
                               const int64_t* pos, const int64_t* active, float* ml, float* o, int32_t batch, int32_t heads,
                               int32_t rank, int32_t rot, int32_t window, int32_t splits, float scale, int32_t f32,
                               int32_t overlap, b200_stream_t stream);
+int b200_latent_decode(const void* q, const void* cache, int64_t num_pages, const int32_t* block_table, int64_t table_stride,
+                       const int64_t* pos, const int64_t* active, float* ml, float* o, int32_t batch, int32_t heads,
+                       int32_t rank, int32_t rot, int32_t window, int32_t splits, float scale, int32_t overlap,
+                       b200_stream_t stream);
 int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* out, int32_t batch, int32_t heads, int32_t rank,
                       int32_t vdim, int32_t splits, int32_t f32, int32_t overlap, b200_stream_t stream);
 

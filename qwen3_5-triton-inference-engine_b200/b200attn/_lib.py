@@ -74,6 +74,8 @@ SIGNATURES: dict[str, list] = {
     "b200_rope_interleaved": [P, I64, I32, I32, I32, I32, P, P, I32, I32, P],
     "b200_latent_gather": [P, P, P, I64, P, P, P, I32, I32, I32, P],
     "b200_latent_prefill_simple": [P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, c_float, I32, P],
+    "b200_latent_prefill": [P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32, c_float, P],
+    "b200_latent_decode": [P, P, I64, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, P],
     "b200_latent_absorb": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, P],
     "b200_latent_decode_simple": [P, P, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_latent_value": [P, P, P, P, I32, I32, I32, I32, I32, I32, I32, P],

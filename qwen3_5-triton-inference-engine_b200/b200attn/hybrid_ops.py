@@ -150,15 +150,22 @@ def latent_gather(cache, block_table, slots, cu_k, k_pos0, keys: int, max_keys: 
     return out
 
 
-def latent_prefill(q, kv, ctx, cu_q, cu_k, q_pos0, k_pos0, max_q: int, vdim: int, rank: int, window: int, scale: float):
+def latent_prefill(q, kv, ctx, cu_q, cu_k, q_pos0, k_pos0, max_q: int, true_dim: int, true_rot: int, vdim: int, rank: int,
+                   window: int, scale: float, simple: bool = False):
     """Windowed causal attention of packed queries q [tokens, heads, dim + rot] over expanded keys and values
-    kv [keys, heads*dim | heads*vdim] and the shared rotated parts in ctx [keys, rank + rot] -> [tokens, heads*vdim]."""
+    kv [keys, heads*dim | heads*vdim] and the shared rotated parts in ctx [keys, rank + rot] -> [tokens, heads*vdim].
+    bf16 heads of up to 256 + 256 dimensions run on the tensor-core kernel; simple=True keeps them off it."""
     tokens, heads, width = q.shape
     rot = ctx.shape[1] - rank
     dim = width - rot
     assert kv.shape == (ctx.shape[0], heads * (dim + vdim)) and q.is_contiguous() and kv.is_contiguous() and ctx.is_contiguous()
     _require_cuda(q, kv, ctx)
     out = torch.empty((tokens, heads * vdim), dtype=q.dtype, device=q.device)
+    if q.dtype == torch.bfloat16 and width <= 256 and vdim <= 256 and not simple:
+        _lib.call("b200_latent_prefill", _ptr(q), _ptr(kv), _ptr(ctx), _ptr(out), _ptr(cu_q), _ptr(cu_k), _ptr(q_pos0),
+                  _ptr(k_pos0), cu_q.numel() - 1, max_q, tokens, ctx.shape[0], heads, dim, true_dim, rot, true_rot, vdim, rank,
+                  min(window, 1 << 30), float(scale), _stream())
+        return out
     _lib.call("b200_latent_prefill_simple", _ptr(q), _ptr(kv), _ptr(ctx), _ptr(out), _ptr(cu_q), _ptr(cu_k), _ptr(q_pos0),
               _ptr(k_pos0), cu_q.numel() - 1, max_q, heads, dim, rot, vdim, rank, min(window, 1 << 30), float(scale), _f32(q),
               _stream())
@@ -183,12 +190,29 @@ def latent_decode_workspace(batch: int, heads: int, rank: int, splits: int, devi
             torch.empty((batch, heads, splits, rank), dtype=torch.float32, device=device))
 
 
-def latent_decode(q, cache, block_table, pos, active, workspace, window: int, scale: float, overlap: int = 0) -> None:
-    """Decode attention of q [B, heads, rank + rot] over the paged rows; leaves the split results in `workspace`."""
+LATENT_DECODE_MAX_ROW = 1344     # widest cache row two stages of the tensor-core kernel's ring hold
+
+
+def latent_decode_splits(batch: int, heads: int, span: int, sm_count: int) -> int:
+    """Key ranges per slot: the count whose launch has the shortest longest SM, at ~64 tokens of fixed cost per CTA."""
+    groups = batch * -(-heads // 16)
+    most = max(1, min(LATENT_MAX_SPLITS, span // (2 * PAGE_SIZE)))
+    return min(range(1, most + 1), key=lambda s: (-(-groups * s // sm_count) * (span / s + 64), s))
+
+
+def latent_decode(q, cache, block_table, pos, active, workspace, window: int, scale: float, overlap: int = 0,
+                  simple: bool = False) -> None:
+    """Decode attention of q [B, heads, rank + rot] over the paged rows; leaves the split results in `workspace`.
+    bf16 rows run on the tensor-core kernel where they fit; simple=True keeps them off it."""
     ml, o = workspace
     batch, heads, splits, rank = o.shape
     assert q.shape == (batch, heads, cache.shape[2]) and q.is_contiguous() and pos.dtype == torch.int64
     _require_cuda(q, cache, block_table, pos, ml, o)
+    if q.dtype == torch.bfloat16 and rank <= 1024 and cache.shape[2] <= LATENT_DECODE_MAX_ROW and not simple:
+        _lib.call("b200_latent_decode", _ptr(q), _ptr(cache), cache.shape[0], _ptr(block_table), block_table.stride(0),
+                  _ptr(pos), _ptr(active), _ptr(ml), _ptr(o), batch, heads, rank, cache.shape[2] - rank, min(window, 1 << 30),
+                  splits, float(scale), int(overlap), _stream())
+        return
     _lib.call("b200_latent_decode_simple", _ptr(q), _ptr(cache), _ptr(block_table), block_table.stride(0), _ptr(pos),
               _ptr(active), _ptr(ml), _ptr(o), batch, heads, rank, cache.shape[2] - rank, min(window, 1 << 30), splits,
               float(scale), _f32(q), int(overlap), _stream())

@@ -137,10 +137,7 @@ class LatentAttention:
         if self.kv_from is None:
             state["cache"] = hops.allocate_latent_cache(engine.num_pages, self.rank_p + self.rot_p, engine.dtype,
                                                         device=engine.device)
-        # enough key ranges for every SM to have work, no shorter than four pages each
-        span = min(self.window, engine.max_context)
-        want = -(-2 * engine.sm_count // (engine.batch * -(-self.heads // 16)))
-        splits = max(1, min(want, span // (4 * ops.PAGE_SIZE), hops.LATENT_MAX_SPLITS))
+        splits = hops.latent_decode_splits(engine.batch, self.heads, min(self.window, engine.max_context), engine.sm_count)
         state["workspace"] = engine.shared_workspace(self.heads, self.rank_p, splits)
         return state
 
@@ -158,8 +155,8 @@ class LatentAttention:
             ctx = hops.latent_gather(cache, engine.block_table, batch.slots, span.cu, span.first, span.keys, span.max_keys)
             batch.kept[self.source, self.window] = ctx
         kv = engine.linear(ctx[:, : self.rank_p], self.ukv)
-        out = hops.latent_prefill(q, kv, ctx, batch.cu, span.cu, batch.start, span.first, batch.max_len, self.vdim_p,
-                                  self.rank_p, self.window, self.scale)
+        out = hops.latent_prefill(q, kv, ctx, batch.cu, span.cu, batch.start, span.first, batch.max_len, self.dim,
+                                  self.rot_dim, self.vdim_p, self.rank_p, self.window, self.scale)
         return engine.linear(out, self.o)
 
     def decode(self, h, engine, states):

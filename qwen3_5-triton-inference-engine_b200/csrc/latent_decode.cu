@@ -1,0 +1,276 @@
+// Decode attention over cached latents on the tensor cores: every head of a token scores the same cache rows
+// [latent | rotated key part], so 16 heads are one MMA M tile and a row is read once per 16 heads.
+//
+// One CTA = (key range of a slot, block of 16 heads).  A producer warp brings 32-token tiles (two 16-token pages, one
+// tensor-map TMA box each, 128-byte swizzle, no multicast) through a ring of mbarrier-tracked stages; eight warps work on
+// a tile together:
+//     S[16 x 32]    = q' . rows^T     a warp takes 8 tokens and every other 32-wide step of the row (two warps per group)
+//     P             = exp2(S - m)     a warp owns two head rows, a lane one token; online maximum and sum in fp32
+//     O[16 x rank] += P . latents     a warp owns rank / 8 columns; accumulators stay in registers
+// The kernel is bound by HBM (about 2 * 16 FLOP per byte), far below what 16-row tiles reach on tcgen05 (M = 128), so
+// mma.sync carries the products, as in the paged decode kernels.  Key ranges leave (max, sum, unnormalised O) in fp32;
+// latent_value merges them.  Rows of a tile outside the visible range are zeroed in shared memory before they are used:
+// whatever a page held for an earlier owner cannot reach the sums.  Every wait is bounded.
+#include <mutex>
+
+#include "latent.cuh"
+#include "umma.cuh"
+
+namespace b200 {
+
+constexpr int LD_WARPS = 8;                      // consumers; one more warp produces
+constexpr int LD_THREADS = (LD_WARPS + 1) * 32;
+constexpr int LD_TOK = 32;
+constexpr int LD_MAX_STAGES = 6;
+constexpr int LD_S_PITCH = 36;                   // floats per score row
+constexpr int LD_P_PITCH = 40;                   // bf16 per probability row (80 bytes: ldmatrix rows in different banks)
+constexpr int LD_SMEM_LIMIT = 216 * 1024;         // dynamic; 6 KiB more are static
+
+// NT: value columns per warp / 8 that the accumulators hold (rank <= 64 * NT)
+template <int NT>
+__global__ void __launch_bounds__(LD_THREADS)
+latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_constant__ CUtensorMap map_rows, int stages) {
+  extern __shared__ __align__(1024) uint8_t ld_smem_raw[];
+  __shared__ uint64_t full[LD_MAX_STAGES], empty[LD_MAX_STAGES];
+  __shared__ float ss[2][16][LD_S_PITCH];
+  __shared__ __align__(16) __nv_bfloat16 ps[16][LD_P_PITCH];
+  __shared__ float alphas[16];
+  const int split = blockIdx.x, hb = blockIdx.y, b = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int pitch = p.rank + p.rot, row_bytes = pitch * 2, tile_bytes = LD_TOK * row_bytes, page_bytes = PAGE * row_bytes;
+  const int q_pitch = row_bytes + 16;
+  uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ld_smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* qs = ring + stages * tile_bytes;
+  if (tid == 0) {
+    for (int s = 0; s < stages; ++s) {
+      mbar_init(&full[s], 1);
+      mbar_init(&empty[s], LD_WARPS);
+    }
+    mbar_fence_init();
+  }
+  if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
+  pdl_wait();
+  int lo, hi;
+  latent_split_range(p, b, split, lo, hi);
+  const int heads_here = min(16, p.heads - hb * 16);
+  const int64_t part0 = (static_cast<int64_t>(b) * p.heads + hb * 16) * p.splits + split;
+  if (lo >= hi) {
+    if (tid < heads_here) p.ml[part0 + static_cast<int64_t>(tid) * p.splits] = make_float2(-INFINITY, 0.f);
+    return;
+  }
+  const int page0 = lo / PAGE, pages = (hi + PAGE - 1) / PAGE - page0, tiles = (pages + 1) / 2;
+  __syncthreads();  // barriers initialised
+  if (warp == LD_WARPS) {
+    const int32_t* table = p.table + b * p.table_stride + page0;
+    bool ok = true;
+    for (int t = 0; t < tiles && ok; ++t) {
+      const int s = t % stages;
+      if (t >= stages) ok = mbar_wait_bounded(&empty[s], (t / stages - 1) & 1);
+      if (!ok) break;
+      if (lane == 0) {
+        const int n = min(2, pages - 2 * t);
+        mbar_expect_tx(&full[s], n * page_bytes);
+        for (int i = 0; i < n; ++i)
+          tma_load_3d(ring + s * tile_bytes + i * page_bytes, &map_rows, 0, table[2 * t + i] * PAGE, 0, &full[s]);
+      }
+      __syncwarp();
+    }
+    if (!ok && lane == 0) atomicExch(p.err, 1);
+    return;
+  }
+  // q' rows of the head block (rows past the last head are zero)
+  {
+    const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) +
+                                                    (static_cast<int64_t>(b) * p.heads + hb * 16) * pitch);
+    const int vecs = row_bytes / 16;
+    for (int i = tid; i < 16 * vecs; i += LD_WARPS * 32) {
+      const int r = i / vecs, c = i % vecs;
+      *reinterpret_cast<uint4*>(qs + r * q_pitch + c * 16) = r < heads_here ? q[r * vecs + c] : make_uint4(0, 0, 0, 0);
+    }
+  }
+  named_barrier(1, LD_WARPS * 32);
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  const float scale_log2 = p.scale * 1.4426950408889634f;
+  const int tg = warp & 3, kh = warp >> 2;
+  const int units = pitch / 32;
+  const int nt = p.rank / 64, col0 = warp * nt * 8;
+  const uint32_t a_base = smem_u32(qs) + (lane & 15) * q_pitch + (lane >> 4) * 16;
+  const int s_row = (tg & 1) * 8 + (lane & 7);
+  const uint32_t s_off = (tg >> 1) * page_bytes + s_row * 128;
+  bool ok = true;
+  for (int t = 0; t < tiles; ++t) {
+    const int s = t % stages;
+    uint8_t* tile = ring + s * tile_bytes;
+    const uint32_t tile_a = smem_u32(tile);
+    const int tok0 = (page0 + 2 * t) * PAGE;  // position of the tile's first row
+    if (ok) ok = __all_sync(0xffffffffu, mbar_wait_bounded(&full[s], (t / stages) & 1));  // uniform in the warp
+    const bool ragged = tok0 < lo || tok0 + LD_TOK > hi;
+    if (ragged) {
+      for (int r = warp; r < LD_TOK; r += LD_WARPS)
+        if (tok0 + r < lo || tok0 + r >= hi)
+          for (int c = lane; c < row_bytes / 16; c += 32)
+            *reinterpret_cast<uint4*>(tile + (r / PAGE) * page_bytes + (c >> 3) * (PAGE * 128) + (r % PAGE) * 128 + (c & 7) * 16) =
+                make_uint4(0, 0, 0, 0);
+      named_barrier(1, LD_WARPS * 32);
+    }
+    // ---- scores
+    if (ok) {
+      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 3
+      for (int u = kh; u < units; u += 2) {
+        uint32_t a0[4], a1[4], bm[4];
+        const int chunk = u * 4 + (lane >> 3);
+        ldmatrix_x4(bm, tile_a + s_off + (chunk >> 3) * (PAGE * 128) + (((chunk & 7) ^ (s_row & 7)) << 4));
+        ldmatrix_x4(a0, a_base + u * 64);
+        ldmatrix_x4(a1, a_base + u * 64 + 32);
+        mma_bf16_16816(c0, a0, bm[0], bm[1]);
+        mma_bf16_16816(c1, a1, bm[2], bm[3]);
+      }
+      const int col = tg * 8 + (lane & 3) * 2, r = lane >> 2;
+      *reinterpret_cast<float2*>(&ss[kh][r][col]) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+      *reinterpret_cast<float2*>(&ss[kh][r + 8][col]) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
+    }
+    named_barrier(1, LD_WARPS * 32);
+    // ---- softmax: rows 2 * warp, 2 * warp + 1; lane = token
+    const bool visible = tok0 + lane >= lo && tok0 + lane < hi;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int r = warp * 2 + i;
+      const float x = visible ? (ss[0][r][lane] + ss[1][r][lane]) * scale_log2 : -INFINITY;
+      const float m_new = fmaxf(m_run[i], warp_max(x));   // a tile holds at least one visible token
+      const float pr = ex2_fast(x - m_new);
+      const float a = ex2_fast(m_run[i] - m_new);
+      l_run[i] = l_run[i] * a + warp_sum(pr);
+      m_run[i] = m_new;
+      ps[r][lane] = __float2bfloat16_rn(pr);
+      if (lane == 0) alphas[r] = a;
+    }
+    named_barrier(1, LD_WARPS * 32);
+    // ---- O: this warp's columns
+    if (ok) {
+      const float al0 = alphas[lane >> 2], al1 = alphas[(lane >> 2) + 8];
+      if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+          acc[i][0] *= al0, acc[i][1] *= al0;
+          acc[i][2] *= al1, acc[i][3] *= al1;
+        }
+      }
+#pragma unroll
+      for (int ks = 0; ks < 2; ++ks) {
+        if (ks * PAGE >= hi - tok0) break;               // the second page of the last tile may be missing
+        uint32_t a[4];
+        ldmatrix_x4(a, smem_u32(&ps[lane & 15][ks * 16 + (lane >> 4) * 8]));
+        const uint32_t v_row = tile_a + ks * page_bytes + (lane & 15) * 128;
+#pragma unroll
+        for (int i = 0; i < NT; i += 2) {
+          if (i < nt) {
+            uint32_t bm[4];
+            const int chunk = col0 / 8 + i + (lane >> 4);
+            ldmatrix_x4_trans(bm, v_row + (chunk >> 3) * (PAGE * 128) + (((chunk & 7) ^ (lane & 7)) << 4));
+            mma_bf16_16816(acc[i], a, bm[0], bm[1]);
+            if (NT > 1 && i + 1 < nt) mma_bf16_16816(acc[i + 1 < NT ? i + 1 : i], a, bm[2], bm[3]);
+          }
+        }
+      }
+    }
+    if (ragged) fence_proxy_async();  // the zeroed rows before the next copy into this stage
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[s]);
+  }
+  if (!ok) {
+    if (lane == 0) atomicExch(p.err, 1);
+    return;
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = warp * 2 + i;
+    // maxima are kept in the log2 domain; latent_value works with natural exponentials
+    if (lane == 0 && r < heads_here)
+      p.ml[part0 + static_cast<int64_t>(r) * p.splits] = make_float2(m_run[i] * 0.6931471805599453f, l_run[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+    if (i < nt) {
+      const int r = lane >> 2, c = col0 + i * 8 + (lane & 3) * 2;
+      float* o = p.o + part0 * p.rank + c;
+      const int64_t step = static_cast<int64_t>(p.splits) * p.rank;
+      if (r < heads_here) *reinterpret_cast<float2*>(o + r * step) = make_float2(acc[i][0], acc[i][1]);
+      if (r + 8 < heads_here) *reinterpret_cast<float2*>(o + (r + 8) * step) = make_float2(acc[i][2], acc[i][3]);
+    }
+}
+
+// One encoded map per cache (base, rows, row width); a handful per engine.
+static bool row_map(CUtensorMap* out, const void* base, int64_t rows, int pitch) {
+  struct Entry {
+    const void* base;
+    int64_t rows;
+    int pitch;
+    CUtensorMap map;
+  };
+  static std::mutex lock;
+  static Entry entries[64];
+  static int used = 0, next = 0;
+  std::lock_guard<std::mutex> guard(lock);
+  for (int i = 0; i < used; ++i)
+    if (entries[i].base == base && entries[i].rows == rows && entries[i].pitch == pitch) {
+      *out = entries[i].map;
+      return true;
+    }
+  Entry e = {base, rows, pitch, {}};
+  if (!encode_tile_map(&e.map, base, static_cast<uint64_t>(rows), pitch, static_cast<uint64_t>(pitch) * 2, PAGE, pitch / 64)) return false;
+  const int at = used < 64 ? used++ : next++ % 64;
+  entries[at] = e;
+  *out = e.map;
+  return true;
+}
+
+template <int NT>
+static int launch_latent_decode(const LatentDecodeParams& p, const CUtensorMap& map, int batch, int stages, int smem,
+                                cudaStream_t st) {
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev >= 0 && dev < 64 && !configured[dev]) {
+    if (cudaFuncSetAttribute(latent_decode_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT) != cudaSuccess)
+      return fail(ERR_RUNTIME, "latent_decode: cannot raise dynamic shared memory to %d", LD_SMEM_LIMIT);
+    configured[dev] = true;
+  }
+  if (launch_pdl((p.overlap & OVERLAP_START) != 0, latent_decode_kernel<NT>, dim3(p.splits, (p.heads + 15) / 16, batch),
+                 dim3(LD_THREADS), smem, st, p, map, stages) != cudaSuccess)
+    return fail(ERR_LAUNCH, "latent_decode: %s", cudaGetErrorString(cudaGetLastError()));
+  return check_launch("latent_decode");
+}
+
+}  // namespace b200
+
+using namespace b200;
+
+extern "C" int b200_latent_decode(const void* q, const void* cache, int64_t num_pages, const int32_t* block_table,
+                                  int64_t table_stride, const int64_t* pos, const int64_t* active, float* ml, float* o,
+                                  int32_t batch, int32_t heads, int32_t rank, int32_t rot, int32_t window, int32_t splits,
+                                  float scale, int32_t overlap, b200_stream_t stream) {
+  if (batch <= 0) return OK;
+  B200_REQUIRE(rank > 0 && rank % 64 == 0 && rank <= 1024 && rot >= 0 && rot % 64 == 0 && heads > 0,
+               "latent_decode: rank and rot must be multiples of 64, rank at most 1024 (got %d, %d)", rank, rot);
+  B200_REQUIRE(window > 0 && splits > 0 && splits <= LATENT_MAX_SPLITS && batch <= 65535 && scale > 0.f && num_pages > 0,
+               "latent_decode: window, scale and splits (at most %d) must be positive", LATENT_MAX_SPLITS);
+  B200_REQUIRE(aligned16(q) && aligned16(cache) && aligned16(o), "latent_decode: unaligned tensor");
+  const int pitch = rank + rot, tile = LD_TOK * pitch * 2, q_bytes = 16 * (pitch * 2 + 16) + 1024;  // incl. alignment of the ring
+  int stages = (LD_SMEM_LIMIT - q_bytes) / tile;
+  if (stages > LD_MAX_STAGES) stages = LD_MAX_STAGES;
+  B200_REQUIRE(stages >= 2, "latent_decode: rows of %d elements do not fit", pitch);
+  LatentDecodeParams p = {q, cache, block_table, table_stride, pos, active, reinterpret_cast<float2*>(ml), o,
+                          heads, rank, rot, window, splits, overlap, scale, wait_timeout_flag()};
+  if (!p.err) return fail(ERR_RUNTIME, "latent_decode: no error flag");
+  CUtensorMap map;
+  if (!row_map(&map, cache, num_pages * PAGE, pitch)) return fail(ERR_RUNTIME, "latent_decode: cannot encode the cache's tensor map");
+  const int smem = stages * tile + q_bytes;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (rank <= 128) return launch_latent_decode<2>(p, map, batch, stages, smem, st);
+  if (rank <= 512) return launch_latent_decode<8>(p, map, batch, stages, smem, st);
+  return launch_latent_decode<16>(p, map, batch, stages, smem, st);
+}
