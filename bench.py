@@ -357,6 +357,16 @@ def hbm_peak():
     return FALLBACK_HBM_GBS, "fallback"
 
 
+def tensor_peak():
+    p = ROOT / "MEASURED_PEAKS.json"
+    if p.exists():
+        try:
+            return float(json.loads(p.read_text())["bf16_tflops"]), "measured"
+        except Exception:
+            pass
+    return 1590.0, "fallback"
+
+
 # --------------------------------------------------------------------------- main
 def aggregate_over_ranks(ms_local: float, units_local: float, dist, device):
     """Whole-job figures of a replicated run: (slowest rank's time, units summed over ranks).  `dist` is
@@ -475,6 +485,10 @@ def main():
     ap.add_argument("--no-graph", action="store_true", help="launch every step from Python instead of one CUDA graph")
     ap.add_argument("--no-model", action="store_true", help="skip the whole-model decode measurement (24-layer random-init model)")
     ap.add_argument("--model-steps", type=int, default=512)
+    ap.add_argument("--hybrid", action="store_true",
+                    help="instead of the default workload: the kernels of the hybrid stacks (latent attention, HGRN2, minGRU, "
+                         "hyper-connections) and whole-model prefill / decode, beside the Qwen3.5 engine at equal size")
+    ap.add_argument("--hybrid-part", default="all", choices=["all", "kernels", "models"])
     ap.add_argument("--workload", default="decode", choices=["decode", "chain", "prefill", "gdn", "gdn_decode", "gemm", "model_prefill"],
                     help="with --kernel-only: which kernel family to run (profiler captures of the other families)")
     args = ap.parse_args()
@@ -500,6 +514,14 @@ def main():
         dist.init_process_group("nccl", device_id=device)
 
     from b200attn import ops
+
+    if args.hybrid:
+        with ClockSampler(local_rank) as clocks:
+            rows = run_hybrid_kernel_rows(ops, device, args.sweep_steps) if args.hybrid_part != "models" else []
+            models = run_hybrid_models(device, args.sweep_steps) if args.hybrid_part != "kernels" else []
+        emit({"workload": "hybrid", "data": "synthetic", "dtype": "bf16", "hbm_peak_gbs": hbm_peak(), "tensor_peak_tflops": tensor_peak(),
+              "clocks": clocks.summary(), "kernels": rows, "models": models})
+        return
 
     if args.kernel_only and args.workload != "decode":
         if args.workload == "gemm":
@@ -1024,6 +1046,233 @@ def run_prefill_sweep(ops, device, steps, only=None):
         ms = time_steps(lambda i: ops.call_gdn_recurrent_prefill_chunked_triton(sq, sk, sv, sb, sg), steps, 3)
         rows.append({"op": "gdn chunk-64 prefill, one sequence (drop-in entry point)", "shape": f"1 x {n_tok}",
                      "tokens": n_tok, "us": ms * 1e3})
+    return rows
+
+
+# --------------------------------------------------------------------------- hybrid stacks
+HYBRID_WINDOW = 4096
+
+
+def hybrid_config(width: int, layers: int, heads: int, vocab: int) -> dict:
+    """A stack of a real model's layer sizes: three recurrent layers (HGRN2, minGRU, HGRN2) and one latent-attention layer in
+    turn, as the Qwen3.5 stack has three Gated-DeltaNet layers and one attention layer; same width, feed-forward and
+    recurrent state per layer."""
+    latent = {"type": "latent_attention",
+              "mixer": {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 3 * width // 4,
+                        "mask": {"size": HYBRID_WINDOW}, "scale": 192 ** -0.5,
+                        "rot": {"base": 1e6, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    hgrn2 = {"type": "hgrn2", "mixer": {"heads": heads, "dim": 128, "vdim": 128}}
+    mingru = {"type": "mingru", "mixer": {"width": 2 * width}}
+    order = [hgrn2, mingru, hgrn2, latent]
+    return {"architecture": "Tofilorn", "vocab": vocab, "width": width, "streams": 2, "norm": {"eps": 1e-6},
+            "layers": [{**order[i % 4], "mlp": {"kind": "dense", "ff": 7 * width // 2}} for i in range(layers)]}
+
+
+def run_hybrid_models(device, steps):
+    """Whole models of random weights: the hybrid stack and the Qwen3.5 stack of the same width, depth, feed-forward and
+    vocabulary.  Decode is one CUDA-graph replay per step after a prefill of the stated prompts; prefill is timed from the
+    first host instruction to the last kernel (median of five)."""
+    from b200attn import models
+    vocab, rows = 65536, []
+    for width, layers, heads in ((1024, 24, 16), (2048, 12, 32)):
+        stacks = {"Tofilorn": hybrid_config(width, layers, heads, vocab),
+                  "Qwen3.5": {"architecture": "Qwen3.5", "hidden": width, "num_layers": layers, "num_q_heads": heads // 2,
+                              "num_kv_heads": heads // 8, "gdn_heads": heads, "intermediate": 7 * width // 2, "vocab": vocab}}
+        for name, config in stacks.items():
+            model = models.random_model(config, seed=4, device=device)
+            for batch, prompt in ((1, 2048), (32, 128), (32, 2048), (8, 4096)):
+                gen = torch.Generator().manual_seed(4)
+                prompts = [torch.randint(0, vocab, (prompt,), generator=gen).tolist() for _ in range(batch)]
+                eng = model.engine(batch, prompt + 2 * steps + 16, device)
+                times = []
+                start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                for i in range(7):
+                    eng.pos.zero_()
+                    torch.cuda.synchronize()
+                    start.record()
+                    eng.prefill(prompts)
+                    end.record()
+                    torch.cuda.synchronize()
+                    times.append(start.elapsed_time(end))
+                prefill_ms = sorted(times[2:])[2]
+                for _ in range(3):
+                    eng.step()
+                eng.capture()
+                for _ in range(3):
+                    eng.step()
+                torch.cuda.synchronize()
+                start.record()
+                for _ in range(steps):
+                    eng.step()
+                end.record()
+                torch.cuda.synchronize()
+                ms = start.elapsed_time(end) / steps
+                rows.append({"model": name, "width": width, "layers": layers, "batch": batch, "prompt": prompt,
+                             "prefill_ms": prefill_ms, "prefill_tok_s": batch * prompt / prefill_ms * 1e3, "decode_ms": ms,
+                             "decode_tok_s": batch / ms * 1e3})
+                print(rows[-1], file=sys.stderr, flush=True)
+                del eng
+                torch.cuda.empty_cache()
+            del model
+            torch.cuda.empty_cache()
+    return rows
+
+
+class _Rows:
+    """What the packed-prefill operators read of a batch of equal whole prompts."""
+
+    def __init__(self, batch, length, device):
+        self.count, self.max_len = batch, length
+        i32 = dict(dtype=torch.int32, device=device)
+        self.cu = torch.arange(batch + 1, **i32) * length
+        self.slots, self.start = torch.arange(batch, **i32), torch.zeros(batch, **i32)
+        self.pos = torch.arange(length, **i32).repeat(batch)
+        self.slot_of = self.slots.repeat_interleave(length)
+
+
+def run_hybrid_kernel_rows(ops, device, steps):
+    """Every kernel of the hybrid stacks at a real layer's sizes beside the like kernel of the Qwen3.5 stack: algorithmic bytes
+    (or FLOPs) over device time.  Inputs rotate over enough copies that no call finds its own in L2."""
+    from b200attn import hybrid_ops as hops
+    from b200attn.mixers import Rotation
+    hbm, tensor = hbm_peak()[0], tensor_peak()[0]
+    bf, f32 = torch.bfloat16, torch.float32
+    rows = []
+
+    def rnd(*shape, dtype=bf):
+        return torch.randn(*shape, dtype=f32, device=device).mul_(0.5).to(dtype)
+
+    def row(op, like, shape, fn, sets, nbytes=None, flops=None):
+        ms = time_steps(fn, max(steps, sets), 3)
+        r = {"op": op, "like": like, "shape": shape, "us": ms * 1e3}
+        if nbytes is not None:
+            r["gbs"], r["frac_hbm"] = nbytes / ms / 1e6, nbytes / ms / 1e6 / hbm
+        if flops is not None:
+            r["tflops"], r["frac_tensor"] = flops / ms / 1e9, flops / ms / 1e9 / tensor
+        rows.append(r)
+        print(r, file=sys.stderr, flush=True)
+        torch.cuda.empty_cache()
+
+    def copies(nbytes):
+        return max(1, min(48, cdiv(3 * L2_BYTES, nbytes)))
+
+    # ---- decode attention
+    for batch, heads, ctx in ((1, 16, 4096), (32, 16, 4096), (32, 32, 4096), (256, 16, 2048), (32, 16, 640)):
+        rank, rot = 512, 64
+        pages = ctx // 16
+        nbytes = batch * (ctx * (rank + rot) * 2 + heads * (rank + rot) * 2 + heads * rank * 2)
+        n = copies(nbytes)
+        caches = [rnd(batch * pages, 16, rank + rot) for _ in range(n)]
+        tables = [torch.randperm(batch * pages, device=device).view(batch, pages).to(torch.int32) for _ in range(n)]
+        q = rnd(batch, heads, rank + rot)
+        pos = torch.full((batch,), ctx - 1, dtype=torch.int64, device=device)
+        splits = hops.latent_decode_splits(batch, heads, min(ctx, HYBRID_WINDOW), torch.cuda.get_device_properties(device).multi_processor_count)
+        ws = hops.latent_decode_workspace(batch, heads, rank, splits, device)
+        row("latent_decode", "fused_decode_attention", f"B={batch} H={heads} ctx={ctx} splits={splits}",
+            lambda i: hops.latent_decode(q, caches[i % n], tables[i % n], pos, None, ws, HYBRID_WINDOW, 0.07), n, nbytes)
+        uks = [rnd(heads, 128, rank) for _ in range(48)]
+        angles = Rotation(64, 1e6).table(ctx, device)
+        qn = rnd(batch, heads, 192)
+        row("latent_absorb", "skinny_gemm", f"B={batch} H={heads}", lambda i: hops.latent_absorb(qn, uks[i % 48], pos, angles), 48,
+            heads * 128 * rank * 2 + batch * heads * (192 + 576) * 2)
+        row("latent_value", "skinny_gemm", f"B={batch} H={heads} splits={splits}",
+            lambda i: hops.latent_value(ws, uks[i % 48], bf), 48, heads * 128 * rank * 2 + batch * heads * (rank * 4 * splits + 256))
+        del caches, uks
+    for batch in (1, 32, 256):
+        w = Workload([2048] * batch, device, max_sets=32)
+        fd = fused_step(ops, w, ops.fused_decode_workspace(device))
+        row("fused_decode_attention", None, f"B={batch} ctx=2048", fd, w.sets, w.bytes)
+        del w, fd
+    # ---- prefill attention
+    for batch, length, heads in ((8, 4096, 16), (32, 128, 16), (1, 2048, 16)):
+        rank, rot, dim, vdim = 512, 64, 128, 128
+        total = batch * length
+        b = _Rows(batch, length, device)
+        q, kv, ctx = rnd(total, heads, dim + rot), rnd(total, heads * (dim + vdim)), rnd(total, rank + rot)
+        for window in (HYBRID_WINDOW, 1024):
+            pairs = sum(min(i + 1, window) for i in range(length)) * batch
+            row("latent_prefill", "gqa_attention_varlen_causal", f"{batch}x{length} H={heads} window={window}",
+                lambda i: hops.latent_prefill(q, kv, ctx, b.cu, b.cu, b.start, b.start, length, dim, rot, vdim, rank, window, 0.07), 1,
+                total * heads * (192 + 256 + 128) * 2 + total * 128, 2 * pairs * heads * (192 + 128))
+        cu, max_len = ops.build_cu_seqlens([length] * batch, device=device)
+        qq, kk, vv = rnd(total, HQ, D), rnd(total, HKV, D), rnd(total, HKV, D)
+        row("gqa_attention_varlen_causal", None, f"{batch}x{length}", lambda i: ops.gqa_attention_varlen_causal(qq, kk, vv, cu, max_len), 1,
+            total * (2 * HQ + 2 * HKV) * D * 2, 4 * HQ * D * batch * length * (length + 1) // 2)
+        angles = Rotation(64, 1e6).table(length, device)
+        row("rope_interleaved", "add_rmsnorm", f"{batch}x{length} H={heads}", lambda i: hops.rope_interleaved(q, dim, b.pos, angles), 1,
+            total * heads * 64 * 2 * 2)
+        fused = rnd(total, 768 + rank + rot)
+        table = torch.arange(batch * cdiv(length, 16), dtype=torch.int32, device=device).view(batch, -1)
+        cache = hops.allocate_latent_cache(table.numel(), rank + rot, bf, device=device)
+        ones = torch.ones(768, device=device)
+        row("latent_prep", "add_rmsnorm", f"{batch}x{length}",
+            lambda i: hops.latent_prep(fused, ones, ones[:rank], b.pos, b.slot_of, None, table, angles, cache, 768, rank, rank, 1e-6), 1,
+            total * (768 + rank + rot) * 2 * 2)
+        row("latent_gather", "add_rmsnorm", f"{batch}x{length}",
+            lambda i: hops.latent_gather(cache, table, b.slots, b.cu, b.start, total, length), 1, total * (rank + rot) * 2 * 2)
+        del q, kv, ctx, qq, kk, vv, fused, cache
+    # ---- recurrences, prefill
+    for batch, length in ((32, 128), (1, 2048), (32, 1024)):
+        total, heads = batch * length, 16
+        b = _Rows(batch, length, device)
+        state = torch.zeros(batch, heads, 128, 128, device=device)
+        nbytes = total * heads * 128 * 2 * 4 + state.numel() * 4
+        n = copies(nbytes)
+        qfv = [rnd(total, 3 * heads * 128) for _ in range(n)]
+        lower, bias, norm = torch.full((heads * 128,), 0.5, device=device), torch.zeros(heads * 128, device=device), torch.ones(128, device=device)
+        row("hgrn2_prefill", "gdn_chunked_prefill", f"{batch}x{length}",
+            lambda i: hops.hgrn2_prefill(qfv[i % n], lower, bias, norm, state, b, 128, 1e-6), n, nbytes)
+        gq = torch.nn.functional.normalize(torch.randn(total, heads, 128, device=device), dim=-1).to(bf)
+        beta, g = torch.rand(total, heads, device=device), -torch.rand(total, heads, device=device)
+        cu, _ = ops.build_cu_seqlens([length] * batch, device=device)
+        row("gdn_chunked_prefill", None, f"{batch}x{length}", lambda i: ops.gdn_chunked_prefill_packed(gq, gq, gq, beta, g, cu), 1,
+            total * heads * (4 * 128 * 2 + 8) + batch * heads * 128 * 128 * 4)
+        del qfv, gq
+        for width in (2048, 4096):
+            nb = total * width * 4 * 2
+            n = copies(nb)
+            zxg = [rnd(total, 3 * width) for _ in range(n)]
+            bias2, st = torch.zeros(2 * width, device=device), torch.zeros(batch, width, device=device)
+            row("mingru_prefill", "depthwise_causal_conv4_prefill", f"{batch}x{length} width={width}",
+                lambda i: hops.mingru_prefill(zxg[i % n], bias2, st, b), n, nb)
+            del zxg
+        from b200attn import glue_ops
+        conv = getattr(glue_ops.depthwise_causal_conv4_prefill, "_init_fn", glue_ops.depthwise_causal_conv4_prefill)
+        nb = total * 6144 * 2 * 2
+        n = copies(nb)
+        x, w4 = [rnd(total, 6144) for _ in range(n)], rnd(6144, 4)
+        seq_start = (b.slot_of * length).to(torch.int32)
+        row("depthwise_causal_conv4_prefill", None, f"{batch}x{length} channels=6144", lambda i: conv(x[i % n], w4, seq_start), n, nb)
+        del x
+    # ---- recurrences, decode
+    for batch in (1, 32, 256):
+        heads = 16
+        nbytes = batch * heads * (2 * 128 * 128 * 4 + 4 * 128 * 2)
+        n = copies(nbytes)
+        states = [torch.zeros(batch, heads, 128, 128, device=device) for _ in range(n)]
+        qfv, pos = rnd(batch, 3 * heads * 128), torch.ones(batch, dtype=torch.int64, device=device)
+        row("hgrn2_decode", "gdn_decode_fused", f"B={batch}",
+            lambda i: hops.hgrn2_decode(qfv, lower, bias, norm, states[i % n], pos, None, 128, 1e-6), n, nbytes)
+        del states
+        zxg, st = rnd(batch, 3 * 4096), torch.zeros(batch, 4096, device=device)
+        bias2 = torch.zeros(8192, device=device)
+        row("mingru_decode", "add_rmsnorm", f"B={batch} width=4096", lambda i: hops.mingru_decode(zxg, bias2, st, pos, None), 1,
+            batch * 4096 * (3 * 2 + 2 + 8))
+    rows += [{**r, "like": None} for r in run_gdn_decode_rows(ops, device, hbm, steps, (1, 32, 256))]
+    # ---- streams
+    for tokens, width in ((32, 1024), (32, 2048), (4096, 1024), (4096, 2048), (32768, 1024)):
+        nbytes = tokens * width * (2 * 2 * 4 + 2 + 2)
+        n = copies(nbytes)
+        xs, y = [rnd(tokens, 2, width, dtype=f32) for _ in range(n)], rnd(tokens, width)
+        joint = torch.tensor([0.9, 0.1, 0.1, 0.9, 0.5, 0.5, 0.5, 0.5, 1.0], device=device)
+        row("hyper_connect", "add_rmsnorm", f"{tokens} rows, width {width}, 2 streams",
+            lambda i: hops.hyper_connect(xs[i % n], joint, width, 1e-6, bf, y=y), n, nbytes)
+        nb = tokens * width * 8
+        n2 = copies(nb)
+        rs = [rnd(tokens, width) for _ in range(n2)]
+        wn = torch.zeros(width, dtype=bf, device=device)
+        row("add_rmsnorm", None, f"{tokens} rows, width {width}", lambda i: ops.add_rmsnorm(y, wn, 1e-6, residual=rs[i % n2]), n2, nb)
+        del xs, rs
     return rows
 
 

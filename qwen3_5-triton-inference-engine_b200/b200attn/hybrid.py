@@ -96,7 +96,7 @@ class HybridWeights:
         after = [[wide(f"l{i}.hc{q}.mix").flatten(), wide(f"l{i}.hc{q}.out")] for i, q in steps]
         before = [[wide(f"l{i}.hc{q}.in"), wide(f"l{i}.norm{q}").view(1)] for i, q in steps]
         before.append([torch.ones(s), wide("final.norm").view(1)])
-        self.joints = [torch.cat(a + b).to(device).contiguous() for a, b in zip([none] + after, before)]
+        self.joints = [torch.cat([t.cpu() for t in a + b]).to(device) for a, b in zip([none] + after, before)]
         return self
 
 
