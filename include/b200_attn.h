@@ -469,11 +469,12 @@ int b200_mingru_decode(const void* zxg, int64_t stride, const float* bias, float
 
 /* HGRN2: qfv = rows of [q heads*dim | f heads*dim | v heads*vdim]; lower, bias fp32 [heads*dim]; norm fp32 [vdim];
  * state fp32 [slots, heads, dim, vdim];  f = l + (1-l) sigmoid(f + bias), S <- diag(f) S + (1-f) v^T, o = S^T silu(q),
- * out = o / sqrt(mean(o^2) + eps) * norm per head.  o_scratch: fp32 [tokens, heads*vdim]. */
+ * out = o / sqrt(mean(o^2) + eps) * norm per head.  o_scratch: fp32 [tokens, heads*vdim].  serial: keep bf16 prefill on the
+ * token-serial kernel (default: 16-token chunks on the tensor cores for dim <= 128). */
 int b200_hgrn2_prefill(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
                        const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start, float* o_scratch, void* out,
                        int32_t batch, int32_t tokens, int32_t heads, int32_t dim, int32_t vdim, int32_t true_vdim, float eps,
-                       int32_t f32, b200_stream_t stream);
+                       int32_t f32, int32_t serial, b200_stream_t stream);
 int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
                       const int64_t* pos, const int64_t* active, void* out, int32_t batch, int32_t heads, int32_t dim,
                       int32_t vdim, int32_t true_vdim, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);
@@ -490,7 +491,7 @@ int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* lower, const
  * b200_latent_absorb: q' = [W_uk^T q_unrotated | rotated part], w_uk [heads, dim, rank].
  * b200_latent_decode(_simple): q' against the paged rows, the visible range split in `splits` runs of pages: ml fp32
  *   [batch, heads, splits, 2] (maximum, sum), o fp32 [batch, heads, splits, rank] unnormalised.
- * b200_latent_value: merges the splits and applies w_uv [heads, vdim, rank]. */
+ * b200_latent_value: merges the splits (merged: E scratch [batch, heads, rank]) and applies w_uv [heads, vdim, rank]. */
 int b200_latent_prep(const void* fused, int64_t stride, const float* q_weight, const float* kv_weight, const void* pos,
                      int32_t pos_is_int64, const int32_t* slot, const int64_t* active, const int32_t* block_table,
                      int64_t table_stride, const float* angles, void* cache, void* cq, int32_t rows, int32_t q_rank,
@@ -520,8 +521,8 @@ int b200_latent_decode(const void* q, const void* cache, int64_t num_pages, cons
                        const int64_t* pos, const int64_t* active, float* ml, float* o, int32_t batch, int32_t heads,
                        int32_t rank, int32_t rot, int32_t window, int32_t splits, float scale, int32_t overlap,
                        b200_stream_t stream);
-int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* out, int32_t batch, int32_t heads, int32_t rank,
-                      int32_t vdim, int32_t splits, int32_t f32, int32_t overlap, b200_stream_t stream);
+int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* merged, void* out, int32_t batch,
+                      int32_t heads, int32_t rank, int32_t vdim, int32_t splits, int32_t f32, int32_t overlap, b200_stream_t stream);
 
 #ifdef __cplusplus
 }

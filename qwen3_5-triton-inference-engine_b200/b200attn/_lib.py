@@ -67,7 +67,7 @@ SIGNATURES: dict[str, list] = {
     "b200_swiglu_f32": [P, I64, P, I32, I32, P],
     "b200_mingru_prefill": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, P],
     "b200_mingru_decode": [P, I64, P, P, P, P, P, I32, I32, I32, I32, P],
-    "b200_hgrn2_prefill": [P, I64, P, P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, P],
+    "b200_hgrn2_prefill": [P, I64, P, P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_hgrn2_decode": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_latent_prep": [P, I64, P, P, P, I32, P, P, P, I64, P, P, P, I32, I32, I32, I32, I32, I32, I32, c_float, I32, I32,
                          P],
@@ -78,7 +78,7 @@ SIGNATURES: dict[str, list] = {
     "b200_latent_decode": [P, P, I64, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, P],
     "b200_latent_absorb": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, P],
     "b200_latent_decode_simple": [P, P, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, P],
-    "b200_latent_value": [P, P, P, P, I32, I32, I32, I32, I32, I32, I32, P],
+    "b200_latent_value": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, P],
 }
 OTHER = {
     "b200_mingru_workspace_bytes": ([I32, I32, I32], c_int64),

@@ -44,8 +44,11 @@ def swiglu_f32(gate_up, intermediate: int):
 
 
 # ------------------------------------------------------------------------------------------------------------- minGRU
-def mingru_chunking(max_len: int) -> tuple[int, int]:
-    """(chunk length, chunks of the longest sequence): at least 64 tokens a chunk, at most 64 chunks."""
+def mingru_chunking(max_len: int, count: int = 1, width: int = 1) -> tuple[int, int]:
+    """(chunk length, chunks of the longest sequence).  A batch wide enough to keep the memory system busy (a thread per
+    two channels) runs each sequence in one pass; otherwise chunks of at least 64 tokens, at most 64 of them."""
+    if count * width >= 65536:
+        return max_len, 1
     chunk = max(64, -(-max_len // 64))
     return chunk, -(-max_len // chunk)
 
@@ -56,7 +59,7 @@ def mingru_prefill(zxg, bias, state, batch):
     assert zxg.shape[1] == 3 * width and zxg.stride(1) == 1 and bias.numel() == 2 * width
     assert state.dtype == bias.dtype == torch.float32 and state.is_contiguous() and bias.is_contiguous()
     _require_cuda(zxg, bias, state)
-    chunk, chunks = mingru_chunking(batch.max_len)
+    chunk, chunks = mingru_chunking(batch.max_len, batch.count, width)
     n = batch.count
     ws = torch.empty(_lib.load().b200_mingru_workspace_bytes(n, chunks, width), dtype=torch.uint8, device=zxg.device)
     out = torch.empty((zxg.shape[0], width), dtype=zxg.dtype, device=zxg.device)
@@ -86,7 +89,7 @@ def _check_hgrn2(qfv, lower, bias, norm, state):
     return heads, dim, vdim
 
 
-def hgrn2_prefill(qfv, lower, bias, norm, state, batch, true_vdim: int, eps: float):
+def hgrn2_prefill(qfv, lower, bias, norm, state, batch, true_vdim: int, eps: float, serial: bool = False):
     """qfv [tokens, 2*heads*dim + heads*vdim]; state [slots, heads, dim, vdim] fp32, in place."""
     heads, dim, vdim = _check_hgrn2(qfv, lower, bias, norm, state)
     tokens = qfv.shape[0]
@@ -94,7 +97,7 @@ def hgrn2_prefill(qfv, lower, bias, norm, state, batch, true_vdim: int, eps: flo
     out = torch.empty((tokens, heads * vdim), dtype=qfv.dtype, device=qfv.device)
     _lib.call("b200_hgrn2_prefill", _ptr(qfv), qfv.stride(0), _ptr(lower), _ptr(bias), _ptr(norm), _ptr(state), _ptr(batch.cu),
               _ptr(batch.slots), _ptr(batch.start), _ptr(scratch), _ptr(out), batch.count, tokens, heads, dim, vdim, true_vdim,
-              float(eps), _f32(qfv), _stream())
+              float(eps), _f32(qfv), int(serial), _stream())
     return out
 
 
@@ -194,10 +197,11 @@ LATENT_DECODE_MAX_ROW = 1344     # widest cache row two stages of the tensor-cor
 
 
 def latent_decode_splits(batch: int, heads: int, span: int, sm_count: int) -> int:
-    """Key ranges per slot: the count whose launch has the shortest longest SM, at ~64 tokens of fixed cost per CTA."""
+    """Key ranges per slot: the count whose launch ends first with two CTAs per SM, at ~100 tokens of fixed cost per CTA and
+    a merge that grows with the number of ranges."""
     groups = batch * -(-heads // 16)
     most = max(1, min(LATENT_MAX_SPLITS, span // (2 * PAGE_SIZE)))
-    return min(range(1, most + 1), key=lambda s: (-(-groups * s // sm_count) * (span / s + 64), s))
+    return min(range(1, most + 1), key=lambda s: (-(-groups * s // (2 * sm_count)) * (span / s + 100) + 4 * s, s))
 
 
 def latent_decode(q, cache, block_table, pos, active, workspace, window: int, scale: float, overlap: int = 0,
@@ -225,6 +229,7 @@ def latent_value(workspace, w_uv, dtype, overlap: int = 0):
     vdim = w_uv.shape[1]
     assert w_uv.shape == (heads, vdim, rank) and w_uv.is_contiguous() and w_uv.dtype == dtype
     out = torch.empty((batch, heads * vdim), dtype=dtype, device=o.device)
-    _lib.call("b200_latent_value", _ptr(ml), _ptr(o), _ptr(w_uv), _ptr(out), batch, heads, rank, vdim, splits, _f32(w_uv),
+    merged = torch.empty((batch, heads, rank), dtype=dtype, device=o.device)
+    _lib.call("b200_latent_value", _ptr(ml), _ptr(o), _ptr(w_uv), _ptr(merged), _ptr(out), batch, heads, rank, vdim, splits, _f32(w_uv),
               int(overlap), _stream())
     return out

@@ -19,6 +19,24 @@ __device__ __forceinline__ float load1(const __nv_bfloat16* p) { return __bfloat
 __device__ __forceinline__ void store1(float* p, float v) { *p = v; }
 __device__ __forceinline__ void store1(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
 
+// eight at a time (16 bytes of bf16, 32 of fp32)
+__device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
+  const float4 a = load4(p), b = load4(p + 4);
+  f[0] = a.x, f[1] = a.y, f[2] = a.z, f[3] = a.w, f[4] = b.x, f[5] = b.y, f[6] = b.z, f[7] = b.w;
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 v = *reinterpret_cast<const uint4*>(p);
+  f[0] = bf16_lo(v.x), f[1] = bf16_hi(v.x), f[2] = bf16_lo(v.y), f[3] = bf16_hi(v.y);
+  f[4] = bf16_lo(v.z), f[5] = bf16_hi(v.z), f[6] = bf16_lo(v.w), f[7] = bf16_hi(v.w);
+}
+__device__ __forceinline__ void store8(float* p, const float (&f)[8]) {
+  store4(p, make_float4(f[0], f[1], f[2], f[3]));
+  store4(p + 4, make_float4(f[4], f[5], f[6], f[7]));
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
+  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+}
+
 // Logistic function in fp32: exact library exponential and division for fp32 activations, the hardware exponential and
 // reciprocal (a few fp32 ulp) next to bf16 ones.
 template <typename E>

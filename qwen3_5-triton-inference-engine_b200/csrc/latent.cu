@@ -7,7 +7,7 @@
 //   b200_latent_prefill_simple   attention over expanded keys/values, any shape, bf16 or fp32 (CUDA cores)
 //   b200_latent_absorb     decode: q' = [W_uk^T q_unrotated | rotated part], so that scores need the cache rows only
 //   b200_latent_decode_simple    decode over the paged rows, split over key ranges, any shape (CUDA cores)
-//   b200_latent_value      decode: merges the splits and applies W_uv
+//   b200_latent_value      decode: merges the splits, then applies W_uv (two launches)
 // The tensor-core forms live in latent_decode.cu and latent_prefill_umma.cu.
 // Padded layout (the weight loader's): kv_rank, rot_dim, dim, vdim and q_rank are rounded up to multiples of 64 with
 // zero rows / columns, a cache row is [latent | rotated part] with both parts padded.  Norms divide by the true widths.
@@ -35,68 +35,87 @@ struct LatentPrepParams {
   float eps;
 };
 
-template <typename E>
-__global__ void __launch_bounds__(128) latent_prep_kernel(const __grid_constant__ LatentPrepParams p) {
+// One CTA per row; a thread holds up to V groups of 8 elements of the row [query latent | kv latent | rotated part] in
+// registers: one pass over memory, one block reduction for both norms.
+template <typename E, int V>
+__global__ void __launch_bounds__(256) latent_prep_kernel(const __grid_constant__ LatentPrepParams p) {
   __shared__ float red[64];
   const int row = blockIdx.x, tid = threadIdx.x;
   if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
   pdl_wait();
   const E* x = static_cast<const E*>(p.fused) + row * p.stride;
-  const E* kv = x + p.q_rank;
-  float sq[2] = {0.f, 0.f};
-  for (int c = tid * 4; c < p.q_rank; c += 512) {
-    const float4 v = load4(x + c);
-    sq[0] += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-  }
   const bool own = p.cache != nullptr;
-  if (own)
-    for (int c = tid * 4; c < p.rank; c += 512) {
-      const float4 v = load4(kv + c);
-      sq[1] += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  const int nq = p.q_rank / 8, nk = nq + p.rank / 8, total = own ? nk + p.rot / 8 : nq;
+  float f[V][8], sq[2] = {0.f, 0.f};
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int i = tid + v * blockDim.x;
+    if (i < total) load8(x + i * 8, f[v]);
+    if (i < nk && i < total) {
+      float part = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) part = fmaf(f[v][j], f[v][j], part);
+      sq[i < nq ? 0 : 1] += part;
     }
+  }
+  const int slot = own && p.slot ? p.slot[row] : row;
+  const bool write = own && !(p.active && p.active[slot] == 0);
+  int64_t pos = 0;
+  E* out = nullptr;
+  if (write) {
+    pos = p.pos_is_int64 ? static_cast<const int64_t*>(p.pos)[row] : static_cast<int64_t>(static_cast<const int32_t*>(p.pos)[row]);
+    const int64_t page = p.table[slot * p.table_stride + pos / PAGE];
+    out = static_cast<E*>(p.cache) + (page * PAGE + pos % PAGE) * (p.rank + p.rot);
+  }
   block_sum<2>(sq, red);
   const float qs = 1.0f / sqrtf(sq[0] / static_cast<float>(p.true_q_rank) + p.eps);
-  E* cq = static_cast<E*>(p.cq) + static_cast<int64_t>(row) * p.q_rank;
-  for (int c = tid * 4; c < p.q_rank; c += 512) {
-    const float4 v = load4(x + c), w = load4(p.q_weight + c);
-    store4(cq + c, make_float4(v.x * qs * w.x, v.y * qs * w.y, v.z * qs * w.z, v.w * qs * w.w));
-  }
-  if (!own) return;
-  const int slot = p.slot ? p.slot[row] : row;
-  if (p.active && p.active[slot] == 0) return;
-  const int64_t pos = p.pos_is_int64 ? static_cast<const int64_t*>(p.pos)[row]
-                                     : static_cast<int64_t>(static_cast<const int32_t*>(p.pos)[row]);
-  const int64_t page = p.table[slot * p.table_stride + pos / PAGE];
-  E* out = static_cast<E*>(p.cache) + (page * PAGE + pos % PAGE) * (p.rank + p.rot);
   const float ks = 1.0f / sqrtf(sq[1] / static_cast<float>(p.true_rank) + p.eps);
-  for (int c = tid * 4; c < p.rank; c += 512) {
-    const float4 v = load4(kv + c), w = load4(p.kv_weight + c);
-    store4(out + c, make_float4(v.x * ks * w.x, v.y * ks * w.y, v.z * ks * w.z, v.w * ks * w.w));
-  }
-  const E* kr = kv + p.rank;
-  for (int i = tid; i < p.rot / 2; i += 128) {
-    float u = load1(kr + 2 * i), v = load1(kr + 2 * i + 1);
-    if (i < p.rot_pairs) rotate_pair(u, v, p.angles[pos * p.rot_pairs + i]);
-    store1(out + p.rank + 2 * i, u);
-    store1(out + p.rank + 2 * i + 1, v);
+  E* cq = static_cast<E*>(p.cq) + static_cast<int64_t>(row) * p.q_rank;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int i = tid + v * blockDim.x;
+    if (i < nq) {
+      float w[8];
+      load8(p.q_weight + i * 8, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[v][j] *= qs * w[j];
+      store8(cq + i * 8, f[v]);
+    } else if (i < total && write) {
+      if (i < nk) {
+        float w[8];
+        load8(p.kv_weight + (i - nq) * 8, w);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[v][j] *= ks * w[j];
+      } else {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int pair = (i - nk) * 4 + j;
+          if (pair < p.rot_pairs) rotate_pair(f[v][2 * j], f[v][2 * j + 1], p.angles[pos * p.rot_pairs + pair]);
+        }
+      }
+      store8(out + (i - nq) * 8, f[v]);
+    }
   }
 }
 
 // ---------------------------------------------------------------------------------------------------------- rotation
-// x [rows, heads, head_stride]: the pairs from offset `off` on
+// x [rows, heads, head_stride]: the pairs from offset `off` on, four per thread; the parts are padded to multiples of 8
 template <typename E>
 __global__ void __launch_bounds__(256) rope_interleaved_kernel(E* x, int64_t row_stride, int head_stride, int off, int heads,
-                                                               int pairs, const int32_t* pos, const float2* angles) {
-  const int row = blockIdx.x;
-  const float2* a = angles + static_cast<int64_t>(pos[row]) * pairs;
-  for (int i = threadIdx.x; i < heads * pairs; i += 256) {
-    const int h = i / pairs, j = i % pairs;
-    E* q = x + row * row_stride + static_cast<int64_t>(h) * head_stride + off + 2 * j;
-    float u = load1(q), v = load1(q + 1);
-    rotate_pair(u, v, a[j]);
-    store1(q, u);
-    store1(q + 1, v);
-  }
+                                                               int pairs, const int32_t* pos, const float2* angles, int rows) {
+  const int quads = (pairs + 3) / 4, per_row = heads * quads;
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  const int64_t row = i / per_row;
+  if (row >= rows) return;
+  const int r = static_cast<int>(i - row * per_row), h = r / quads, j = (r - h * quads) * 4;
+  E* q = x + row * row_stride + static_cast<int64_t>(h) * head_stride + off + 2 * j;
+  const float2* a = angles + static_cast<int64_t>(pos[row]) * pairs + j;
+  float f[8];
+  load8(q, f);
+#pragma unroll
+  for (int k = 0; k < 4; ++k)
+    if (j + k < pairs) rotate_pair(f[2 * k], f[2 * k + 1], a[k]);
+  store8(q, f);
 }
 
 // ------------------------------------------------------------------------------------------------------------ gather
@@ -257,147 +276,161 @@ __global__ void __launch_bounds__(128) latent_absorb_f32_kernel(const __grid_con
   if (blockIdx.y == 0) absorb_rotated_part<float>(p, h, b0);
 }
 
-// bf16: one m16 tile of slots, W tile [64 k][64 n] at a time in shared memory, a warp per 16 columns
-constexpr int LA_PITCH = 144;  // bytes of a 64-element row plus 16: ldmatrix rows fall into different banks
-__global__ void __launch_bounds__(128) latent_absorb_bf16_kernel(const __grid_constant__ LatentAbsorbParams p) {
-  __shared__ __align__(16) uint8_t ws[2][64 * LA_PITCH];
-  __shared__ __align__(16) uint8_t qs[2][16 * LA_PITCH];
-  const int h = blockIdx.x, n0 = blockIdx.y * 64, b0 = blockIdx.z * 16;
+// bf16 products of up to 16 slots with a head's own matrix: out[b, h, n] = sum_k x[b, h, k] W_h[k, n], a CTA per
+// (head, 64 columns, 16 slots), a warp per 16 columns.  The whole [K x 64] slice of W is requested at once (cp.async,
+// before the predecessor has finished), the slots' rows after it: one memory round trip.
+// K_ROWS: W_h is stored [K, N] (absorb), else [N, K] (value).
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+constexpr int HG_PITCH = 144;                              // bytes of a 64-element row plus 16
+constexpr int HG_STEP = (64 + 16) * HG_PITCH;              // bytes of one 64-wide step of K: W tile, then the slots' tile
+
+template <bool K_ROWS>
+__device__ __forceinline__ void head_gemm(const __nv_bfloat16* w, int ldw, const __nv_bfloat16* x, int64_t x_stride, int slots,
+                                          int steps, int n0, bool trigger, uint8_t* smem, float (&acc)[2][4]) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int width = p.dim + p.rot, pitch = p.rank + p.rot, steps = p.dim / 64;
-  const uint8_t* w = reinterpret_cast<const uint8_t*>(static_cast<const __nv_bfloat16*>(p.w) +
-                                                      static_cast<int64_t>(h) * p.dim * p.rank + n0);
-  uint4 wr[4];
-  auto fetch_w = [&](int s) {
+  for (int s = 0; s < steps; ++s)
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int r = (tid + i * 128) >> 3, c = tid & 7;
-      wr[i] = *reinterpret_cast<const uint4*>(w + (static_cast<int64_t>(s * 64 + r) * p.rank + c * 8) * 2);
+      const __nv_bfloat16* src = K_ROWS ? w + static_cast<int64_t>(s * 64 + r) * ldw + n0 + c * 8
+                                        : w + static_cast<int64_t>(n0 + r) * ldw + s * 64 + c * 8;
+      cp_async16(smem + s * HG_STEP + r * HG_PITCH + c * 16, src);
     }
-  };
-  fetch_w(0);  // a weight: may be read before the predecessor has finished
-  if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
+  if (trigger) pdl_trigger();
   pdl_wait();
-  float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
   for (int s = 0; s < steps; ++s) {
-    uint8_t *wb = ws[s & 1], *qb = qs[s & 1];
-    {
-      const int r = tid >> 3, c = tid & 7, b = b0 + r;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (b < p.batch)
-        v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) +
-                                            (static_cast<int64_t>(b) * p.heads + h) * width + s * 64 + c * 8);
-      *reinterpret_cast<uint4*>(qb + r * LA_PITCH + c * 16) = v;
-    }
-#pragma unroll
-    for (int i = 0; i < 4; ++i) *reinterpret_cast<uint4*>(wb + ((tid + i * 128) >> 3) * LA_PITCH + (tid & 7) * 16) = wr[i];
-    __syncthreads();  // two buffers: a warp may still read the other one
-    if (s + 1 < steps) fetch_w(s + 1);
+    const int r = tid >> 3, c = tid & 7;
+    uint8_t* dst = smem + s * HG_STEP + (64 + r) * HG_PITCH + c * 16;
+    if (r < slots) cp_async16(dst, x + r * x_stride + s * 64 + c * 8);
+    else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+  for (int s = 0; s < steps; ++s) {
+    const uint32_t wb = smem_u32(smem + s * HG_STEP), xb = wb + 64 * HG_PITCH;
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t a[4], bm[4];
-      ldmatrix_x4(a, smem_u32(qb) + (lane & 15) * LA_PITCH + ks * 32 + (lane >> 4) * 16);
-      // k rows x n columns, transposed on the way in: matrices (k 0-7, n 0-7), (k 8-15, n 0-7), (k 0-7, n 8-15), ...
-      ldmatrix_x4_trans(bm, smem_u32(wb) + (ks * 16 + (lane & 15)) * LA_PITCH + warp * 32 + (lane >> 4) * 16);
+      ldmatrix_x4(a, xb + (lane & 15) * HG_PITCH + ks * 32 + (lane >> 4) * 16);
+      // matrices (k 0-7, n 0-7), (k 8-15, n 0-7), (k 0-7, n 8-15), (k 8-15, n 8-15)
+      if (K_ROWS) ldmatrix_x4_trans(bm, wb + (ks * 16 + (lane & 15)) * HG_PITCH + warp * 32 + (lane >> 4) * 16);
+      else ldmatrix_x4(bm, wb + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * HG_PITCH + ks * 32 + ((lane >> 3) & 1) * 16);
       mma_bf16_16816(acc[0], a, bm[0], bm[1]);
       mma_bf16_16816(acc[1], a, bm[2], bm[3]);
     }
   }
-  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
+}
+__device__ __forceinline__ void head_gemm_store(const float (&acc)[2][4], __nv_bfloat16* out, int64_t stride, int slots) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 #pragma unroll
   for (int t = 0; t < 2; ++t)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int b = b0 + (lane >> 2) + half * 8;
-      if (b < p.batch)
-        *reinterpret_cast<uint32_t*>(out + (static_cast<int64_t>(b) * p.heads + h) * pitch + n0 + warp * 16 + t * 8 + (lane & 3) * 2) =
-            pack_bf16(acc[t][half * 2], acc[t][half * 2 + 1]);
+      const int r = (lane >> 2) + half * 8;
+      if (r < slots)
+        *reinterpret_cast<uint32_t*>(out + r * stride + warp * 16 + t * 8 + (lane & 3) * 2) = pack_bf16(acc[t][half * 2], acc[t][half * 2 + 1]);
     }
+}
+
+__global__ void __launch_bounds__(128) latent_absorb_bf16_kernel(const __grid_constant__ LatentAbsorbParams p) {
+  extern __shared__ __align__(16) uint8_t hg_smem[];
+  const int h = blockIdx.x, n0 = blockIdx.y * 64, b0 = blockIdx.z * 16, slots = min(16, p.batch - b0);
+  const int width = p.dim + p.rot, pitch = p.rank + p.rot;
+  float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+  head_gemm<true>(static_cast<const __nv_bfloat16*>(p.w) + static_cast<int64_t>(h) * p.dim * p.rank, p.rank,
+                  static_cast<const __nv_bfloat16*>(p.q) + (static_cast<int64_t>(b0) * p.heads + h) * width,
+                  static_cast<int64_t>(p.heads) * width, slots, p.dim / 64, n0, (p.overlap & OVERLAP_TRIGGER) != 0, hg_smem, acc);
+  head_gemm_store(acc, static_cast<__nv_bfloat16*>(p.out) + (static_cast<int64_t>(b0) * p.heads + h) * pitch + n0,
+                  static_cast<int64_t>(p.heads) * pitch, slots);
   if (blockIdx.y == 0) absorb_rotated_part<__nv_bfloat16>(p, h, b0);
 }
 
 // --------------------------------------------------------------------------------------- decode: merge splits, W_uv
-// grid (heads, vdim / 64, ceil(batch / 16)).  Merged latents of up to 16 slots go to shared memory (E), then W_uv.
+// merged[b, h, :] = sum_s w_s o_s with w_s = exp(m_s - m) / sum exp(m_s - m) l_s; an idle slot gives zeros.
+// grid (heads, batch)
 template <typename E>
-__global__ void __launch_bounds__(128) latent_value_kernel(const __grid_constant__ LatentValueParams p) {
-  extern __shared__ __align__(16) uint8_t lv_smem[];
-  __shared__ float weight[16][LATENT_MAX_SPLITS];
-  const int h = blockIdx.x, n0 = blockIdx.y * 64, b0 = blockIdx.z * 16;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int pitch = p.rank * static_cast<int>(sizeof(E)) + 16;  // bytes of a merged row
+__global__ void __launch_bounds__(128) latent_merge_kernel(const __grid_constant__ LatentValueParams p) {
+  __shared__ float weight[LATENT_MAX_SPLITS];
+  const int64_t bh = static_cast<int64_t>(blockIdx.y) * p.heads + blockIdx.x;
+  const int tid = threadIdx.x;
   if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
   pdl_wait();
-  for (int r = warp; r < 16; r += 4) {
-    const int b = b0 + r;
-    float m = -INFINITY;
-    const float2* ml = p.ml + (static_cast<int64_t>(b) * p.heads + h) * p.splits;
-    if (b < p.batch)
-      for (int s = lane; s < p.splits; s += 32) m = fmaxf(m, ml[s].x);
+  if (tid < 32) {
+    constexpr int N = LATENT_MAX_SPLITS / 32;
+    float2 a[N];
+    float m = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      a[i] = tid + i * 32 < p.splits ? p.ml[bh * p.splits + tid + i * 32] : make_float2(-INFINITY, 0.f);
+      m = fmaxf(m, a[i].x);
+    }
     m = warp_max(m);
-    float l = 0.f;
-    for (int s = lane; s < p.splits; s += 32) {
-      const float2 a = b < p.batch ? ml[s] : make_float2(-INFINITY, 0.f);
-      const float e = a.y > 0.f ? expf(a.x - m) : 0.f;
-      weight[r][s] = e;
-      l += e * a.y;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      a[i].x = a[i].y > 0.f ? expf(a[i].x - m) : 0.f;
+      l += a[i].x * a[i].y;
     }
     l = warp_sum(l);
     const float inv = l > 0.f ? 1.0f / l : 0.f;
-    for (int s = lane; s < p.splits; s += 32) weight[r][s] *= inv;
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (tid + i * 32 < p.splits) weight[tid + i * 32] = a[i].x * inv;
   }
   __syncthreads();
-  const int quads = p.rank / 4;
-  for (int i = tid; i < 16 * quads; i += 128) {
-    const int r = i / quads, c = (i % quads) * 4, b = b0 + r;
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (b < p.batch) {
-      const float* o = p.o + ((static_cast<int64_t>(b) * p.heads + h) * p.splits) * p.rank + c;
-#pragma unroll 4
-      for (int s = 0; s < p.splits; ++s) {
-        const float w = weight[r][s];
-        if (w != 0.f) {
-          const float4 v = load4(o + static_cast<int64_t>(s) * p.rank);
-          a.x = fmaf(w, v.x, a.x), a.y = fmaf(w, v.y, a.y), a.z = fmaf(w, v.z, a.z), a.w = fmaf(w, v.w, a.w);
+  for (int c = tid * 4; c < p.rank; c += 512) {
+    const float* o = p.o + bh * p.splits * p.rank + c;
+    float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+    constexpr int U = 8;
+    for (int s0 = 0; s0 < p.splits; s0 += U) {
+      float4 v[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (s0 + u < p.splits) v[u] = load4(o + static_cast<int64_t>(s0 + u) * p.rank);
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (s0 + u < p.splits && weight[s0 + u] != 0.f) {  // an empty range left its part of the workspace unwritten
+          const float w = weight[s0 + u];
+          sum.x = fmaf(w, v[u].x, sum.x), sum.y = fmaf(w, v[u].y, sum.y);
+          sum.z = fmaf(w, v[u].z, sum.z), sum.w = fmaf(w, v[u].w, sum.w);
         }
-      }
     }
-    store4(reinterpret_cast<E*>(lv_smem + r * pitch) + c, a);
+    store4(static_cast<E*>(p.merged) + bh * p.rank + c, sum);
   }
-  __syncthreads();
-  const E* w = static_cast<const E*>(p.w) + (static_cast<int64_t>(h) * p.vdim + n0) * p.rank;
-  E* out = static_cast<E*>(p.out);
-  if constexpr (sizeof(E) == 2) {
-    // a warp per 16 value columns; the B operand comes straight from W_uv rows (K contiguous): lane (n = lane / 4,
-    // k pair = lane % 4) loads its own 32-bit words
-    float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-    const uint32_t* w0 = reinterpret_cast<const uint32_t*>(w + static_cast<int64_t>(warp * 16 + (lane >> 2)) * p.rank) + (lane & 3);
-    const uint32_t* w1 = w0 + static_cast<int64_t>(8) * p.rank / 2;
-#pragma unroll 8
-    for (int ks = 0; ks < p.rank / 16; ++ks) {
-      uint32_t a[4];
-      ldmatrix_x4(a, smem_u32(lv_smem) + (lane & 15) * pitch + ks * 32 + (lane >> 4) * 16);
-      mma_bf16_16816(acc[0], a, w0[ks * 8], w0[ks * 8 + 4]);
-      mma_bf16_16816(acc[1], a, w1[ks * 8], w1[ks * 8 + 4]);
-    }
-#pragma unroll
-    for (int t = 0; t < 2; ++t)
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        const int b = b0 + (lane >> 2) + half * 8;
-        if (b < p.batch)
-          *reinterpret_cast<uint32_t*>(out + (static_cast<int64_t>(b) * p.heads + h) * p.vdim + n0 + warp * 16 + t * 8 + (lane & 3) * 2) =
-              pack_bf16(acc[t][half * 2], acc[t][half * 2 + 1]);
-      }
-  } else {
-    for (int i = tid; i < 16 * 64; i += 128) {
-      const int r = i / 64, n = i % 64, b = b0 + r;
-      if (b >= p.batch) break;
-      const float* x = reinterpret_cast<const float*>(lv_smem + r * pitch);
-      float s = 0.f;
-      for (int k = 0; k < p.rank; ++k) s = fmaf(x[k], w[static_cast<int64_t>(n) * p.rank + k], s);
-      out[(static_cast<int64_t>(b) * p.heads + h) * p.vdim + n0 + n] = s;
-    }
+}
+
+__global__ void __launch_bounds__(128) latent_value_bf16_kernel(const __grid_constant__ LatentValueParams p) {
+  extern __shared__ __align__(16) uint8_t hg_smem[];
+  const int h = blockIdx.x, n0 = blockIdx.y * 64, b0 = blockIdx.z * 16, slots = min(16, p.batch - b0);
+  float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+  head_gemm<false>(static_cast<const __nv_bfloat16*>(p.w) + static_cast<int64_t>(h) * p.vdim * p.rank, p.rank,
+                   static_cast<const __nv_bfloat16*>(p.merged) + (static_cast<int64_t>(b0) * p.heads + h) * p.rank,
+                   static_cast<int64_t>(p.heads) * p.rank, slots, p.rank / 64, n0, (p.overlap & OVERLAP_TRIGGER) != 0, hg_smem, acc);
+  head_gemm_store(acc, static_cast<__nv_bfloat16*>(p.out) + (static_cast<int64_t>(b0) * p.heads + h) * p.vdim + n0,
+                  static_cast<int64_t>(p.heads) * p.vdim, slots);
+}
+__global__ void __launch_bounds__(128) latent_value_f32_kernel(const __grid_constant__ LatentValueParams p) {
+  const int h = blockIdx.x, n0 = blockIdx.y * 64, b0 = blockIdx.z * 16;
+  for (int i = threadIdx.x; i < 16 * 64; i += 128) {
+    const int b = b0 + i / 64, n = n0 + i % 64;
+    if (b >= p.batch) break;
+    const float* x = static_cast<const float*>(p.merged) + (static_cast<int64_t>(b) * p.heads + h) * p.rank;
+    const float* w = static_cast<const float*>(p.w) + (static_cast<int64_t>(h) * p.vdim + n) * p.rank;
+    float s = 0.f;
+    for (int k = 0; k < p.rank; ++k) s = fmaf(x[k], w[k], s);
+    static_cast<float*>(p.out)[(static_cast<int64_t>(b) * p.heads + h) * p.vdim + n] = s;
   }
+}
+
+static bool head_gemm_configure(const void* kernel, int which) {
+  static bool configured[2][64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev < 0 || dev >= 64 || configured[which][dev]) return true;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 16 * HG_STEP) != cudaSuccess) return false;
+  configured[which][dev] = true;
+  return true;
 }
 
 }  // namespace b200
@@ -410,16 +443,30 @@ extern "C" int b200_latent_prep(const void* fused, int64_t stride, const float* 
                                 int32_t rows, int32_t q_rank, int32_t true_q_rank, int32_t rank, int32_t true_rank,
                                 int32_t rot, int32_t rot_pairs, float eps, int32_t f32, int32_t overlap, b200_stream_t stream) {
   if (rows <= 0) return OK;
-  B200_REQUIRE(q_rank > 0 && q_rank % 4 == 0 && rank % 4 == 0 && rot % 2 == 0 && stride % 4 == 0 && rot_pairs * 2 <= rot,
-               "latent_prep: widths must be multiples of 4 and cover the rotated pairs");
-  B200_REQUIRE(aligned16(fused) && aligned16(cq) && aligned16(cache), "latent_prep: unaligned tensor");
+  B200_REQUIRE(q_rank > 0 && q_rank % 8 == 0 && rank % 8 == 0 && rot % 8 == 0 && stride % 8 == 0 && rot_pairs * 2 <= rot,
+               "latent_prep: widths must be multiples of 8 and cover the rotated pairs");
+  B200_REQUIRE(aligned16(fused) && aligned16(cq) && aligned16(cache) && aligned16(q_weight) && aligned16(kv_weight),
+               "latent_prep: unaligned tensor");
   LatentPrepParams p = {fused, stride, q_weight, kv_weight, pos, pos_is_int64, slot, active, block_table, table_stride,
                         reinterpret_cast<const float2*>(angles), cache, cq, q_rank, true_q_rank, rank, true_rank, rot,
                         rot_pairs, overlap, eps};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const bool early = (overlap & OVERLAP_START) != 0;
-  const cudaError_t e = f32 ? launch_pdl(early, latent_prep_kernel<float>, dim3(rows), dim3(128), 0, st, p)
-                            : launch_pdl(early, latent_prep_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, st, p);
+  const int vecs = (q_rank + (cache ? rank + rot : 0)) / 8;
+  int v = 1;
+  while (v < 4 && vecs > 256 * v) v *= 2;
+  B200_REQUIRE(vecs <= 1024, "latent_prep: at most 8192 elements per row (got %d)", vecs * 8);
+  const dim3 block(((vecs + v - 1) / v + 31) / 32 * 32);
+  cudaError_t e;
+  if (f32) {
+    e = v == 1 ? launch_pdl(early, latent_prep_kernel<float, 1>, dim3(rows), block, 0, st, p)
+        : v == 2 ? launch_pdl(early, latent_prep_kernel<float, 2>, dim3(rows), block, 0, st, p)
+                 : launch_pdl(early, latent_prep_kernel<float, 4>, dim3(rows), block, 0, st, p);
+  } else {
+    e = v == 1 ? launch_pdl(early, latent_prep_kernel<__nv_bfloat16, 1>, dim3(rows), block, 0, st, p)
+        : v == 2 ? launch_pdl(early, latent_prep_kernel<__nv_bfloat16, 2>, dim3(rows), block, 0, st, p)
+                 : launch_pdl(early, latent_prep_kernel<__nv_bfloat16, 4>, dim3(rows), block, 0, st, p);
+  }
   if (e != cudaSuccess) return fail(ERR_LAUNCH, "latent_prep: %s", cudaGetErrorString(e));
   return check_launch("latent_prep");
 }
@@ -428,13 +475,14 @@ extern "C" int b200_rope_interleaved(void* x, int64_t row_stride, int32_t head_s
                                      int32_t pairs, const int32_t* pos, const float* angles, int32_t rows, int32_t f32,
                                      b200_stream_t stream) {
   if (rows <= 0 || pairs <= 0) return OK;
+  B200_REQUIRE(row_stride % 8 == 0 && head_stride % 8 == 0 && offset % 8 == 0 && aligned16(x) && offset + (2 * pairs + 7) / 8 * 8 <= head_stride,
+               "rope_interleaved: the rotated part must start and end on groups of 8 elements");
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  if (f32)
-    rope_interleaved_kernel<float><<<rows, 256, 0, st>>>(static_cast<float*>(x), row_stride, head_stride, offset, heads, pairs,
-                                                         pos, reinterpret_cast<const float2*>(angles));
-  else
-    rope_interleaved_kernel<__nv_bfloat16><<<rows, 256, 0, st>>>(static_cast<__nv_bfloat16*>(x), row_stride, head_stride, offset,
-                                                                 heads, pairs, pos, reinterpret_cast<const float2*>(angles));
+  const int64_t items = static_cast<int64_t>(rows) * heads * ((pairs + 3) / 4);
+  const unsigned grid = static_cast<unsigned>((items + 255) / 256);
+  const float2* a = reinterpret_cast<const float2*>(angles);
+  if (f32) rope_interleaved_kernel<float><<<grid, 256, 0, st>>>(static_cast<float*>(x), row_stride, head_stride, offset, heads, pairs, pos, a, rows);
+  else rope_interleaved_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(static_cast<__nv_bfloat16*>(x), row_stride, head_stride, offset, heads, pairs, pos, a, rows);
   return check_launch("rope_interleaved");
 }
 
@@ -467,15 +515,17 @@ extern "C" int b200_latent_absorb(const void* q, const void* w_uk, const int64_t
                                   int32_t batch, int32_t heads, int32_t dim, int32_t rot, int32_t rot_pairs, int32_t rank,
                                   int32_t f32, int32_t overlap, b200_stream_t stream) {
   if (batch <= 0) return OK;
-  B200_REQUIRE(dim % 64 == 0 && rank % 64 == 0 && rot % 2 == 0 && rot_pairs * 2 <= rot && (batch + 15) / 16 <= 65535,
-               "latent_absorb: dim and rank must be multiples of 64");
+  B200_REQUIRE(dim % 64 == 0 && dim <= 1024 && rank % 64 == 0 && rot % 2 == 0 && rot_pairs * 2 <= rot && (batch + 15) / 16 <= 65535,
+               "latent_absorb: dim (at most 1024) and rank must be multiples of 64");
   B200_REQUIRE(aligned16(q) && aligned16(w_uk) && aligned16(out), "latent_absorb: unaligned tensor");
   LatentAbsorbParams p = {q, w_uk, pos, reinterpret_cast<const float2*>(angles), out, batch, heads, dim, rot, rot_pairs, rank, overlap};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid(heads, rank / 64, (batch + 15) / 16);
   if (f32) latent_absorb_f32_kernel<<<grid, 128, 0, st>>>(p);
   else {
-    const cudaError_t e = launch_pdl((overlap & OVERLAP_START) != 0, latent_absorb_bf16_kernel, grid, dim3(128), 0, st, p);
+    if (!head_gemm_configure(reinterpret_cast<const void*>(latent_absorb_bf16_kernel), 0))
+      return fail(ERR_RUNTIME, "latent_absorb: cannot raise dynamic shared memory");
+    const cudaError_t e = launch_pdl((overlap & OVERLAP_START) != 0, latent_absorb_bf16_kernel, grid, dim3(128), dim / 64 * HG_STEP, st, p);
     if (e != cudaSuccess) return fail(ERR_LAUNCH, "latent_absorb: %s", cudaGetErrorString(e));
   }
   return check_launch("latent_absorb");
@@ -500,29 +550,31 @@ extern "C" int b200_latent_decode_simple(const void* q, const void* cache, const
   return check_launch("latent_decode_simple");
 }
 
-extern "C" int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* out, int32_t batch, int32_t heads,
-                                 int32_t rank, int32_t vdim, int32_t splits, int32_t f32, int32_t overlap, b200_stream_t stream) {
+extern "C" int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* merged, void* out, int32_t batch,
+                                 int32_t heads, int32_t rank, int32_t vdim, int32_t splits, int32_t f32, int32_t overlap,
+                                 b200_stream_t stream) {
   if (batch <= 0) return OK;
-  B200_REQUIRE(rank % 64 == 0 && rank <= LS_MAX_COLS && vdim % 64 == 0 && splits > 0 && splits <= LATENT_MAX_SPLITS,
+  B200_REQUIRE(rank % 64 == 0 && rank <= LS_MAX_COLS && vdim % 64 == 0 && splits > 0 && splits <= LATENT_MAX_SPLITS && batch <= 65535,
                "latent_value: rank and vdim must be multiples of 64, rank at most %d, splits at most %d", LS_MAX_COLS,
                LATENT_MAX_SPLITS);
-  LatentValueParams p = {reinterpret_cast<const float2*>(ml), o, w_uv, out, batch, heads, rank, vdim, splits, overlap};
+  B200_REQUIRE(aligned16(o) && aligned16(w_uv) && aligned16(merged) && aligned16(out), "latent_value: unaligned tensor");
+  LatentValueParams p = {reinterpret_cast<const float2*>(ml), o, w_uv, merged, out, batch, heads, rank, vdim, splits, overlap};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const dim3 grid(heads, vdim / 64, (batch + 15) / 16);
-  const int smem = 16 * (rank * (f32 ? 4 : 2) + 16);
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev >= 0 && dev < 64 && !configured[dev]) {
-    constexpr int most = 16 * (LS_MAX_COLS * 4 + 16);
-    if (cudaFuncSetAttribute(latent_value_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess ||
-        cudaFuncSetAttribute(latent_value_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess)
-      return fail(ERR_RUNTIME, "latent_value: cannot raise dynamic shared memory");
-    configured[dev] = true;
-  }
+  const dim3 grid(heads, vdim / 64, (batch + 15) / 16), merge_grid(heads, batch);
   const bool early = (overlap & OVERLAP_START) != 0;
-  const cudaError_t e = f32 ? launch_pdl(early, latent_value_kernel<float>, grid, dim3(128), smem, st, p)
-                            : launch_pdl(early, latent_value_kernel<__nv_bfloat16>, grid, dim3(128), smem, st, p);
-  if (e != cudaSuccess) return fail(ERR_LAUNCH, "latent_value: %s", cudaGetErrorString(e));
+  LatentValueParams merge = p;
+  if (f32) {
+    merge.overlap &= ~OVERLAP_TRIGGER;  // the fp32 product behind it is launched plainly
+    if (launch_pdl(early, latent_merge_kernel<float>, merge_grid, dim3(128), 0, st, merge) != cudaSuccess)
+      return fail(ERR_LAUNCH, "latent_value: %s", cudaGetErrorString(cudaGetLastError()));
+    latent_value_f32_kernel<<<grid, 128, 0, st>>>(p);
+    return check_launch("latent_value");
+  }
+  if (!head_gemm_configure(reinterpret_cast<const void*>(latent_value_bf16_kernel), 1))
+    return fail(ERR_RUNTIME, "latent_value: cannot raise dynamic shared memory");
+  merge.overlap |= OVERLAP_TRIGGER;     // its successor is the product below, which waits
+  if (launch_pdl(early, latent_merge_kernel<__nv_bfloat16>, merge_grid, dim3(128), 0, st, merge) != cudaSuccess ||
+      launch_pdl(true, latent_value_bf16_kernel, grid, dim3(128), rank / 64 * HG_STEP, st, p) != cudaSuccess)
+    return fail(ERR_LAUNCH, "latent_value: %s", cudaGetErrorString(cudaGetLastError()));
   return check_launch("latent_value");
 }

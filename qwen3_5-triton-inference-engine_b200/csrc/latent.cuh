@@ -49,6 +49,7 @@ struct LatentValueParams {
   const float2* ml;
   const float* o;
   const void* w;         // [heads, vdim, rank]
+  void* merged;          // [batch, heads, rank] E
   void* out;             // [batch, heads, vdim]
   int batch, heads, rank, vdim, splits, overlap;
 };

@@ -25,10 +25,11 @@ constexpr int LD_MAX_STAGES = 6;
 constexpr int LD_S_PITCH = 36;                   // floats per score row
 constexpr int LD_P_PITCH = 40;                   // bf16 per probability row (80 bytes: ldmatrix rows in different banks)
 constexpr int LD_SMEM_LIMIT = 216 * 1024;         // dynamic; 6 KiB more are static
+constexpr int LD_SMEM_PAIR = 105 * 1024;          // ... when two CTAs share an SM
 
 // NT: value columns per warp / 8 that the accumulators hold (rank <= 64 * NT)
 template <int NT>
-__global__ void __launch_bounds__(LD_THREADS)
+__global__ void __launch_bounds__(LD_THREADS, NT <= 8 ? 2 : 1)
 latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_constant__ CUtensorMap map_rows, int stages) {
   extern __shared__ __align__(1024) uint8_t ld_smem_raw[];
   __shared__ uint64_t full[LD_MAX_STAGES], empty[LD_MAX_STAGES];
@@ -92,7 +93,8 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
   float acc[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  float m_run = -INFINITY, l_run = 0.f;   // of head row sm_row: the maximum, and this lane's part of the sum
+  const int sm_row = warp * 2 + (lane >> 4), sm_tok = (lane & 15) * 2;
   const float scale_log2 = p.scale * 1.4426950408889634f;
   const int tg = warp & 3, kh = warp >> 2;
   const int units = pitch / 32;
@@ -134,19 +136,22 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
       *reinterpret_cast<float2*>(&ss[kh][r + 8][col]) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
     named_barrier(1, LD_WARPS * 32);
-    // ---- softmax: rows 2 * warp, 2 * warp + 1; lane = token
-    const bool visible = tok0 + lane >= lo && tok0 + lane < hi;
+    // ---- softmax: half a warp per head row, two tokens per lane
+    {
+      const float2 a = *reinterpret_cast<const float2*>(&ss[0][sm_row][sm_tok]), c = *reinterpret_cast<const float2*>(&ss[1][sm_row][sm_tok]);
+      const int at = tok0 + sm_tok;
+      const float x0 = at >= lo && at < hi ? (a.x + c.x) * scale_log2 : -INFINITY;
+      const float x1 = at + 1 >= lo && at + 1 < hi ? (a.y + c.y) * scale_log2 : -INFINITY;
+      float mx = fmaxf(x0, x1);
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int r = warp * 2 + i;
-      const float x = visible ? (ss[0][r][lane] + ss[1][r][lane]) * scale_log2 : -INFINITY;
-      const float m_new = fmaxf(m_run[i], warp_max(x));   // a tile holds at least one visible token
-      const float pr = ex2_fast(x - m_new);
-      const float a = ex2_fast(m_run[i] - m_new);
-      l_run[i] = l_run[i] * a + warp_sum(pr);
-      m_run[i] = m_new;
-      ps[r][lane] = __float2bfloat16_rn(pr);
-      if (lane == 0) alphas[r] = a;
+      for (int bit = 8; bit >= 1; bit >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, bit));
+      const float m_new = fmaxf(m_run, mx);               // a tile holds at least one visible token
+      const float alpha = ex2_fast(m_run - m_new);
+      const float p0 = ex2_fast(x0 - m_new), p1 = ex2_fast(x1 - m_new);
+      l_run = fmaf(l_run, alpha, p0 + p1);
+      m_run = m_new;
+      *reinterpret_cast<uint32_t*>(&ps[sm_row][sm_tok]) = pack_bf16(p0, p1);
+      if ((lane & 15) == 0) alphas[sm_row] = alpha;
     }
     named_barrier(1, LD_WARPS * 32);
     // ---- O: this warp's columns
@@ -186,12 +191,10 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
     return;
   }
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int r = warp * 2 + i;
-    // maxima are kept in the log2 domain; latent_value works with natural exponentials
-    if (lane == 0 && r < heads_here)
-      p.ml[part0 + static_cast<int64_t>(r) * p.splits] = make_float2(m_run[i] * 0.6931471805599453f, l_run[i]);
-  }
+  for (int bit = 8; bit >= 1; bit >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, bit);
+  // maxima are kept in the log2 domain; the merge works with natural exponentials
+  if ((lane & 15) == 0 && sm_row < heads_here)
+    p.ml[part0 + static_cast<int64_t>(sm_row) * p.splits] = make_float2(m_run * 0.6931471805599453f, l_run);
 #pragma unroll
   for (int i = 0; i < NT; ++i)
     if (i < nt) {
@@ -260,7 +263,8 @@ extern "C" int b200_latent_decode(const void* q, const void* cache, int64_t num_
                "latent_decode: window, scale and splits (at most %d) must be positive", LATENT_MAX_SPLITS);
   B200_REQUIRE(aligned16(q) && aligned16(cache) && aligned16(o), "latent_decode: unaligned tensor");
   const int pitch = rank + rot, tile = LD_TOK * pitch * 2, q_bytes = 16 * (pitch * 2 + 16) + 1024;  // incl. alignment of the ring
-  int stages = (LD_SMEM_LIMIT - q_bytes) / tile;
+  int stages = rank <= 512 ? (LD_SMEM_PAIR - q_bytes) / tile : 0;   // two CTAs on an SM cover each other's latencies
+  if (stages < 2) stages = (LD_SMEM_LIMIT - q_bytes) / tile;
   if (stages > LD_MAX_STAGES) stages = LD_MAX_STAGES;
   B200_REQUIRE(stages >= 2, "latent_decode: rows of %d elements do not fit", pitch);
   LatentDecodeParams p = {q, cache, block_table, table_stride, pos, active, reinterpret_cast<float2*>(ml), o,

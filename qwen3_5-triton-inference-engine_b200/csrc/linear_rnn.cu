@@ -8,11 +8,13 @@
 //     pass 2 folds the chunks in front of its own and replays its chunk.  HBM bound; both passes stream 16-byte rows.
 //   Forget-gated outer-product recurrence (HGRN2 form):  f = l + (1 - l) sigmoid(f' + fb), q = silu(q')
 //                           S_t = diag(f) S_(t-1) + (1 - f) v^T,   o = S_t^T q,   out = rms(o) * w per head
-//     Prefill is token-serial in fp32 (no cumulative products of gates, so nothing can under- or overflow): a warp owns
-//     COLS state columns, a lane dim/32 rows of each as packed fp32 pairs (fma.rn.f32x2); 16 tokens of gates are staged
-//     in shared memory at a time, the next 16 are loaded while they are worked on.
+//     Prefill of bf16 activations runs in chunks on the tensor cores (linear_rnn_chunk.cu).  The token-serial form here is
+//     plain fp32, for fp32 activations and for heads wider than 128: a warp owns COLS state columns, a lane dim/32 rows
+//     of each as packed fp32 pairs (fma.rn.f32x2); 16 tokens of gates are staged in shared memory at a time, the next 16
+//     are loaded while they are worked on.
 #include "b200_attn.h"
 #include "elem.cuh"
+#include "linear_rnn.cuh"
 
 namespace b200 {
 
@@ -75,28 +77,29 @@ __global__ void __launch_bounds__(128) mingru_scan_kernel(const __grid_constant_
       return *reinterpret_cast<const float2*>(q);
     }
   };
-  constexpr int U = 8;  // rows in flight
-  for (int t = t0; t < t1; t += U) {
-    float2 z[U], x[U], g[U];
+  constexpr int U = 8;  // rows per group; the next group's loads are in flight while one is worked on
+  float2 z[2][U], x[2][U], g[2][U];
+  auto fetch = [&](int buf, int t) {
 #pragma unroll
-    for (int i = 0; i < U; ++i)
-      if (t + i < t1) {
-        const E* r = base + static_cast<int64_t>(t + i) * p.stride;
-        z[i] = two(r);
-        x[i] = two(r + p.width);
-        if (REPLAY) g[i] = two(r + 2 * p.width);
-      }
+    for (int i = 0; i < U; ++i) {
+      const E* r = base + static_cast<int64_t>(min(t + i, t1 - 1)) * p.stride;  // past the end: a row read again
+      z[buf][i] = two(r);
+      x[buf][i] = two(r + p.width);
+      if (REPLAY) g[buf][i] = two(r + 2 * p.width);
+    }
+  };
+  auto work = [&](int buf, int t) {
 #pragma unroll
-    for (int i = 0; i < U; ++i)
+    for (int i = 0; i < U; ++i) {
+      float k0, k1, b0, b1;
+      mingru_gate<E>(z[buf][i].x, x[buf][i].x, zb.x, xb.x, k0, b0);
+      mingru_gate<E>(z[buf][i].y, x[buf][i].y, zb.y, xb.y, k1, b1);
       if (t + i < t1) {
-        float k0, k1, b0, b1;
-        mingru_gate<E>(z[i].x, x[i].x, zb.x, xb.x, k0, b0);
-        mingru_gate<E>(z[i].y, x[i].y, zb.y, xb.y, k1, b1);
         s0 = fmaf(k0, s0, b0);
         s1 = fmaf(k1, s1, b1);
         if (REPLAY) {
           E* o = static_cast<E*>(p.out) + static_cast<int64_t>(row0 + t + i) * p.width + c;
-          const float o0 = s0 * silu_f<E>(g[i].x), o1 = s1 * silu_f<E>(g[i].y);
+          const float o0 = s0 * silu_f<E>(g[buf][i].x), o1 = s1 * silu_f<E>(g[buf][i].y);
           if constexpr (sizeof(E) == 2) *reinterpret_cast<uint32_t*>(o) = pack_bf16(o0, o1);
           else *reinterpret_cast<float2*>(o) = make_float2(o0, o1);
         } else {
@@ -104,6 +107,16 @@ __global__ void __launch_bounds__(128) mingru_scan_kernel(const __grid_constant_
           a1 *= k1;
         }
       }
+    }
+  };
+  fetch(0, t0);
+  for (int t = t0; t < t1; t += 2 * U) {
+    if (t + U < t1) fetch(1, t + U);
+    work(0, t);
+    if (t + U < t1) {
+      if (t + 2 * U < t1) fetch(0, t + 2 * U);
+      work(1, t + U);
+    }
   }
   if (!REPLAY) *reinterpret_cast<float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(chunk) * p.width) = make_float4(a0, s0, a1, s1);
   else if (t1 == len) {
@@ -171,19 +184,6 @@ __device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
   asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
   return r;
 }
-
-struct OuterRnnParams {
-  const void* qfv;         // [rows, stride] E: [q heads*dim | f heads*dim | v heads*vdim]
-  int64_t stride;
-  const float* lower;      // [heads*dim]
-  const float* bias;       // [heads*dim]
-  float* state;            // [slots, heads, dim, vdim]
-  const int32_t* cu;
-  const int32_t* slots;
-  const int32_t* start;
-  float* o;                // [rows, heads*vdim] fp32, before the head norm
-  int heads, dim, vdim;    // padded sizes: dim a multiple of 32, vdim a multiple of 16
-};
 
 constexpr int OR_TB = 16;        // tokens staged at a time
 constexpr int OR_WARPS = 4;
@@ -484,7 +484,9 @@ template <typename E, int RP>
 static int launch_outer(const OuterRnnParams& p, int n, cudaStream_t st) {
   // wide columns share the gates of a token among more state; narrow ones give more CTAs when there are few heads
   const int64_t wide = static_cast<int64_t>((p.vdim + 31) / 32) * p.heads * n;
-  if (RP <= 2 && wide >= 2 * sm_count()) return launch_outer_cols<E, RP, 8>(p, n, st);
+  if constexpr (RP <= 2) {
+    if (wide >= 2 * sm_count()) return launch_outer_cols<E, RP, 8>(p, n, st);
+  }
   return launch_outer_cols<E, RP, 4>(p, n, st);
 }
 
@@ -547,15 +549,22 @@ extern "C" int b200_mingru_decode(const void* zxg, int64_t stride, const float* 
 extern "C" int b200_hgrn2_prefill(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm,
                                   float* state, const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start,
                                   float* o_scratch, void* out, int32_t batch, int32_t tokens, int32_t heads, int32_t dim,
-                                  int32_t vdim, int32_t true_vdim, float eps, int32_t f32, b200_stream_t stream) {
+                                  int32_t vdim, int32_t true_vdim, float eps, int32_t f32, int32_t serial,
+                                  b200_stream_t stream) {
   if (batch <= 0 || tokens <= 0) return OK;
   B200_REQUIRE(dim > 0 && dim <= 256 && vdim > 0 && vdim % 4 == 0 && vdim <= OD_MAX_VDIM && true_vdim <= vdim,
                "hgrn2_prefill: dim at most 256, vdim a multiple of 4 and at most %d (got %d, %d)", OD_MAX_VDIM, dim, vdim);
   B200_REQUIRE(heads > 0 && heads <= 65535 && batch <= 65535, "hgrn2_prefill: at most 65535 heads and sequences");
   B200_REQUIRE(aligned16(o_scratch) && aligned16(out) && aligned16(norm), "hgrn2_prefill: unaligned tensor");
-  OuterRnnParams p = {qfv, stride, lower, bias, state, cu_seqlens, slots, start, o_scratch, heads, dim, vdim};
+  OuterRnnParams p = {qfv, stride, lower, bias, state, cu_seqlens, slots, start, o_scratch, heads, dim, vdim,
+                      norm, nullptr, true_vdim, eps};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const int rc = f32 ? launch_outer_rows<float>(p, batch, st) : launch_outer_rows<__nv_bfloat16>(p, batch, st);
+  const bool chunked = !f32 && !serial && outer_rnn_chunk_supports(dim, vdim) && stride % 8 == 0 && heads * dim % 8 == 0 && aligned16(qfv);
+  if (chunked && vdim <= 128) {  // the head norm inside: one launch
+    p.out = out;
+    return outer_rnn_chunk_launch(p, batch, st);
+  }
+  const int rc = chunked ? outer_rnn_chunk_launch(p, batch, st) : f32 ? launch_outer_rows<float>(p, batch, st) : launch_outer_rows<__nv_bfloat16>(p, batch, st);
   if (rc != OK) return rc;
   const int64_t rows = static_cast<int64_t>(tokens) * heads;
   const unsigned grid = static_cast<unsigned>((rows + 7) / 8);

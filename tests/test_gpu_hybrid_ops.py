@@ -149,19 +149,19 @@ def _hgrn2_inputs(tokens, heads, dim, vdim, dtype, seed):
     return qfv, lower, bias, 1.0 + rnd(vdim, seed=seed + 3, scale=0.3)
 
 
-HGRN2_SIZES = [(3, 32, 48), (1, 16, 16), (2, 128, 128), (5, 64, 32), (2, 208, 80), (1, 256, 512)]
+HGRN2_SIZES = [(3, 32, 48), (1, 16, 16), (2, 48, 144), (4, 112, 64), (2, 128, 128), (5, 64, 32), (2, 208, 80), (1, 256, 512)]
 
 
-@pytest.mark.parametrize("dt", DT)
+@pytest.mark.parametrize("form", ["f32", "bf16", "bf16-serial"])
 @pytest.mark.parametrize("heads,dim,vdim", HGRN2_SIZES)
-def test_hgrn2_prefill(hops, dt, heads, dim, vdim):
-    dtype, eps = DT[dt], 1e-5
+def test_hgrn2_prefill(hops, form, heads, dim, vdim):
+    dtype, eps = DT[form.split("-")[0]], 1e-5
     lengths, slots, starts = [1, 15, 16, 33, 70], [2, 0, 4, 5, 1], [0, 3, 0, 16, 0]
     qfv, lower, bias, norm = _hgrn2_inputs(sum(lengths), heads, dim, vdim, dtype, 11)
     before = rnd(6, heads, dim, vdim, seed=17)
     state = before.to(DEV)
     dev = [t.to(DEV) for t in (qfv, lower, bias, norm)]
-    out = hops.hgrn2_prefill(*dev, state, Batch(slots, starts, lengths), vdim, eps)
+    out = hops.hgrn2_prefill(*dev, state, Batch(slots, starts, lengths), vdim, eps, serial=form.endswith("serial"))
     row = 0
     for slot, start, n in zip(slots, starts, lengths):
         want, last = _hgrn2_want(qfv[row: row + n], lower, bias, norm, heads, dim, vdim,
@@ -172,12 +172,14 @@ def test_hgrn2_prefill(hops, dt, heads, dim, vdim):
     assert torch.equal(state[3].cpu(), before[3])
 
 
-def test_hgrn2_wide_batch(hops):
-    """Enough heads and sequences for the wide-column form of the prefill kernel."""
+@pytest.mark.parametrize("serial", [False, True])
+def test_hgrn2_wide_batch(hops, serial):
+    """A batch of many heads (the wide-column form of the token-serial kernel among them)."""
     heads, dim, vdim, lengths = 16, 128, 128, [20 + i for i in range(9)]
     qfv, lower, bias, norm = _hgrn2_inputs(sum(lengths), heads, dim, vdim, torch.bfloat16, 3)
     state = torch.zeros(9, heads, dim, vdim, device=DEV)
-    out = hops.hgrn2_prefill(*[t.to(DEV) for t in (qfv, lower, bias, norm)], state, Batch(list(range(9)), [0] * 9, lengths), vdim, 1e-5)
+    out = hops.hgrn2_prefill(*[t.to(DEV) for t in (qfv, lower, bias, norm)], state, Batch(list(range(9)), [0] * 9, lengths), vdim, 1e-5,
+                             serial=serial)
     row = 0
     for i, n in enumerate(lengths):
         want, last = _hgrn2_want(qfv[row: row + n], lower, bias, norm, heads, dim, vdim, torch.zeros(heads, dim, vdim), 1e-5, vdim)
