@@ -470,11 +470,15 @@ int b200_mingru_decode(const void* zxg, int64_t stride, const float* bias, float
 /* HGRN2: qfv = rows of [q heads*dim | f heads*dim | v heads*vdim]; lower, bias fp32 [heads*dim]; norm fp32 [vdim];
  * state fp32 [slots, heads, dim, vdim];  f = l + (1-l) sigmoid(f + bias), S <- diag(f) S + (1-f) v^T, o = S^T silu(q),
  * out = o / sqrt(mean(o^2) + eps) * norm per head.  o_scratch: fp32 [tokens, heads*vdim].  serial: keep bf16 prefill on the
- * token-serial kernel (default: 16-token chunks on the tensor cores for dim <= 128). */
+ * token-serial kernel (default: 16-token chunks on the tensor cores for dim <= 128).  The chunked form may cut sequences
+ * into at most `segments` segments of `segment` tokens (a multiple of 16) that run side by side; segments = 1 with
+ * segment >= the longest sequence does not, more take a workspace of b200_hgrn2_workspace_bytes(). */
+int64_t b200_hgrn2_workspace_bytes(int32_t batch, int32_t segments, int32_t heads, int32_t dim, int32_t vdim);
 int b200_hgrn2_prefill(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
                        const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start, float* o_scratch, void* out,
                        int32_t batch, int32_t tokens, int32_t heads, int32_t dim, int32_t vdim, int32_t true_vdim, float eps,
-                       int32_t f32, int32_t serial, b200_stream_t stream);
+                       int32_t f32, int32_t serial, int32_t segment, int32_t segments, float* workspace,
+                       b200_stream_t stream);
 int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
                       const int64_t* pos, const int64_t* active, void* out, int32_t batch, int32_t heads, int32_t dim,
                       int32_t vdim, int32_t true_vdim, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);

@@ -67,7 +67,8 @@ SIGNATURES: dict[str, list] = {
     "b200_swiglu_f32": [P, I64, P, I32, I32, P],
     "b200_mingru_prefill": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, P],
     "b200_mingru_decode": [P, I64, P, P, P, P, P, I32, I32, I32, I32, P],
-    "b200_hgrn2_prefill": [P, I64, P, P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, P],
+    "b200_hgrn2_prefill": [P, I64, P, P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, I32, I32, P,
+                           P],
     "b200_hgrn2_decode": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_latent_prep": [P, I64, P, P, P, I32, P, P, P, I64, P, P, P, I32, I32, I32, I32, I32, I32, I32, c_float, I32, I32,
                          P],
@@ -82,6 +83,7 @@ SIGNATURES: dict[str, list] = {
 }
 OTHER = {
     "b200_mingru_workspace_bytes": ([I32, I32, I32], c_int64),
+    "b200_hgrn2_workspace_bytes": ([I32, I32, I32, I32, I32], c_int64),
     "b200_last_error": ([], c_char_p),
     "b200_abi_version": ([], c_int),
     "b200_wait_timed_out": ([], c_int),

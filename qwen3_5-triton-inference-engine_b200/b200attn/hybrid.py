@@ -204,10 +204,21 @@ class HybridEngine(SlotEngine):
         return (self.dtype == torch.bfloat16 and weight.shape[1] <= ops.SKINNY_GEMM_PAIR_MAX_K
                 and ops.skinny_gemm_supports(self.batch, n, weight.shape[1], swiglu))
 
-    def proj(self, x, weight):
+    def then(self, own_next: bool) -> int:
+        """Overlap flags of a decode-step kernel whose successor is (not) one of this package's."""
+        return ops.OVERLAP_START | ops.OVERLAP_TRIGGER if own_next else ops.OVERLAP_START
+
+    def proj(self, x, weight, own_next: bool):
+        """Decode-step projection: the weight-streaming kernel where it takes the shape, cuBLAS otherwise."""
         if self.streams_weight(weight):
-            return ops.skinny_gemm(x, weight)
+            return ops.skinny_gemm(x, weight, overlap=self.then(own_next))
         return F.linear(x, weight)
+
+    def fuses_head(self) -> bool:
+        """Whether LM head and greedy choice run as one launch on the decode batch."""
+        head = self.w.head
+        return (self.dtype == torch.bfloat16 and self.w.vocab_p == self.cfg.vocab and head.shape[1] <= ops.SKINNY_GEMM_MAX_K
+                and ops.skinny_gemm_supports(self.batch, head.shape[0], head.shape[1]))
 
     def logits(self, h) -> torch.Tensor:
         """fp32 logits [rows, padded vocab] of normed final rows; padding columns are -inf."""
@@ -220,29 +231,28 @@ class HybridEngine(SlotEngine):
             out[:, self.cfg.vocab:] = float("-inf")
         return out
 
-    def _joint(self, k: int, streams, y=None, ids=None):
+    def _joint(self, k: int, streams, y=None, ids=None, overlap: int = 0):
         return hops.hyper_connect(streams, self.w.joints[k], self.cfg.width, self.cfg.eps, self.dtype, y=y, ids=ids,
-                                  table=self.w.embed if ids is not None else None)
+                                  table=self.w.embed if ids is not None else None, overlap=overlap)
 
-    def _run(self, streams, ids, mix, feed):
-        """The stack over rows of `streams`: returns the final normed hidden rows."""
-        h = self._joint(0, streams, ids=ids)
-        k = 1
-        for i, mlp in enumerate(self.w.mlps):
-            h = self._joint(k, streams, y=mix(self.w.mixers[i], h))
-            k += 1
-            if mlp is not None:
-                h = self._joint(k, streams, y=feed(mlp, h))
-                k += 1
-            if self.trace is not None:
-                self.trace.append(streams.sum(1)[:, : self.cfg.width].clone())
-        return h
+    def _traced(self, streams) -> None:
+        if self.trace is not None:
+            self.trace.append(streams.sum(1)[:, : self.cfg.width].clone())
 
     # ------------------------------------------------------------------------------------------------------ prefill
     def _forward(self, batch: PackedBatch) -> torch.Tensor:
+        """The stack over a packed batch: the final normed hidden rows."""
         streams = torch.empty(batch.tokens, self.cfg.streams, self.w.width_p, dtype=torch.float32, device=self.device)
-        return self._run(streams, batch.ids, lambda m, h: m.prefill(h, batch, self, self.states),
-                         lambda m, h: m.prefill(h, self))
+        h = self._joint(0, streams, ids=batch.ids)
+        k = 1
+        for mixer, mlp in zip(self.w.mixers, self.w.mlps):
+            h = self._joint(k, streams, y=mixer.prefill(h, batch, self, self.states))
+            k += 1
+            if mlp is not None:
+                h = self._joint(k, streams, y=mlp.prefill(h, self))
+                k += 1
+            self._traced(streams)
+        return h
 
     def _set_pos(self, slots, ends) -> None:
         at = torch.tensor([slots, ends], dtype=torch.int64, device=self.device)
@@ -282,7 +292,8 @@ class HybridEngine(SlotEngine):
         at = torch.tensor([slots, starts, [p[0] for p in portions]], dtype=torch.int64, device=self.device)
         self.pos.index_copy_(0, at[0], at[1])
         tok = self.tok.index_copy(0, at[0], at[2])
-        h = self._decode_hidden(tok)
+        h = self._decode_hidden(tok, False)
+        self._move_on()
         self.active.copy_(others)
         rows = [s for s, w in zip(slots, want) for _ in w]
         if not rows:
@@ -309,18 +320,40 @@ class HybridEngine(SlotEngine):
         return first.clone()
 
     # ------------------------------------------------------------------------------------------------------- decode
-    def _decode_hidden(self, tok) -> torch.Tensor:
-        """One token per slot; `pos` moves on for the active ones.  Idle slots ride along and touch nothing."""
-        h = self._run(self.streams, tok, lambda m, h: m.decode(h, self, self.states), lambda m, h: m.decode(h, self))
-        self.pos.add_(1 if self.active is None else self.active)
+    def _decode_hidden(self, tok, own_head: bool) -> torch.Tensor:
+        """The stack over one token per slot; idle slots ride along and touch nothing.  Every kernel of this package that
+        follows another one starts early; what the next sublayer's first projection runs on decides a joint's flags."""
+        steps = list(self.w.sublayers())
+
+        def first_own(k: int) -> bool:               # does a kernel of ours read the output of joint k?
+            if k == len(steps):
+                return own_head
+            i, q = steps[k]
+            if q == 1:
+                return self.streams_weight(self.w.mixers[i].first_weight())
+            return self.streams_weight(self.w.mlps[i].gate_up, swiglu=True)
+
+        streams, untraced = self.streams, self.trace is None
+        h = self._joint(0, streams, ids=tok, overlap=self.then(first_own(0)))
+        for k, (i, q) in enumerate(steps, start=1):
+            last = k == len(steps) or steps[k][0] != i          # the layer ends here
+            y = self.w.mixers[i].decode(h, self, self.states, True) if q == 1 else self.w.mlps[i].decode(h, self, True)
+            h = self._joint(k, streams, y=y, overlap=self.then(first_own(k) and untraced))
+            if last:
+                self._traced(streams)
         return h
+
+    def _move_on(self) -> None:
+        self.pos.add_(1 if self.active is None else self.active)
 
     @torch.no_grad()
     def _decode(self, tok):
-        h = self._decode_hidden(tok)
-        head = self.w.head
-        if (self.dtype == torch.bfloat16 and self.w.vocab_p == self.cfg.vocab and head.shape[1] <= ops.SKINNY_GEMM_MAX_K
-                and ops.skinny_gemm_supports(self.batch, head.shape[0], head.shape[1])):
+        own_head = self.fuses_head()
+        h = self._decode_hidden(tok, own_head)
+        if own_head:
             in_place = tok.data_ptr() == self.tok.data_ptr()
-            return ops.lm_head_argmax(h, head, self.argmax_ws, out=tok if in_place else None)
-        return ops.argmax_rows(self.logits(h), self.argmax_ws)
+            nxt = ops.lm_head_argmax(h, self.w.head, self.argmax_ws, out=tok if in_place else None, overlap=ops.OVERLAP_START)
+        else:
+            nxt = ops.argmax_rows(self.logits(h), self.argmax_ws)
+        self._move_on()
+        return nxt

@@ -44,12 +44,16 @@ def swiglu_f32(gate_up, intermediate: int):
 
 
 # ------------------------------------------------------------------------------------------------------------- minGRU
-def mingru_chunking(max_len: int, count: int = 1, width: int = 1) -> tuple[int, int]:
-    """(chunk length, chunks of the longest sequence).  A batch wide enough to keep the memory system busy (a thread per
-    two channels) runs each sequence in one pass; otherwise chunks of at least 64 tokens, at most 64 of them."""
-    if count * width >= 65536:
+MINGRU_THREADS = 65536           # threads (two channels each) that keep the memory system busy
+
+
+def mingru_chunking(max_len: int, count: int, width: int) -> tuple[int, int]:
+    """(chunk length, chunks of the longest sequence).  A batch wide enough runs each sequence in one pass; otherwise chunks
+    short enough to fill the device twice over, at least 16 tokens long and at most 128 of them."""
+    threads = count * width // 2
+    if threads >= MINGRU_THREADS:
         return max_len, 1
-    chunk = max(64, -(-max_len // 64))
+    chunk = max(16, -(-max_len * threads // (2 * MINGRU_THREADS)), -(-max_len // 128))
     return chunk, -(-max_len // chunk)
 
 
@@ -89,15 +93,44 @@ def _check_hgrn2(qfv, lower, bias, norm, state):
     return heads, dim, vdim
 
 
-def hgrn2_prefill(qfv, lower, bias, norm, state, batch, true_vdim: int, eps: float, serial: bool = False):
-    """qfv [tokens, 2*heads*dim + heads*vdim]; state [slots, heads, dim, vdim] fp32, in place."""
+def hgrn2_segments(max_len: int, groups: int, sm_count: int) -> tuple[int, int]:
+    """(segment length, segments of the longest sequence).  `groups` CTAs work on whole sequences; when they leave half of
+    the slots (two per SM) empty, sequences are cut into segments of at least 128 tokens that run side by side, at the
+    price of a second pass over the rows."""
+    parts = min(2 * sm_count // groups, max_len // 128)
+    if parts < 3:
+        return max_len, 1
+    segment = -(-max_len // parts // 16) * 16 + (0 if max_len % parts == 0 and (max_len // parts) % 16 == 0 else 16)
+    return segment, -(-max_len // segment)
+
+
+_sm_counts: dict = {}
+
+
+def sm_count(device) -> int:
+    key = torch.device(device).index or 0
+    if key not in _sm_counts:
+        _sm_counts[key] = torch.cuda.get_device_properties(device).multi_processor_count
+    return _sm_counts[key]
+
+
+def hgrn2_prefill(qfv, lower, bias, norm, state, batch, true_vdim: int, eps: float, serial: bool = False, segments=None):
+    """qfv [tokens, 2*heads*dim + heads*vdim]; state [slots, heads, dim, vdim] fp32, in place.  segments: (length, count) to
+    pin how sequences are cut."""
     heads, dim, vdim = _check_hgrn2(qfv, lower, bias, norm, state)
     tokens = qfv.shape[0]
-    scratch = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=qfv.device)
+    chunked = qfv.dtype == torch.bfloat16 and dim <= 128 and not serial
+    segment, count = (batch.max_len, 1) if not chunked else segments or hgrn2_segments(
+        batch.max_len, batch.count * heads * -(-vdim // 128), sm_count(qfv.device))
+    ws = None
+    if count > 1:
+        nbytes = _lib.load().b200_hgrn2_workspace_bytes(batch.count, count, heads, dim, vdim)
+        ws = torch.empty(nbytes // 4, dtype=torch.float32, device=qfv.device)
+    scratch = None if chunked and vdim <= 128 else torch.empty((tokens, heads * vdim), dtype=torch.float32, device=qfv.device)
     out = torch.empty((tokens, heads * vdim), dtype=qfv.dtype, device=qfv.device)
     _lib.call("b200_hgrn2_prefill", _ptr(qfv), qfv.stride(0), _ptr(lower), _ptr(bias), _ptr(norm), _ptr(state), _ptr(batch.cu),
               _ptr(batch.slots), _ptr(batch.start), _ptr(scratch), _ptr(out), batch.count, tokens, heads, dim, vdim, true_vdim,
-              float(eps), _f32(qfv), int(serial), _stream())
+              float(eps), _f32(qfv), int(serial), segment, count, _ptr(ws), _stream())
     return out
 
 

@@ -4,7 +4,9 @@ edge) and knows what a slot keeps for it:
 
     allocate(engine)                        the layer's cache or state, indexed by page or by slot
     prefill(h, batch, engine, states)       packed tokens of several sequences (`hybrid.PackedBatch`)
-    decode(h, engine, states, then)         one token per slot; no host value changes from step to step
+    decode(h, engine, states, nxt)          one token per slot; no host value changes from step to step.  Kernels of this
+                                            package that follow one another start early (`engine.then(own)`: whether the
+                                            kernel behind is one of them); nxt: what follows the mixer
 
 `shapes(width)` lists a layer's tensors (name -> shape) for loading and for random initialisation.
 """
@@ -18,9 +20,6 @@ import torch.nn.functional as F
 
 from . import hybrid_ops as hops
 from . import ops
-
-START, TRIGGER = ops.OVERLAP_START, ops.OVERLAP_TRIGGER
-
 
 def round_up(n: int, to: int) -> int:
     return -(-n // to) * to
@@ -159,17 +158,22 @@ class LatentAttention:
                                   self.rot_dim, self.vdim_p, self.rank_p, self.window, self.scale)
         return engine.linear(out, self.o)
 
-    def decode(self, h, engine, states):
-        state, cache = states[self.index], states[self.source]["cache"]
+    def first_weight(self):
+        return self.down
+
+    def decode(self, h, engine, states, nxt: bool):
+        state, cache, then = states[self.index], states[self.source]["cache"], engine.then
         own = self.kv_from is None
-        fused = engine.proj(h, self.down)
+        fused = engine.proj(h, self.down, True)
         cq = hops.latent_prep(fused, self.q_norm, self.kv_norm, engine.pos, None, engine.active, engine.block_table,
-                              state["angles"], cache if own else None, self.q_rank, self.rank_p, self.rank, self.eps)
-        q = engine.proj(cq, self.uq).view(-1, self.heads, self.dim_p + self.rot_p)
-        q = hops.latent_absorb(q, self.uk, engine.pos, state["angles"])
-        hops.latent_decode(q, cache, engine.block_table, engine.pos, engine.active, state["workspace"], self.window, self.scale)
-        out = hops.latent_value(state["workspace"], self.uv, engine.dtype)
-        return engine.proj(out, self.o)
+                              state["angles"], cache if own else None, self.q_rank, self.rank_p, self.rank, self.eps,
+                              overlap=then(engine.streams_weight(self.uq)))
+        q = engine.proj(cq, self.uq, True).view(-1, self.heads, self.dim_p + self.rot_p)
+        q = hops.latent_absorb(q, self.uk, engine.pos, state["angles"], overlap=then(True))
+        hops.latent_decode(q, cache, engine.block_table, engine.pos, engine.active, state["workspace"], self.window, self.scale,
+                           overlap=then(True))
+        out = hops.latent_value(state["workspace"], self.uv, engine.dtype, overlap=then(engine.streams_weight(self.o)))
+        return engine.proj(out, self.o, nxt)
 
 
 # -------------------------------------------------------------------------------------------------------------- minGRU
@@ -199,9 +203,13 @@ class MinGRU:
         out = hops.mingru_prefill(engine.linear(h, self.zxg), self.bias, states[self.index]["state"], batch)
         return engine.linear(out, self.o)
 
-    def decode(self, h, engine, states):
-        out = hops.mingru_decode(engine.proj(h, self.zxg), self.bias, states[self.index]["state"], engine.pos, engine.active)
-        return engine.proj(out, self.o)
+    def first_weight(self):
+        return self.zxg
+
+    def decode(self, h, engine, states, nxt: bool):
+        out = hops.mingru_decode(engine.proj(h, self.zxg, True), self.bias, states[self.index]["state"], engine.pos,
+                                 engine.active, overlap=engine.then(engine.streams_weight(self.o)))
+        return engine.proj(out, self.o, nxt)
 
 
 # --------------------------------------------------------------------------------------------------------------- HGRN2
@@ -243,10 +251,14 @@ class HGRN2:
                                  batch, self.vdim, self.eps)
         return engine.linear(out, self.o)
 
-    def decode(self, h, engine, states):
-        out = hops.hgrn2_decode(engine.proj(h, self.qfv), self.lower, self.bias, self.norm, states[self.index]["state"],
-                                engine.pos, engine.active, self.vdim, self.eps)
-        return engine.proj(out, self.o)
+    def first_weight(self):
+        return self.qfv
+
+    def decode(self, h, engine, states, nxt: bool):
+        out = hops.hgrn2_decode(engine.proj(h, self.qfv, True), self.lower, self.bias, self.norm, states[self.index]["state"],
+                                engine.pos, engine.active, self.vdim, self.eps,
+                                overlap=engine.then(engine.streams_weight(self.o)))
+        return engine.proj(out, self.o, nxt)
 
 
 # -------------------------------------------------------------------------------------------------------- feed-forward
@@ -261,20 +273,21 @@ class SwiGLU:
         self.gate_up = torch.cat([padded(get(n), self.ff_p, width_p) for n in ("gate", "up")]).to(device, dtype)
         self.down = padded(get("down"), width_p, self.ff_p).to(device, dtype)
 
-    def _act(self, gate_up):
+    def _act(self, gate_up, overlap: int = 0):
         if gate_up.dtype == torch.float32:
             return hops.swiglu_f32(gate_up, self.ff_p)
-        return ops.swiglu_fused(gate_up, self.ff_p)
+        return ops.swiglu_fused(gate_up, self.ff_p, overlap=overlap)
 
     def prefill(self, h, engine):
         return engine.linear(self._act(engine.linear(h, self.gate_up)), self.down)
 
-    def decode(self, h, engine):
+    def decode(self, h, engine, nxt: bool):
+        flags = engine.then(engine.streams_weight(self.down))
         if engine.streams_weight(self.gate_up, swiglu=True):
-            act = ops.skinny_gemm(h, self.gate_up, swiglu=True)
+            act = ops.skinny_gemm(h, self.gate_up, swiglu=True, overlap=flags)
         else:
-            act = self._act(F.linear(h, self.gate_up))
-        return engine.proj(act, self.down)
+            act = self._act(F.linear(h, self.gate_up), overlap=flags)
+        return engine.proj(act, self.down, nxt)
 
 
 MIXERS = {cls.kind: cls for cls in (LatentAttention, MinGRU, HGRN2)}

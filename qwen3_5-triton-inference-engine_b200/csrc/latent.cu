@@ -98,6 +98,68 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const __grid_constant_
   }
 }
 
+// Prompt-sized batches: one warp per row, eight rows per CTA, no block barrier; the same arithmetic.
+template <typename E, int V>
+__global__ void __launch_bounds__(256) latent_prep_rows_kernel(const __grid_constant__ LatentPrepParams p, int rows) {
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const E* x = static_cast<const E*>(p.fused) + row * p.stride;
+  const bool own = p.cache != nullptr;
+  const int nq = p.q_rank / 8, nk = nq + p.rank / 8, total = own ? nk + p.rot / 8 : nq;
+  const int slot = own && p.slot ? p.slot[row] : row;
+  const int64_t pos = !own ? 0 : p.pos_is_int64 ? static_cast<const int64_t*>(p.pos)[row]
+                                                : static_cast<int64_t>(static_cast<const int32_t*>(p.pos)[row]);
+  uint4 raw[V][sizeof(E) / 2];
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int i = lane + v * 32;
+    if (i < total) {
+#pragma unroll
+      for (int k = 0; k < static_cast<int>(sizeof(E) / 2); ++k) raw[v][k] = reinterpret_cast<const uint4*>(x + i * 8)[k];
+    }
+  }
+  const bool write = own && !(p.active && p.active[slot] == 0);
+  E* out = nullptr;
+  if (write) out = static_cast<E*>(p.cache) + (static_cast<int64_t>(p.table[slot * p.table_stride + pos / PAGE]) * PAGE + pos % PAGE) * (p.rank + p.rot);
+  auto unpack = [&](int v, float (&f)[8]) { load8(reinterpret_cast<const E*>(&raw[v][0]), f); };
+  float sq0 = 0.f, sq1 = 0.f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int i = lane + v * 32;
+    if (i < nk && i < total) {
+      float f[8], part = 0.f;
+      unpack(v, f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) part = fmaf(f[j], f[j], part);
+      if (i < nq) sq0 += part;
+      else sq1 += part;
+    }
+  }
+  const float qs = 1.0f / sqrtf(warp_sum(sq0) / static_cast<float>(p.true_q_rank) + p.eps);
+  const float ks = 1.0f / sqrtf(warp_sum(sq1) / static_cast<float>(p.true_rank) + p.eps);
+  E* cq = static_cast<E*>(p.cq) + static_cast<int64_t>(row) * p.q_rank;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int i = lane + v * 32;
+    if (i >= total || (i >= nq && !write)) continue;
+    float f[8], w[8];
+    unpack(v, f);
+    if (i < nk) {
+      const float s = i < nq ? qs : ks;
+      load8(i < nq ? p.q_weight + i * 8 : p.kv_weight + (i - nq) * 8, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] *= s * w[j];
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int pair = (i - nk) * 4 + j;
+        if (pair < p.rot_pairs) rotate_pair(f[2 * j], f[2 * j + 1], p.angles[pos * p.rot_pairs + pair]);
+      }
+    }
+    store8(i < nq ? cq + i * 8 : out + (i - nq) * 8, f);
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------- rotation
 // x [rows, heads, head_stride]: the pairs from offset `off` on, four per thread; the parts are padded to multiples of 8
 template <typename E>
@@ -458,6 +520,14 @@ extern "C" int b200_latent_prep(const void* fused, int64_t stride, const float* 
   B200_REQUIRE(vecs <= 1024, "latent_prep: at most 8192 elements per row (got %d)", vecs * 8);
   const dim3 block(((vecs + v - 1) / v + 31) / 32 * 32);
   cudaError_t e;
+  if (!f32 && rows >= GLUE_WIDE_ROWS && vecs <= 256) {
+    const unsigned grid = (rows + 7) / 8;
+    if (vecs <= 64) latent_prep_rows_kernel<__nv_bfloat16, 2><<<grid, 256, 0, st>>>(p, rows);
+    else if (vecs <= 128) latent_prep_rows_kernel<__nv_bfloat16, 4><<<grid, 256, 0, st>>>(p, rows);
+    else if (vecs <= 192) latent_prep_rows_kernel<__nv_bfloat16, 6><<<grid, 256, 0, st>>>(p, rows);
+    else latent_prep_rows_kernel<__nv_bfloat16, 8><<<grid, 256, 0, st>>>(p, rows);
+    return check_launch("latent_prep");
+  }
   if (f32) {
     e = v == 1 ? launch_pdl(early, latent_prep_kernel<float, 1>, dim3(rows), block, 0, st, p)
         : v == 2 ? launch_pdl(early, latent_prep_kernel<float, 2>, dim3(rows), block, 0, st, p)

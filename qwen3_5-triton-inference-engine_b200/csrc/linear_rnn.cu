@@ -61,7 +61,7 @@ __global__ void __launch_bounds__(128) mingru_scan_kernel(const __grid_constant_
       s0 = s.x;
       s1 = s.y;
     }
-#pragma unroll 4
+#pragma unroll 8
     for (int i = 0; i < chunk; ++i) {
       const float4 ab = *reinterpret_cast<const float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(i) * p.width);
       s0 = fmaf(ab.x, s0, ab.y);
@@ -546,18 +546,26 @@ extern "C" int b200_mingru_decode(const void* zxg, int64_t stride, const float* 
   return check_launch("mingru_decode");
 }
 
+extern "C" int64_t b200_hgrn2_workspace_bytes(int32_t batch, int32_t segments, int32_t heads, int32_t dim, int32_t vdim) {
+  return static_cast<int64_t>(batch) * segments * heads * dim * (vdim + 1) * 4;
+}
+
 extern "C" int b200_hgrn2_prefill(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm,
                                   float* state, const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start,
                                   float* o_scratch, void* out, int32_t batch, int32_t tokens, int32_t heads, int32_t dim,
                                   int32_t vdim, int32_t true_vdim, float eps, int32_t f32, int32_t serial,
-                                  b200_stream_t stream) {
+                                  int32_t segment, int32_t segments, float* workspace, b200_stream_t stream) {
   if (batch <= 0 || tokens <= 0) return OK;
+  B200_REQUIRE(segment > 0 && segments > 0 && (segments == 1 || (segment % 16 == 0 && workspace && aligned16(workspace))),
+               "hgrn2_prefill: segments must be multiples of 16 tokens and have a workspace");
+  B200_REQUIRE(static_cast<int64_t>(batch) * segments <= 65535, "hgrn2_prefill: too many segments");
   B200_REQUIRE(dim > 0 && dim <= 256 && vdim > 0 && vdim % 4 == 0 && vdim <= OD_MAX_VDIM && true_vdim <= vdim,
                "hgrn2_prefill: dim at most 256, vdim a multiple of 4 and at most %d (got %d, %d)", OD_MAX_VDIM, dim, vdim);
   B200_REQUIRE(heads > 0 && heads <= 65535 && batch <= 65535, "hgrn2_prefill: at most 65535 heads and sequences");
   B200_REQUIRE(aligned16(o_scratch) && aligned16(out) && aligned16(norm), "hgrn2_prefill: unaligned tensor");
   OuterRnnParams p = {qfv, stride, lower, bias, state, cu_seqlens, slots, start, o_scratch, heads, dim, vdim,
-                      norm, nullptr, true_vdim, eps};
+                      norm, nullptr, true_vdim, eps, segment, segments, workspace,
+                      workspace ? workspace + static_cast<int64_t>(batch) * segments * heads * dim * vdim : nullptr};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const bool chunked = !f32 && !serial && outer_rnn_chunk_supports(dim, vdim) && stride % 8 == 0 && heads * dim % 8 == 0 && aligned16(qfv);
   if (chunked && vdim <= 128) {  // the head norm inside: one launch

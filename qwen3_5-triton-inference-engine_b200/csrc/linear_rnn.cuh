@@ -21,6 +21,10 @@ struct OuterRnnParams {
   void* out;
   int true_vdim;
   float eps;
+  // chunked form over segments of `segment` tokens (a multiple of 16), at most `segments` per sequence (1: none)
+  int segment, segments;
+  float* seg_state;        // [sequences, segments, heads, dim, vdim]
+  float* seg_decay;        // [sequences, segments, heads, dim]
 };
 
 bool outer_rnn_chunk_supports(int dim, int vdim);

@@ -172,6 +172,27 @@ def test_hgrn2_prefill(hops, form, heads, dim, vdim):
     assert torch.equal(state[3].cpu(), before[3])
 
 
+@pytest.mark.parametrize("heads,dim,vdim", [(2, 128, 128), (1, 48, 144), (3, 32, 48)])
+@pytest.mark.parametrize("segments", [None, (16, 40), (64, 10), (320, 2)])
+def test_hgrn2_segments(hops, heads, dim, vdim, segments):
+    """Sequences cut into segments that run side by side: unequal lengths (some with a single segment), carried states,
+    gates that never forget across segments."""
+    lengths, slots, starts, eps = [600, 16, 33, 320, 1], [2, 0, 4, 5, 1], [0, 3, 0, 16, 9], 1e-5
+    qfv, lower, bias, norm = _hgrn2_inputs(sum(lengths), heads, dim, vdim, torch.bfloat16, 41)
+    before = rnd(6, heads, dim, vdim, seed=42)
+    state = before.to(DEV)
+    out = hops.hgrn2_prefill(*[t.to(DEV) for t in (qfv, lower, bias, norm)], state, Batch(slots, starts, lengths), vdim, eps,
+                             segments=segments)
+    row = 0
+    for slot, start, n in zip(slots, starts, lengths):
+        want, last = _hgrn2_want(qfv[row: row + n], lower, bias, norm, heads, dim, vdim,
+                                 before[slot] if start else torch.zeros(heads, dim, vdim), eps, vdim)
+        close(out[row: row + n], want, torch.bfloat16, f"length {n}", 2.0)
+        close(state[slot], last, torch.float32, f"state after {n}", 8.0)
+        row += n
+    assert torch.equal(state[3].cpu(), before[3])
+
+
 @pytest.mark.parametrize("serial", [False, True])
 def test_hgrn2_wide_batch(hops, serial):
     """A batch of many heads (the wide-column form of the token-serial kernel among them)."""
@@ -221,12 +242,14 @@ def test_rope_interleaved(hops):
     close(got, want, torch.float32)
 
 
+@pytest.mark.parametrize("repeat,q_rank", [(1, 128), (1, 2944), (200, 128), (200, 640), (200, 1152), (200, 1792)])
 @pytest.mark.parametrize("dt", DT)
-def test_latent_prep_writes_pages(hops, dt):
+def test_latent_prep_writes_pages(hops, dt, repeat, q_rank):
+    """A few rows and prompt-sized batches (the same six rows over and over), narrow and wide query latents."""
     from b200attn.mixers import Rotation
     dtype, eps = DT[dt], 1e-5
     rot = {"base": 300.0, "dims": 24}
-    q_rank, true_q, rank, true_rank, rotw = 128, 88, 64, 40, 64
+    true_q, rank, true_rank, rotw = q_rank - 40, 64, 40, 64
     pos = torch.tensor([0, 15, 16, 31, 47, 5], dtype=torch.int32)
     slot = torch.tensor([1, 1, 1, 0, 0, 2], dtype=torch.int32)
     fused = rnd(6, q_rank + rank + rotw, seed=1, dtype=dtype)
@@ -238,8 +261,10 @@ def test_latent_prep_writes_pages(hops, dt):
     cache = torch.full((9, 16, rank + rotw), 5.0, dtype=dtype, device=DEV)
     active = torch.tensor([1, 1, 0], device=DEV)
     angles = Rotation.from_config(rot).table(64, DEV)
-    cq = hops.latent_prep(fused.to(DEV), qw.to(DEV), kw.to(DEV), pos.to(DEV), slot.to(DEV), active, table, angles, cache, true_q, rank,
-                          true_rank, eps)
+    cq = hops.latent_prep(fused.repeat(repeat, 1).to(DEV), qw.to(DEV), kw.to(DEV), pos.repeat(repeat).to(DEV),
+                          slot.repeat(repeat).to(DEV), active, table, angles, cache, true_q, rank, true_rank, eps)
+    assert torch.equal(cq[:6].repeat(repeat, 1), cq)
+    cq = cq[:6]
     f = fused.double()
     close(cq[:, :true_q], R.rms(f[:, :true_q], eps) * qw[:true_q].double(), dtype)
     want = torch.full((9, 16, rank + rotw), 5.0, dtype=torch.float64)

@@ -108,9 +108,14 @@ def test_padding_keeps_heads_apart():
 def test_chunking_and_splits():
     from b200attn import hybrid_ops as hops
 
-    for n in (1, 2, 63, 64, 65, 4096, 4097, 100000):
-        chunk, chunks = hops.mingru_chunking(n)
-        assert chunk >= 64 and chunks <= 64 and (chunks - 1) * chunk < n <= chunks * chunk
+    for n in (1, 2, 63, 64, 65, 2048, 4096, 4097, 100000):
+        for count, width in ((1, 64), (1, 2048), (32, 2048), (64, 4096)):
+            chunk, chunks = hops.mingru_chunking(n, count, width)
+            assert chunks <= 128 and (chunks - 1) * chunk < n <= chunks * chunk
+        for groups in (1, 16, 32, 500):
+            seg, segs = hops.hgrn2_segments(n, groups, 148)
+            assert (segs - 1) * seg < n <= segs * seg and (segs == 1 or (seg % 16 == 0 and seg >= 128))
+            assert segs == 1 or segs * groups <= 2 * 148
     for batch, heads, span in [(1, 1, 16), (1, 16, 4096), (32, 16, 4096), (256, 128, 512), (1, 1, 1)]:
         s = hops.latent_decode_splits(batch, heads, span, 148)
         assert 1 <= s <= hops.LATENT_MAX_SPLITS and (s == 1 or span // s >= 16)
