@@ -458,11 +458,12 @@ int b200_swiglu_f32(const float* gate_up, int64_t row_stride, float* out, int32_
 
 /* minGRU: zxg = rows of [z | x | g] projections, each `width` wide; bias fp32 [2*width] (z, x); state fp32 [slots, width];
  *   z = sigmoid(z + zb), u = x + xb, c = u >= 0 ? u + 1/2 : sigmoid(u), S <- (1-z) S + z c, out = S * silu(g).
- * Prefill cuts sequences into `chunks` chunks of `chunk` tokens; workspace of b200_mingru_workspace_bytes(). */
-int64_t b200_mingru_workspace_bytes(int32_t batch, int32_t chunks, int32_t width);
+ * Prefill may cut sequences into at most `segments` segments of `segment` tokens that run side by side (1: none, segment
+ * >= the longest sequence); more than one take a workspace of b200_mingru_workspace_bytes(). */
+int64_t b200_mingru_workspace_bytes(int32_t batch, int32_t segments, int32_t width);
 int b200_mingru_prefill(const void* zxg, int64_t stride, const float* bias, float* state, const int32_t* cu_seqlens,
-                        const int32_t* slots, const int32_t* start, void* workspace, void* out, int32_t batch, int32_t chunk,
-                        int32_t chunks, int32_t width, int32_t f32, b200_stream_t stream);
+                        const int32_t* slots, const int32_t* start, void* workspace, void* out, int32_t batch, int32_t segment,
+                        int32_t segments, int32_t width, int32_t f32, b200_stream_t stream);
 int b200_mingru_decode(const void* zxg, int64_t stride, const float* bias, float* state, const int64_t* pos,
                        const int64_t* active, void* out, int32_t batch, int32_t width, int32_t f32, int32_t overlap,
                        b200_stream_t stream);

@@ -44,31 +44,45 @@ def swiglu_f32(gate_up, intermediate: int):
 
 
 # ------------------------------------------------------------------------------------------------------------- minGRU
-MINGRU_THREADS = 65536           # threads (two channels each) that keep the memory system busy
+MINGRU_BLOCK, MINGRU_COLS = 128, 64
 
 
-def mingru_chunking(max_len: int, count: int, width: int) -> tuple[int, int]:
-    """(chunk length, chunks of the longest sequence).  A batch wide enough runs each sequence in one pass; otherwise chunks
-    short enough to fill the device twice over, at least 16 tokens long and at most 128 of them."""
-    threads = count * width // 2
-    if threads >= MINGRU_THREADS:
+def sm_count(device) -> int:
+    key = torch.device(device).index or 0
+    if key not in _sm_counts:
+        _sm_counts[key] = torch.cuda.get_device_properties(device).multi_processor_count
+    return _sm_counts[key]
+
+
+_sm_counts: dict = {}
+
+
+def mingru_segments(max_len: int, groups: int, sm_count: int) -> tuple[int, int]:
+    """(segment length, segments of the longest sequence).  `groups` CTAs walk whole sequences in blocks of 128 tokens; when
+    they do not fill the device (two per SM), sequences are cut into runs of whole blocks, at the price of a second pass."""
+    blocks = -(-max_len // MINGRU_BLOCK)
+    parts = min(-(-2 * sm_count // groups), blocks, 64)
+    if parts < 2:
         return max_len, 1
-    chunk = max(16, -(-max_len * threads // (2 * MINGRU_THREADS)), -(-max_len // 128))
-    return chunk, -(-max_len // chunk)
+    per = -(-blocks // parts)
+    return per * MINGRU_BLOCK, -(-blocks // per)
 
 
-def mingru_prefill(zxg, bias, state, batch):
-    """zxg [tokens, 3*width] projections of a packed batch (`batch`: PackedBatch); state [slots, width] fp32, in place."""
+def mingru_prefill(zxg, bias, state, batch, segments=None):
+    """zxg [tokens, 3*width] projections of a packed batch (`batch`: PackedBatch); state [slots, width] fp32, in place.
+    segments: (length, count) to pin how sequences are cut."""
     width = state.shape[1]
     assert zxg.shape[1] == 3 * width and zxg.stride(1) == 1 and bias.numel() == 2 * width
     assert state.dtype == bias.dtype == torch.float32 and state.is_contiguous() and bias.is_contiguous()
     _require_cuda(zxg, bias, state)
-    chunk, chunks = mingru_chunking(batch.max_len, batch.count, width)
     n = batch.count
-    ws = torch.empty(_lib.load().b200_mingru_workspace_bytes(n, chunks, width), dtype=torch.uint8, device=zxg.device)
+    segment, count = segments or mingru_segments(batch.max_len, n * -(-width // MINGRU_COLS), sm_count(zxg.device))
+    ws = None
+    if count > 1:
+        ws = torch.empty(_lib.load().b200_mingru_workspace_bytes(n, count, width), dtype=torch.uint8, device=zxg.device)
     out = torch.empty((zxg.shape[0], width), dtype=zxg.dtype, device=zxg.device)
     _lib.call("b200_mingru_prefill", _ptr(zxg), zxg.stride(0), _ptr(bias), _ptr(state), _ptr(batch.cu), _ptr(batch.slots),
-              _ptr(batch.start), _ptr(ws), _ptr(out), n, chunk, chunks, width, _f32(zxg), _stream())
+              _ptr(batch.start), _ptr(ws), _ptr(out), n, segment, count, width, _f32(zxg), _stream())
     return out
 
 
@@ -102,16 +116,6 @@ def hgrn2_segments(max_len: int, groups: int, sm_count: int) -> tuple[int, int]:
         return max_len, 1
     segment = -(-max_len // parts // 16) * 16 + (0 if max_len % parts == 0 and (max_len // parts) % 16 == 0 else 16)
     return segment, -(-max_len // segment)
-
-
-_sm_counts: dict = {}
-
-
-def sm_count(device) -> int:
-    key = torch.device(device).index or 0
-    if key not in _sm_counts:
-        _sm_counts[key] = torch.cuda.get_device_properties(device).multi_processor_count
-    return _sm_counts[key]
 
 
 def hgrn2_prefill(qfv, lower, bias, norm, state, batch, true_vdim: int, eps: float, serial: bool = False, segments=None):

@@ -37,6 +37,12 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
   *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
 }
 
+__device__ __forceinline__ float rcp_fast(float x) {  // 1 / x, one hardware instruction (about an ulp; 1 / inf = 0)
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // Logistic function in fp32: exact library exponential and division for fp32 activations, the hardware exponential and
 // reciprocal (a few fp32 ulp) next to bf16 ones.
 template <typename E>
@@ -44,7 +50,7 @@ __device__ __forceinline__ float sigmoid_f(float x);
 template <>
 __device__ __forceinline__ float sigmoid_f<float>(float x) { return 1.0f / (1.0f + expf(-x)); }
 template <>
-__device__ __forceinline__ float sigmoid_f<__nv_bfloat16>(float x) { return __fdividef(1.0f, 1.0f + __expf(-x)); }
+__device__ __forceinline__ float sigmoid_f<__nv_bfloat16>(float x) { return rcp_fast(1.0f + ex2_fast(-1.4426950408889634f * x)); }
 template <typename E>
 __device__ __forceinline__ float silu_f(float x) { return x * sigmoid_f<E>(x); }
 

@@ -4,8 +4,8 @@
 // One CTA = (key range of a slot, block of 16 heads).  A producer warp brings 32-token tiles (two 16-token pages, one
 // tensor-map TMA box each, 128-byte swizzle, no multicast) through a ring of mbarrier-tracked stages; eight warps work on
 // a tile together:
-//     S[16 x 32]    = q' . rows^T     a warp takes 8 tokens and every other 32-wide step of the row (two warps per group)
-//     P             = exp2(S - m)     a warp owns two head rows, a lane one token; online maximum and sum in fp32
+//     S[16 x 32]    = q' . rows^T     a warp takes 16 tokens and every fourth 32-wide step of the row
+//     P             = exp2(S - m)     half a warp per head row, two tokens per lane; online maximum and sum in fp32
 //     O[16 x rank] += P . latents     a warp owns rank / 8 columns; accumulators stay in registers
 // The kernel is bound by HBM (about 2 * 16 FLOP per byte), far below what 16-row tiles reach on tcgen05 (M = 128), so
 // mma.sync carries the products, as in the paged decode kernels.  Key ranges leave (max, sum, unnormalised O) in fp32;
@@ -24,8 +24,8 @@ constexpr int LD_TOK = 32;
 constexpr int LD_MAX_STAGES = 6;
 constexpr int LD_S_PITCH = 36;                   // floats per score row
 constexpr int LD_P_PITCH = 40;                   // bf16 per probability row (80 bytes: ldmatrix rows in different banks)
-constexpr int LD_SMEM_LIMIT = 216 * 1024;         // dynamic; 6 KiB more are static
-constexpr int LD_SMEM_PAIR = 105 * 1024;          // ... when two CTAs share an SM
+constexpr int LD_SMEM_LIMIT = 216 * 1024;         // dynamic; 11 KiB more are static
+constexpr int LD_SMEM_PAIR = 102 * 1024;          // ... when two CTAs share an SM
 
 // NT: value columns per warp / 8 that the accumulators hold (rank <= 64 * NT)
 template <int NT>
@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(LD_THREADS, NT <= 8 ? 2 : 1)
 latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_constant__ CUtensorMap map_rows, int stages) {
   extern __shared__ __align__(1024) uint8_t ld_smem_raw[];
   __shared__ uint64_t full[LD_MAX_STAGES], empty[LD_MAX_STAGES];
-  __shared__ float ss[2][16][LD_S_PITCH];
+  __shared__ float ss[4][16][LD_S_PITCH];            // partial scores of the four quarters of a row
   __shared__ __align__(16) __nv_bfloat16 ps[16][LD_P_PITCH];
   __shared__ float alphas[16];
   const int split = blockIdx.x, hb = blockIdx.y, b = blockIdx.z;
@@ -96,12 +96,12 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
   float m_run = -INFINITY, l_run = 0.f;   // of head row sm_row: the maximum, and this lane's part of the sum
   const int sm_row = warp * 2 + (lane >> 4), sm_tok = (lane & 15) * 2;
   const float scale_log2 = p.scale * 1.4426950408889634f;
-  const int tg = warp & 3, kh = warp >> 2;
+  const int tg = warp & 1, kq = warp >> 1;
   const int units = pitch / 32;
   const int nt = p.rank / 64, col0 = warp * nt * 8;
   const uint32_t a_base = smem_u32(qs) + (lane & 15) * q_pitch + (lane >> 4) * 16;
-  const int s_row = (tg & 1) * 8 + (lane & 7);
-  const uint32_t s_off = (tg >> 1) * page_bytes + s_row * 128;
+  const int s_row = lane & 7;   // rows s_row and s_row + 8 of page tg
+  const uint32_t s_off = tg * page_bytes + s_row * 128;
   bool ok = true;
   for (int t = 0; t < tiles; ++t) {
     const int s = t % stages;
@@ -120,28 +120,40 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
     }
     // ---- scores
     if (ok) {
-      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+      float c[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll 3
-      for (int u = kh; u < units; u += 2) {
-        uint32_t a0[4], a1[4], bm[4];
+      for (int u = kq; u < units; u += 4) {
+        uint32_t a0[4], a1[4], b0[4], b1[4];
         const int chunk = u * 4 + (lane >> 3);
-        ldmatrix_x4(bm, tile_a + s_off + (chunk >> 3) * (PAGE * 128) + (((chunk & 7) ^ (s_row & 7)) << 4));
+        const uint32_t at = tile_a + s_off + (chunk >> 3) * (PAGE * 128) + (((chunk & 7) ^ s_row) << 4);
         ldmatrix_x4(a0, a_base + u * 64);
+        ldmatrix_x4(b0, at);
+        ldmatrix_x4(b1, at + 8 * 128);
         ldmatrix_x4(a1, a_base + u * 64 + 32);
-        mma_bf16_16816(c0, a0, bm[0], bm[1]);
-        mma_bf16_16816(c1, a1, bm[2], bm[3]);
+        mma_bf16_16816(c[0], a0, b0[0], b0[1]);
+        mma_bf16_16816(c[1], a0, b1[0], b1[1]);
+        mma_bf16_16816(c[0], a1, b0[2], b0[3]);
+        mma_bf16_16816(c[1], a1, b1[2], b1[3]);
       }
-      const int col = tg * 8 + (lane & 3) * 2, r = lane >> 2;
-      *reinterpret_cast<float2*>(&ss[kh][r][col]) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
-      *reinterpret_cast<float2*>(&ss[kh][r + 8][col]) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int col = tg * 16 + i * 8 + (lane & 3) * 2, r = lane >> 2;
+        *reinterpret_cast<float2*>(&ss[kq][r][col]) = make_float2(c[i][0], c[i][1]);
+        *reinterpret_cast<float2*>(&ss[kq][r + 8][col]) = make_float2(c[i][2], c[i][3]);
+      }
     }
     named_barrier(1, LD_WARPS * 32);
     // ---- softmax: half a warp per head row, two tokens per lane
     {
-      const float2 a = *reinterpret_cast<const float2*>(&ss[0][sm_row][sm_tok]), c = *reinterpret_cast<const float2*>(&ss[1][sm_row][sm_tok]);
+      float2 a = make_float2(0.f, 0.f);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 part = *reinterpret_cast<const float2*>(&ss[k][sm_row][sm_tok]);
+        a.x += part.x, a.y += part.y;
+      }
       const int at = tok0 + sm_tok;
-      const float x0 = at >= lo && at < hi ? (a.x + c.x) * scale_log2 : -INFINITY;
-      const float x1 = at + 1 >= lo && at + 1 < hi ? (a.y + c.y) * scale_log2 : -INFINITY;
+      const float x0 = at >= lo && at < hi ? a.x * scale_log2 : -INFINITY;
+      const float x1 = at + 1 >= lo && at + 1 < hi ? a.y * scale_log2 : -INFINITY;
       float mx = fmaxf(x0, x1);
 #pragma unroll
       for (int bit = 8; bit >= 1; bit >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, bit));

@@ -4,8 +4,9 @@
 //
 //   minGRU (element-wise):  z = sigmoid(z' + zb), u = x' + xb, c = u >= 0 ? u + 1/2 : sigmoid(u)
 //                           S_t = (1 - z) S_(t-1) + z c,   out = S_t * silu(g)
-//     Prefill cuts every sequence into chunks: pass 1 reduces a chunk to (product of 1 - z, state it leaves from zero),
-//     pass 2 folds the chunks in front of its own and replays its chunk.  HBM bound; both passes stream 16-byte rows.
+//     Prefill: a CTA walks a sequence in blocks of 128 tokens, its warps scan 16 tokens each in parallel.  Too few CTAs:
+//     sequences are cut into segments; pass 1 reduces a segment to (product of 1 - z, state it leaves from zero), pass 2
+//     folds the segments in front of its own.  HBM bound.
 //   Forget-gated outer-product recurrence (HGRN2 form):  f = l + (1 - l) sigmoid(f' + fb), q = silu(q')
 //                           S_t = diag(f) S_(t-1) + (1 - f) v^T,   o = S_t^T q,   out = rms(o) * w per head
 //     Prefill of bf16 activations runs in chunks on the tensor cores (linear_rnn_chunk.cu).  The token-serial form here is
@@ -27,9 +28,10 @@ struct MinGruParams {
   const int32_t* cu;        // [n + 1] packed rows of the sequences
   const int32_t* slots;     // [n]
   const int32_t* start;     // [n] position of each sequence's first packed token
-  float2* chunk_ab;         // [n, chunks, width] workspace of pass 1
+  float2* ab;               // [n, segments + 1, width]: (product of 1 - z, state from zero) per segment; the last entry
+                            // keeps the sequence's initial state
   void* out;                // [rows, width] E
-  int width, chunk, chunks;
+  int width, segment, segments;
 };
 
 template <typename E>
@@ -41,96 +43,103 @@ __device__ __forceinline__ void mingru_gate(float z_raw, float u, float zb, floa
   add = z * cand;
 }
 
-// grid (width / (128 * 2), chunks, sequences); thread = 2 channels
-template <typename E, bool REPLAY>
-__global__ void __launch_bounds__(128) mingru_scan_kernel(const __grid_constant__ MinGruParams p) {
-  const int seq = blockIdx.z, chunk = blockIdx.y;
-  const int c = (blockIdx.x * 128 + threadIdx.x) * 2;
-  const int row0 = p.cu[seq], len = p.cu[seq + 1] - row0;
-  const int t0 = chunk * p.chunk, t1 = min(t0 + p.chunk, len);
-  if (t0 >= len || c >= p.width) return;
-  if (!REPLAY && t1 == len) return;  // nobody folds the last chunk
-  const float2 zb = *reinterpret_cast<const float2*>(p.bias + c), xb = *reinterpret_cast<const float2*>(p.bias + p.width + c);
-  float s0 = 0.f, s1 = 0.f, a0 = 1.f, a1 = 1.f;
-  float* state = p.state + static_cast<int64_t>(p.slots[seq]) * p.width + c;
-  const int64_t ab_base = static_cast<int64_t>(seq) * p.chunks * p.width + c;
-  if (REPLAY) {
-    if (p.start[seq] > 0) {
-      // (unchanged during this launch: the commit kernel behind it writes the slot)
-      const float2 s = *reinterpret_cast<const float2*>(state);
-      s0 = s.x;
-      s1 = s.y;
-    }
+__device__ __forceinline__ float2 load2(const __nv_bfloat16* q) {
+  const uint32_t v = *reinterpret_cast<const uint32_t*>(q);
+  return make_float2(bf16_lo(v), bf16_hi(v));
+}
+__device__ __forceinline__ float2 load2(const float* q) { return *reinterpret_cast<const float2*>(q); }
+
+constexpr int MG_WARPS = 8, MG_RUN = 16;            // a warp's run of consecutive tokens
+constexpr int MG_BLOCK = MG_WARPS * MG_RUN;         // tokens a CTA takes at a time
+constexpr int MG_COLS = 64;                         // channels of a CTA, two per lane
+
+// A CTA walks its segment in blocks of 128 tokens.  Every warp turns 16 of them into (keep, add) pairs in registers, leaves
+// their product and sum in shared memory, folds the runs in front of its own and replays its run: inputs are read once.
+// grid (width / 64, segments, sequences).  REDUCE: only the segment's (product, state from zero).
+template <typename E, bool REDUCE>
+__global__ void __launch_bounds__(MG_WARPS * 32) mingru_prefill_kernel(const __grid_constant__ MinGruParams p) {
+  __shared__ float4 runs[2][MG_WARPS][32];
+  const int seq = blockIdx.z, seg = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c = blockIdx.x * MG_COLS + lane * 2;
+  const int row0 = p.cu[seq], all = p.cu[seq + 1] - row0;
+  const int s0 = seg * p.segment, s1 = min(s0 + p.segment, all);
+  const bool last = s1 == all;
+  if (s0 >= all || (REDUCE && last)) return;        // nobody folds a last segment
+  const bool on = c < p.width;
+  const int cc = on ? c : 0;
+  const float2 zb = load2(p.bias + cc), xb = load2(p.bias + p.width + cc);
+  float* state = p.state + static_cast<int64_t>(p.slots[seq]) * p.width + cc;
+  float2* ab = p.ab + static_cast<int64_t>(seq) * (p.segments + 1) * p.width + cc;
+  float2 carry = make_float2(0.f, 0.f);
+  if (REDUCE || (s0 == 0 && last)) {
+    if (!(REDUCE && s0 > 0) && p.start[seq] > 0) carry = load2(state);
+    if (REDUCE && s0 == 0 && warp == 0 && on) *reinterpret_cast<float4*>(ab + static_cast<int64_t>(p.segments) * p.width) = make_float4(carry.x, 0.f, carry.y, 0.f);
+    if (REDUCE) carry = make_float2(0.f, 0.f);
+  } else {
+    const float4 init = *reinterpret_cast<const float4*>(ab + static_cast<int64_t>(p.segments) * p.width);
+    carry = make_float2(init.x, init.z);
 #pragma unroll 8
-    for (int i = 0; i < chunk; ++i) {
-      const float4 ab = *reinterpret_cast<const float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(i) * p.width);
-      s0 = fmaf(ab.x, s0, ab.y);
-      s1 = fmaf(ab.z, s1, ab.w);
+    for (int i = 0; i < seg; ++i) {
+      const float4 x = *reinterpret_cast<const float4*>(ab + static_cast<int64_t>(i) * p.width);
+      carry.x = fmaf(x.x, carry.x, x.y);
+      carry.y = fmaf(x.z, carry.y, x.w);
     }
   }
-  const E* base = static_cast<const E*>(p.zxg) + static_cast<int64_t>(row0) * p.stride + c;
-  auto two = [](const E* q) {
-    if constexpr (sizeof(E) == 2) {
-      const uint32_t v = *reinterpret_cast<const uint32_t*>(q);
-      return make_float2(bf16_lo(v), bf16_hi(v));
-    } else {
-      return *reinterpret_cast<const float2*>(q);
-    }
-  };
-  constexpr int U = 8;  // rows per group; the next group's loads are in flight while one is worked on
-  float2 z[2][U], x[2][U], g[2][U];
-  auto fetch = [&](int buf, int t) {
+  float2 product = make_float2(1.f, 1.f);
+  const E* base = static_cast<const E*>(p.zxg) + static_cast<int64_t>(row0) * p.stride + cc;
+  for (int tb = s0, buf = 0; tb < s1; tb += MG_BLOCK, buf ^= 1) {
+    const int t0 = tb + warp * MG_RUN;
+    float2 keep[MG_RUN], add[MG_RUN], g[MG_RUN];
+    const E *rz = base + static_cast<int64_t>(t0) * p.stride, *rx = rz + p.width, *rg = rx + p.width;
+    const int stride = static_cast<int>(p.stride), lim = s1 - 1 - t0;
 #pragma unroll
-    for (int i = 0; i < U; ++i) {
-      const E* r = base + static_cast<int64_t>(min(t + i, t1 - 1)) * p.stride;  // past the end: a row read again
-      z[buf][i] = two(r);
-      x[buf][i] = two(r + p.width);
-      if (REPLAY) g[buf][i] = two(r + 2 * p.width);
+    for (int i = 0; i < MG_RUN; ++i) {
+      const int off = min(i, lim) * stride;  // past the end: a row read again
+      keep[i] = load2(rz + off);
+      add[i] = load2(rx + off);
+      if (!REDUCE) g[i] = load2(rg + off);
     }
-  };
-  auto work = [&](int buf, int t) {
+    float4 run = make_float4(1.f, 0.f, 1.f, 0.f);
 #pragma unroll
-    for (int i = 0; i < U; ++i) {
-      float k0, k1, b0, b1;
-      mingru_gate<E>(z[buf][i].x, x[buf][i].x, zb.x, xb.x, k0, b0);
-      mingru_gate<E>(z[buf][i].y, x[buf][i].y, zb.y, xb.y, k1, b1);
-      if (t + i < t1) {
-        s0 = fmaf(k0, s0, b0);
-        s1 = fmaf(k1, s1, b1);
-        if (REPLAY) {
-          E* o = static_cast<E*>(p.out) + static_cast<int64_t>(row0 + t + i) * p.width + c;
-          const float o0 = s0 * silu_f<E>(g[buf][i].x), o1 = s1 * silu_f<E>(g[buf][i].y);
+    for (int i = 0; i < MG_RUN; ++i) {
+      float k0, b0, k1, b1;
+      mingru_gate<E>(keep[i].x, add[i].x, zb.x, xb.x, k0, b0);
+      mingru_gate<E>(keep[i].y, add[i].y, zb.y, xb.y, k1, b1);
+      const bool in = i <= lim;
+      keep[i] = in ? make_float2(k0, k1) : make_float2(1.f, 1.f);
+      add[i] = in ? make_float2(b0, b1) : make_float2(0.f, 0.f);
+      run.x *= keep[i].x, run.y = fmaf(keep[i].x, run.y, add[i].x);
+      run.z *= keep[i].y, run.w = fmaf(keep[i].y, run.w, add[i].y);
+    }
+    runs[buf][warp][lane] = run;
+    __syncthreads();  // two buffers: the next block's runs go to the other one
+    float2 s = carry;
+#pragma unroll
+    for (int w = 0; w < MG_WARPS; ++w) {
+      if (w == warp) s = carry;
+      const float4 x = runs[buf][w][lane];
+      carry.x = fmaf(x.x, carry.x, x.y);
+      carry.y = fmaf(x.z, carry.y, x.w);
+      if (REDUCE) product = make_float2(product.x * x.x, product.y * x.z);
+    }
+    if (!REDUCE && on) {
+      E* const out = static_cast<E*>(p.out) + static_cast<int64_t>(row0 + t0) * p.width + c;
+#pragma unroll
+      for (int i = 0; i < MG_RUN; ++i) {
+        s.x = fmaf(keep[i].x, s.x, add[i].x);
+        s.y = fmaf(keep[i].y, s.y, add[i].y);
+        if (i <= lim) {
+          E* o = out + i * p.width;
+          const float o0 = s.x * silu_f<E>(g[i].x), o1 = s.y * silu_f<E>(g[i].y);
           if constexpr (sizeof(E) == 2) *reinterpret_cast<uint32_t*>(o) = pack_bf16(o0, o1);
           else *reinterpret_cast<float2*>(o) = make_float2(o0, o1);
-        } else {
-          a0 *= k0;
-          a1 *= k1;
         }
       }
     }
-  };
-  fetch(0, t0);
-  for (int t = t0; t < t1; t += 2 * U) {
-    if (t + U < t1) fetch(1, t + U);
-    work(0, t);
-    if (t + U < t1) {
-      if (t + 2 * U < t1) fetch(0, t + 2 * U);
-      work(1, t + U);
-    }
   }
-  if (!REPLAY) *reinterpret_cast<float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(chunk) * p.width) = make_float4(a0, s0, a1, s1);
-  else if (t1 == len) {
-    // final state into the workspace's last chunk slot; a copy kernel behind this one moves it to the slot, so that no
-    // chunk of this launch can see it
-    *reinterpret_cast<float4*>(p.chunk_ab + ab_base + static_cast<int64_t>(p.chunks - 1) * p.width) = make_float4(s0, 0.f, s1, 0.f);
-  }
-}
-
-__global__ void __launch_bounds__(256) mingru_commit_kernel(const __grid_constant__ MinGruParams p) {
-  const int seq = blockIdx.y, c = blockIdx.x * 256 + threadIdx.x;
-  if (c >= p.width || p.cu[seq + 1] == p.cu[seq]) return;
-  p.state[static_cast<int64_t>(p.slots[seq]) * p.width + c] =
-      p.chunk_ab[(static_cast<int64_t>(seq) * p.chunks + p.chunks - 1) * p.width + c].x;
+  if (warp != 0 || !on) return;
+  if (REDUCE) *reinterpret_cast<float4*>(ab + static_cast<int64_t>(seg) * p.width) = make_float4(product.x, carry.x, product.y, carry.y);
+  else if (last) *reinterpret_cast<float2*>(state) = carry;  // with several segments nobody else reads the slot in this launch
 }
 
 // one token per slot; thread = 4 channels
@@ -501,29 +510,28 @@ static int launch_outer_rows(const OuterRnnParams& p, int n, cudaStream_t st) {
 
 using namespace b200;
 
-extern "C" int64_t b200_mingru_workspace_bytes(int32_t batch, int32_t chunks, int32_t width) {
-  return static_cast<int64_t>(batch) * chunks * width * 8;
+extern "C" int64_t b200_mingru_workspace_bytes(int32_t batch, int32_t segments, int32_t width) {
+  return segments > 1 ? static_cast<int64_t>(batch) * (segments + 1) * width * 8 : 0;
 }
 
 extern "C" int b200_mingru_prefill(const void* zxg, int64_t stride, const float* bias, float* state, const int32_t* cu_seqlens,
                                    const int32_t* slots, const int32_t* start, void* workspace, void* out, int32_t batch,
-                                   int32_t chunk, int32_t chunks, int32_t width, int32_t f32, b200_stream_t stream) {
-  if (batch <= 0 || chunks <= 0) return OK;
-  B200_REQUIRE(width > 0 && width % 4 == 0 && stride % 4 == 0 && chunk > 0 && batch <= 65535 && chunks <= 65535,
-               "mingru_prefill: width and stride must be multiples of 4, at most 65535 sequences and chunks");
-  B200_REQUIRE(aligned16(zxg) && aligned16(bias) && aligned16(state) && aligned16(workspace) && aligned16(out),
-               "mingru_prefill: tensors must be 16-byte aligned");
-  MinGruParams p = {zxg, stride, bias, state, cu_seqlens, slots, start, static_cast<float2*>(workspace), out, width, chunk, chunks};
+                                   int32_t segment, int32_t segments, int32_t width, int32_t f32, b200_stream_t stream) {
+  if (batch <= 0) return OK;
+  B200_REQUIRE(width > 0 && width % 4 == 0 && stride % 4 == 0 && stride < (1 << 26) && segment > 0 && segments > 0 && batch <= 65535 && segments <= 65535,
+               "mingru_prefill: width and stride must be multiples of 4, at most 65535 sequences and segments");
+  B200_REQUIRE(aligned16(zxg) && aligned16(bias) && aligned16(state) && aligned16(out) && (segments == 1 || (workspace && aligned16(workspace))),
+               "mingru_prefill: tensors must be 16-byte aligned, several segments need a workspace");
+  MinGruParams p = {zxg, stride, bias, state, cu_seqlens, slots, start, static_cast<float2*>(workspace), out, width, segment, segments};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const dim3 grid((width / 2 + 127) / 128, chunks, batch);
+  const dim3 grid((width + MG_COLS - 1) / MG_COLS, segments, batch);
   if (f32) {
-    if (chunks > 1) mingru_scan_kernel<float, false><<<grid, 128, 0, st>>>(p);
-    mingru_scan_kernel<float, true><<<grid, 128, 0, st>>>(p);
+    if (segments > 1) mingru_prefill_kernel<float, true><<<grid, MG_WARPS * 32, 0, st>>>(p);
+    mingru_prefill_kernel<float, false><<<grid, MG_WARPS * 32, 0, st>>>(p);
   } else {
-    if (chunks > 1) mingru_scan_kernel<__nv_bfloat16, false><<<grid, 128, 0, st>>>(p);
-    mingru_scan_kernel<__nv_bfloat16, true><<<grid, 128, 0, st>>>(p);
+    if (segments > 1) mingru_prefill_kernel<__nv_bfloat16, true><<<grid, MG_WARPS * 32, 0, st>>>(p);
+    mingru_prefill_kernel<__nv_bfloat16, false><<<grid, MG_WARPS * 32, 0, st>>>(p);
   }
-  mingru_commit_kernel<<<dim3((width + 255) / 256, batch), 256, 0, st>>>(p);
   return check_launch("mingru_prefill");
 }
 

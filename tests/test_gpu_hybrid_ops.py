@@ -87,8 +87,9 @@ def _mingru_want(zxg, bias, width, state0):
 
 
 @pytest.mark.parametrize("dt", DT)
-@pytest.mark.parametrize("lengths", [[1], [2, 63, 64, 65], [128, 1, 300], [4097]])
-def test_mingru_prefill(hops, dt, lengths):
+@pytest.mark.parametrize("lengths", [[1], [2, 15, 16, 17], [127, 128, 129], [128, 1, 300], [4097]])
+@pytest.mark.parametrize("segments", [None, (10 ** 6, 1), (128, 33), (256, 17)])
+def test_mingru_prefill(hops, dt, lengths, segments):
     dtype, width = DT[dt], 68
     zxg = rnd(sum(lengths), 3 * width, seed=5, dtype=dtype, scale=2.0)
     zxg[:, :width] -= 3.0                                   # gates that keep most of the state: far tokens matter
@@ -97,7 +98,7 @@ def test_mingru_prefill(hops, dt, lengths):
     starts = [0, 7, 0, 40][: len(lengths)]
     before = rnd(6, width, seed=7, scale=3.0)
     state = before.to(DEV)
-    out = hops.mingru_prefill(zxg.to(DEV), bias.to(DEV), state, Batch(slots, starts, lengths))
+    out = hops.mingru_prefill(zxg.to(DEV), bias.to(DEV), state, Batch(slots, starts, lengths), segments=segments)
     row = 0
     for slot, start, n in zip(slots, starts, lengths):
         want, last = _mingru_want(zxg[row: row + n], bias, width, before[slot] if start else torch.zeros(width))

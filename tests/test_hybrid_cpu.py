@@ -109,9 +109,9 @@ def test_chunking_and_splits():
     from b200attn import hybrid_ops as hops
 
     for n in (1, 2, 63, 64, 65, 2048, 4096, 4097, 100000):
-        for count, width in ((1, 64), (1, 2048), (32, 2048), (64, 4096)):
-            chunk, chunks = hops.mingru_chunking(n, count, width)
-            assert chunks <= 128 and (chunks - 1) * chunk < n <= chunks * chunk
+        for groups in (1, 32, 1000):
+            seg, segs = hops.mingru_segments(n, groups, 148)
+            assert segs <= 64 and (segs - 1) * seg < n <= segs * seg and (segs == 1 or seg % hops.MINGRU_BLOCK == 0)
         for groups in (1, 16, 32, 500):
             seg, segs = hops.hgrn2_segments(n, groups, 148)
             assert (segs - 1) * seg < n <= segs * seg and (segs == 1 or (seg % 16 == 0 and seg >= 128))
