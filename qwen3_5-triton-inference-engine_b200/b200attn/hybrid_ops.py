@@ -44,7 +44,7 @@ def swiglu_f32(gate_up, intermediate: int):
 
 
 # ------------------------------------------------------------------------------------------------------------- minGRU
-MINGRU_BLOCK, MINGRU_COLS = 128, 64
+MINGRU_BLOCK, MINGRU_COLS = 64, 64
 
 
 def sm_count(device) -> int:
@@ -58,10 +58,10 @@ _sm_counts: dict = {}
 
 
 def mingru_segments(max_len: int, groups: int, sm_count: int) -> tuple[int, int]:
-    """(segment length, segments of the longest sequence).  `groups` CTAs walk whole sequences in blocks of 128 tokens; when
-    they do not fill the device (two per SM), sequences are cut into runs of whole blocks, at the price of a second pass."""
+    """(segment length, segments of the longest sequence).  `groups` CTAs walk whole sequences in blocks of 64 tokens; when
+    they do not fill the device (three per SM), sequences are cut into runs of whole blocks, at the price of a second pass."""
     blocks = -(-max_len // MINGRU_BLOCK)
-    parts = min(-(-2 * sm_count // groups), blocks, 64)
+    parts = min(-(-3 * sm_count // groups), blocks, 64)
     if parts < 2:
         return max_len, 1
     per = -(-blocks // parts)

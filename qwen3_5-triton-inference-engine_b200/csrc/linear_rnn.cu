@@ -4,7 +4,7 @@
 //
 //   minGRU (element-wise):  z = sigmoid(z' + zb), u = x' + xb, c = u >= 0 ? u + 1/2 : sigmoid(u)
 //                           S_t = (1 - z) S_(t-1) + z c,   out = S_t * silu(g)
-//     Prefill: a CTA walks a sequence in blocks of 128 tokens, its warps scan 16 tokens each in parallel.  Too few CTAs:
+//     Prefill: a CTA walks a sequence in blocks of 64 tokens, its warps scan 8 tokens each in parallel.  Too few CTAs:
 //     sequences are cut into segments; pass 1 reduces a segment to (product of 1 - z, state it leaves from zero), pass 2
 //     folds the segments in front of its own.  HBM bound.
 //   Forget-gated outer-product recurrence (HGRN2 form):  f = l + (1 - l) sigmoid(f' + fb), q = silu(q')
@@ -49,15 +49,15 @@ __device__ __forceinline__ float2 load2(const __nv_bfloat16* q) {
 }
 __device__ __forceinline__ float2 load2(const float* q) { return *reinterpret_cast<const float2*>(q); }
 
-constexpr int MG_WARPS = 8, MG_RUN = 16;            // a warp's run of consecutive tokens
+constexpr int MG_WARPS = 8, MG_RUN = 8;             // a warp's run of consecutive tokens
 constexpr int MG_BLOCK = MG_WARPS * MG_RUN;         // tokens a CTA takes at a time
 constexpr int MG_COLS = 64;                         // channels of a CTA, two per lane
 
-// A CTA walks its segment in blocks of 128 tokens.  Every warp turns 16 of them into (keep, add) pairs in registers, leaves
+// A CTA walks its segment in blocks of 64 tokens.  Every warp turns 8 of them into (keep, add) pairs in registers, leaves
 // their product and sum in shared memory, folds the runs in front of its own and replays its run: inputs are read once.
 // grid (width / 64, segments, sequences).  REDUCE: only the segment's (product, state from zero).
 template <typename E, bool REDUCE>
-__global__ void __launch_bounds__(MG_WARPS * 32) mingru_prefill_kernel(const __grid_constant__ MinGruParams p) {
+__global__ void __launch_bounds__(MG_WARPS * 32, sizeof(E) == 2 ? 3 : 2) mingru_prefill_kernel(const __grid_constant__ MinGruParams p) {
   __shared__ float4 runs[2][MG_WARPS][32];
   const int seq = blockIdx.z, seg = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int c = blockIdx.x * MG_COLS + lane * 2;

@@ -88,7 +88,7 @@ def _mingru_want(zxg, bias, width, state0):
 
 @pytest.mark.parametrize("dt", DT)
 @pytest.mark.parametrize("lengths", [[1], [2, 15, 16, 17], [127, 128, 129], [128, 1, 300], [4097]])
-@pytest.mark.parametrize("segments", [None, (10 ** 6, 1), (128, 33), (256, 17)])
+@pytest.mark.parametrize("segments", [None, (10 ** 6, 1), (64, 65), (256, 17)])
 def test_mingru_prefill(hops, dt, lengths, segments):
     dtype, width = DT[dt], 68
     zxg = rnd(sum(lengths), 3 * width, seed=5, dtype=dtype, scale=2.0)
