@@ -447,11 +447,18 @@ int b200_swiglu_pair(const void* gate, int64_t gate_stride, const void* up, int6
  *
  * b200_hyper_connect: S residual streams (fp32 [rows, S, width]) between two sublayers:
  *     x_t <- sum_s mix[s,t] x_s + out[t] * y;   h = (sum_s in[s] x_s) / sqrt(mean(.^2) + eps) * gain
- *   weights = [mix S*S | out S | in S | gain] fp32.  ids != NULL: the streams are first set to table[ids[row]] (y NULL).
+ *   weights = [mix S*S | out S | in S | gain] fp32; gains fp32 [width] or NULL: h is multiplied by it as well.  ids != NULL: the streams are first set to table[ids[row]] (y NULL).
  *   y == NULL, ids == NULL: streams are only read. */
 int b200_hyper_connect(const void* ids, int32_t ids_are_int64, const void* table, float* streams, const void* y,
-                       const float* weights, void* h, int32_t rows, int32_t num_streams,
-                       int32_t width, int32_t true_width, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);
+                       const float* weights, const float* gains, void* h, int32_t rows, int32_t num_streams, int32_t width,
+                       int32_t true_width, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);
+/* b200_gated_act: out[r,c] = act(x[r,c]) * x[r, up + c], c < width, over strided rows (8-element groups).
+ * b200_softcap: logits[r,c] <- cap * tanh(logits[r,c] / cap) in place for c < vocab, -inf for vocab <= c < width. */
+#define B200_ACT_SILU 0
+#define B200_ACT_GELU_TANH 1
+int b200_gated_act(const void* x, int64_t stride, int32_t up, void* out, int64_t out_stride, int32_t rows, int32_t width,
+                   int32_t act, int32_t f32, int32_t overlap, b200_stream_t stream);
+int b200_softcap(float* logits, int64_t stride, int32_t rows, int32_t vocab, int32_t width, float cap, b200_stream_t stream);
 /* b200_swiglu for fp32 activations. */
 int b200_swiglu_f32(const float* gate_up, int64_t row_stride, float* out, int32_t rows, int32_t intermediate,
                     b200_stream_t stream);
@@ -484,12 +491,30 @@ int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* lower, const
                       const int64_t* pos, const int64_t* active, void* out, int32_t batch, int32_t heads, int32_t dim,
                       int32_t vdim, int32_t true_vdim, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);
 
+/* Gated linear attention: qkv = rows of [q heads*dim | k heads*dim | v heads*vdim]; state fp32 [slots, heads, dim, vdim];
+ *   f = sigmoid(z + bias)^inv_tau, S <- diag(f) S + k v^T, o = S^T q * q_scale, out = o / sqrt(mean(o^2) + eps) * norm per head,
+ *   times silu(gate) when a gate is given (rows gate_stride apart, heads*vdim wide); out rows are out_stride apart.
+ * Prefill: z fp32 rows, z_stride apart; serial, o_scratch (NULL when vdim <= 128 and the chunked form applies), segments and
+ *   the workspace (b200_hgrn2_workspace_bytes) as for b200_hgrn2_prefill.
+ * Decode: z = w_low . low with low rows of `rank` elements (qkv's stride), w_low [heads*dim, rank]. */
+int b200_gla_prefill(const void* qkv, int64_t stride, const float* z, int64_t z_stride, const float* bias, const float* norm,
+                     const void* gate, int64_t gate_stride, float* state, const int32_t* cu_seqlens, const int32_t* slots,
+                     const int32_t* start, float* o_scratch, void* out, int64_t out_stride, int32_t batch, int32_t tokens,
+                     int32_t heads, int32_t dim, int32_t vdim, int32_t true_vdim, float q_scale, float inv_tau, float eps,
+                     int32_t f32, int32_t serial, int32_t segment, int32_t segments, float* workspace, b200_stream_t stream);
+int b200_gla_decode(const void* qkv, int64_t stride, const void* low, const void* w_low, int32_t rank, const float* bias,
+                    const float* norm, const void* gate, int64_t gate_stride, float* state, const int64_t* pos,
+                    const int64_t* active, void* out, int64_t out_stride, int32_t batch, int32_t heads, int32_t dim,
+                    int32_t vdim, int32_t true_vdim, float q_scale, float inv_tau, float eps, int32_t f32, int32_t overlap,
+                    b200_stream_t stream);
+
 /* Latent attention.  Cache rows are [latent rank | rotated key part rot] in pages of 16 tokens; rank, dim, vdim, rot and
  * q_rank padded to multiples of 64.  angles: fp32 (cos, sin) pairs [positions, rot_pairs], amplitude included.
  * b200_latent_prep: fused rows [query latent | kv latent | rotated part] -> cq = rms(query latent) * q_weight, and, when
  *   cache is given, the cache row of position pos[row] of slot[row] (NULL: slot = row).
  * b200_rope_interleaved: rotates pairs (x[offset+2i], x[offset+2i+1]) of every head in place.
- * b200_latent_gather: packed cache rows of positions k_pos0[s] + (0 .. cu_k[s+1]-cu_k[s]-1).
+ * b200_latent_gather: packed cache rows (kv_heads per token; latent: 1) of positions k_pos0[s] + i, i below
+ *   min(cu_k[s+1] - cu_k[s], max_keys rounded up to 16).
  * b200_latent_prefill(_simple): q [tokens, heads, dim+rot] (rotated) against kv [keys, heads*dim | heads*vdim] and the
  *   rotated parts of ctx [keys, rank+rot]; query i of sequence s sits at position q_pos0[s] + i and sees positions
  *   (p - window, p].  _simple: any shape, bf16 or fp32; the other: bf16, tcgen05, dim + rot <= 256, vdim <= 256.
@@ -505,8 +530,8 @@ int b200_latent_prep(const void* fused, int64_t stride, const float* q_weight, c
 int b200_rope_interleaved(void* x, int64_t row_stride, int32_t head_stride, int32_t offset, int32_t heads, int32_t pairs,
                           const int32_t* pos, const float* angles, int32_t rows, int32_t f32, b200_stream_t stream);
 int b200_latent_gather(const void* cache, void* out, const int32_t* block_table, int64_t table_stride, const int32_t* slots,
-                       const int32_t* cu_k, const int32_t* k_pos0, int32_t batch, int32_t max_keys, int32_t row_bytes,
-                       b200_stream_t stream);
+                       const int32_t* cu_k, const int32_t* k_pos0, int32_t batch, int32_t max_keys,
+                       int32_t kv_heads, int32_t row_bytes, b200_stream_t stream);
 int b200_latent_prefill_simple(const void* q, const void* kv, const void* ctx, void* out, const int32_t* cu_q,
                                const int32_t* cu_k, const int32_t* q_pos0, const int32_t* k_pos0, int32_t batch, int32_t max_q,
                                int32_t heads, int32_t dim, int32_t rot, int32_t vdim, int32_t rank, int32_t window, float scale,
@@ -528,6 +553,36 @@ int b200_latent_decode(const void* q, const void* cache, int64_t num_pages, cons
                        b200_stream_t stream);
 int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* merged, void* out, int32_t batch,
                       int32_t heads, int32_t rank, int32_t vdim, int32_t splits, int32_t f32, int32_t overlap, b200_stream_t stream);
+
+/* Windowed attention with grouped heads.  Projection rows x = [q heads*dim | k kv_heads*dim | v kv_heads*vdim | ...] (stride
+ * elements apart); cache rows [key dim | value vdim | padding up to pitch], one per key/value head: [pages, kv_heads, 16,
+ * pitch].  dim a multiple of 32, vdim and pitch of 64.  Query head h reads key/value head h / (heads / kv_heads).
+ * b200_window_prep: adds bias fp32 [(heads + kv_heads)*dim + kv_heads*vdim], rotates the pairs (i, i + rot_pairs) of q and k
+ *   by angles fp32 (cos, sin) [positions, rot_pairs]; q in place, k and v to the cache row of position pos[row] of slot[row]
+ *   (NULL: slot = row) and, when ctx is given, to ctx[ctx_row[row]] ([keys, kv_heads, pitch], packed keys of a prefill).
+ * b200_window_prefill: q (rotated, in x's layout) against ctx; sequence s: queries cu_q, keys cu_k from position k_pos0[s] on;
+ *   query i sits at q_pos0[s] + i and sees (p - window, p].  out[t, h*vdim + c] = o * sigmoid(gate) * out_scale.  simple
+ *   or f32: CUDA cores, any shape; else tcgen05, dim and vdim at most 256 (64-column blocks are read from every head's
+ *   start on: a row must be at least heads*dim + 32 elements wide).
+ * b200_window_decode: one token per slot against the paged rows, the visible range in `splits` runs of pages: ml fp32
+ *   [batch, heads, splits, 2], o fp32 [batch, heads, splits, vdim] unnormalised.
+ * b200_window_merge: merges them; out[b, h*vdim + c] = o * sigmoid(gate) * out_scale. */
+int b200_window_prep(void* x, int64_t stride, const float* bias, const void* pos, int32_t pos_is_int64, const int32_t* slot,
+                     const int64_t* active, const int32_t* block_table, int64_t table_stride, const float* angles, void* cache,
+                     void* ctx, const int32_t* ctx_row, int32_t rows, int32_t heads, int32_t kv_heads, int32_t dim,
+                     int32_t rot_pairs, int32_t vdim, int32_t pitch, int32_t f32, int32_t overlap, b200_stream_t stream);
+int b200_window_prefill(const void* q, int64_t q_stride, const void* ctx, const void* gate, int64_t gate_stride, void* out,
+                        int64_t out_stride, const int32_t* cu_q, const int32_t* cu_k, const int32_t* q_pos0,
+                        const int32_t* k_pos0, int32_t batch, int32_t max_q, int32_t tokens, int32_t keys, int32_t heads,
+                        int32_t kv_heads, int32_t dim, int32_t true_dim, int32_t vdim, int32_t pitch, int32_t window,
+                        float scale, float out_scale, int32_t simple, int32_t f32, b200_stream_t stream);
+int b200_window_decode(const void* q, int64_t q_stride, const void* cache, int64_t num_pages, const int32_t* block_table,
+                       int64_t table_stride, const int64_t* pos, const int64_t* active, float* ml, float* o, int32_t batch,
+                       int32_t heads, int32_t kv_heads, int32_t dim, int32_t vdim, int32_t pitch, int32_t window,
+                       int32_t splits, float scale, int32_t simple, int32_t f32, int32_t overlap, b200_stream_t stream);
+int b200_window_merge(const float* ml, const float* o, const void* gate, int64_t gate_stride, void* out, int64_t out_stride,
+                      int32_t batch, int32_t heads, int32_t vdim, int32_t splits, float out_scale, int32_t f32,
+                      int32_t overlap, b200_stream_t stream);
 
 #ifdef __cplusplus
 }

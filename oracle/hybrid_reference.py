@@ -1,7 +1,8 @@
-"""Plain, slow restatement of the hybrid decoder stack (latent attention / HGRN2 / minGRU mixers, hyper-connected
-residual streams, scalar-gain RMS norms) in eager PyTorch on the CPU, written from the equations of the design: one
-function per mechanism, whole sequences only, no cache, no chunks.  Tests compare the CUDA path with it; the product
-never imports it.
+"""Plain, slow restatement of the hybrid decoder stacks in eager PyTorch on the CPU, written from the equations of the
+designs: one function per mechanism, whole sequences only, no cache, no chunks.  Tofilorn: latent attention / HGRN2 /
+minGRU mixers, hyper-connected residual streams, scalar-gain RMS norms.  Dugilorn: windowed attention beside a state-space
+mixer, gated linear attention, mixer and feed-forward reading one norm.  Tests compare the CUDA path with it; the
+product never imports it.
 
 Everything is computed in the dtype of the weights handed in (tests use float64).  `weights` maps tensor names
 ("l0.mix.dq", ...) to tensors; `config` is the parsed config.json dictionary.
@@ -134,6 +135,126 @@ def swiglu_mlp(h, w, pre):
     return (silu(h @ w[pre + "gate"].T) * (h @ w[pre + "up"].T)) @ w[pre + "down"].T
 
 
+# ------------------------------------------------------------------------------- windowed attention, state space, gla
+def rotate_halves(x, rot, positions):
+    """Rotation of the first rot.dims entries of the last axis, entry i paired with entry i + dims/2."""
+    n = rot["dims"] // 2
+    freqs, _ = rotary_frequencies(rot)
+    angle = positions.double()[:, None] * freqs[None, :]
+    shape = (x.shape[0],) + (1,) * (x.dim() - 2) + (n,)
+    cos, sin = torch.cos(angle).view(shape).to(x.dtype), torch.sin(angle).view(shape).to(x.dtype)
+    u, v = x[..., :n], x[..., n: 2 * n]
+    return torch.cat((u * cos - v * sin, v * cos + u * sin, x[..., 2 * n:]), dim=-1)
+
+
+def biased(h, w, name):
+    return h @ w[name].T + w[name + ".b"]
+
+
+def gated_window_attention(h, w, pre, m):
+    """Grouped query heads over a sliding window, the heads' outputs times sigmoid of a gate, W_o."""
+    T, heads, kv = h.shape[0], m["heads"], m["kv_heads"]
+    at = torch.arange(T)
+    q = rotate_halves(biased(h, w, pre + "q").view(T, heads, m["dim"]), m["rot"], at)
+    k = rotate_halves(biased(h, w, pre + "k").view(T, kv, m["dim"]), m["rot"], at)
+    v = biased(h, w, pre + "v").view(T, kv, m["vdim"])
+    owner = torch.tensor([i // (heads // kv) for i in range(heads)])
+    o = window_attention(q, k[:, owner], v[:, owner], m["scale"], m["mask"]["size"]).reshape(T, -1)
+    return (o * sigmoid(h @ w[pre + "g"].T)) @ w[pre + "o"].T
+
+
+def causal_conv(x, taps, bias):
+    """out[t] = sum_j taps[:, K-1-j] x[t-j] + bias with zeros before the start; x [T, channels], taps [channels, K]."""
+    out = torch.zeros_like(x)
+    for j in range(taps.shape[1]):
+        moved = torch.zeros_like(x)
+        moved[j:] = x[: x.shape[0] - j]
+        out = out + moved * taps[:, taps.shape[1] - 1 - j]
+    return out + bias
+
+
+def softplus(u):
+    return torch.clamp(u, min=0) + torch.log1p(torch.exp(-u.abs()))
+
+
+def state_space_recurrence(x, B, C, dt, A_log, D):
+    """S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T, y_t = S_t^T C_t + D x_t; x [T, H, P], B, C [T, H, N], dt [T, H]."""
+    T, heads, vdim = x.shape
+    S, out = torch.zeros(heads, B.shape[-1], vdim, dtype=x.dtype), []
+    for t in range(T):
+        keep = torch.exp(-torch.exp(A_log) * dt[t])
+        S = keep[:, None, None] * S + dt[t][:, None, None] * B[t][:, :, None] * x[t][:, None, :]
+        out.append(torch.einsum("hnp,hn->hp", S, C[t]) + D[:, None] * x[t])
+    return torch.stack(out)
+
+
+def grouped_rms(x, groups, eps):
+    return rms(x.view(*x.shape[:-1], groups, -1), eps).reshape(x.shape)
+
+
+def state_space(h, w, pre, m, eps):
+    T, heads, vdim, N, G = h.shape[0], m["heads"], m["vdim"], m["state"], m["groups"]
+    inner = heads * vdim
+    z, xbc, dt = (h @ w[pre + "in"].T).split([inner, inner + 2 * G * N, heads], dim=-1)
+    xbc = silu(causal_conv(xbc, w[pre + "conv"], w[pre + "conv.b"]))
+    x, B, C = xbc.split([inner, G * N, G * N], dim=-1)
+    owner = torch.tensor([i // (heads // G) for i in range(heads)])
+    y = state_space_recurrence(x.view(T, heads, vdim), B.view(T, G, N)[:, owner], C.view(T, G, N)[:, owner],
+                               softplus(dt + w[pre + "dt_bias"]), w[pre + "A_log"], w[pre + "D"]).reshape(T, inner)
+    y = grouped_rms(y * silu(z), m["norm_groups"], eps) * w[pre + "norm"]
+    return y @ w[pre + "o"].T
+
+
+def decayed_outer_recurrence(q, k, v, keep):
+    """S_t = diag(keep_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t; q, k, keep [T, H, D], v [T, H, Dv]."""
+    S, out = torch.zeros(q.shape[1], q.shape[2], v.shape[-1], dtype=q.dtype), []
+    for t in range(q.shape[0]):
+        S = keep[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+        out.append(torch.einsum("hdv,hd->hv", S, q[t]))
+    return torch.stack(out)
+
+
+def gated_linear_attention(h, w, pre, m, eps):
+    T, heads, dim, vdim = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    q = (h @ w[pre + "q"].T).view(T, heads, dim) * dim ** -0.5
+    k = (h @ w[pre + "k"].T).view(T, heads, dim)
+    v = (h @ w[pre + "v"].T).view(T, heads, vdim)
+    z = (h @ w[pre + "a1"].T) @ w[pre + "a2"].T + w[pre + "a2.b"]
+    keep = torch.exp(-softplus(-z) / m["tau"]).view(T, heads, dim)          # sigmoid(z) ** (1 / tau)
+    o = rms(decayed_outer_recurrence(q, k, v, keep), eps) * w[pre + "norm"]
+    return (o.reshape(T, -1) * silu(h @ w[pre + "g"].T)) @ w[pre + "o"].T
+
+
+def side_by_side(h, w, pre, m, eps):
+    return (m["left_scale"] * gated_window_attention(h, w, pre + "left.", m["left"])
+            + m["right_scale"] * state_space(h, w, pre + "right.", m["right"], eps))
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def geglu_mlp(h, w, pre):
+    return (gelu_tanh(h @ w[pre + "gate"].T) * (h @ w[pre + "up"].T)) @ w[pre + "down"].T
+
+
+def forward_dugilorn(config, w, tokens):
+    """(logits [T, vocab], residual stream after every layer) of a stack whose layers add mixer(h) + ff(h), h = norm(x)."""
+    eps = config["norm"]["eps"]
+    x, trail = w["embed"][torch.tensor(tokens)], []
+    for i, layer in enumerate(config["layers"]):
+        pre = f"l{i}."
+        h = rms(x, eps) * w[pre + "norm1"]
+        y = {"parallel": side_by_side, "gla": gated_linear_attention}[layer["type"]](h, w, pre + "mix.", layer["mixer"], eps)
+        if layer["mlp"] is not None:
+            y = y + geglu_mlp(h, w, pre + "mlp.")
+        x = x + y
+        trail.append(x)
+    logits = (rms(x, eps) * w["final.norm"]) @ w["head"].T
+    cap = config["logit_softcap"]
+    return cap * torch.tanh(logits / cap), torch.stack(trail)
+
+
 # ------------------------------------------------------------------------------------------------------------- stack
 def hyper_connect(streams, w, pre, sublayer):
     """u = sum_s in[s] x_s; y = sublayer(u); x_t <- sum_s mix[s, t] x_s + out[t] y.  streams [S, T, width]."""
@@ -144,6 +265,8 @@ def hyper_connect(streams, w, pre, sublayer):
 
 def forward(config, w, tokens):
     """(logits [T, vocab], residual stream after every layer [layers, T, width]) of one sequence."""
+    if config["architecture"] == "Dugilorn":
+        return forward_dugilorn(config, w, tokens)
     eps = config["norm"]["eps"]
     x = w["embed"][torch.tensor(tokens)]
     streams = x[None].repeat(config["streams"], 1, 1)

@@ -63,7 +63,7 @@ SIGNATURES: dict[str, list] = {
     "b200_swiglu_pair": [P, I64, P, I64, P, I32, I32, P],
     "b200_gdn_chunked_prefill_fused": [P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I32, I32,
                                        P, P, I64, I64, I32, I32, I32, P],
-    "b200_hyper_connect": [P, I32, P, P, P, P, P, I32, I32, I32, I32, c_float, I32, I32, P],
+    "b200_hyper_connect": [P, I32, P, P, P, P, P, P, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_swiglu_f32": [P, I64, P, I32, I32, P],
     "b200_mingru_prefill": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, P],
     "b200_mingru_decode": [P, I64, P, P, P, P, P, I32, I32, I32, I32, P],
@@ -73,13 +73,24 @@ SIGNATURES: dict[str, list] = {
     "b200_latent_prep": [P, I64, P, P, P, I32, P, P, P, I64, P, P, P, I32, I32, I32, I32, I32, I32, I32, c_float, I32, I32,
                          P],
     "b200_rope_interleaved": [P, I64, I32, I32, I32, I32, P, P, I32, I32, P],
-    "b200_latent_gather": [P, P, P, I64, P, P, P, I32, I32, I32, P],
+    "b200_latent_gather": [P, P, P, I64, P, P, P, I32, I32, I32, I32, P],
     "b200_latent_prefill_simple": [P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, c_float, I32, P],
     "b200_latent_prefill": [P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32, c_float, P],
     "b200_latent_decode": [P, P, I64, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, P],
     "b200_latent_absorb": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, P],
     "b200_latent_decode_simple": [P, P, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_latent_value": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, P],
+    "b200_gated_act": [P, I64, I32, P, I64, I32, I32, I32, I32, I32, P],
+    "b200_softcap": [P, I64, I32, I32, I32, c_float, P],
+    "b200_window_prep": [P, I64, P, P, I32, P, P, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, I32, P],
+    "b200_window_prefill": [P, I64, P, P, I64, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32, I32,
+                            c_float, c_float, I32, I32, P],
+    "b200_window_decode": [P, I64, P, I64, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, c_float, I32, I32, I32, P],
+    "b200_window_merge": [P, P, P, I64, P, I64, I32, I32, I32, I32, c_float, I32, I32, P],
+    "b200_gla_prefill": [P, I64, P, I64, P, P, P, I64, P, P, P, P, P, P, I64, I32, I32, I32, I32, I32, I32, c_float, c_float,
+                         c_float, I32, I32, I32, I32, P, P],
+    "b200_gla_decode": [P, I64, P, P, I32, P, P, P, I64, P, P, P, P, I64, I32, I32, I32, I32, I32, c_float, c_float, c_float, I32,
+                        I32, P],
 }
 OTHER = {
     "b200_mingru_workspace_bytes": ([I32, I32, I32], c_int64),

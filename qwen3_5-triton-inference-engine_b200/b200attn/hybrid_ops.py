@@ -16,12 +16,14 @@ def _f32(t) -> int:
     return int(t.dtype == torch.float32)
 
 
-def hyper_connect(streams, weights, true_width: int, eps: float, dtype, y=None, ids=None, table=None, overlap: int = 0):
+def hyper_connect(streams, weights, true_width: int, eps: float, dtype, y=None, ids=None, table=None, overlap: int = 0, gains=None):
     """One step between two sublayers (b200_hyper_connect): mixes `y` into `streams` [rows, S, width] (in place), or sets
-    them from `table[ids]`; returns the next sublayer's normed input [rows, width]."""
+    them from `table[ids]`; returns the next sublayer's normed input [rows, width].  gains: fp32 [width] norm weights on top
+    of the single gain."""
     assert streams.dtype == weights.dtype == torch.float32 and streams.is_contiguous() and weights.is_contiguous()
     rows, s, width = streams.shape
     assert weights.numel() == s * s + 2 * s + 1
+    assert gains is None or (gains.dtype == torch.float32 and gains.numel() == width and gains.is_contiguous())
     h = torch.empty((rows, width), dtype=dtype, device=streams.device)
     if y is not None:
         assert y.shape == (rows, width) and y.is_contiguous() and y.dtype == dtype
@@ -30,7 +32,7 @@ def hyper_connect(streams, weights, true_width: int, eps: float, dtype, y=None, 
         assert table.dtype == dtype and table.shape[1] == width and table.is_contiguous()
     _require_cuda(streams, weights)
     _lib.call("b200_hyper_connect", _ptr(ids), int(ids is not None and ids.dtype == torch.int64), _ptr(table), _ptr(streams),
-              _ptr(y), _ptr(weights), _ptr(h), rows, s, width, true_width, float(eps), _f32(h), int(overlap),
+              _ptr(y), _ptr(weights), _ptr(gains), _ptr(h), rows, s, width, true_width, float(eps), _f32(h), int(overlap),
               _stream())
     return h
 
@@ -186,7 +188,7 @@ def latent_gather(cache, block_table, slots, cu_k, k_pos0, keys: int, max_keys: 
     out = torch.empty((keys, cache.shape[2]), dtype=cache.dtype, device=cache.device)
     _require_cuda(cache, block_table, slots, cu_k, k_pos0)
     _lib.call("b200_latent_gather", _ptr(cache), _ptr(out), _ptr(block_table), block_table.stride(0), _ptr(slots), _ptr(cu_k),
-              _ptr(k_pos0), slots.numel(), max_keys, cache.shape[2] * cache.element_size(), _stream())
+              _ptr(k_pos0), slots.numel(), max_keys, 1, cache.shape[2] * cache.element_size(), _stream())
     return out
 
 

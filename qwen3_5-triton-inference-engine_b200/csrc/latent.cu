@@ -6,8 +6,8 @@
 //   b200_latent_gather     cache rows of a range of positions per sequence into a packed buffer (prefill context)
 //   b200_latent_prefill_simple   attention over expanded keys/values, any shape, bf16 or fp32 (CUDA cores)
 //   b200_latent_absorb     decode: q' = [W_uk^T q_unrotated | rotated part], so that scores need the cache rows only
-//   b200_latent_decode_simple    decode over the paged rows, split over key ranges, any shape (CUDA cores)
-//   b200_latent_value      decode: merges the splits, then applies W_uv (two launches)
+//   b200_latent_decode_simple    decode over the paged rows, split over key ranges, any shape (row_attention.cu)
+//   b200_latent_value      decode: merges the splits (row_attention.cu), then applies W_uv (two launches)
 // The tensor-core forms live in latent_decode.cu and latent_prefill_umma.cu.
 // Padded layout (the weight loader's): kv_rank, rot_dim, dim, vdim and q_rank are rounded up to multiples of 64 with
 // zero rows / columns, a cache row is [latent | rotated part] with both parts padded.  Norms divide by the true widths.
@@ -181,63 +181,23 @@ __global__ void __launch_bounds__(256) rope_interleaved_kernel(E* x, int64_t row
 }
 
 // ------------------------------------------------------------------------------------------------------------ gather
-// out[cu_k[s] + i] = cache row of position k_pos0[s] + i of sequence s; grid (16-row groups, sequences)
+// out[cu_k[s] + i] = cache rows (one per key/value head) of position k_pos0[s] + i of sequence s; grid (16-row groups,
+// sequences)
 __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4* cache, uint4* out, const int32_t* table,
                                                             int64_t table_stride, const int32_t* slots, const int32_t* cu_k,
-                                                            const int32_t* k_pos0, int row_vecs) {
+                                                            const int32_t* k_pos0, int kv_heads, int row_vecs) {
   const int seq = blockIdx.y, row0 = cu_k[seq], len = cu_k[seq + 1] - row0, base = k_pos0[seq];
   const int32_t* t = table + slots[seq] * table_stride;
   const int r_lo = blockIdx.x * 16, r_hi = min(r_lo + 16, len);
-  for (int i = r_lo * row_vecs + threadIdx.x; i < r_hi * row_vecs; i += 256) {
-    const int r = i / row_vecs, c = i % row_vecs, pos = base + r;
-    out[static_cast<int64_t>(row0 + r) * row_vecs + c] =
-        cache[(static_cast<int64_t>(t[pos / PAGE]) * PAGE + pos % PAGE) * row_vecs + c];
+  const int token_vecs = kv_heads * row_vecs;
+  for (int i = r_lo * token_vecs + threadIdx.x; i < r_hi * token_vecs; i += 256) {
+    const int r = i / token_vecs, gc = i - r * token_vecs, g = gc / row_vecs, pos = base + r;
+    out[static_cast<int64_t>(row0 + r) * token_vecs + gc] =
+        cache[((static_cast<int64_t>(t[pos / PAGE]) * kv_heads + g) * PAGE + pos % PAGE) * row_vecs + gc - g * row_vecs];
   }
 }
 
 // ------------------------------------------------------------------------------- attention on CUDA cores, any shape
-constexpr int LS_TILE = 64;
-constexpr int LS_MAX_COLS = 1024;  // value columns: 8 per thread
-
-// One query row against keys [0, n): scores of a 64-key tile by warps, then every thread owns columns of the sum.
-// key(j, c) / rkey(j, c) / val(j, c) return fp32 elements.
-template <typename KeyDot, typename Val>
-__device__ __forceinline__ void simple_attend(int j_lo, int j_hi, int cols, float scale, KeyDot dot, Val val, float* ps,
-                                              float& m_out, float& l_out, float (&acc)[LS_MAX_COLS / 128]) {
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  float m = -INFINITY, l = 0.f;
-#pragma unroll
-  for (int i = 0; i < LS_MAX_COLS / 128; ++i) acc[i] = 0.f;
-  for (int j0 = j_lo; j0 < j_hi; j0 += LS_TILE) {
-    const int n = min(LS_TILE, j_hi - j0);
-    for (int j = warp; j < n; j += 4) {
-      const float s = warp_sum(dot(j0 + j, lane)) * scale;
-      if (lane == 0) ps[j] = s;
-    }
-    __syncthreads();
-    float tile_max = -INFINITY;
-    for (int j = lane; j < n; j += 32) tile_max = fmaxf(tile_max, ps[j]);
-    tile_max = warp_max(tile_max);
-    const float m_new = fmaxf(m, tile_max);
-    const float alpha = expf(m - m_new);
-    float part = 0.f;
-    for (int j = lane; j < n; j += 32) part += expf(ps[j] - m_new);
-    l = l * alpha + warp_sum(part);
-    m = m_new;
-#pragma unroll
-    for (int i = 0; i < LS_MAX_COLS / 128; ++i) acc[i] *= alpha;
-    for (int j = 0; j < n; ++j) {
-      const float w = expf(ps[j] - m_new);
-#pragma unroll
-      for (int i = 0; i < LS_MAX_COLS / 128; ++i)
-        if (tid + i * 128 < cols) acc[i] = fmaf(w, val(j0 + j, tid + i * 128), acc[i]);
-    }
-    __syncthreads();
-  }
-  m_out = m;
-  l_out = l;
-}
-
 template <typename E>
 __global__ void __launch_bounds__(128) latent_prefill_simple_kernel(const __grid_constant__ LatentPrefillParams p) {
   __shared__ float ps[LS_TILE];
@@ -270,40 +230,6 @@ __global__ void __launch_bounds__(128) latent_prefill_simple_kernel(const __grid
 #pragma unroll
   for (int c = 0; c < LS_MAX_COLS / 128; ++c)
     if (threadIdx.x + c * 128 < p.vdim) store1(out + threadIdx.x + c * 128, acc[c] / l);
-}
-
-template <typename E>
-__global__ void __launch_bounds__(128) latent_decode_simple_kernel(const __grid_constant__ LatentDecodeParams p) {
-  __shared__ float ps[LS_TILE];
-  const int split = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
-  if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
-  pdl_wait();
-  int lo, hi;
-  latent_split_range(p, b, split, lo, hi);
-  const int64_t part = (static_cast<int64_t>(b) * p.heads + h) * p.splits + split;
-  if (lo >= hi) {
-    if (threadIdx.x == 0) p.ml[part] = make_float2(-INFINITY, 0.f);
-    return;
-  }
-  const int pitch = p.rank + p.rot;
-  const E* q = static_cast<const E*>(p.q) + (static_cast<int64_t>(b) * p.heads + h) * pitch;
-  const E* cache = static_cast<const E*>(p.cache);
-  const int32_t* table = p.table + b * p.table_stride;
-  auto row = [&](int j) { return cache + (static_cast<int64_t>(table[j / PAGE]) * PAGE + j % PAGE) * pitch; };
-  float m, l, acc[LS_MAX_COLS / 128];
-  simple_attend(
-      lo, hi, p.rank, p.scale,
-      [&](int j, int lane) {
-        const E* k = row(j);
-        float s = 0.f;
-        for (int c = lane; c < pitch; c += 32) s = fmaf(load1(q + c), load1(k + c), s);
-        return s;
-      },
-      [&](int j, int c) { return load1(row(j) + c); }, ps, m, l, acc);
-  if (threadIdx.x == 0) p.ml[part] = make_float2(m, l);
-#pragma unroll
-  for (int c = 0; c < LS_MAX_COLS / 128; ++c)
-    if (threadIdx.x + c * 128 < p.rank) p.o[part * p.rank + threadIdx.x + c * 128] = acc[c];
 }
 
 // ------------------------------------------------------------------------------------------------ decode: q' = W_uk^T q
@@ -410,58 +336,6 @@ __global__ void __launch_bounds__(128) latent_absorb_bf16_kernel(const __grid_co
 }
 
 // --------------------------------------------------------------------------------------- decode: merge splits, W_uv
-// merged[b, h, :] = sum_s w_s o_s with w_s = exp(m_s - m) / sum exp(m_s - m) l_s; an idle slot gives zeros.
-// grid (heads, batch)
-template <typename E>
-__global__ void __launch_bounds__(128) latent_merge_kernel(const __grid_constant__ LatentValueParams p) {
-  __shared__ float weight[LATENT_MAX_SPLITS];
-  const int64_t bh = static_cast<int64_t>(blockIdx.y) * p.heads + blockIdx.x;
-  const int tid = threadIdx.x;
-  if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
-  pdl_wait();
-  if (tid < 32) {
-    constexpr int N = LATENT_MAX_SPLITS / 32;
-    float2 a[N];
-    float m = -INFINITY, l = 0.f;
-#pragma unroll
-    for (int i = 0; i < N; ++i) {
-      a[i] = tid + i * 32 < p.splits ? p.ml[bh * p.splits + tid + i * 32] : make_float2(-INFINITY, 0.f);
-      m = fmaxf(m, a[i].x);
-    }
-    m = warp_max(m);
-#pragma unroll
-    for (int i = 0; i < N; ++i) {
-      a[i].x = a[i].y > 0.f ? expf(a[i].x - m) : 0.f;
-      l += a[i].x * a[i].y;
-    }
-    l = warp_sum(l);
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
-#pragma unroll
-    for (int i = 0; i < N; ++i)
-      if (tid + i * 32 < p.splits) weight[tid + i * 32] = a[i].x * inv;
-  }
-  __syncthreads();
-  for (int c = tid * 4; c < p.rank; c += 512) {
-    const float* o = p.o + bh * p.splits * p.rank + c;
-    float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
-    constexpr int U = 8;
-    for (int s0 = 0; s0 < p.splits; s0 += U) {
-      float4 v[U];
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-        if (s0 + u < p.splits) v[u] = load4(o + static_cast<int64_t>(s0 + u) * p.rank);
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-        if (s0 + u < p.splits && weight[s0 + u] != 0.f) {  // an empty range left its part of the workspace unwritten
-          const float w = weight[s0 + u];
-          sum.x = fmaf(w, v[u].x, sum.x), sum.y = fmaf(w, v[u].y, sum.y);
-          sum.z = fmaf(w, v[u].z, sum.z), sum.w = fmaf(w, v[u].w, sum.w);
-        }
-    }
-    store4(static_cast<E*>(p.merged) + bh * p.rank + c, sum);
-  }
-}
-
 __global__ void __launch_bounds__(128) latent_value_bf16_kernel(const __grid_constant__ LatentValueParams p) {
   extern __shared__ __align__(16) uint8_t hg_smem[];
   const int h = blockIdx.x, n0 = blockIdx.y * 64, b0 = blockIdx.z * 16, slots = min(16, p.batch - b0);
@@ -558,11 +432,12 @@ extern "C" int b200_rope_interleaved(void* x, int64_t row_stride, int32_t head_s
 
 extern "C" int b200_latent_gather(const void* cache, void* out, const int32_t* block_table, int64_t table_stride,
                                   const int32_t* slots, const int32_t* cu_k, const int32_t* k_pos0, int32_t batch,
-                                  int32_t max_keys, int32_t row_bytes, b200_stream_t stream) {
+                                  int32_t max_keys, int32_t kv_heads, int32_t row_bytes, b200_stream_t stream) {
   if (batch <= 0 || max_keys <= 0) return OK;
-  B200_REQUIRE(row_bytes % 16 == 0 && aligned16(cache) && aligned16(out) && batch <= 65535, "latent_gather: unaligned rows");
+  B200_REQUIRE(row_bytes % 16 == 0 && aligned16(cache) && aligned16(out) && batch <= 65535 && kv_heads > 0, "latent_gather: unaligned rows");
   latent_gather_kernel<<<dim3((max_keys + 15) / 16, batch), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
-      static_cast<const uint4*>(cache), static_cast<uint4*>(out), block_table, table_stride, slots, cu_k, k_pos0, row_bytes / 16);
+      static_cast<const uint4*>(cache), static_cast<uint4*>(out), block_table, table_stride, slots, cu_k, k_pos0,
+      kv_heads, row_bytes / 16);
   return check_launch("latent_gather");
 }
 
@@ -606,18 +481,10 @@ extern "C" int b200_latent_decode_simple(const void* q, const void* cache, const
                                          int32_t heads, int32_t rank, int32_t rot, int32_t window, int32_t splits, float scale,
                                          int32_t f32, int32_t overlap, b200_stream_t stream) {
   if (batch <= 0) return OK;
-  B200_REQUIRE(rank > 0 && rank <= LS_MAX_COLS && window > 0 && splits > 0 && splits <= LATENT_MAX_SPLITS && heads <= 65535 &&
-                   batch <= 65535,
-               "latent_decode_simple: rank at most %d, splits at most %d", LS_MAX_COLS, LATENT_MAX_SPLITS);
-  LatentDecodeParams p = {q, cache, block_table, table_stride, pos, active, reinterpret_cast<float2*>(ml), o,
-                          heads, rank, rot, window, splits, overlap, scale, nullptr};
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const dim3 grid(splits, heads, batch);
-  const bool early = (overlap & OVERLAP_START) != 0;
-  const cudaError_t e = f32 ? launch_pdl(early, latent_decode_simple_kernel<float>, grid, dim3(128), 0, st, p)
-                            : launch_pdl(early, latent_decode_simple_kernel<__nv_bfloat16>, grid, dim3(128), 0, st, p);
-  if (e != cudaSuccess) return fail(ERR_LAUNCH, "latent_decode_simple: %s", cudaGetErrorString(e));
-  return check_launch("latent_decode_simple");
+  const RowDecodeParams p = {q, static_cast<int64_t>(heads) * (rank + rot), cache, block_table, table_stride, pos, active,
+                             reinterpret_cast<float2*>(ml), o, heads, 1, heads, rank + rot, 0, rank, rank + rot, window, splits,
+                             overlap, scale, nullptr};
+  return row_decode_simple_launch(p, batch, f32 != 0, "latent_decode_simple", reinterpret_cast<cudaStream_t>(stream));
 }
 
 extern "C" int b200_latent_value(const float* ml, const float* o, const void* w_uv, void* merged, void* out, int32_t batch,
@@ -628,23 +495,22 @@ extern "C" int b200_latent_value(const float* ml, const float* o, const void* w_
                "latent_value: rank and vdim must be multiples of 64, rank at most %d, splits at most %d", LS_MAX_COLS,
                LATENT_MAX_SPLITS);
   B200_REQUIRE(aligned16(o) && aligned16(w_uv) && aligned16(merged) && aligned16(out), "latent_value: unaligned tensor");
-  LatentValueParams p = {reinterpret_cast<const float2*>(ml), o, w_uv, merged, out, batch, heads, rank, vdim, splits, overlap};
+  const LatentValueParams p = {w_uv, merged, out, batch, heads, rank, vdim, overlap};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const dim3 grid(heads, vdim / 64, (batch + 15) / 16), merge_grid(heads, batch);
-  const bool early = (overlap & OVERLAP_START) != 0;
-  LatentValueParams merge = p;
+  const dim3 grid(heads, vdim / 64, (batch + 15) / 16);
+  // the product behind the merge: in bf16 it starts early and waits, in fp32 it is launched plainly
+  const int merge_overlap = f32 ? overlap & ~OVERLAP_TRIGGER : overlap | OVERLAP_TRIGGER;
+  const RowMergeParams merge = {reinterpret_cast<const float2*>(ml), o, nullptr, 0, merged, static_cast<int64_t>(heads) * rank,
+                                heads, rank, splits, merge_overlap, 1.f};
+  const int rc = row_merge_launch(merge, batch, f32 != 0, "latent_value", st);
+  if (rc != OK) return rc;
   if (f32) {
-    merge.overlap &= ~OVERLAP_TRIGGER;  // the fp32 product behind it is launched plainly
-    if (launch_pdl(early, latent_merge_kernel<float>, merge_grid, dim3(128), 0, st, merge) != cudaSuccess)
-      return fail(ERR_LAUNCH, "latent_value: %s", cudaGetErrorString(cudaGetLastError()));
     latent_value_f32_kernel<<<grid, 128, 0, st>>>(p);
     return check_launch("latent_value");
   }
   if (!head_gemm_configure(reinterpret_cast<const void*>(latent_value_bf16_kernel), 1))
     return fail(ERR_RUNTIME, "latent_value: cannot raise dynamic shared memory");
-  merge.overlap |= OVERLAP_TRIGGER;     // its successor is the product below, which waits
-  if (launch_pdl(early, latent_merge_kernel<__nv_bfloat16>, merge_grid, dim3(128), 0, st, merge) != cudaSuccess ||
-      launch_pdl(true, latent_value_bf16_kernel, grid, dim3(128), rank / 64 * HG_STEP, st, p) != cudaSuccess)
+  if (launch_pdl(true, latent_value_bf16_kernel, grid, dim3(128), rank / 64 * HG_STEP, st, p) != cudaSuccess)
     return fail(ERR_LAUNCH, "latent_value: %s", cudaGetErrorString(cudaGetLastError()));
   return check_launch("latent_value");
 }

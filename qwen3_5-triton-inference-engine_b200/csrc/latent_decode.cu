@@ -1,15 +1,16 @@
-// Decode attention over cached latents on the tensor cores: every head of a token scores the same cache rows
-// [latent | rotated key part], so 16 heads are one MMA M tile and a row is read once per 16 heads.
+// Decode attention over paged rows on the tensor cores (latent.cuh, RowDecodeParams): the heads that share a row are one MMA
+// M tile of 16, so a row is read once per 16 heads.  Latent attention: all heads share the rows [latent | rotated key part]
+// and sum their first `rank` elements.  Grouped heads: rows [key | value] per key/value head.
 //
-// One CTA = (key range of a slot, block of 16 heads).  A producer warp brings 32-token tiles (two 16-token pages, one
+// One CTA = (key range of a slot, block of up to 16 heads of one key/value head).  A producer warp brings 32-token tiles (two 16-token pages, one
 // tensor-map TMA box each, 128-byte swizzle, no multicast) through a ring of mbarrier-tracked stages; eight warps work on
 // a tile together:
-//     S[16 x 32]    = q' . rows^T     a warp takes 16 tokens and every fourth 32-wide step of the row
+//     S[16 x 32]    = q . keys^T      a warp takes 16 tokens and every fourth 32-wide step of the key part
 //     P             = exp2(S - m)     half a warp per head row, two tokens per lane; online maximum and sum in fp32
-//     O[16 x rank] += P . latents     a warp owns rank / 8 columns; accumulators stay in registers
-// The kernel is bound by HBM (about 2 * 16 FLOP per byte), far below what 16-row tiles reach on tcgen05 (M = 128), so
+//     O[16 x rank] += P . values      a warp owns rank / 8 columns; accumulators stay in registers
+// The kernel is bound by HBM (at most 2 * 16 FLOP per byte), far below what 16-row tiles reach on tcgen05 (M = 128), so
 // mma.sync carries the products, as in the paged decode kernels.  Key ranges leave (max, sum, unnormalised O) in fp32;
-// latent_value merges them.  Rows of a tile outside the visible range are zeroed in shared memory before they are used:
+// row_merge_kernel merges them.  Rows of a tile outside the visible range are zeroed in shared memory before they are used:
 // whatever a page held for an earlier owner cannot reach the sums.  Every wait is bounded.
 #include <mutex>
 
@@ -30,16 +31,16 @@ constexpr int LD_SMEM_PAIR = 102 * 1024;          // ... when two CTAs share an 
 // NT: value columns per warp / 8 that the accumulators hold (rank <= 64 * NT)
 template <int NT>
 __global__ void __launch_bounds__(LD_THREADS, NT <= 8 ? 2 : 1)
-latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_constant__ CUtensorMap map_rows, int stages) {
+row_decode_kernel(const __grid_constant__ RowDecodeParams p, const __grid_constant__ CUtensorMap map_rows, int stages) {
   extern __shared__ __align__(1024) uint8_t ld_smem_raw[];
   __shared__ uint64_t full[LD_MAX_STAGES], empty[LD_MAX_STAGES];
   __shared__ float ss[4][16][LD_S_PITCH];            // partial scores of the four quarters of a row
   __shared__ __align__(16) __nv_bfloat16 ps[16][LD_P_PITCH];
   __shared__ float alphas[16];
-  const int split = blockIdx.x, hb = blockIdx.y, b = blockIdx.z;
+  const int blocks = (p.group + 15) / 16, split = blockIdx.x, g = blockIdx.y / blocks, hb = blockIdx.y % blocks, b = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int pitch = p.rank + p.rot, row_bytes = pitch * 2, tile_bytes = LD_TOK * row_bytes, page_bytes = PAGE * row_bytes;
-  const int q_pitch = row_bytes + 16;
+  const int row_bytes = p.pitch * 2, tile_bytes = LD_TOK * row_bytes, page_bytes = PAGE * row_bytes;
+  const int q_pitch = p.key * 2 + 16;
   uint8_t* ring = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ld_smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* qs = ring + stages * tile_bytes;
   if (tid == 0) {
@@ -53,8 +54,8 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
   pdl_wait();
   int lo, hi;
   latent_split_range(p, b, split, lo, hi);
-  const int heads_here = min(16, p.heads - hb * 16);
-  const int64_t part0 = (static_cast<int64_t>(b) * p.heads + hb * 16) * p.splits + split;
+  const int heads_here = min(16, p.group - hb * 16), head0 = g * p.group + hb * 16;
+  const int64_t part0 = (static_cast<int64_t>(b) * p.heads + head0) * p.splits + split;
   if (lo >= hi) {
     if (tid < heads_here) p.ml[part0 + static_cast<int64_t>(tid) * p.splits] = make_float2(-INFINITY, 0.f);
     return;
@@ -72,18 +73,17 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
         const int n = min(2, pages - 2 * t);
         mbar_expect_tx(&full[s], n * page_bytes);
         for (int i = 0; i < n; ++i)
-          tma_load_3d(ring + s * tile_bytes + i * page_bytes, &map_rows, 0, table[2 * t + i] * PAGE, 0, &full[s]);
+          tma_load_3d(ring + s * tile_bytes + i * page_bytes, &map_rows, 0, (table[2 * t + i] * p.kv_heads + g) * PAGE, 0, &full[s]);
       }
       __syncwarp();
     }
     if (!ok && lane == 0) atomicExch(p.err, 1);
     return;
   }
-  // q' rows of the head block (rows past the last head are zero)
+  // q rows of the head block (rows past the last head are zero)
   {
-    const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) +
-                                                    (static_cast<int64_t>(b) * p.heads + hb * 16) * pitch);
-    const int vecs = row_bytes / 16;
+    const uint4* q = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q) + b * p.q_stride + static_cast<int64_t>(head0) * p.key);
+    const int vecs = p.key / 8;
     for (int i = tid; i < 16 * vecs; i += LD_WARPS * 32) {
       const int r = i / vecs, c = i % vecs;
       *reinterpret_cast<uint4*>(qs + r * q_pitch + c * 16) = r < heads_here ? q[r * vecs + c] : make_uint4(0, 0, 0, 0);
@@ -97,8 +97,9 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
   const int sm_row = warp * 2 + (lane >> 4), sm_tok = (lane & 15) * 2;
   const float scale_log2 = p.scale * 1.4426950408889634f;
   const int tg = warp & 1, kq = warp >> 1;
-  const int units = pitch / 32;
+  const int units = p.key / 32;
   const int nt = p.rank / 64, col0 = warp * nt * 8;
+  const int v_chunk = (p.v_off + col0) / 8, last_chunk = p.pitch / 8 - 1;
   const uint32_t a_base = smem_u32(qs) + (lane & 15) * q_pitch + (lane >> 4) * 16;
   const int s_row = lane & 7;   // rows s_row and s_row + 8 of page tg
   const uint32_t s_off = tg * page_bytes + s_row * 128;
@@ -186,7 +187,7 @@ latent_decode_kernel(const __grid_constant__ LatentDecodeParams p, const __grid_
         for (int i = 0; i < NT; i += 2) {
           if (i < nt) {
             uint32_t bm[4];
-            const int chunk = col0 / 8 + i + (lane >> 4);
+            const int chunk = min(v_chunk + i + (lane >> 4), last_chunk);  // an odd last pair's second half is not used
             ldmatrix_x4_trans(bm, v_row + (chunk >> 3) * (PAGE * 128) + (((chunk & 7) ^ (lane & 7)) << 4));
             mma_bf16_16816(acc[i], a, bm[0], bm[1]);
             if (NT > 1 && i + 1 < nt) mma_bf16_16816(acc[i + 1 < NT ? i + 1 : i], a, bm[2], bm[3]);
@@ -244,20 +245,46 @@ static bool row_map(CUtensorMap* out, const void* base, int64_t rows, int pitch)
 }
 
 template <int NT>
-static int launch_latent_decode(const LatentDecodeParams& p, const CUtensorMap& map, int batch, int stages, int smem,
+static int launch_row_decode(const RowDecodeParams& p, const CUtensorMap& map, int batch, int stages, int smem,
                                 cudaStream_t st) {
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(latent_decode_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT) != cudaSuccess)
-      return fail(ERR_RUNTIME, "latent_decode: cannot raise dynamic shared memory to %d", LD_SMEM_LIMIT);
+    if (cudaFuncSetAttribute(row_decode_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT) != cudaSuccess)
+      return fail(ERR_RUNTIME, "row_decode: cannot raise dynamic shared memory to %d", LD_SMEM_LIMIT);
     configured[dev] = true;
   }
-  if (launch_pdl((p.overlap & OVERLAP_START) != 0, latent_decode_kernel<NT>, dim3(p.splits, (p.heads + 15) / 16, batch),
-                 dim3(LD_THREADS), smem, st, p, map, stages) != cudaSuccess)
-    return fail(ERR_LAUNCH, "latent_decode: %s", cudaGetErrorString(cudaGetLastError()));
-  return check_launch("latent_decode");
+  const dim3 grid(p.splits, p.kv_heads * ((p.group + 15) / 16), batch);
+  if (launch_pdl((p.overlap & OVERLAP_START) != 0, row_decode_kernel<NT>, grid, dim3(LD_THREADS), smem, st, p, map, stages) != cudaSuccess)
+    return fail(ERR_LAUNCH, "row_decode: %s", cudaGetErrorString(cudaGetLastError()));
+  return check_launch("row_decode");
+}
+
+int row_decode_launch(const RowDecodeParams& in, int64_t num_pages, int batch, const char* name, cudaStream_t st) {
+  B200_REQUIRE(in.key > 0 && in.key % 32 == 0 && in.rank > 0 && in.rank % 64 == 0 && in.rank <= 1024 && in.pitch % 64 == 0 &&
+                   in.v_off % 8 == 0 && in.key <= in.pitch && in.v_off + in.rank <= in.pitch && in.q_stride % 8 == 0,
+               "%s: keys must be a multiple of 32, values and rows of 64, at most 1024 value columns (got %d, %d, %d)", name, in.key,
+               in.rank, in.pitch);
+  B200_REQUIRE(in.window > 0 && in.splits > 0 && in.splits <= LATENT_MAX_SPLITS && batch <= 65535 && in.scale > 0.f && num_pages > 0 &&
+                   in.kv_heads > 0 && in.heads == in.kv_heads * in.group && num_pages * in.kv_heads * PAGE < (1ll << 31),
+               "%s: window, scale and splits (at most %d) must be positive, heads a multiple of the key/value heads", name,
+               LATENT_MAX_SPLITS);
+  B200_REQUIRE(aligned16(in.q) && aligned16(in.cache) && aligned16(in.o), "%s: unaligned tensor", name);
+  RowDecodeParams p = in;
+  const int tile = LD_TOK * p.pitch * 2, q_bytes = 16 * (p.key * 2 + 16) + 1024;  // incl. alignment of the ring
+  int stages = p.rank <= 512 ? (LD_SMEM_PAIR - q_bytes) / tile : 0;   // two CTAs on an SM cover each other's latencies
+  if (stages < 2) stages = (LD_SMEM_LIMIT - q_bytes) / tile;
+  if (stages > LD_MAX_STAGES) stages = LD_MAX_STAGES;
+  B200_REQUIRE(stages >= 2, "%s: rows of %d elements do not fit", name, p.pitch);
+  p.err = wait_timeout_flag();
+  if (!p.err) return fail(ERR_RUNTIME, "%s: no error flag", name);
+  CUtensorMap map;
+  if (!row_map(&map, p.cache, num_pages * p.kv_heads * PAGE, p.pitch)) return fail(ERR_RUNTIME, "%s: cannot encode the cache's tensor map", name);
+  const int smem = stages * tile + q_bytes;
+  if (p.rank <= 128) return launch_row_decode<2>(p, map, batch, stages, smem, st);
+  if (p.rank <= 512) return launch_row_decode<8>(p, map, batch, stages, smem, st);
+  return launch_row_decode<16>(p, map, batch, stages, smem, st);
 }
 
 }  // namespace b200
@@ -269,24 +296,10 @@ extern "C" int b200_latent_decode(const void* q, const void* cache, int64_t num_
                                   int32_t batch, int32_t heads, int32_t rank, int32_t rot, int32_t window, int32_t splits,
                                   float scale, int32_t overlap, b200_stream_t stream) {
   if (batch <= 0) return OK;
-  B200_REQUIRE(rank > 0 && rank % 64 == 0 && rank <= 1024 && rot >= 0 && rot % 64 == 0 && heads > 0,
-               "latent_decode: rank and rot must be multiples of 64, rank at most 1024 (got %d, %d)", rank, rot);
-  B200_REQUIRE(window > 0 && splits > 0 && splits <= LATENT_MAX_SPLITS && batch <= 65535 && scale > 0.f && num_pages > 0,
-               "latent_decode: window, scale and splits (at most %d) must be positive", LATENT_MAX_SPLITS);
-  B200_REQUIRE(aligned16(q) && aligned16(cache) && aligned16(o), "latent_decode: unaligned tensor");
-  const int pitch = rank + rot, tile = LD_TOK * pitch * 2, q_bytes = 16 * (pitch * 2 + 16) + 1024;  // incl. alignment of the ring
-  int stages = rank <= 512 ? (LD_SMEM_PAIR - q_bytes) / tile : 0;   // two CTAs on an SM cover each other's latencies
-  if (stages < 2) stages = (LD_SMEM_LIMIT - q_bytes) / tile;
-  if (stages > LD_MAX_STAGES) stages = LD_MAX_STAGES;
-  B200_REQUIRE(stages >= 2, "latent_decode: rows of %d elements do not fit", pitch);
-  LatentDecodeParams p = {q, cache, block_table, table_stride, pos, active, reinterpret_cast<float2*>(ml), o,
-                          heads, rank, rot, window, splits, overlap, scale, wait_timeout_flag()};
-  if (!p.err) return fail(ERR_RUNTIME, "latent_decode: no error flag");
-  CUtensorMap map;
-  if (!row_map(&map, cache, num_pages * PAGE, pitch)) return fail(ERR_RUNTIME, "latent_decode: cannot encode the cache's tensor map");
-  const int smem = stages * tile + q_bytes;
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  if (rank <= 128) return launch_latent_decode<2>(p, map, batch, stages, smem, st);
-  if (rank <= 512) return launch_latent_decode<8>(p, map, batch, stages, smem, st);
-  return launch_latent_decode<16>(p, map, batch, stages, smem, st);
+  B200_REQUIRE(rank > 0 && rank % 64 == 0 && rot >= 0 && rot % 64 == 0 && heads > 0,
+               "latent_decode: rank and rot must be multiples of 64 (got %d, %d)", rank, rot);
+  const RowDecodeParams p = {q, static_cast<int64_t>(heads) * (rank + rot), cache, block_table, table_stride, pos, active,
+                             reinterpret_cast<float2*>(ml), o, heads, 1, heads, rank + rot, 0, rank, rank + rot, window, splits,
+                             overlap, scale, nullptr};
+  return row_decode_launch(p, num_pages, batch, "latent_decode", reinterpret_cast<cudaStream_t>(stream));
 }

@@ -1,8 +1,11 @@
-// Windowed causal attention of packed prompt portions over expanded latents, on tcgen05 (bf16, accumulators in TMEM).
+// Windowed causal attention of packed prompt portions on tcgen05 (bf16, accumulators in TMEM), over expanded latents or over
+// the keys and values of grouped heads.
 //
-// One CTA = 128 query tokens of one head of one sequence.  Keys are [expanded part of the head | rotated part shared by
-// all heads]: two TMA boxes per 128-key tile land side by side as the column blocks of one K-major operand, so the shared
-// part is never copied per head.  Per tile:
+// One CTA = 128 query tokens of one head of one sequence.  Latent keys are [expanded part of the head | rotated part shared
+// by all heads]: two TMA boxes per 128-key tile land side by side as the column blocks of one K-major operand, so the shared
+// part is never copied per head.  Grouped heads: `group` query heads read the same key/value head, keys are one box; a key
+// size that is no multiple of 64 brings columns of its neighbour along, which no product reads.  The epilogue may multiply
+// by sigmoid(gate) and a constant.  Per tile:
 //     S[128 x 128]   = Q . K^T            tcgen05.mma, both operands in shared memory, two S buffers in TMEM
 //     P              = exp2(S*scale - m)  two softmax threads per row, TMEM -> registers -> TMEM (bf16 over S)
 //     O[128 x vdim] += P . V              tcgen05.mma, P from TMEM, V as an MN-major operand
@@ -25,8 +28,11 @@ constexpr int LP_SMEM_LIMIT = 220 * 1024;
 
 struct LatentUmmaParams {
   __nv_bfloat16* out;
+  const __nv_bfloat16* gate;      // [tokens, gate_stride] or NULL
+  int64_t out_stride, gate_stride;
+  float out_scale;
   const int32_t *cu_q, *cu_k, *q_pos0, *k_pos0;
-  int heads, vdim, dim_blocks, rot_blocks, dim_steps, rot_steps, window, k_stages, v_stages;
+  int group, vdim, dim_blocks, rot_blocks, dim_steps, rot_steps, window, k_stages, v_stages;
   float scale_log2;
   int* err;
 };
@@ -40,7 +46,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   __shared__ uint32_t tmem_slot;
   __shared__ float xm[2][2][128];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int qb = gridDim.x - 1 - blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+  const int qb = gridDim.x - 1 - blockIdx.x, h = blockIdx.y, b = blockIdx.z, g = h / p.group;
   const int q_row0 = p.cu_q[b], len = p.cu_q[b + 1] - q_row0;
   const int q0 = qb * LP_TILE;
   if (q0 >= len) return;
@@ -84,8 +90,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (i >= 0) ok = mbar_wait_bounded(&bar_s[i & 1], (i >> 1) & 1);  // S of the tile that used this stage is done
         if (!ok) break;
         mbar_expect_tx(&bar_k[st], k_bytes);
-        tma_load_4d(k_s + st * k_bytes, &map_k, 0, k_row0 + j * LP_TILE, 0, h, &bar_k[st]);
-        tma_load_3d(k_s + st * k_bytes + p.dim_blocks * LP_BLOCK_BYTES, &map_r, 0, k_row0 + j * LP_TILE, 0, &bar_k[st]);
+        tma_load_4d(k_s + st * k_bytes, &map_k, 0, k_row0 + j * LP_TILE, 0, g, &bar_k[st]);
+        if (p.rot_blocks > 0) tma_load_3d(k_s + st * k_bytes + p.dim_blocks * LP_BLOCK_BYTES, &map_r, 0, k_row0 + j * LP_TILE, 0, &bar_k[st]);
       }
       if (!ok) atomicExch(p.err, 1);
     }
@@ -97,7 +103,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (i >= 0) ok = mbar_wait_bounded(&bar_pv[i & 1], (i >> 1) & 1);
         if (!ok) break;
         mbar_expect_tx(&bar_v[st], v_bytes);
-        tma_load_4d(v_s + st * v_bytes, &map_v, 0, k_row0 + j * LP_TILE, 0, h, &bar_v[st]);
+        tma_load_4d(v_s + st * v_bytes, &map_v, 0, k_row0 + j * LP_TILE, 0, g, &bar_v[st]);
       }
       if (!ok) atomicExch(p.err, 1);
     }
@@ -257,15 +263,91 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       const int vecs = p.vdim / 8;
       for (int i = tid; i < LP_TILE * vecs; i += LP_SOFTMAX_THREADS) {
         const int r = i / vecs, c = i % vecs;
-        if (q0 + r < len)
-          *reinterpret_cast<uint4*>(p.out + (static_cast<int64_t>(q_row0 + q0 + r) * p.heads + h) * p.vdim + c * 8) =
-              *reinterpret_cast<const uint4*>(smem + r * out_pitch + c * 16);
+        if (q0 + r >= len) continue;
+        const int64_t row_at = q_row0 + q0 + r;
+        uint4 o = *reinterpret_cast<const uint4*>(smem + r * out_pitch + c * 16);
+        if (p.gate) {
+          float f[8], z[8];
+          load8(reinterpret_cast<const __nv_bfloat16*>(&o), f);
+          load8(p.gate + row_at * p.gate_stride + h * p.vdim + c * 8, z);
+#pragma unroll
+          for (int k = 0; k < 8; ++k) f[k] *= sigmoid_f<__nv_bfloat16>(z[k]) * p.out_scale;
+          store8(reinterpret_cast<__nv_bfloat16*>(&o), f);
+        }
+        *reinterpret_cast<uint4*>(p.out + row_at * p.out_stride + h * p.vdim + c * 8) = o;
       }
     }
   }
   tc_fence_before_sync();
   __syncthreads();
   if (warp == 0) tmem_dealloc(tmem, LP_TMEM_COLS);
+}
+
+// A strided matrix of `heads` parts, `blocks` column blocks of 64 each, as the 4-D tensor {64, rows, blocks, heads}
+static bool head_map(CUtensorMap* map, const void* base, uint64_t rows, int64_t row_stride, int blocks, int64_t head_stride, int heads) {
+  const uint64_t dims[4] = {64, rows, static_cast<uint64_t>(blocks), static_cast<uint64_t>(heads)};
+  const uint64_t st[3] = {static_cast<uint64_t>(row_stride) * 2, 128, static_cast<uint64_t>(head_stride) * 2};
+  const uint32_t box[4] = {64, LP_TILE, static_cast<uint32_t>(blocks), 1};
+  return encode_map_bf16_sw128(map, base, 4, dims, st, box);
+}
+
+int row_prefill_launch(const RowPrefillOperands& a, const char* name, cudaStream_t st) {
+  B200_REQUIRE(a.dim > 0 && a.rot % 64 == 0 && a.vdim > 0 && a.vdim % 64 == 0 && a.dim + a.rot <= 256 && a.vdim <= 256 &&
+                   (a.rot == 0 || a.dim % 64 == 0),
+               "%s: keys and values of at most 256, in multiples of 64 (got %d, %d, %d)", name, a.dim, a.rot, a.vdim);
+  B200_REQUIRE(a.true_dim > 0 && a.true_dim <= a.dim && a.true_rot <= a.rot && a.window > 0 && a.scale > 0.f && a.tokens > 0 && a.keys > 0,
+               "%s: bad true sizes, window or scale", name);
+  B200_REQUIRE(a.heads > 0 && a.heads <= 65535 && a.batch <= 65535 && a.group > 0 && a.heads % a.group == 0,
+               "%s: at most 65535 heads and sequences", name);
+  B200_REQUIRE(aligned16(a.q) && aligned16(a.k) && aligned16(a.r) && aligned16(a.v) && aligned16(a.out) && aligned16(a.gate) &&
+                   a.out_stride % 8 == 0 && a.gate_stride % 8 == 0,
+               "%s: unaligned tensor", name);
+  const int dim_blocks = (a.dim + 63) / 64, rot_blocks = a.rot / 64, kv_heads = a.heads / a.group;
+  const int head_width = a.dim + a.rot;
+  B200_REQUIRE(a.q_stride >= static_cast<int64_t>(a.heads - 1) * head_width + (dim_blocks + rot_blocks) * 64,
+               "%s: rows of q end inside the last head's column blocks", name);
+  CUtensorMap map_q, map_k, map_r = {}, map_v;
+  if (!head_map(&map_q, a.q, a.tokens, a.q_stride, dim_blocks + rot_blocks, head_width, a.heads) ||
+      !head_map(&map_k, a.k, a.keys, a.k_stride, dim_blocks, a.k_head, kv_heads) ||
+      !head_map(&map_v, a.v, a.keys, a.v_stride, a.vdim / 64, a.v_head, kv_heads))
+    return fail(ERR_RUNTIME, "%s: cannot encode a tensor map", name);
+  if (rot_blocks > 0) {
+    const uint64_t dims[3] = {64, static_cast<uint64_t>(a.keys), static_cast<uint64_t>(rot_blocks)};
+    const uint64_t strides[2] = {static_cast<uint64_t>(a.r_stride) * 2, 128};
+    const uint32_t box[3] = {64, LP_TILE, static_cast<uint32_t>(rot_blocks)};
+    if (!encode_map_bf16_sw128(&map_r, a.r, 3, dims, strides, box))
+      return fail(ERR_RUNTIME, "%s: cannot encode the shared part's tensor map", name);
+  }
+  LatentUmmaParams p = {};
+  p.out = static_cast<__nv_bfloat16*>(a.out);
+  p.gate = static_cast<const __nv_bfloat16*>(a.gate);
+  p.out_stride = a.out_stride, p.gate_stride = a.gate_stride, p.out_scale = a.out_scale;
+  p.cu_q = a.cu_q, p.cu_k = a.cu_k, p.q_pos0 = a.q_pos0, p.k_pos0 = a.k_pos0;
+  p.group = a.group, p.vdim = a.vdim, p.dim_blocks = dim_blocks, p.rot_blocks = rot_blocks;
+  p.dim_steps = (a.true_dim + 15) / 16, p.rot_steps = (a.true_rot + 15) / 16;
+  p.window = a.window;
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.err = wait_timeout_flag();
+  if (!p.err) return fail(ERR_RUNTIME, "%s: no error flag", name);
+  const int k_bytes = (dim_blocks + rot_blocks) * LP_BLOCK_BYTES, v_bytes = a.vdim / 64 * LP_BLOCK_BYTES;
+  p.k_stages = 2, p.v_stages = 2;
+  auto smem_for = [&] { return k_bytes * (1 + p.k_stages) + v_bytes * p.v_stages + 1024; };
+  if (smem_for() > LP_SMEM_LIMIT) p.v_stages = 1;
+  if (smem_for() > LP_SMEM_LIMIT) p.k_stages = 1;
+  int smem = smem_for();
+  // the epilogue stages rows of vdim * 2 + 16 bytes over the operands
+  if (smem < LP_TILE * (a.vdim * 2 + 16) + 1024) smem = LP_TILE * (a.vdim * 2 + 16) + 1024;
+  static bool configured[64] = {false};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (dev >= 0 && dev < 64 && !configured[dev]) {
+    if (cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LP_SMEM_LIMIT) != cudaSuccess)
+      return fail(ERR_RUNTIME, "%s: cannot raise dynamic shared memory to %d", name, LP_SMEM_LIMIT);
+    configured[dev] = true;
+  }
+  latent_prefill_kernel<<<dim3((a.max_q + LP_TILE - 1) / LP_TILE, a.heads, a.batch), LP_THREADS, smem, st>>>(map_q, map_k, map_r,
+                                                                                                            map_v, p);
+  return check_launch(name);
 }
 
 }  // namespace b200
@@ -278,63 +360,17 @@ extern "C" int b200_latent_prefill(const void* q, const void* kv, const void* ct
                                    int32_t rot, int32_t true_rot, int32_t vdim, int32_t rank, int32_t window, float scale,
                                    b200_stream_t stream) {
   if (batch <= 0 || max_q <= 0) return OK;
-  B200_REQUIRE(dim > 0 && rot > 0 && vdim > 0 && dim % 64 == 0 && rot % 64 == 0 && vdim % 64 == 0 && rank % 64 == 0 &&
-                   dim + rot <= 256 && vdim <= 256,
-               "latent_prefill: sizes must be multiples of 64, dim + rot and vdim at most 256 (got %d, %d, %d)", dim, rot, vdim);
-  B200_REQUIRE(true_dim > 0 && true_dim <= dim && true_rot > 0 && true_rot <= rot && window > 0 && scale > 0.f &&
-                   tokens > 0 && keys > 0,
-               "latent_prefill: bad true sizes, window or scale");
-  B200_REQUIRE(heads > 0 && heads <= 65535 && batch <= 65535, "latent_prefill: at most 65535 heads and sequences");
-  B200_REQUIRE(aligned16(q) && aligned16(kv) && aligned16(ctx) && aligned16(out), "latent_prefill: unaligned tensor");
-  const uint64_t H = heads, T = tokens, K = keys;
-  const uint64_t width = dim + rot, kv_row = H * (dim + vdim) * 2;
-  CUtensorMap map_q, map_k, map_r, map_v;
-  {
-    const uint64_t dims[4] = {64, T, width / 64, H}, st[3] = {H * width * 2, 128, width * 2};
-    const uint32_t box[4] = {64, LP_TILE, static_cast<uint32_t>(width / 64), 1};
-    if (!encode_map_bf16_sw128(&map_q, q, 4, dims, st, box)) return fail(ERR_RUNTIME, "latent_prefill: cannot encode q's tensor map");
-  }
-  {
-    const uint64_t dims[4] = {64, K, static_cast<uint64_t>(dim / 64), H}, st[3] = {kv_row, 128, static_cast<uint64_t>(dim) * 2};
-    const uint32_t box[4] = {64, LP_TILE, static_cast<uint32_t>(dim / 64), 1};
-    if (!encode_map_bf16_sw128(&map_k, kv, 4, dims, st, box)) return fail(ERR_RUNTIME, "latent_prefill: cannot encode k's tensor map");
-  }
-  {
-    const uint64_t dims[3] = {64, K, static_cast<uint64_t>(rot / 64)}, st[2] = {static_cast<uint64_t>(rank + rot) * 2, 128};
-    const uint32_t box[3] = {64, LP_TILE, static_cast<uint32_t>(rot / 64)};
-    if (!encode_map_bf16_sw128(&map_r, static_cast<const __nv_bfloat16*>(ctx) + rank, 3, dims, st, box))
-      return fail(ERR_RUNTIME, "latent_prefill: cannot encode the rotated part's tensor map");
-  }
-  {
-    const uint64_t dims[4] = {64, K, static_cast<uint64_t>(vdim / 64), H}, st[3] = {kv_row, 128, static_cast<uint64_t>(vdim) * 2};
-    const uint32_t box[4] = {64, LP_TILE, static_cast<uint32_t>(vdim / 64), 1};
-    if (!encode_map_bf16_sw128(&map_v, static_cast<const __nv_bfloat16*>(kv) + H * dim, 4, dims, st, box))
-      return fail(ERR_RUNTIME, "latent_prefill: cannot encode v's tensor map");
-  }
-  LatentUmmaParams p = {};
-  p.out = static_cast<__nv_bfloat16*>(out);
-  p.cu_q = cu_q, p.cu_k = cu_k, p.q_pos0 = q_pos0, p.k_pos0 = k_pos0;
-  p.heads = heads, p.vdim = vdim, p.dim_blocks = dim / 64, p.rot_blocks = rot / 64;
-  p.dim_steps = (true_dim + 15) / 16, p.rot_steps = (true_rot + 15) / 16;
-  p.window = window;
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.err = wait_timeout_flag();
-  if (!p.err) return fail(ERR_RUNTIME, "latent_prefill: no error flag");
-  const int k_bytes = (p.dim_blocks + p.rot_blocks) * LP_BLOCK_BYTES, v_bytes = vdim / 64 * LP_BLOCK_BYTES;
-  p.k_stages = 2, p.v_stages = 2;
-  auto smem_for = [&] { return k_bytes * (1 + p.k_stages) + v_bytes * p.v_stages + 1024; };
-  if (smem_for() > LP_SMEM_LIMIT) p.v_stages = 1;
-  if (smem_for() > LP_SMEM_LIMIT) p.k_stages = 1;
-  const int smem = smem_for();
-  static bool configured[64] = {false};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, LP_SMEM_LIMIT) != cudaSuccess)
-      return fail(ERR_RUNTIME, "latent_prefill: cannot raise dynamic shared memory to %d", LP_SMEM_LIMIT);
-    configured[dev] = true;
-  }
-  latent_prefill_kernel<<<dim3((max_q + LP_TILE - 1) / LP_TILE, heads, batch), LP_THREADS, smem,
-                          reinterpret_cast<cudaStream_t>(stream)>>>(map_q, map_k, map_r, map_v, p);
-  return check_launch("latent_prefill");
+  B200_REQUIRE(dim > 0 && dim % 64 == 0 && rot > 0 && rank % 64 == 0 && true_rot > 0, "latent_prefill: sizes must be multiples of 64");
+  const int64_t kv_row = static_cast<int64_t>(heads) * (dim + vdim), ctx_row = rank + rot;
+  RowPrefillOperands a = {};
+  a.q = q, a.q_stride = static_cast<int64_t>(heads) * (dim + rot);
+  a.k = kv, a.k_stride = kv_row, a.k_head = dim;
+  a.r = static_cast<const __nv_bfloat16*>(ctx) + rank, a.r_stride = ctx_row;
+  a.v = static_cast<const __nv_bfloat16*>(kv) + static_cast<int64_t>(heads) * dim, a.v_stride = kv_row, a.v_head = vdim;
+  a.out = out, a.out_stride = static_cast<int64_t>(heads) * vdim;
+  a.cu_q = cu_q, a.cu_k = cu_k, a.q_pos0 = q_pos0, a.k_pos0 = k_pos0;
+  a.batch = batch, a.max_q = max_q, a.tokens = tokens, a.keys = keys, a.heads = heads, a.group = 1;
+  a.dim = dim, a.true_dim = true_dim, a.rot = rot, a.true_rot = true_rot, a.vdim = vdim, a.window = window;
+  a.scale = scale, a.out_scale = 1.f;
+  return row_prefill_launch(a, "latent_prefill", reinterpret_cast<cudaStream_t>(stream));
 }

@@ -7,12 +7,11 @@
 //     Prefill: a CTA walks a sequence in blocks of 64 tokens, its warps scan 8 tokens each in parallel.  Too few CTAs:
 //     sequences are cut into segments; pass 1 reduces a segment to (product of 1 - z, state it leaves from zero), pass 2
 //     folds the segments in front of its own.  HBM bound.
-//   Forget-gated outer-product recurrence (HGRN2 form):  f = l + (1 - l) sigmoid(f' + fb), q = silu(q')
-//                           S_t = diag(f) S_(t-1) + (1 - f) v^T,   o = S_t^T q,   out = rms(o) * w per head
-//     Prefill of bf16 activations runs in chunks on the tensor cores (linear_rnn_chunk.cu).  The token-serial form here is
-//     plain fp32, for fp32 activations and for heads wider than 128: a warp owns COLS state columns, a lane dim/32 rows
-//     of each as packed fp32 pairs (fma.rn.f32x2); 16 tokens of gates are staged in shared memory at a time, the next 16
-//     are loaded while they are worked on.
+//   Outer-product recurrences (linear_rnn.cuh: HGRN2, gated linear attention, state space).
+//     Prefill of bf16 activations runs in chunks on the tensor cores (linear_rnn_chunk.cu, ssd.cu).  The token-serial form
+//     here is plain fp32, for fp32 activations and for heads wider than 128: a warp owns COLS state columns, a lane dim/32
+//     rows of each as packed fp32 pairs (fma.rn.f32x2); 16 tokens of gates are staged in shared memory at a time, the next
+//     16 are loaded while they are worked on.
 #include "b200_attn.h"
 #include "elem.cuh"
 #include "linear_rnn.cuh"
@@ -168,7 +167,7 @@ __global__ void __launch_bounds__(128) mingru_decode_kernel(const E* zxg, int64_
          make_float4(s.x * silu_f<E>(g.x), s.y * silu_f<E>(g.y), s.z * silu_f<E>(g.z), s.w * silu_f<E>(g.w)));
 }
 
-// ------------------------------------------------------------------------------------------------------------- HGRN2
+// ------------------------------------------------------------------------------------------ outer-product recurrences
 // packed fp32 pairs
 struct F2 {
   uint64_t v;
@@ -201,31 +200,34 @@ constexpr int OR_THREADS = OR_WARPS * 32;
 // RP = row pairs per lane (dim = 64 * RP, or dim = 32 with RP = 1 and the second row of a pair absent -> dim is padded
 // to a multiple of 64 by the caller of this template), COLS = columns per warp.
 // grid (vdim / (4 * COLS), heads, sequences)
-template <typename E, int RP, int COLS>
+template <typename E, int RP, int COLS, RnnKind KIND>
 __global__ void __launch_bounds__(OR_THREADS) outer_rnn_prefill_kernel(const __grid_constant__ OuterRnnParams p) {
   constexpr int DIM = 64 * RP;                       // rows incl. padding
   constexpr int CT = OR_WARPS * COLS;                // columns of the CTA
   constexpr int CPT = (DIM + OR_THREADS - 1) / OR_THREADS;  // gate channels per thread
+  constexpr bool KEYS = KIND != RNN_FORGET;          // keys of their own
   extern __shared__ __align__(16) float or_smem[];
   float* fs = or_smem;                               // [2][TB][DIM]
   float* qs = fs + 2 * OR_TB * DIM;                  // [2][TB][DIM]
-  float* vs = qs + 2 * OR_TB * DIM;                  // [2][TB][CT][2]  every v twice: a ready-made pair
+  float* ks = qs + 2 * OR_TB * DIM;                  // [2][TB][DIM] when KEYS
+  float* vs = ks + (KEYS ? 2 * OR_TB * DIM : 0);     // [2][TB][CT][2]  every v twice: a ready-made pair
   float* os = vs + 2 * OR_TB * CT * 2;               // [TB][CT]
   const int seq = blockIdx.z, head = blockIdx.y, col0 = blockIdx.x * CT;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int row0 = p.cu[seq], len = p.cu[seq + 1] - row0;
   if (len <= 0) return;
-  const int hd = p.heads * p.dim;
-  const E* base = static_cast<const E*>(p.qfv) + static_cast<int64_t>(row0) * p.stride;
-  float low[CPT], fb[CPT];
+  const E* base = static_cast<const E*>(p.x) + static_cast<int64_t>(row0) * p.stride;
+  const int qk_col = (head / p.per_group) * p.dim, v_col = p.v_off + head * p.vdim;
+  float low[CPT], fb[CPT], dt_b = 0.f, rate = 0.f, skip = 0.f;
 #pragma unroll
   for (int i = 0; i < CPT; ++i) {
     const int ch = tid + i * OR_THREADS;
-    low[i] = ch < p.dim ? p.lower[head * p.dim + ch] : 0.f;
-    fb[i] = ch < p.dim ? p.bias[head * p.dim + ch] : 0.f;
+    low[i] = KIND == RNN_FORGET && ch < p.dim ? p.lower[head * p.dim + ch] : 0.f;
+    fb[i] = KIND != RNN_SSD && ch < p.dim ? p.bias[head * p.dim + ch] : 0.f;
   }
+  if (KIND == RNN_SSD) dt_b = p.bias[head], rate = expf(p.a_log[head]), skip = p.skip[head];
   // the raw rows of the next block travel in registers
-  float rq[CPT][OR_TB], rf[CPT][OR_TB], rv[(OR_TB * CT + OR_THREADS - 1) / OR_THREADS];
+  float rq[CPT][OR_TB], rf[CPT][OR_TB], rz[KIND == RNN_KEYED ? CPT : 1][OR_TB], rv[(OR_TB * CT + OR_THREADS - 1) / OR_THREADS];
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < CPT; ++i) {
@@ -234,34 +236,57 @@ __global__ void __launch_bounds__(OR_THREADS) outer_rnn_prefill_kernel(const __g
 #pragma unroll
         for (int t = 0; t < OR_TB; ++t)
           if (t0 + t < len) {
-            const E* r = base + static_cast<int64_t>(t0 + t) * p.stride + head * p.dim + ch;
-            rq[i][t] = load1(r);
-            rf[i][t] = load1(r + hd);
+            const E* r = base + static_cast<int64_t>(t0 + t) * p.stride + qk_col + ch;
+            rq[i][t] = load1(r + p.q_off);
+            rf[i][t] = load1(r + p.k_off);
+            if constexpr (KIND == RNN_KEYED) rz[i][t] = p.z[static_cast<int64_t>(row0 + t0 + t) * p.z_stride + head * p.dim + ch];
           }
       }
+    }
+    if constexpr (KIND == RNN_SSD) {
+#pragma unroll
+      for (int t = 0; t < OR_TB; ++t)
+        if (t0 + t < len) rz[0][t] = load1(static_cast<const E*>(p.dt) + static_cast<int64_t>(row0 + t0 + t) * p.dt_stride + head);
     }
 #pragma unroll
     for (int i = 0; i < (OR_TB * CT + OR_THREADS - 1) / OR_THREADS; ++i) {
       const int e = tid + i * OR_THREADS, t = e / CT, c = e % CT;
       rv[i] = 0.f;
       if (e < OR_TB * CT && t0 + t < len && col0 + c < p.vdim)
-        rv[i] = load1(base + static_cast<int64_t>(t0 + t) * p.stride + 2 * hd + head * p.vdim + col0 + c);
+        rv[i] = load1(base + static_cast<int64_t>(t0 + t) * p.stride + v_col + col0 + c);
     }
   };
   auto stage = [&](int t0, int buf) {
 #pragma unroll
-    for (int i = 0; i < CPT; ++i) {
-      const int ch = tid + i * OR_THREADS;
-      if (ch < DIM) {
+    for (int t = 0; t < OR_TB; ++t) {
+      const bool in = t0 + t < len;
+      float dt = 0.f, decay = 1.f;
+      if (KIND == RNN_SSD && in) {
+        dt = softplus_f(rz[0][t] + dt_b);
+        decay = expf(-rate * dt);
+      }
 #pragma unroll
-        for (int t = 0; t < OR_TB; ++t) {
-          float q = 0.f, f = 1.f;                    // padding rows and tokens: keep the state, read nothing
-          if (ch < p.dim && t0 + t < len) {
-            q = silu_f<E>(rq[i][t]);
-            f = low[i] + (1.0f - low[i]) * sigmoid_f<E>(rf[i][t] + fb[i]);
+      for (int i = 0; i < CPT; ++i) {
+        const int ch = tid + i * OR_THREADS;
+        if (ch < DIM) {
+          float q = 0.f, f = 1.f, k = 0.f;           // padding rows and tokens: keep the state, read and add nothing
+          if (ch < p.dim && in) {
+            if constexpr (KIND == RNN_FORGET) {
+              q = silu_f<E>(rq[i][t]);
+              f = low[i] + (1.0f - low[i]) * sigmoid_f<E>(rf[i][t] + fb[i]);
+            } else if constexpr (KIND == RNN_KEYED) {
+              q = rq[i][t] * p.q_scale;
+              k = rf[i][t];
+              f = sigmoid_root<E>(rz[i][t] + fb[i], p.inv_tau);
+            } else {
+              q = rq[i][t];
+              k = rf[i][t] * dt;
+              f = decay;
+            }
           }
           fs[(buf * OR_TB + t) * DIM + ch] = f;
           qs[(buf * OR_TB + t) * DIM + ch] = q;
+          if (KEYS) ks[(buf * OR_TB + t) * DIM + ch] = k;
         }
       }
     }
@@ -298,6 +323,7 @@ __global__ void __launch_bounds__(OR_THREADS) outer_rnn_prefill_kernel(const __g
     const int n = min(OR_TB, len - t0);
     const float* fsb = fs + buf * OR_TB * DIM + lane * 2 * RP;
     const float* qsb = qs + buf * OR_TB * DIM + lane * 2 * RP;
+    const float* ksb = ks + buf * OR_TB * DIM + lane * 2 * RP;
     const float* vsb = vs + (buf * OR_TB * CT + warp * COLS) * 2;
 #pragma unroll 2
     for (int t = 0; t < n; ++t) {
@@ -308,7 +334,12 @@ __global__ void __launch_bounds__(OR_THREADS) outer_rnn_prefill_kernel(const __g
         const float2 b = *reinterpret_cast<const float2*>(qsb + t * DIM + 2 * i);
         f[i] = f2(a.x, a.y);
         q[i] = f2(b.x, b.y);
-        k[i] = f2(1.0f - a.x, 1.0f - a.y);
+        if constexpr (KEYS) {
+          const float2 c = *reinterpret_cast<const float2*>(ksb + t * DIM + 2 * i);
+          k[i] = f2(c.x, c.y);
+        } else {
+          k[i] = f2(1.0f - a.x, 1.0f - a.y);
+        }
       }
 #pragma unroll
       for (int c = 0; c < COLS; c += 2) {
@@ -349,7 +380,8 @@ __global__ void __launch_bounds__(OR_THREADS) outer_rnn_prefill_kernel(const __g
     __syncthreads();
     for (int e = tid; e < n * CT; e += OR_THREADS) {
       const int t = e / CT, c = e % CT;
-      if (col0 + c < p.vdim) p.o[static_cast<int64_t>(row0 + t0 + t) * p.heads * p.vdim + head * p.vdim + col0 + c] = os[e];
+      if (col0 + c < p.vdim) p.o[static_cast<int64_t>(row0 + t0 + t) * p.heads * p.vdim + head * p.vdim + col0 + c] =
+            KIND == RNN_SSD ? fmaf(skip, vs[(buf * OR_TB * CT + e) * 2], os[e]) : os[e];
     }
     __syncthreads();
   }
@@ -366,58 +398,100 @@ __global__ void __launch_bounds__(OR_THREADS) outer_rnn_prefill_kernel(const __g
     }
 }
 
-// out[r, :] = o[r, :] / sqrt(mean(o^2) + eps) * w for rows (token, head); one warp per row
+// out = o / sqrt(mean(o^2) + eps) * w (* silu(gate)) for rows (token, head); one warp per row
 template <typename E>
-__global__ void __launch_bounds__(256) head_rms_kernel(const float* o, const float* w, E* out, int64_t rows, int vdim,
-                                                       int true_vdim, float eps) {
+__global__ void __launch_bounds__(256) head_rms_kernel(const __grid_constant__ OuterRnnParams p, int64_t rows) {
   const int64_t r = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (r >= rows) return;
-  const float* x = o + r * vdim;
+  const float* x = p.o + r * p.vdim;
+  const int64_t token = r / p.heads;
+  const int col = static_cast<int>(r - token * p.heads) * p.vdim;
+  const E* gate = p.gate ? static_cast<const E*>(p.gate) + token * p.gate_stride + col : nullptr;
+  E* out = static_cast<E*>(p.out) + token * p.out_stride + col;
   float sq = 0.f;
-  for (int c = lane * 4; c < vdim; c += 128) {
+  for (int c = lane * 4; c < p.vdim; c += 128) {
     const float4 a = load4(x + c);
     sq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
   }
-  const float scale = 1.0f / sqrtf(warp_sum(sq) / static_cast<float>(true_vdim) + eps);
-  for (int c = lane * 4; c < vdim; c += 128) {
-    const float4 a = load4(x + c), g = load4(w + c);
-    store4(out + r * vdim + c, make_float4(a.x * scale * g.x, a.y * scale * g.y, a.z * scale * g.z, a.w * scale * g.w));
+  const float scale = 1.0f / sqrtf(warp_sum(sq) / static_cast<float>(p.true_vdim) + p.eps);
+  for (int c = lane * 4; c < p.vdim; c += 128) {
+    const float4 a = load4(x + c), w = load4(p.norm + c);
+    float4 y = make_float4(a.x * scale * w.x, a.y * scale * w.y, a.z * scale * w.z, a.w * scale * w.w);
+    if (gate) {
+      const float4 g = load4(gate + c);
+      y.x *= silu_f<E>(g.x), y.y *= silu_f<E>(g.y), y.z *= silu_f<E>(g.z), y.w *= silu_f<E>(g.w);
+    }
+    store4(out + c, y);
   }
 }
 
 // One token per slot, one CTA per (head, slot): state in, state out, head norm inside.  A warp walks rows, its lanes
-// cover the columns four at a time (several rows at once when vdim < 128).
+// cover the columns four at a time (several rows at once when vdim < 128).  State space: the convolution of the head's
+// inputs is inside; a ring of `taps` raw inputs per channel is written at pos % taps, which no CTA reads in this step.
 constexpr int OD_WARPS = 8;
 constexpr int OD_MAX_VDIM = 512;
-template <typename E>
-__global__ void __launch_bounds__(OD_WARPS * 32)
-outer_rnn_decode_kernel(const E* qfv, int64_t stride, const float* lower, const float* bias, const float* norm, float* state,
-                        const int64_t* pos, const int64_t* active, E* out, int heads, int dim, int vdim, int true_vdim,
-                        float eps, int lanes_per_row, int overlap) {
+template <typename E, RnnKind KIND>
+__global__ void __launch_bounds__(OD_WARPS * 32) outer_rnn_decode_kernel(const __grid_constant__ OuterRnnParams p) {
+  constexpr bool KEYS = KIND != RNN_FORGET;
   extern __shared__ __align__(16) float od_smem[];
+  const int dim = p.dim, vdim = p.vdim, heads = p.heads;
   float* fs = od_smem;            // [dim]
   float* qs = fs + dim;           // [dim]
-  float* vv = qs + dim;           // [vdim]
+  float* ks = qs + dim;           // [dim] when KEYS
+  float* vv = ks + (KEYS ? dim : 0);   // [vdim]
   float* part = vv + vdim;        // [OD_WARPS][vdim]
   __shared__ float red[32];
   const int head = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  if (overlap & OVERLAP_TRIGGER) pdl_trigger();
+  if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
   pdl_wait();
-  const bool on = !active || active[b] != 0;
-  const bool fresh = pos[b] == 0;
-  const E* row = qfv + b * stride;
-  const int hd = heads * dim;
-  for (int i = tid; i < dim; i += OD_WARPS * 32) {
-    const int ch = head * dim + i;
-    const float l = lower[ch];
-    qs[i] = silu_f<E>(load1(row + ch));
-    fs[i] = l + (1.0f - l) * sigmoid_f<E>(load1(row + hd + ch) + bias[ch]);
+  const bool on = !p.active || p.active[b] != 0;
+  const int64_t pos = p.pos[b];
+  const bool fresh = pos == 0;
+  const E* row = static_cast<const E*>(p.x) + b * p.stride;
+  const int qk_col = (head / p.per_group) * dim, v_col = p.v_off + head * vdim;
+  if constexpr (KIND == RNN_SSD) {
+    const float dt = softplus_f(load1(static_cast<const E*>(p.dt) + b * p.dt_stride + head) + p.bias[head]);
+    const float decay = expf(-expf(p.a_log[head]) * dt);
+    const int now = static_cast<int>(pos % p.taps), back = static_cast<int>(pos < p.taps - 1 ? pos : p.taps - 1);
+    float* ring = p.ring + static_cast<int64_t>(b) * p.taps * p.channels;
+    const bool first = head % p.per_group == 0;       // writes the group's inputs
+    for (int i = tid; i < 2 * dim + vdim; i += OD_WARPS * 32) {
+      const int c = i < dim ? p.q_off + qk_col + i : i < 2 * dim ? p.k_off + qk_col + i - dim : v_col + i - 2 * dim;
+      const float raw = load1(row + c);
+      float acc = fmaf(p.taps_w[c], raw, p.taps_b[c]);
+      for (int j = 1; j <= back; ++j)
+        acc = fmaf(p.taps_w[j * p.channels + c], ring[static_cast<int64_t>(now - j < 0 ? now - j + p.taps : now - j) * p.channels + c], acc);
+      const float y = silu_f<E>(acc);
+      if (i < dim) qs[i] = y, fs[i] = decay;
+      else if (i < 2 * dim) ks[i - dim] = y * dt;
+      else vv[i - 2 * dim] = y;
+      if (on && (i >= 2 * dim || first)) ring[static_cast<int64_t>(now) * p.channels + c] = raw;
+    }
+  } else {
+    for (int i = tid; i < dim; i += OD_WARPS * 32) {
+      const int ch = head * dim + i;
+      if constexpr (KIND == RNN_FORGET) {
+        const float l = p.lower[ch];
+        qs[i] = silu_f<E>(load1(row + p.q_off + ch));
+        fs[i] = l + (1.0f - l) * sigmoid_f<E>(load1(row + p.k_off + ch) + p.bias[ch]);
+      } else {
+        float z = p.bias[ch];
+        const E *w = static_cast<const E*>(p.w_low) + static_cast<int64_t>(ch) * p.rank, *a = static_cast<const E*>(p.low) + b * p.stride;
+        for (int r = 0; r < p.rank; r += 4) {
+          const float4 x = load4(a + r), y = load4(w + r);
+          z = fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, z))));
+        }
+        qs[i] = load1(row + p.q_off + ch) * p.q_scale;
+        ks[i] = load1(row + p.k_off + ch);
+        fs[i] = sigmoid_root<E>(z, p.inv_tau);
+      }
+    }
+    for (int i = tid; i < vdim; i += OD_WARPS * 32) vv[i] = load1(row + v_col + i);
   }
-  for (int i = tid; i < vdim; i += OD_WARPS * 32) vv[i] = load1(row + 2 * hd + head * vdim + i);
   __syncthreads();
-  float* st = state + (static_cast<int64_t>(b) * heads + head) * dim * vdim;
-  const int rows_at_once = 32 / lanes_per_row, sub = lane / lanes_per_row, cl = (lane % lanes_per_row) * 4;
+  float* st = p.state + (static_cast<int64_t>(b) * heads + head) * dim * vdim;
+  const int rows_at_once = 32 / p.lanes_per_row, sub = lane / p.lanes_per_row, cl = (lane % p.lanes_per_row) * 4;
   for (int c0 = 0; c0 < vdim; c0 += 128) {
     const int c = c0 + cl;
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -436,7 +510,7 @@ outer_rnn_decode_kernel(const E* qfv, int64_t stride, const float* lower, const 
         for (int u = 0; u < U; ++u) {
           const int r = r0 + u * step;
           if (r < dim) {
-            const float f = fs[r], k = 1.0f - f, q = qs[r];
+            const float f = fs[r], k = KEYS ? ks[r] : 1.0f - f, q = qs[r];
             s[u].x = fmaf(f, s[u].x, k * v.x), s[u].y = fmaf(f, s[u].y, k * v.y);
             s[u].z = fmaf(f, s[u].z, k * v.z), s[u].w = fmaf(f, s[u].w, k * v.w);
             if (on) store4(st + static_cast<int64_t>(r) * vdim + c, s[u]);
@@ -446,7 +520,7 @@ outer_rnn_decode_kernel(const E* qfv, int64_t stride, const float* lower, const 
         }
       }
     }
-    for (int bit = lanes_per_row; bit < 32; bit <<= 1) {
+    for (int bit = p.lanes_per_row; bit < 32; bit <<= 1) {
       o.x += __shfl_xor_sync(0xffffffffu, o.x, bit), o.y += __shfl_xor_sync(0xffffffffu, o.y, bit);
       o.z += __shfl_xor_sync(0xffffffffu, o.z, bit), o.w += __shfl_xor_sync(0xffffffffu, o.w, bit);
     }
@@ -463,47 +537,105 @@ outer_rnn_decode_kernel(const E* qfv, int64_t stride, const float* lower, const 
       for (int w = 0; w < OD_WARPS; ++w) sum[i] += part[w * vdim + c];
     sq[0] += sum[i] * sum[i];
   }
+  if constexpr (KIND == RNN_SSD) {
+#pragma unroll
+    for (int i = 0; i < OD_MAX_VDIM / (OD_WARPS * 32); ++i) {
+      const int c = tid + i * OD_WARPS * 32;
+      if (c < vdim) p.o[(static_cast<int64_t>(b) * heads + head) * vdim + c] = fmaf(p.skip[head], vv[c], sum[i]);
+    }
+    return;
+  }
   block_sum<1>(sq, red);
-  const float scale = 1.0f / sqrtf(sq[0] / static_cast<float>(true_vdim) + eps);
+  const float scale = 1.0f / sqrtf(sq[0] / static_cast<float>(p.true_vdim) + p.eps);
 #pragma unroll
   for (int i = 0; i < OD_MAX_VDIM / (OD_WARPS * 32); ++i) {
     const int c = tid + i * OD_WARPS * 32;
-    if (c < vdim) store1(out + (static_cast<int64_t>(b) * heads + head) * vdim + c, sum[i] * scale * norm[c]);
+    if (c < vdim) {
+      float y = sum[i] * scale * p.norm[c];
+      if (p.gate) y *= silu_f<E>(load1(static_cast<const E*>(p.gate) + b * p.gate_stride + head * vdim + c));
+      store1(static_cast<E*>(p.out) + b * p.out_stride + head * vdim + c, y);
+    }
   }
 }
 
-template <typename E, int RP, int COLS>
+template <typename E, int RP, int COLS, RnnKind KIND>
 static int launch_outer_cols(const OuterRnnParams& p, int n, cudaStream_t st) {
   constexpr int DIM = 64 * RP, CT = OR_WARPS * COLS;
-  constexpr int smem = (4 * OR_TB * DIM + 2 * OR_TB * CT * 2 + OR_TB * CT) * 4;
+  constexpr int smem = ((KIND == RNN_FORGET ? 4 : 6) * OR_TB * DIM + 2 * OR_TB * CT * 2 + OR_TB * CT) * 4;
   static_assert(smem <= 200 * 1024, "staging must fit");
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (smem > 48 * 1024 && dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(outer_rnn_prefill_kernel<E, RP, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
-      return fail(ERR_RUNTIME, "hgrn2_prefill: cannot raise dynamic shared memory to %d", smem);
+    if (cudaFuncSetAttribute(outer_rnn_prefill_kernel<E, RP, COLS, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      return fail(ERR_RUNTIME, "outer_rnn: cannot raise dynamic shared memory to %d", smem);
     configured[dev] = true;
   }
-  outer_rnn_prefill_kernel<E, RP, COLS><<<dim3((p.vdim + CT - 1) / CT, p.heads, n), OR_THREADS, smem, st>>>(p);
-  return check_launch("hgrn2_prefill");
+  outer_rnn_prefill_kernel<E, RP, COLS, KIND><<<dim3((p.vdim + CT - 1) / CT, p.heads, n), OR_THREADS, smem, st>>>(p);
+  return check_launch("outer_rnn (token by token)");
 }
 
-template <typename E, int RP>
+template <typename E, int RP, RnnKind KIND>
 static int launch_outer(const OuterRnnParams& p, int n, cudaStream_t st) {
   // wide columns share the gates of a token among more state; narrow ones give more CTAs when there are few heads
   const int64_t wide = static_cast<int64_t>((p.vdim + 31) / 32) * p.heads * n;
   if constexpr (RP <= 2) {
-    if (wide >= 2 * sm_count()) return launch_outer_cols<E, RP, 8>(p, n, st);
+    if (wide >= 2 * sm_count()) return launch_outer_cols<E, RP, 8, KIND>(p, n, st);
   }
-  return launch_outer_cols<E, RP, 4>(p, n, st);
+  return launch_outer_cols<E, RP, 4, KIND>(p, n, st);
 }
 
-template <typename E>
+template <typename E, RnnKind KIND>
 static int launch_outer_rows(const OuterRnnParams& p, int n, cudaStream_t st) {
-  if (p.dim <= 64) return launch_outer<E, 1>(p, n, st);
-  if (p.dim <= 128) return launch_outer<E, 2>(p, n, st);
-  return launch_outer<E, 4>(p, n, st);
+  if (p.dim <= 64) return launch_outer<E, 1, KIND>(p, n, st);
+  if (p.dim <= 128) return launch_outer<E, 2, KIND>(p, n, st);
+  return launch_outer<E, 4, KIND>(p, n, st);
+}
+
+int outer_rnn_serial_launch(const OuterRnnParams& p, RnnKind kind, bool f32, int n, cudaStream_t st) {
+  B200_REQUIRE(p.dim <= 256, "outer_rnn: at most 256 state rows (got %d)", p.dim);
+  if (kind == RNN_FORGET) return f32 ? launch_outer_rows<float, RNN_FORGET>(p, n, st) : launch_outer_rows<__nv_bfloat16, RNN_FORGET>(p, n, st);
+  if (kind == RNN_KEYED) return f32 ? launch_outer_rows<float, RNN_KEYED>(p, n, st) : launch_outer_rows<__nv_bfloat16, RNN_KEYED>(p, n, st);
+  return f32 ? launch_outer_rows<float, RNN_SSD>(p, n, st) : launch_outer_rows<__nv_bfloat16, RNN_SSD>(p, n, st);
+}
+
+template <typename E, RnnKind KIND>
+static cudaError_t launch_outer_decode(const OuterRnnParams& p, int batch, int smem, cudaStream_t st) {
+  return launch_pdl((p.overlap & OVERLAP_START) != 0, outer_rnn_decode_kernel<E, KIND>, dim3(p.heads, batch), dim3(OD_WARPS * 32), smem, st, p);
+}
+
+int outer_rnn_decode_launch(OuterRnnParams p, RnnKind kind, bool f32, int batch, const char* name, cudaStream_t st) {
+  B200_REQUIRE(p.dim > 0 && p.dim <= 1024 && p.vdim > 0 && p.vdim % 4 == 0 && p.vdim <= OD_MAX_VDIM && p.true_vdim <= p.vdim,
+               "%s: dim at most 1024, vdim a multiple of 4 and at most %d (got %d, %d)", name, OD_MAX_VDIM, p.dim, p.vdim);
+  B200_REQUIRE(p.heads > 0 && p.per_group > 0 && batch <= 65535 && aligned16(p.state), "%s: unaligned state or too many slots", name);
+  p.lanes_per_row = 1;
+  while (p.lanes_per_row < 32 && p.lanes_per_row * 4 < p.vdim) p.lanes_per_row <<= 1;
+  const int smem = ((kind == RNN_FORGET ? 2 : 3) * p.dim + p.vdim + OD_WARPS * p.vdim) * 4 + 16;
+  cudaError_t e;
+  if (kind == RNN_FORGET) e = f32 ? launch_outer_decode<float, RNN_FORGET>(p, batch, smem, st) : launch_outer_decode<__nv_bfloat16, RNN_FORGET>(p, batch, smem, st);
+  else if (kind == RNN_KEYED) e = f32 ? launch_outer_decode<float, RNN_KEYED>(p, batch, smem, st) : launch_outer_decode<__nv_bfloat16, RNN_KEYED>(p, batch, smem, st);
+  else e = f32 ? launch_outer_decode<float, RNN_SSD>(p, batch, smem, st) : launch_outer_decode<__nv_bfloat16, RNN_SSD>(p, batch, smem, st);
+  if (e != cudaSuccess) return fail(ERR_LAUNCH, "%s: %s", name, cudaGetErrorString(e));
+  return check_launch(name);
+}
+
+// FORGET and KEYED, any length: chunks where the shape fits, else token by token; the head norm inside or behind
+static int outer_rnn_prefill(OuterRnnParams p, RnnKind kind, bool f32, bool serial, int n, int tokens, cudaStream_t st) {
+  float* const scratch = p.o;
+  const bool chunked = !f32 && !serial && outer_rnn_chunk_supports(p.dim, p.vdim) && p.stride % 8 == 0 && p.q_off % 8 == 0 &&
+                       p.k_off % 8 == 0 && p.v_off % 8 == 0 && p.z_stride % 4 == 0 && aligned16(p.x);
+  void* const out = p.out;
+  if (chunked && p.vdim <= 128) return outer_rnn_chunk_launch(p, kind, n, st);  // the head norm inside: one launch
+  B200_REQUIRE(scratch, "outer_rnn: this shape needs a scratch tensor");
+  p.out = nullptr;
+  const int rc = chunked ? outer_rnn_chunk_launch(p, kind, n, st) : outer_rnn_serial_launch(p, kind, f32, n, st);
+  if (rc != OK) return rc;
+  p.out = out;
+  const int64_t rows = static_cast<int64_t>(tokens) * p.heads;
+  const unsigned grid = static_cast<unsigned>((rows + 7) / 8);
+  if (f32) head_rms_kernel<float><<<grid, 256, 0, st>>>(p, rows);
+  else head_rms_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(p, rows);
+  return check_launch("outer_rnn (norm)");
 }
 
 }  // namespace b200
@@ -571,22 +703,13 @@ extern "C" int b200_hgrn2_prefill(const void* qfv, int64_t stride, const float* 
                "hgrn2_prefill: dim at most 256, vdim a multiple of 4 and at most %d (got %d, %d)", OD_MAX_VDIM, dim, vdim);
   B200_REQUIRE(heads > 0 && heads <= 65535 && batch <= 65535, "hgrn2_prefill: at most 65535 heads and sequences");
   B200_REQUIRE(aligned16(o_scratch) && aligned16(out) && aligned16(norm), "hgrn2_prefill: unaligned tensor");
-  OuterRnnParams p = {qfv, stride, lower, bias, state, cu_seqlens, slots, start, o_scratch, heads, dim, vdim,
-                      norm, nullptr, true_vdim, eps, segment, segments, workspace,
-                      workspace ? workspace + static_cast<int64_t>(batch) * segments * heads * dim * vdim : nullptr};
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const bool chunked = !f32 && !serial && outer_rnn_chunk_supports(dim, vdim) && stride % 8 == 0 && heads * dim % 8 == 0 && aligned16(qfv);
-  if (chunked && vdim <= 128) {  // the head norm inside: one launch
-    p.out = out;
-    return outer_rnn_chunk_launch(p, batch, st);
-  }
-  const int rc = chunked ? outer_rnn_chunk_launch(p, batch, st) : f32 ? launch_outer_rows<float>(p, batch, st) : launch_outer_rows<__nv_bfloat16>(p, batch, st);
-  if (rc != OK) return rc;
-  const int64_t rows = static_cast<int64_t>(tokens) * heads;
-  const unsigned grid = static_cast<unsigned>((rows + 7) / 8);
-  if (f32) head_rms_kernel<float><<<grid, 256, 0, st>>>(o_scratch, norm, static_cast<float*>(out), rows, vdim, true_vdim, eps);
-  else head_rms_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(o_scratch, norm, static_cast<__nv_bfloat16*>(out), rows, vdim, true_vdim, eps);
-  return check_launch("hgrn2_prefill (norm)");
+  OuterRnnParams p = {};
+  p.x = qfv, p.stride = stride, p.q_off = 0, p.k_off = heads * dim, p.v_off = 2 * heads * dim, p.per_group = 1;
+  p.lower = lower, p.bias = bias, p.state = state, p.cu = cu_seqlens, p.slots = slots, p.start = start, p.o = o_scratch;
+  p.heads = heads, p.dim = dim, p.vdim = vdim, p.norm = norm, p.out = out, p.out_stride = static_cast<int64_t>(heads) * vdim;
+  p.true_vdim = true_vdim, p.eps = eps, p.segment = segment, p.segments = segments, p.seg_state = workspace;
+  p.seg_decay = workspace ? workspace + static_cast<int64_t>(batch) * segments * heads * dim * vdim : nullptr;
+  return outer_rnn_prefill(p, RNN_FORGET, f32 != 0, serial != 0, batch, tokens, reinterpret_cast<cudaStream_t>(stream));
 }
 
 extern "C" int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* lower, const float* bias, const float* norm,
@@ -594,22 +717,53 @@ extern "C" int b200_hgrn2_decode(const void* qfv, int64_t stride, const float* l
                                  int32_t heads, int32_t dim, int32_t vdim, int32_t true_vdim, float eps, int32_t f32,
                                  int32_t overlap, b200_stream_t stream) {
   if (batch <= 0) return OK;
-  B200_REQUIRE(dim > 0 && dim <= 1024 && vdim > 0 && vdim % 4 == 0 && vdim <= OD_MAX_VDIM && true_vdim <= vdim,
-               "hgrn2_decode: dim at most 1024, vdim a multiple of 4 and at most %d (got %d, %d)", OD_MAX_VDIM, dim, vdim);
-  B200_REQUIRE(heads > 0 && batch <= 65535 && aligned16(state), "hgrn2_decode: unaligned state or too many slots");
-  int lanes = 1;
-  while (lanes < 32 && lanes * 4 < vdim) lanes <<= 1;
-  const int smem = (2 * dim + vdim + OD_WARPS * vdim) * 4 + 16;
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  const bool early = (overlap & OVERLAP_START) != 0;
-  const dim3 grid(heads, batch);
-  const cudaError_t e =
-      f32 ? launch_pdl(early, outer_rnn_decode_kernel<float>, grid, dim3(OD_WARPS * 32), smem, st, static_cast<const float*>(qfv),
-                       stride, lower, bias, norm, state, pos, active, static_cast<float*>(out), heads, dim, vdim, true_vdim,
-                       eps, lanes, overlap)
-          : launch_pdl(early, outer_rnn_decode_kernel<__nv_bfloat16>, grid, dim3(OD_WARPS * 32), smem, st,
-                       static_cast<const __nv_bfloat16*>(qfv), stride, lower, bias, norm, state, pos, active,
-                       static_cast<__nv_bfloat16*>(out), heads, dim, vdim, true_vdim, eps, lanes, overlap);
-  if (e != cudaSuccess) return fail(ERR_LAUNCH, "hgrn2_decode: %s", cudaGetErrorString(e));
-  return check_launch("hgrn2_decode");
+  OuterRnnParams p = {};
+  p.x = qfv, p.stride = stride, p.q_off = 0, p.k_off = heads * dim, p.v_off = 2 * heads * dim, p.per_group = 1;
+  p.lower = lower, p.bias = bias, p.state = state, p.heads = heads, p.dim = dim, p.vdim = vdim, p.norm = norm;
+  p.out = out, p.out_stride = static_cast<int64_t>(heads) * vdim, p.true_vdim = true_vdim, p.eps = eps;
+  p.pos = pos, p.active = active, p.overlap = overlap;
+  return outer_rnn_decode_launch(p, RNN_FORGET, f32 != 0, batch, "hgrn2_decode", reinterpret_cast<cudaStream_t>(stream));
+}
+
+extern "C" int b200_gla_prefill(const void* qkv, int64_t stride, const float* z, int64_t z_stride, const float* bias,
+                                const float* norm, const void* gate, int64_t gate_stride, float* state,
+                                const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start, float* o_scratch,
+                                void* out, int64_t out_stride, int32_t batch, int32_t tokens, int32_t heads, int32_t dim,
+                                int32_t vdim, int32_t true_vdim, float q_scale, float inv_tau, float eps, int32_t f32,
+                                int32_t serial, int32_t segment, int32_t segments, float* workspace, b200_stream_t stream) {
+  if (batch <= 0 || tokens <= 0) return OK;
+  B200_REQUIRE(segment > 0 && segments > 0 && (segments == 1 || (segment % 16 == 0 && workspace && aligned16(workspace))),
+               "gla_prefill: segments must be multiples of 16 tokens and have a workspace");
+  B200_REQUIRE(dim > 0 && dim <= 256 && vdim > 0 && vdim % 4 == 0 && vdim <= OD_MAX_VDIM && true_vdim <= vdim,
+               "gla_prefill: dim at most 256, vdim a multiple of 4 and at most %d (got %d, %d)", OD_MAX_VDIM, dim, vdim);
+  B200_REQUIRE(heads > 0 && heads <= 65535 && static_cast<int64_t>(batch) * segments <= 65535, "gla_prefill: too many heads or segments");
+  B200_REQUIRE(aligned16(z) && aligned16(gate) && aligned16(o_scratch) && aligned16(out) && aligned16(norm) &&
+                   gate_stride % 8 == 0 && out_stride % 8 == 0,
+               "gla_prefill: unaligned tensor");
+  OuterRnnParams p = {};
+  p.x = qkv, p.stride = stride, p.q_off = 0, p.k_off = heads * dim, p.v_off = 2 * heads * dim, p.per_group = 1;
+  p.z = z, p.z_stride = z_stride, p.bias = bias, p.q_scale = q_scale, p.inv_tau = inv_tau;
+  p.state = state, p.cu = cu_seqlens, p.slots = slots, p.start = start, p.o = o_scratch;
+  p.heads = heads, p.dim = dim, p.vdim = vdim, p.norm = norm, p.gate = gate, p.gate_stride = gate_stride;
+  p.out = out, p.out_stride = out_stride, p.true_vdim = true_vdim, p.eps = eps;
+  p.segment = segment, p.segments = segments, p.seg_state = workspace;
+  p.seg_decay = workspace ? workspace + static_cast<int64_t>(batch) * segments * heads * dim * vdim : nullptr;
+  return outer_rnn_prefill(p, RNN_KEYED, f32 != 0, serial != 0, batch, tokens, reinterpret_cast<cudaStream_t>(stream));
+}
+
+extern "C" int b200_gla_decode(const void* qkv, int64_t stride, const void* low, const void* w_low, int32_t rank,
+                               const float* bias, const float* norm, const void* gate, int64_t gate_stride, float* state,
+                               const int64_t* pos, const int64_t* active, void* out, int64_t out_stride, int32_t batch,
+                               int32_t heads, int32_t dim, int32_t vdim, int32_t true_vdim, float q_scale, float inv_tau,
+                               float eps, int32_t f32, int32_t overlap, b200_stream_t stream) {
+  if (batch <= 0) return OK;
+  B200_REQUIRE(rank > 0 && rank % 4 == 0 && stride % 4 == 0 && aligned16(low) && aligned16(w_low),
+               "gla_decode: the rank and the stride must be multiples of 4, tensors 16-byte aligned");
+  OuterRnnParams p = {};
+  p.x = qkv, p.stride = stride, p.q_off = 0, p.k_off = heads * dim, p.v_off = 2 * heads * dim, p.per_group = 1;
+  p.low = low, p.w_low = w_low, p.rank = rank, p.bias = bias, p.q_scale = q_scale, p.inv_tau = inv_tau;
+  p.state = state, p.heads = heads, p.dim = dim, p.vdim = vdim, p.norm = norm, p.gate = gate, p.gate_stride = gate_stride;
+  p.out = out, p.out_stride = out_stride, p.true_vdim = true_vdim, p.eps = eps;
+  p.pos = pos, p.active = active, p.overlap = overlap;
+  return outer_rnn_decode_launch(p, RNN_KEYED, f32 != 0, batch, "gla_decode", reinterpret_cast<cudaStream_t>(stream));
 }

@@ -1,12 +1,12 @@
-// Prefill of the forget-gated outer-product recurrence (HGRN2 form, linear_rnn.cu) in chunks of 16 tokens on the tensor
-// cores, for bf16 activations and head sizes up to 128:
-//     S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T,   o_t = S_t^T q_t,   out = rms(o) * w per head
+// Prefill of the outer-product recurrences with a decay per key channel (linear_rnn.cuh, FORGET and KEYED) in chunks of 16
+// tokens on the tensor cores, for bf16 activations and head sizes up to 128:
+//     S_t = diag(f_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   out = rms(o) * w (* silu(gate)) per head
 // With B_t = f_1 .. f_t and R_s = f_(s+1) .. f_16 inside a chunk (products of numbers <= 1: they can only shrink, no
 // quotient of them is ever formed):
-//     o_t    = S_0^T (q_t B_t) + sum_(s<=t) A_ts v_s,     A_ts = sum_d q_td (1 - f_sd) f_(s+1)d .. f_td
-//     S_16^T = S_0^T diag(B_16) + V^T (K R),              K = 1 - f
+//     o_t    = S_0^T (q_t B_t) + sum_(s<=t) A_ts v_s,     A_ts = sum_d q_td k_sd f_(s+1)d .. f_td
+//     S_16^T = S_0^T diag(B_16) + V^T (K R),              FORGET: k = 1 - f
 // One CTA = one head of one sequence (and up to 128 value columns).  Per chunk:
-//   gates   silu, forget gates and biases of the chunk's raw rows (brought in by cp.async a chunk ahead) -> shared fp32
+//   gates   activations, decays and biases of the chunk's raw rows (brought in by cp.async a chunk ahead) -> shared fp32
 //   decays  running products forward (q B) and backward (K R) per channel, by half of the warps; A on the CUDA cores in
 //           fp32, half a warp per key token with the decayed key carried in registers from query to query
 //   mma     a warp owns 16 value columns of S^T as fp32 accumulators of m16n8k16; the same registers, split into bf16
@@ -42,13 +42,14 @@ __device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, b
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(on ? 16 : 0) : "memory");
 }
 
-template <int D>
+template <int D, bool KEYED>
 struct ChunkSmem {
   static constexpr int FP = D + 4;   // fp32 row pitch
   static constexpr int BP = D + 8;   // bf16 row pitch: ldmatrix rows in different banks
   float fs[OC_C * FP], qs[OC_C * FP];
   __nv_bfloat16 qh[OC_C * BP], ql[OC_C * BP], kh[OC_C * BP], kl[OC_C * BP];
-  __nv_bfloat16 raw[2][OC_C * D];    // the next chunk's q and f rows as they come
+  __nv_bfloat16 raw[2][OC_C * D];    // the next chunk's q and f' (KEYED: k) rows as they come
+  float ks[KEYED ? OC_C * FP : 4], zs[KEYED ? OC_C * D : 4];   // keys; the next chunk's z rows
   __nv_bfloat16 vs[2][OC_C * OC_VP];
   float am[OC_C][OC_C + 2];
   float bc[D], total[D];
@@ -57,9 +58,9 @@ struct ChunkSmem {
 
 // D: channels incl. padding (32, 64 or 128).  LOCAL: only the state from zero and the total decay of every segment.
 // grid (vdim / 128, heads, sequences * segments)
-template <int D, bool LOCAL>
+template <int D, bool LOCAL, bool KEYED>
 __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __grid_constant__ OuterRnnParams p) {
-  using Smem = ChunkSmem<D>;
+  using Smem = ChunkSmem<D, KEYED>;
   constexpr int FP = Smem::FP, BP = Smem::BP;
   constexpr int ROW_VECS = D / 8, V_VECS = OC_VCOLS / 8;
   extern __shared__ __align__(16) uint8_t oc_smem[];
@@ -69,20 +70,26 @@ __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __
   const int all = p.cu[seq + 1] - p.cu[seq], seg0 = seg * p.segment;
   const int row0 = p.cu[seq] + seg0, len = min(all - seg0, p.segment);
   if (len <= 0 || (LOCAL && seg0 + len == all)) return;  // nothing follows a sequence's last segment
-  const int hd = p.heads * p.dim;
-  const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.qfv) + static_cast<int64_t>(row0) * p.stride;
+  const __nv_bfloat16* base = static_cast<const __nv_bfloat16*>(p.x) + static_cast<int64_t>(row0) * p.stride;
   auto fetch = [&](int t0, int buf) {
     for (int i = tid; i < OC_C * ROW_VECS; i += OC_THREADS) {
       const int t = i / ROW_VECS, c = (i % ROW_VECS) * 8;
       const bool on = t0 + t < len && c < p.dim;
       const __nv_bfloat16* r = base + static_cast<int64_t>(on ? t0 + t : 0) * p.stride + head * p.dim + (on ? c : 0);
-      if (!LOCAL) cp_async16_or_zero(&sm.raw[0][t * D + c], r, on);
-      cp_async16_or_zero(&sm.raw[1][t * D + c], r + hd, on);
+      if (!LOCAL) cp_async16_or_zero(&sm.raw[0][t * D + c], r + p.q_off, on);
+      cp_async16_or_zero(&sm.raw[1][t * D + c], r + p.k_off, on);
+    }
+    if constexpr (KEYED) {
+      for (int i = tid; i < OC_C * (D / 4); i += OC_THREADS) {
+        const int t = i / (D / 4), c = (i % (D / 4)) * 4;
+        const bool on = t0 + t < len && c < p.dim;
+        cp_async16_or_zero(&sm.zs[t * D + c], p.z + static_cast<int64_t>(row0 + (on ? t0 + t : 0)) * p.z_stride + head * p.dim + (on ? c : 0), on);
+      }
     }
     const int t = tid / V_VECS, c = (tid % V_VECS) * 8;
     const bool on = t0 + t < len && col0 + c < p.vdim;
     cp_async16_or_zero(&sm.vs[buf][t * OC_VP + c],
-                       base + static_cast<int64_t>(on ? t0 + t : 0) * p.stride + 2 * hd + head * p.vdim + (on ? col0 + c : 0), on);
+                       base + static_cast<int64_t>(on ? t0 + t : 0) * p.stride + p.v_off + head * p.vdim + (on ? col0 + c : 0), on);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   fetch(0, 0);
@@ -91,7 +98,7 @@ __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __
   const int ch = (tid % (D / 2)) * 2, grp = tid / (D / 2);
   float low0 = 0.f, low1 = 0.f, fb0 = 0.f, fb1 = 0.f;
   if (ch < p.dim) {
-    low0 = p.lower[head * p.dim + ch], low1 = p.lower[head * p.dim + ch + 1];
+    if (!KEYED) low0 = p.lower[head * p.dim + ch], low1 = p.lower[head * p.dim + ch + 1];
     fb0 = p.bias[head * p.dim + ch], fb1 = p.bias[head * p.dim + ch + 1];
   }
   for (int i = tid; i < OC_C * (OC_C + 2); i += OC_THREADS) (&sm.am[0][0])[i] = 0.f;  // A above the diagonal stays zero
@@ -123,16 +130,24 @@ __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __
     __syncthreads();  // the chunk's rows are here; everybody is done with the previous chunk
     // ---- gates
     for (int t = grp; t < OC_C; t += GROUPS) {
-      float2 q = make_float2(0.f, 0.f), f = make_float2(1.f, 1.f);   // padding keeps the state and reads nothing
+      float2 q = make_float2(0.f, 0.f), f = make_float2(1.f, 1.f), k = q;   // padding keeps the state and reads nothing
       if (ch < p.dim && t0 + t < len) {
         const uint32_t rf = *reinterpret_cast<const uint32_t*>(&sm.raw[1][t * D + ch]);
-        f = make_float2(low0 + (1.0f - low0) * sigmoid_f<__nv_bfloat16>(bf16_lo(rf) + fb0),
-                        low1 + (1.0f - low1) * sigmoid_f<__nv_bfloat16>(bf16_hi(rf) + fb1));
+        if constexpr (KEYED) {
+          const float2 z = *reinterpret_cast<const float2*>(&sm.zs[t * D + ch]);
+          f = make_float2(sigmoid_root<__nv_bfloat16>(z.x + fb0, p.inv_tau), sigmoid_root<__nv_bfloat16>(z.y + fb1, p.inv_tau));
+          k = make_float2(bf16_lo(rf), bf16_hi(rf));
+        } else {
+          f = make_float2(low0 + (1.0f - low0) * sigmoid_f<__nv_bfloat16>(bf16_lo(rf) + fb0),
+                          low1 + (1.0f - low1) * sigmoid_f<__nv_bfloat16>(bf16_hi(rf) + fb1));
+        }
         if (!LOCAL) {
           const uint32_t rq = *reinterpret_cast<const uint32_t*>(&sm.raw[0][t * D + ch]);
-          q = make_float2(silu_f<__nv_bfloat16>(bf16_lo(rq)), silu_f<__nv_bfloat16>(bf16_hi(rq)));
+          if constexpr (KEYED) q = make_float2(bf16_lo(rq) * p.q_scale, bf16_hi(rq) * p.q_scale);
+          else q = make_float2(silu_f<__nv_bfloat16>(bf16_lo(rq)), silu_f<__nv_bfloat16>(bf16_hi(rq)));
         }
       }
+      if constexpr (KEYED) *reinterpret_cast<float2*>(&sm.ks[t * FP + ch]) = k;
       *reinterpret_cast<float2*>(&sm.fs[t * FP + ch]) = f;
       if (!LOCAL) *reinterpret_cast<float2*>(&sm.qs[t * FP + ch]) = q;
     }
@@ -146,7 +161,7 @@ __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __
         for (int t = 0; t < OC_C; ++t) f[t] = sm.fs[t * FP + c];
 #pragma unroll
         for (int t = OC_C - 1; t >= 0; --t) {
-          split_store(&sm.kh[t * BP + c], &sm.kl[t * BP + c], (1.0f - f[t]) * run);
+          split_store(&sm.kh[t * BP + c], &sm.kl[t * BP + c], (KEYED ? sm.ks[t * FP + c] : 1.0f - f[t]) * run);
           run *= f[t];
         }
         sm.bc[c] = run;
@@ -179,9 +194,11 @@ __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __
             x[0] = a.x, x[1] = a.y;
           }
       };
-      row(sm.fs, s, g);
+      row(KEYED ? sm.ks : sm.fs, s, g);
+      if (!KEYED) {
 #pragma unroll
-      for (int c = 0; c < LC; ++c) g[c] = 1.0f - g[c];
+        for (int c = 0; c < LC; ++c) g[c] = 1.0f - g[c];
+      }
 #pragma unroll 4
       for (int t = 2 * warp; t < OC_C; ++t) {
         float f[LC], q[LC];
@@ -253,7 +270,6 @@ __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __
     if (LOCAL) continue;
     // ---- output rows lane / 4 and + 8, columns out_col (+ 1), + 8 (+ 9)
     const int t_lo = t0 + (lane >> 2), t_hi = t_lo + 8;
-    const int64_t step = static_cast<int64_t>(p.heads) * p.vdim;
     if (fused_norm) {
       float s_lo = o[0][0] * o[0][0] + o[0][1] * o[0][1] + o[1][0] * o[1][0] + o[1][1] * o[1][1];
       float s_hi = o[0][2] * o[0][2] + o[0][3] * o[0][3] + o[1][2] * o[1][2] + o[1][3] * o[1][3];
@@ -275,16 +291,24 @@ __global__ void __launch_bounds__(OC_THREADS, 2) outer_rnn_chunk_kernel(const __
       }
       const float r_lo = 1.0f / sqrtf(s_lo / static_cast<float>(p.true_vdim) + p.eps);
       const float r_hi = 1.0f / sqrtf(s_hi / static_cast<float>(p.true_vdim) + p.eps);
-      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + static_cast<int64_t>(row0) * step + head * p.vdim + out_col;
+      const int col = head * p.vdim + out_col;
+      auto put = [&](int t, int c, float x, float y) {
+        if (p.gate) {
+          const uint32_t g = *reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(p.gate) + (row0 + t) * p.gate_stride + c);
+          x *= silu_f<__nv_bfloat16>(bf16_lo(g)), y *= silu_f<__nv_bfloat16>(bf16_hi(g));
+        }
+        *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + (row0 + t) * p.out_stride + c) = pack_bf16(x, y);
+      };
       if (out_col < p.vdim) {
-        if (t_lo < len) *reinterpret_cast<uint32_t*>(out + t_lo * step) = pack_bf16(o[0][0] * r_lo * w0, o[0][1] * r_lo * w1);
-        if (t_hi < len) *reinterpret_cast<uint32_t*>(out + t_hi * step) = pack_bf16(o[0][2] * r_hi * w0, o[0][3] * r_hi * w1);
+        if (t_lo < len) put(t_lo, col, o[0][0] * r_lo * w0, o[0][1] * r_lo * w1);
+        if (t_hi < len) put(t_hi, col, o[0][2] * r_hi * w0, o[0][3] * r_hi * w1);
       }
       if (out_col + 8 < p.vdim) {
-        if (t_lo < len) *reinterpret_cast<uint32_t*>(out + t_lo * step + 8) = pack_bf16(o[1][0] * r_lo * w2, o[1][1] * r_lo * w3);
-        if (t_hi < len) *reinterpret_cast<uint32_t*>(out + t_hi * step + 8) = pack_bf16(o[1][2] * r_hi * w2, o[1][3] * r_hi * w3);
+        if (t_lo < len) put(t_lo, col + 8, o[1][0] * r_lo * w2, o[1][1] * r_lo * w3);
+        if (t_hi < len) put(t_hi, col + 8, o[1][2] * r_hi * w2, o[1][3] * r_hi * w3);
       }
     } else {
+      const int64_t step = static_cast<int64_t>(p.heads) * p.vdim;
       float* out = p.o + static_cast<int64_t>(row0) * step + head * p.vdim + out_col;
 #pragma unroll
       for (int n = 0; n < 2; ++n)
@@ -334,31 +358,40 @@ __global__ void __launch_bounds__(256) outer_rnn_fold_kernel(const __grid_consta
 
 bool outer_rnn_chunk_supports(int dim, int vdim) { return dim <= 128 && dim % 8 == 0 && vdim % 8 == 0; }
 
-template <int D>
+void outer_rnn_fold_launch(const OuterRnnParams& p, int n, cudaStream_t st) {
+  outer_rnn_fold_kernel<<<dim3((p.dim * p.vdim / 4 + 255) / 256, p.heads, n), 256, 0, st>>>(p);
+}
+
+template <int D, bool KEYED>
 static int launch_chunks(const OuterRnnParams& p, int n, cudaStream_t st) {
-  constexpr int smem = sizeof(ChunkSmem<D>);
+  constexpr int smem = sizeof(ChunkSmem<D, KEYED>);
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(outer_rnn_chunk_kernel<D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess ||
-        cudaFuncSetAttribute(outer_rnn_chunk_kernel<D, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
-      return fail(ERR_RUNTIME, "hgrn2_prefill: cannot raise dynamic shared memory to %d", smem);
+    if (cudaFuncSetAttribute(outer_rnn_chunk_kernel<D, false, KEYED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess ||
+        cudaFuncSetAttribute(outer_rnn_chunk_kernel<D, true, KEYED>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      return fail(ERR_RUNTIME, "outer_rnn: cannot raise dynamic shared memory to %d", smem);
     configured[dev] = true;
   }
   const dim3 grid((p.vdim + OC_VCOLS - 1) / OC_VCOLS, p.heads, n * p.segments);
   if (p.segments > 1) {
-    outer_rnn_chunk_kernel<D, true><<<grid, OC_THREADS, smem, st>>>(p);
-    outer_rnn_fold_kernel<<<dim3((p.dim * p.vdim / 4 + 255) / 256, p.heads, n), 256, 0, st>>>(p);
+    outer_rnn_chunk_kernel<D, true, KEYED><<<grid, OC_THREADS, smem, st>>>(p);
+    outer_rnn_fold_launch(p, n, st);
   }
-  outer_rnn_chunk_kernel<D, false><<<grid, OC_THREADS, smem, st>>>(p);
-  return check_launch("hgrn2_prefill (chunks)");
+  outer_rnn_chunk_kernel<D, false, KEYED><<<grid, OC_THREADS, smem, st>>>(p);
+  return check_launch("outer_rnn (chunks)");
 }
 
-int outer_rnn_chunk_launch(const OuterRnnParams& p, int n, cudaStream_t st) {
-  if (p.dim <= 32) return launch_chunks<32>(p, n, st);
-  if (p.dim <= 64) return launch_chunks<64>(p, n, st);
-  return launch_chunks<128>(p, n, st);
+int outer_rnn_chunk_launch(const OuterRnnParams& p, RnnKind kind, int n, cudaStream_t st) {
+  if (kind == RNN_KEYED) {
+    if (p.dim <= 32) return launch_chunks<32, true>(p, n, st);
+    if (p.dim <= 64) return launch_chunks<64, true>(p, n, st);
+    return launch_chunks<128, true>(p, n, st);
+  }
+  if (p.dim <= 32) return launch_chunks<32, false>(p, n, st);
+  if (p.dim <= 64) return launch_chunks<64, false>(p, n, st);
+  return launch_chunks<128, false>(p, n, st);
 }
 
 }  // namespace b200

@@ -3,7 +3,8 @@
 // sublayer's input and its RMS norm with a single gain:
 //     x_t <- sum_s mix[s, t] x_s + out[t] * y        (all streams from the old ones)
 //     h   = (sum_s in[s] x_s) / sqrt(mean(.^2) + eps) * gain
-// Streams live in fp32 [rows, S, width]; y and h are bf16 or fp32 activations.  Without y the streams come from the
+// (gains: an optional vector over the width on top of the single gain; one stream with unit weights and a gain vector is
+// the plain residual with an RMS norm).  Streams live in fp32 [rows, S, width]; y and h are bf16 or fp32 activations.  Without y the streams come from the
 // embedding table (every stream equal to the token's row), or are only read.
 // HBM / latency bound: one CTA per row, a thread owns 4 columns of every stream per step, all loads before the
 // reduction.  Width is padded to a multiple of 4 with zero columns; the mean runs over the true width.
@@ -22,6 +23,7 @@ struct HyperParams {
   float* streams;         // [rows, S, width]
   const void* y;          // [rows, width] E or NULL
   const float* weights;   // [mix S*S | out S | in S | gain]
+  const float* gains;     // [width] or NULL
   void* h;                // [rows, width] E
   int s, width, true_width, overlap;
   float eps;
@@ -100,7 +102,9 @@ __global__ void __launch_bounds__(512) hyper_connect_kernel(const __grid_constan
 #pragma unroll
   for (int v = 0; v < V; ++v) {
     const int c = (tid + v * blockDim.x) * 4;
-    if (c < width) store4(h + c, make_float4(u[v].x * scale, u[v].y * scale, u[v].z * scale, u[v].w * scale));
+    if (c >= width) continue;
+    const float4 g = p.gains ? load4(p.gains + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+    store4(h + c, make_float4(u[v].x * scale * g.x, u[v].y * scale * g.y, u[v].z * scale * g.z, u[v].w * scale * g.w));
   }
 }
 
@@ -122,6 +126,51 @@ static cudaError_t launch_hyper_e(const HyperParams& p, int rows, cudaStream_t s
   return launch_hyper<E, HC_MAX_STREAMS>(p, rows, st);
 }
 
+// out[r, c] = act(x[r, c]) * x[r, up + c] over strided rows; act: silu or the tanh form of gelu.  A thread takes 8 columns
+// of ROWS consecutive rows, all loads before the first use.
+template <typename E>
+__device__ __forceinline__ float gate_act(float z, int act) {
+  if (act == B200_ACT_SILU) return silu_f<E>(z);
+  // 0.5 z (1 + tanh(u)) = z * sigmoid(2 u)
+  return z * sigmoid_f<E>(1.5957691216057308f * fmaf(0.044715f * z * z, z, z));
+}
+
+template <typename E, int ROWS>
+__global__ void __launch_bounds__(128) gated_act_kernel(const E* x, int64_t stride, int up, E* out, int64_t out_stride, int rows,
+                                                        int width, int act, int overlap) {
+  if (overlap & OVERLAP_TRIGGER) pdl_trigger();
+  pdl_wait();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (c >= width) return;
+  float g[ROWS][8], u[ROWS][8];
+  const int64_t r0 = static_cast<int64_t>(blockIdx.y) * ROWS;
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    const E* row = x + min(r0 + i, static_cast<int64_t>(rows) - 1) * stride + c;
+    load8(row, g[i]);
+    load8(row + up, u[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) {
+    if (r0 + i >= rows) break;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) g[i][j] = gate_act<E>(g[i][j], act) * u[i][j];
+    store8(out + (r0 + i) * out_stride + c, g[i]);
+  }
+}
+
+// logits <- cap * tanh(logits / cap), columns behind `vocab` become -inf
+__global__ void __launch_bounds__(256) softcap_kernel(float* logits, int64_t stride, int vocab, int width, float cap) {
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
+  if (c >= width) return;
+  float* at = logits + static_cast<int64_t>(blockIdx.y) * stride + c;
+  const float4 a = load4(at);
+  float f[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) f[i] = c + i < vocab ? cap * tanhf(f[i] / cap) : -INFINITY;
+  store4(at, make_float4(f[0], f[1], f[2], f[3]));
+}
+
 // out[r, c] = silu(gate_up[r, c]) * gate_up[r, width + c] for fp32 activations (the bf16 form is b200_swiglu)
 __global__ void __launch_bounds__(256) swiglu_f32_kernel(const float* gate_up, int64_t stride, float* out, int width) {
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -137,18 +186,18 @@ __global__ void __launch_bounds__(256) swiglu_f32_kernel(const float* gate_up, i
 using namespace b200;
 
 extern "C" int b200_hyper_connect(const void* ids, int32_t ids_are_int64, const void* table, float* streams, const void* y,
-                                  const float* weights, void* h, int32_t rows, int32_t num_streams, int32_t width, int32_t true_width, float eps, int32_t f32,
-                                  int32_t overlap, b200_stream_t stream) {
+                                  const float* weights, const float* gains, void* h, int32_t rows, int32_t num_streams, int32_t width,
+                                  int32_t true_width, float eps, int32_t f32, int32_t overlap, b200_stream_t stream) {
   if (rows <= 0) return OK;
   B200_REQUIRE(num_streams >= 1 && num_streams <= HC_MAX_STREAMS, "hyper_connect: 1 to %d streams (got %d)",
                HC_MAX_STREAMS, num_streams);
   B200_REQUIRE(width > 0 && width % 4 == 0 && width <= HC_MAX_WIDTH && true_width > 0 && true_width <= width,
                "hyper_connect: width must be a multiple of 4, at most %d, and cover the true width (got %d, %d)",
                HC_MAX_WIDTH, width, true_width);
-  B200_REQUIRE(streams && weights && h && aligned16(streams) && aligned16(h) && (!y || aligned16(y)),
+  B200_REQUIRE(streams && weights && h && aligned16(streams) && aligned16(h) && aligned16(y) && aligned16(gains),
                "hyper_connect: NULL or unaligned tensor");
   B200_REQUIRE(!ids || (table && aligned16(table) && !y), "hyper_connect: the embedding form takes a table, no y");
-  HyperParams p = {ids, ids_are_int64, table, streams, y, weights, h, num_streams, width, true_width, overlap, eps};
+  HyperParams p = {ids, ids_are_int64, table, streams, y, weights, gains, h, num_streams, width, true_width, overlap, eps};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = f32 ? launch_hyper_e<float>(p, rows, st) : launch_hyper_e<__nv_bfloat16>(p, rows, st);
   if (e != cudaSuccess) return fail(ERR_LAUNCH, "hyper_connect: %s", cudaGetErrorString(e));
@@ -166,4 +215,47 @@ extern "C" int b200_swiglu_f32(const float* gate_up, int64_t row_stride, float* 
         gate_up + r0 * row_stride, row_stride, out + static_cast<int64_t>(r0) * intermediate, intermediate);
   }
   return check_launch("swiglu_f32");
+}
+
+extern "C" int b200_gated_act(const void* x, int64_t stride, int32_t up, void* out, int64_t out_stride, int32_t rows,
+                              int32_t width, int32_t act, int32_t f32, int32_t overlap, b200_stream_t stream) {
+  if (rows <= 0) return OK;
+  B200_REQUIRE(width > 0 && width % 8 == 0 && stride % 8 == 0 && up % 8 == 0 && out_stride % 8 == 0 && aligned16(x) && aligned16(out),
+               "gated_act: width, offset and strides must be multiples of 8, tensors 16-byte aligned");
+  B200_REQUIRE(act == B200_ACT_SILU || act == B200_ACT_GELU_TANH, "gated_act: unknown activation %d", act);
+  const bool early = (overlap & OVERLAP_START) != 0;
+  const int per = rows >= GLUE_WIDE_ROWS ? 4 : 1;
+  const unsigned cols = (width / 8 + 127) / 128;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  for (int64_t r0 = 0; r0 < rows; r0 += 65535ll * per) {
+    const int n = static_cast<int>(rows - r0 < 65535ll * per ? rows - r0 : 65535ll * per);
+    const dim3 grid(cols, (n + per - 1) / per), block(128);
+    cudaError_t e;
+    if (f32) {
+      const float* a = static_cast<const float*>(x) + r0 * stride;
+      float* o = static_cast<float*>(out) + r0 * out_stride;
+      e = per == 4 ? launch_pdl(early, gated_act_kernel<float, 4>, grid, block, 0, st, a, stride, up, o, out_stride, n, width, act, overlap)
+                   : launch_pdl(early, gated_act_kernel<float, 1>, grid, block, 0, st, a, stride, up, o, out_stride, n, width, act, overlap);
+    } else {
+      const __nv_bfloat16* a = static_cast<const __nv_bfloat16*>(x) + r0 * stride;
+      __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out) + r0 * out_stride;
+      e = per == 4 ? launch_pdl(early, gated_act_kernel<__nv_bfloat16, 4>, grid, block, 0, st, a, stride, up, o, out_stride, n, width, act, overlap)
+                   : launch_pdl(early, gated_act_kernel<__nv_bfloat16, 1>, grid, block, 0, st, a, stride, up, o, out_stride, n, width, act, overlap);
+    }
+    if (e != cudaSuccess) return fail(ERR_LAUNCH, "gated_act: %s", cudaGetErrorString(e));
+  }
+  return check_launch("gated_act");
+}
+
+extern "C" int b200_softcap(float* logits, int64_t stride, int32_t rows, int32_t vocab, int32_t width, float cap,
+                            b200_stream_t stream) {
+  if (rows <= 0) return OK;
+  B200_REQUIRE(width > 0 && width % 4 == 0 && stride % 4 == 0 && vocab > 0 && vocab <= width && cap > 0.f && aligned16(logits),
+               "softcap: width and stride must be multiples of 4, the cap positive");
+  for (int r0 = 0; r0 < rows; r0 += 65535) {
+    const int n = rows - r0 < 65535 ? rows - r0 : 65535;
+    softcap_kernel<<<dim3((width / 4 + 255) / 256, n), 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
+        logits + r0 * stride, stride, vocab, width, cap);
+  }
+  return check_launch("softcap");
 }
