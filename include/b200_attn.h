@@ -508,6 +508,34 @@ int b200_gla_decode(const void* qkv, int64_t stride, const void* low, const void
                     int32_t vdim, int32_t true_vdim, float q_scale, float inv_tau, float eps, int32_t f32, int32_t overlap,
                     b200_stream_t stream);
 
+/* State-space mixer: rows [x heads*vdim | B groups*dim | C groups*dim] (stride elements apart), head h in group
+ * h / (heads / groups); dt one column per head; state fp32 [slots, heads, dim, vdim];
+ *   dt <- softplus(dt + dt_bias), S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + skip * x.
+ * b200_conv_prefill: causal convolution over a packed batch, silu; weight fp32 [taps, channels] (first row: the current token's),
+ *   taps 4, 8 or 16 (pad with zero rows); ring fp32 [slots, taps, channels] holds the input of position p at p % taps: read
+ *   for the tokens in front of a portion, then written.
+ * b200_ssd_prefill: rows after the convolution.  bf16 and b200_ssd_chunked(dim, vdim): 32-token chunks on the tensor cores,
+ *   y bf16 [tokens, heads*vdim], optionally in segments (multiples of 32 tokens, workspace as for b200_hgrn2_prefill);
+ *   f32, serial or other shapes: token by token, y fp32.
+ * b200_ssd_decode: one token per slot, rows before the convolution, which is inside; y fp32 [batch, heads*vdim].
+ * b200_gated_group_norm: f = y * silu(z), out = f / sqrt(mean(f^2) + eps) * weight, the mean over each of `groups` equal parts
+ *   of the heads * true_vdim channels; heads are vdim columns wide, padding columns of out become zero. */
+int b200_conv_prefill(const void* x, int64_t stride, const float* weight, const float* bias, float* ring,
+                      const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start, void* out, int64_t out_stride,
+                      int32_t batch, int32_t max_len, int32_t channels, int32_t taps, int32_t f32, b200_stream_t stream);
+int32_t b200_ssd_chunked(int32_t dim, int32_t vdim);
+int b200_ssd_prefill(const void* xbc, int64_t stride, const void* dt, int64_t dt_stride, const float* dt_bias, const float* a_log,
+                     const float* skip, float* state, const int32_t* cu_seqlens, const int32_t* slots, const int32_t* start,
+                     void* y, int32_t batch, int32_t heads, int32_t groups, int32_t dim, int32_t vdim, int32_t f32,
+                     int32_t serial, int32_t segment, int32_t segments, float* workspace, b200_stream_t stream);
+int b200_ssd_decode(const void* xbc, int64_t stride, const void* dt, int64_t dt_stride, const float* dt_bias, const float* a_log,
+                    const float* skip, const float* conv_weight, const float* conv_bias, float* ring, int32_t taps, float* state,
+                    const int64_t* pos, const int64_t* active, float* y, int32_t batch, int32_t heads, int32_t groups,
+                    int32_t dim, int32_t vdim, int32_t f32, int32_t overlap, b200_stream_t stream);
+int b200_gated_group_norm(const void* y, int64_t y_stride, const void* z, int64_t z_stride, const float* weight, void* out,
+                          int64_t out_stride, int32_t rows, int32_t heads, int32_t vdim, int32_t true_vdim, int32_t groups,
+                          float eps, int32_t y_f32, int32_t f32, int32_t overlap, b200_stream_t stream);
+
 /* Latent attention.  Cache rows are [latent rank | rotated key part rot] in pages of 16 tokens; rank, dim, vdim, rot and
  * q_rank padded to multiples of 64.  angles: fp32 (cos, sin) pairs [positions, rot_pairs], amplitude included.
  * b200_latent_prep: fused rows [query latent | kv latent | rotated part] -> cq = rms(query latent) * q_weight, and, when

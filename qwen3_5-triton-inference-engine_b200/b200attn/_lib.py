@@ -80,6 +80,10 @@ SIGNATURES: dict[str, list] = {
     "b200_latent_absorb": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, P],
     "b200_latent_decode_simple": [P, P, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_latent_value": [P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, P],
+    "b200_conv_prefill": [P, I64, P, P, P, P, P, P, P, I64, I32, I32, I32, I32, I32, P],
+    "b200_ssd_prefill": [P, I64, P, I64, P, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, I32, P, P],
+    "b200_ssd_decode": [P, I64, P, I64, P, P, P, P, P, P, I32, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, P],
+    "b200_gated_group_norm": [P, I64, P, I64, P, P, I64, I32, I32, I32, I32, I32, c_float, I32, I32, I32, P],
     "b200_gated_act": [P, I64, I32, P, I64, I32, I32, I32, I32, I32, P],
     "b200_softcap": [P, I64, I32, I32, I32, c_float, P],
     "b200_window_prep": [P, I64, P, P, I32, P, P, P, I64, P, P, P, P, I32, I32, I32, I32, I32, I32, I32, I32, I32, P],
@@ -93,6 +97,7 @@ SIGNATURES: dict[str, list] = {
                         I32, P],
 }
 OTHER = {
+    "b200_ssd_chunked": ([I32, I32], c_int32),
     "b200_mingru_workspace_bytes": ([I32, I32, I32], c_int64),
     "b200_hgrn2_workspace_bytes": ([I32, I32, I32, I32, I32], c_int64),
     "b200_last_error": ([], c_char_p),

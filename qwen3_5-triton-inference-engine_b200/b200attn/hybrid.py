@@ -1,8 +1,11 @@
-"""Decoder stacks whose layers are listed one by one in config.json: any order of the mixers of `mixers.py`, an optional
-feed-forward per layer, several residual streams joined by hyper-connections, RMS norms with a single gain.  Served by
-`HybridEngine` through the same slots, pages, graph capture and batcher as every other engine of the package.
+"""Decoder stacks whose layers are listed one by one in config.json: any order of the mixers of `mixers.py` and `cores.py`, an
+optional feed-forward per layer.  What a family of such stacks fixes is its `Design`: several residual streams joined by
+hyper-connections or one plain residual, norms with a single gain or a weight per channel, the feed-forward behind the mixer
+or beside it on the same norm.  Served by `HybridEngine` through the same slots, pages, graph capture and batcher as every
+other engine of the package.
 
-config.json:  architecture, vocab, width, streams, norm.eps, layers = [{type, mixer, mlp | null}, ...].
+config.json:  architecture, vocab, width, norm.eps, layers = [{type, mixer, mlp | null}, ...]; hyper-connected: streams;
+optional: logit_softcap.
 """
 from __future__ import annotations
 
@@ -14,8 +17,24 @@ import torch.nn.functional as F
 
 from . import hybrid_ops as hops
 from . import ops
+from . import cores
+from .cores import CoreMixer, FusedUnit, GatedMLP
 from .mixers import FEED_FORWARDS, MIXERS, padded, round_up
 from .slots import SlotEngine
+
+MIXERS = MIXERS | {cls.kind: cls for cls in (cores.SideBySide, cores.GatedLinearMixer)}
+
+
+@dataclass(frozen=True)
+class Design:
+    """What config.json does not say."""
+    hyper: bool            # hyper-connected streams and norms with a single gain; else one residual and norm weights
+    parallel: bool         # mixer and feed-forward read one norm and are added together; else one behind the other
+    activation: str        # of the feed-forward's gate
+
+
+DESIGNS = {"Tofilorn": Design(hyper=True, parallel=False, activation="silu"),
+           "Dugilorn": Design(hyper=False, parallel=True, activation="gelu_tanh")}
 
 
 @dataclass(frozen=True)
@@ -25,11 +44,56 @@ class HybridConfig:
     streams: int
     eps: float
     layers: tuple          # of the raw layer dictionaries
+    design: Design
+    softcap: float | None = None
 
     @classmethod
     def from_config(cls, config: dict) -> "HybridConfig":
-        return cls(int(config["vocab"]), int(config["width"]), int(config["streams"]), float(config["norm"]["eps"]),
-                   tuple(config["layers"]))
+        design, cap = DESIGNS[config["architecture"]], config.get("logit_softcap")
+        return cls(int(config["vocab"]), int(config["width"]), int(config["streams"]) if design.hyper else 1,
+                   float(config["norm"]["eps"]), tuple(config["layers"]), design, None if cap is None else float(cap))
+
+
+# Units: what runs between two joints.  prefill(h, batch, engine, states) and decode(h, engine, states, nxt) give the
+# sublayer's output; starts_own(engine): whether its first decode-step kernel is one of this package.
+class MixerUnit:
+    def __init__(self, layer: int, mixer):
+        self.layer, self.mixer = layer, mixer
+
+    def load(self, get, width_p, dtype, device) -> None:
+        self.mixer.load(lambda n: get(f"mix.{n}"), width_p, dtype, device)
+
+    def allocate(self, engine) -> dict:
+        return {self.mixer.index: self.mixer.allocate(engine)}
+
+    def prefill(self, h, batch, engine, states):
+        return self.mixer.prefill(h, batch, engine, states)
+
+    def starts_own(self, engine) -> bool:
+        return engine.streams_weight(self.mixer.first_weight())
+
+    def decode(self, h, engine, states, nxt: bool):
+        return self.mixer.decode(h, engine, states, nxt)
+
+
+class FeedForwardUnit:
+    def __init__(self, layer: int, mlp):
+        self.layer, self.mlp = layer, mlp
+
+    def load(self, get, width_p, dtype, device) -> None:
+        self.mlp.load(lambda n: get(f"mlp.{n}"), width_p, dtype, device)
+
+    def allocate(self, engine) -> dict:
+        return {}
+
+    def prefill(self, h, batch, engine, states):
+        return self.mlp.prefill(h, engine)
+
+    def starts_own(self, engine) -> bool:
+        return engine.streams_weight(self.mlp.gate_up, swiglu=True)
+
+    def decode(self, h, engine, states, nxt: bool):
+        return self.mlp.decode(h, engine, nxt)
 
 
 class HybridWeights:
@@ -46,16 +110,28 @@ class HybridWeights:
             mlp = layer["mlp"]
             if mlp is not None and mlp["kind"] not in FEED_FORWARDS:
                 raise ValueError(f"layer {i}: unknown feed-forward '{mlp['kind']}'")
-            self.mlps.append(None if mlp is None else FEED_FORWARDS[mlp["kind"]](mlp))
+            fused = cfg.design.parallel or cfg.design.activation != "silu"
+            self.mlps.append(None if mlp is None else GatedMLP(mlp, cfg.design.activation) if fused else FEED_FORWARDS[mlp["kind"]](mlp))
         for mixer in self.mixers:
             mixer.check(self.mixers)
+        self.units = [unit for i in range(len(self.mixers)) for unit in self._layer_units(i)]
+
+    def _layer_units(self, i: int) -> list:
+        mixer, mlp = self.mixers[i], self.mlps[i]
+        ff = [("mlp.", mlp)] if mlp is not None else []
+        if not isinstance(mixer, CoreMixer):
+            if self.cfg.design.parallel and ff:
+                raise ValueError(f"layer {i}: this mixer cannot share its norm with a feed-forward")
+            return [MixerUnit(i, mixer)] + [FusedUnit(i, ff) if isinstance(mlp, GatedMLP) else FeedForwardUnit(i, mlp) for _ in ff]
+        mix = [("mix." + core.prefix, core) for core in mixer.cores]
+        if self.cfg.design.parallel:
+            return [FusedUnit(i, mix + ff)]
+        return [FusedUnit(i, mix)] + [FeedForwardUnit(i, mlp) if not isinstance(mlp, GatedMLP) else FusedUnit(i, ff) for _ in ff]
 
     def sublayers(self):
-        """(layer, 1 = mixer / 2 = feed-forward) in the order they run."""
-        for i, mlp in enumerate(self.mlps):
-            yield i, 1
-            if mlp is not None:
-                yield i, 2
+        """(layer, 1 = mixer, with the feed-forward where they share a norm / 2 = feed-forward) in the order they run."""
+        for k, unit in enumerate(self.units):
+            yield unit.layer, 2 if k and self.units[k - 1].layer == unit.layer else 1
 
     def shapes(self) -> dict:
         """name -> shape of every tensor of the checkpoint."""
@@ -65,11 +141,17 @@ class HybridWeights:
             out |= {f"l{i}.mix.{n}": shape for n, shape in mixer.shapes(cfg.width).items()}
             if mlp is not None:
                 out |= {f"l{i}.mlp.{n}": shape for n, shape in mlp.shapes(cfg.width).items()}
-            for q in (1, 2) if mlp is not None else (1,):
-                out |= {f"l{i}.norm{q}": (), f"l{i}.hc{q}.in": (s,), f"l{i}.hc{q}.out": (s,), f"l{i}.hc{q}.mix": (s, s)}
-        return out | {"final.norm": (), "head": (cfg.vocab, cfg.width)}
+        gain = () if cfg.design.hyper else (cfg.width,)
+        for i, q in self.sublayers():
+            out[f"l{i}.norm{q}"] = gain
+            if cfg.design.hyper:
+                out |= {f"l{i}.hc{q}.in": (s,), f"l{i}.hc{q}.out": (s,), f"l{i}.hc{q}.mix": (s, s)}
+        return out | {"final.norm": gain, "head": (cfg.vocab, cfg.width)}
 
     def load(self, tensors: dict, dtype, device) -> "HybridWeights":
+        for i, mixer in enumerate(self.mixers):
+            if isinstance(mixer, CoreMixer):
+                mixer.measure(lambda n, i=i: tensors[f"l{i}.mix.{n}"].shape)
         want = self.shapes()
         missing = sorted(set(want) - set(tensors))
         if missing:
@@ -85,24 +167,30 @@ class HybridWeights:
 
         self.embed = padded(wide("embed"), cfg.vocab, width_p).to(device, dtype)
         self.head = padded(wide("head"), self.vocab_p, width_p).to(device, dtype)
-        for i, (mixer, mlp) in enumerate(zip(self.mixers, self.mlps)):
-            mixer.load(lambda n, i=i: wide(f"l{i}.mix.{n}"), width_p, dtype, device)
-            if mlp is not None:
-                mlp.load(lambda n, i=i: wide(f"l{i}.mlp.{n}"), width_p, dtype, device)
-        # joints: what happens to the streams between two sublayers, as one fp32 vector [mix | out | in | gain] each
+        for unit in self.units:
+            unit.load(lambda n, i=unit.layer: wide(f"l{i}.{n}"), width_p, dtype, device)
+        # joints: what happens to the streams between two sublayers, as one fp32 vector [mix | out | in | gain] each, and the
+        # norm weights where a norm has more than a single gain
         steps = list(self.sublayers())
+        norms = [f"l{i}.norm{q}" for i, q in steps] + ["final.norm"]
         s = cfg.streams
+        if not cfg.design.hyper:
+            plain = torch.ones(4, device=device)
+            self.joints = [plain] * len(norms)
+            self.gains = [padded(wide(n), width_p).to(device).contiguous() for n in norms]
+            return self
         none = [torch.zeros(s * s), torch.zeros(s)]
         after = [[wide(f"l{i}.hc{q}.mix").flatten(), wide(f"l{i}.hc{q}.out")] for i, q in steps]
-        before = [[wide(f"l{i}.hc{q}.in"), wide(f"l{i}.norm{q}").view(1)] for i, q in steps]
+        before = [[wide(f"l{i}.hc{q}.in"), wide(n).view(1)] for (i, q), n in zip(steps, norms)]
         before.append([torch.ones(s), wide("final.norm").view(1)])
         self.joints = [torch.cat([t.cpu() for t in a + b]).to(device) for a, b in zip([none] + after, before)]
+        self.gains = [None] * len(norms)
         return self
 
 
 def random_tensors(weights: HybridWeights, seed: int, device="cpu", std: float = 0.02) -> dict:
     """Random checkpoint of a stack's shapes: N(0, std) projections, unit norm weights, forget-gate floors in [0, 1),
-    streams mixed by a matrix near the identity."""
+    streams mixed by a matrix near the identity, decays that forget within tens to hundreds of tokens."""
     gen = torch.Generator(device=device).manual_seed(seed)
     out = {}
     for name, shape in weights.shapes().items():
@@ -118,17 +206,22 @@ def random_tensors(weights: HybridWeights, seed: int, device="cpu", std: float =
             noise = noise + 1.0 / shape[0]
         elif leaf == "out":
             noise = noise + 1.0
+        elif leaf == "dt_bias":
+            noise = noise * 50.0 - 3.0
         out[name] = noise.to(torch.bfloat16)
     return out
 
 
 @dataclass
 class KeySpan:
-    """Cached positions a packed batch's queries can see: packed row offsets and the first position per sequence."""
+    """Cached positions a packed batch's queries can see: packed row offsets and the first position per sequence, the row of
+    every token of the batch itself, the most positions of a sequence that earlier passes wrote."""
     cu: torch.Tensor
     first: torch.Tensor
+    rows: torch.Tensor
     keys: int
     max_keys: int
+    max_old: int
 
 
 class PackedBatch:
@@ -156,9 +249,13 @@ class PackedBatch:
         if span is None:
             first = [max(0, s - window + 1) for s in self.starts]
             counts = [s + n - f for s, n, f in zip(self.starts, self.lengths, first)]
-            host = np.concatenate(([0], np.cumsum(counts), first)).astype(np.int32)
-            cu, pos = torch.from_numpy(host).to(self.device).split([self.count + 1, self.count])
-            span = self._spans[window] = KeySpan(cu, pos, sum(counts), max(counts))
+            cu = np.concatenate(([0], np.cumsum(counts)))
+            old = [s - f for s, f in zip(self.starts, first)]
+            ends = np.cumsum(self.lengths)
+            rows = np.arange(self.tokens) + np.repeat(cu[:-1] + old - (ends - self.lengths), self.lengths)
+            host = torch.from_numpy(np.concatenate((cu, first, rows)).astype(np.int32)).to(self.device)
+            cu, pos, rows = host.split([self.count + 1, self.count, self.tokens])
+            span = self._spans[window] = KeySpan(cu, pos, rows, sum(counts), max(counts), max(old))
         return span
 
 
@@ -177,8 +274,10 @@ class HybridEngine(SlotEngine):
         # 32-bit means 32-bit: no TF32 products, no 16-bit partial sums
         torch.backends.cuda.matmul.allow_tf32 = False
         torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
-        self._tables, self._workspaces = {}, {}
-        self.states = [mixer.allocate(self) for mixer in weights.mixers]
+        self._tables, self._workspaces, self._scratch = {}, {}, {}
+        self.states: dict = {}               # caches and states of the units, by the unit's own keys (a mixer's: its layer)
+        for unit in weights.units:
+            self.states |= unit.allocate(self)
         self.streams = torch.zeros(batch, self.cfg.streams, weights.width_p, dtype=torch.float32, device=self.device)
         self.trace: list | None = None       # a list: the residual (sum of the streams) after every layer is appended
 
@@ -194,6 +293,12 @@ class HybridEngine(SlotEngine):
         if key not in self._workspaces:
             self._workspaces[key] = hops.latent_decode_workspace(self.batch, heads, rank, splits, self.device)
         return self._workspaces[key]
+
+    def zero_scratch(self, used: int, pad: int):
+        """[batch, used + pad] activations of a decode step whose last `pad` columns nobody writes: they stay zero."""
+        if (used, pad) not in self._scratch:
+            self._scratch[used, pad] = torch.zeros(self.batch, used + pad, dtype=self.dtype, device=self.device)
+        return self._scratch[used, pad]
 
     def linear(self, x, weight):
         return F.linear(x, weight)
@@ -220,20 +325,23 @@ class HybridEngine(SlotEngine):
         return (self.dtype == torch.bfloat16 and self.w.vocab_p == self.cfg.vocab and head.shape[1] <= ops.SKINNY_GEMM_MAX_K
                 and ops.skinny_gemm_supports(self.batch, head.shape[0], head.shape[1]))
 
-    def logits(self, h) -> torch.Tensor:
-        """fp32 logits [rows, padded vocab] of normed final rows; padding columns are -inf."""
+    def logits(self, h, cap: bool = True) -> torch.Tensor:
+        """fp32 logits [rows, padded vocab] of normed final rows; padding columns are -inf.  cap=False leaves a soft cap out: it
+        does not change the order (a choice needs it not, and cannot be misled by values that saturate)."""
         head = self.w.head
         if self.dtype == torch.float32:
             out = F.linear(h, head)
         else:
             out = torch.mm(h, head.t(), out_dtype=torch.float32)
+        if cap and self.cfg.softcap is not None:
+            return hops.softcap(out, self.cfg.vocab, self.cfg.softcap)
         if self.w.vocab_p != self.cfg.vocab:
             out[:, self.cfg.vocab:] = float("-inf")
         return out
 
     def _joint(self, k: int, streams, y=None, ids=None, overlap: int = 0):
         return hops.hyper_connect(streams, self.w.joints[k], self.cfg.width, self.cfg.eps, self.dtype, y=y, ids=ids,
-                                  table=self.w.embed if ids is not None else None, overlap=overlap)
+                                  table=self.w.embed if ids is not None else None, overlap=overlap, gains=self.w.gains[k])
 
     def _traced(self, streams) -> None:
         if self.trace is not None:
@@ -244,14 +352,11 @@ class HybridEngine(SlotEngine):
         """The stack over a packed batch: the final normed hidden rows."""
         streams = torch.empty(batch.tokens, self.cfg.streams, self.w.width_p, dtype=torch.float32, device=self.device)
         h = self._joint(0, streams, ids=batch.ids)
-        k = 1
-        for mixer, mlp in zip(self.w.mixers, self.w.mlps):
-            h = self._joint(k, streams, y=mixer.prefill(h, batch, self, self.states))
-            k += 1
-            if mlp is not None:
-                h = self._joint(k, streams, y=mlp.prefill(h, self))
-                k += 1
-            self._traced(streams)
+        units = self.w.units
+        for k, unit in enumerate(units, start=1):
+            h = self._joint(k, streams, y=unit.prefill(h, batch, self, self.states))
+            if k == len(units) or units[k].layer != unit.layer:
+                self._traced(streams)
         return h
 
     def _set_pos(self, slots, ends) -> None:
@@ -313,7 +418,7 @@ class HybridEngine(SlotEngine):
             done = [k for k, i in enumerate(live) if len(prompts[i]) <= start + cut]
             if done:
                 rows = batch.cu[1:].long()[torch.tensor(done, device=self.device)] - 1
-                ids = ops.argmax_rows(self.logits(h.index_select(0, rows)), self.argmax_ws)
+                ids = ops.argmax_rows(self.logits(h.index_select(0, rows), cap=False), self.argmax_ws)
                 first[torch.tensor([live[k] for k in done], device=self.device)] = ids
         self._set_pos(slots, [len(p) for p in prompts])
         self.tok.index_copy_(0, torch.tensor(slots, dtype=torch.int64, device=self.device), first)
@@ -323,23 +428,16 @@ class HybridEngine(SlotEngine):
     def _decode_hidden(self, tok, own_head: bool) -> torch.Tensor:
         """The stack over one token per slot; idle slots ride along and touch nothing.  Every kernel of this package that
         follows another one starts early; what the next sublayer's first projection runs on decides a joint's flags."""
-        steps = list(self.w.sublayers())
+        units = self.w.units
 
         def first_own(k: int) -> bool:               # does a kernel of ours read the output of joint k?
-            if k == len(steps):
-                return own_head
-            i, q = steps[k]
-            if q == 1:
-                return self.streams_weight(self.w.mixers[i].first_weight())
-            return self.streams_weight(self.w.mlps[i].gate_up, swiglu=True)
+            return own_head if k == len(units) else units[k].starts_own(self)
 
         streams, untraced = self.streams, self.trace is None
         h = self._joint(0, streams, ids=tok, overlap=self.then(first_own(0)))
-        for k, (i, q) in enumerate(steps, start=1):
-            last = k == len(steps) or steps[k][0] != i          # the layer ends here
-            y = self.w.mixers[i].decode(h, self, self.states, True) if q == 1 else self.w.mlps[i].decode(h, self, True)
-            h = self._joint(k, streams, y=y, overlap=self.then(first_own(k) and untraced))
-            if last:
+        for k, unit in enumerate(units, start=1):
+            h = self._joint(k, streams, y=unit.decode(h, self, self.states, True), overlap=self.then(first_own(k) and untraced))
+            if k == len(units) or units[k].layer != unit.layer:          # the layer ends here
                 self._traced(streams)
         return h
 
@@ -354,6 +452,6 @@ class HybridEngine(SlotEngine):
             in_place = tok.data_ptr() == self.tok.data_ptr()
             nxt = ops.lm_head_argmax(h, self.w.head, self.argmax_ws, out=tok if in_place else None, overlap=ops.OVERLAP_START)
         else:
-            nxt = ops.argmax_rows(self.logits(h), self.argmax_ws)
+            nxt = ops.argmax_rows(self.logits(h, cap=False), self.argmax_ws)
         self._move_on()
         return nxt

@@ -272,3 +272,227 @@ def latent_value(workspace, w_uv, dtype, overlap: int = 0):
     _lib.call("b200_latent_value", _ptr(ml), _ptr(o), _ptr(w_uv), _ptr(merged), _ptr(out), batch, heads, rank, vdim, splits, _f32(w_uv),
               int(overlap), _stream())
     return out
+
+
+# ------------------------------------------------------------------------------------- gated activations and soft cap
+ACT_SILU, ACT_GELU_TANH = 0, 1
+
+
+def _rows(t) -> bool:
+    """A matrix whose rows may be further apart than they are long."""
+    return t.ndim == 2 and t.stride(1) == 1
+
+
+def gated_act(gate_up, width: int, out, act: int, overlap: int = 0):
+    """out = act(gate_up[:, :width]) * gate_up[:, width: 2*width]; both may be column ranges of wider matrices."""
+    assert _rows(gate_up) and gate_up.shape[1] >= 2 * width and _rows(out) and out.shape == (gate_up.shape[0], width)
+    assert out.dtype == gate_up.dtype
+    _require_cuda(gate_up, out)
+    _lib.call("b200_gated_act", _ptr(gate_up), gate_up.stride(0), width, _ptr(out), out.stride(0), out.shape[0], width, act,
+              _f32(gate_up), int(overlap), _stream())
+    return out
+
+
+def softcap(logits, vocab: int, cap: float):
+    """logits <- cap * tanh(logits / cap) in place; columns from `vocab` on become -inf."""
+    assert logits.dtype == torch.float32 and _rows(logits)
+    _require_cuda(logits)
+    _lib.call("b200_softcap", _ptr(logits), logits.stride(0), logits.shape[0], vocab, logits.shape[1], float(cap), _stream())
+    return logits
+
+
+# ------------------------------------------------------------------------------------------------- windowed attention
+def allocate_window_cache(num_pages: int, kv_heads: int, pitch: int, dtype, *, device="cuda"):
+    """Zero-filled pages of [key | value] rows, one per key/value head and token."""
+    return torch.zeros((num_pages, kv_heads, PAGE_SIZE, pitch), dtype=dtype, device=device)
+
+
+def window_prep(x, bias, pos, slot, active, block_table, angles, cache, heads: int, dim: int, vdim: int, ctx=None, ctx_row=None,
+                overlap: int = 0) -> None:
+    """Biases and rotation on the rows x = [q | k | v | ...] of projections: q in place, [k | v] to the pages and to `ctx`."""
+    _, kv_heads, _, pitch = cache.shape
+    assert _rows(x) and x.shape[1] >= (heads + kv_heads) * dim + kv_heads * vdim and x.dtype == cache.dtype
+    assert bias.dtype == torch.float32 and bias.numel() == (heads + kv_heads) * dim + kv_heads * vdim
+    assert angles.dtype == torch.float32 and angles.is_contiguous() and cache.is_contiguous() and pos.dtype in (torch.int32, torch.int64)
+    if ctx is not None:
+        assert ctx.shape[1:] == (kv_heads, pitch) and ctx.dtype == x.dtype and ctx.is_contiguous() and ctx_row.dtype == torch.int32
+    _require_cuda(x, bias, pos, block_table, angles, cache)
+    _lib.call("b200_window_prep", _ptr(x), x.stride(0), _ptr(bias), _ptr(pos), int(pos.dtype == torch.int64), _ptr(slot),
+              _ptr(active), _ptr(block_table), block_table.stride(0), _ptr(angles), _ptr(cache), _ptr(ctx), _ptr(ctx_row), x.shape[0],
+              heads, kv_heads, dim, angles.shape[1], vdim, pitch, _f32(x), int(overlap), _stream())
+
+
+def window_gather(cache, ctx, block_table, slots, cu_k, k_pos0, max_keys: int) -> None:
+    """The first max_keys keys (rounded up to 16) of every sequence, from the pages to ctx [keys, kv_heads, pitch]."""
+    _, kv_heads, _, pitch = cache.shape
+    _require_cuda(cache, ctx, block_table, slots, cu_k, k_pos0)
+    _lib.call("b200_latent_gather", _ptr(cache), _ptr(ctx), _ptr(block_table), block_table.stride(0), _ptr(slots), _ptr(cu_k),
+              _ptr(k_pos0), slots.numel(), max_keys, kv_heads, pitch * cache.element_size(), _stream())
+
+
+def window_prefill(q, ctx, gate, out, cu_q, cu_k, q_pos0, k_pos0, max_q: int, heads: int, dim: int, true_dim: int, vdim: int,
+                   window: int, scale: float, out_scale: float = 1.0, simple: bool = False):
+    """Windowed causal attention of the packed queries in the first heads*dim columns of q over ctx [keys, kv_heads, pitch];
+    out [tokens, heads*vdim] = o * sigmoid(gate) * out_scale.  bf16 heads of up to 256 + 256 dimensions run on the
+    tensor-core kernel; simple=True keeps them off it."""
+    keys, kv_heads, pitch = ctx.shape
+    assert _rows(q) and _rows(gate) and _rows(out) and out.shape == gate.shape == (q.shape[0], heads * vdim) and ctx.is_contiguous()
+    assert q.dtype == ctx.dtype == gate.dtype == out.dtype and q.shape[1] >= heads * dim
+    _require_cuda(q, ctx, gate, out)
+    simple = simple or dim > 256 or vdim > 256
+    _lib.call("b200_window_prefill", _ptr(q), q.stride(0), _ptr(ctx), _ptr(gate), gate.stride(0), _ptr(out), out.stride(0),
+              _ptr(cu_q), _ptr(cu_k), _ptr(q_pos0), _ptr(k_pos0), cu_q.numel() - 1, max_q, q.shape[0], keys, heads, kv_heads, dim,
+              true_dim, vdim, pitch, min(window, 1 << 30), float(scale), float(out_scale), int(simple), _f32(q), _stream())
+    return out
+
+
+def window_decode_splits(batch: int, heads: int, kv_heads: int, span: int, sm_count: int) -> int:
+    """Key ranges per slot (as for latent attention: a CTA takes up to 16 query heads of one key/value head)."""
+    return latent_decode_splits(batch * kv_heads, heads // kv_heads, span, sm_count)
+
+
+def window_decode(q, cache, block_table, pos, active, workspace, dim: int, window: int, scale: float, overlap: int = 0,
+                  simple: bool = False) -> None:
+    """One token per slot: the heads in the first heads*dim columns of q (rotated) over the pages; leaves the split results in
+    `workspace`."""
+    ml, o = workspace
+    batch, heads, splits, vdim = o.shape
+    _, kv_heads, _, pitch = cache.shape
+    assert _rows(q) and q.shape[0] == batch and q.shape[1] >= heads * dim and pos.dtype == torch.int64 and q.dtype == cache.dtype
+    _require_cuda(q, cache, block_table, pos, ml, o)
+    simple = simple or vdim > 1024 or pitch > LATENT_DECODE_MAX_ROW
+    _lib.call("b200_window_decode", _ptr(q), q.stride(0), _ptr(cache), cache.shape[0], _ptr(block_table), block_table.stride(0),
+              _ptr(pos), _ptr(active), _ptr(ml), _ptr(o), batch, heads, kv_heads, dim, vdim, pitch, min(window, 1 << 30), splits,
+              float(scale), int(simple), _f32(q), int(overlap), _stream())
+
+
+def window_merge(workspace, gate, out, out_scale: float = 1.0, overlap: int = 0):
+    """Merges the splits: out [B, heads*vdim] = o * sigmoid(gate) * out_scale."""
+    ml, o = workspace
+    batch, heads, splits, vdim = o.shape
+    assert _rows(gate) and _rows(out) and out.shape == gate.shape == (batch, heads * vdim) and out.dtype == gate.dtype
+    _require_cuda(ml, o, gate, out)
+    _lib.call("b200_window_merge", _ptr(ml), _ptr(o), _ptr(gate), gate.stride(0), _ptr(out), out.stride(0), batch, heads, vdim,
+              splits, float(out_scale), _f32(out), int(overlap), _stream())
+    return out
+
+
+# --------------------------------------------------------------------------------------------------------- state space
+def conv_taps(taps: int) -> int:
+    """Taps of the kernels' convolution that hold `taps` of a model's."""
+    assert 1 <= taps <= 16, f"convolutions of 1 to 16 taps (got {taps})"
+    return 4 if taps <= 4 else 8 if taps <= 8 else 16
+
+
+def conv_prefill(x, weight, bias, ring, batch):
+    """Causal convolution with silu over a packed batch; x [tokens, channels] (a column range), weight fp32 [taps, channels] with
+    the current token's row first, ring fp32 [slots, taps, channels] in place."""
+    slots, taps, channels = ring.shape
+    assert _rows(x) and x.shape[1] == channels and weight.shape == (taps, channels) and bias.numel() == channels
+    for t in (weight, bias, ring):
+        assert t.dtype == torch.float32 and t.is_contiguous()
+    _require_cuda(x, weight, bias, ring)
+    out = torch.empty((x.shape[0], channels), dtype=x.dtype, device=x.device)
+    _lib.call("b200_conv_prefill", _ptr(x), x.stride(0), _ptr(weight), _ptr(bias), _ptr(ring), _ptr(batch.cu), _ptr(batch.slots),
+              _ptr(batch.start), _ptr(out), out.stride(0), batch.count, batch.max_len, channels, taps, _f32(x), _stream())
+    return out
+
+
+def ssd_segments(max_len: int, groups: int, sm_count: int) -> tuple[int, int]:
+    """(segment length, segments of the longest sequence) of the chunked state-space prefill, as `hgrn2_segments`."""
+    parts = min(2 * sm_count // groups, max_len // 128)
+    if parts < 3:
+        return max_len, 1
+    segment = -(-max_len // (parts * 32)) * 32
+    return segment, -(-max_len // segment)
+
+
+def ssd_prefill(xbc, dt, dt_bias, a_log, skip, state, groups: int, batch, serial: bool = False, segments=None):
+    """State-space recurrence of a packed batch: xbc [tokens, x | B | C] after the convolution, dt [tokens, heads] (a column
+    range), state fp32 [slots, heads, dim, vdim] in place -> y [tokens, heads*vdim] (bf16 from the chunked kernel, else
+    fp32).  segments: (length, count) to pin how sequences are cut."""
+    _, heads, dim, vdim = state.shape
+    assert _rows(xbc) and xbc.shape[1] == heads * vdim + 2 * groups * dim and _rows(dt) and dt.shape[1] >= heads and dt.dtype == xbc.dtype
+    for t in (dt_bias, a_log, skip, state):
+        assert t.dtype == torch.float32 and t.is_contiguous()
+    _require_cuda(xbc, dt, dt_bias, a_log, skip, state)
+    tokens = xbc.shape[0]
+    chunked = xbc.dtype == torch.bfloat16 and not serial and bool(_lib.load().b200_ssd_chunked(dim, vdim))
+    segment, count = (batch.max_len, 1) if not chunked else segments or ssd_segments(
+        batch.max_len, batch.count * max(1, heads * vdim // 128), sm_count(xbc.device))
+    ws = None
+    if count > 1:
+        ws = torch.empty(_lib.load().b200_hgrn2_workspace_bytes(batch.count, count, heads, dim, vdim) // 4, dtype=torch.float32,
+                         device=xbc.device)
+    y = torch.empty((tokens, heads * vdim), dtype=torch.bfloat16 if chunked else torch.float32, device=xbc.device)
+    _lib.call("b200_ssd_prefill", _ptr(xbc), xbc.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(state),
+              _ptr(batch.cu), _ptr(batch.slots), _ptr(batch.start), _ptr(y), batch.count, heads, groups, dim, vdim, _f32(xbc),
+              int(not chunked), segment, count, _ptr(ws), _stream())
+    return y
+
+
+def ssd_decode(xbc, dt, dt_bias, a_log, skip, weight, bias, ring, state, groups: int, pos, active, overlap: int = 0):
+    """One token per slot: convolution (ring) and recurrence (state) -> y fp32 [B, heads*vdim]; xbc rows are raw projections."""
+    rows, heads, dim, vdim = state.shape
+    assert _rows(xbc) and xbc.shape == (rows, heads * vdim + 2 * groups * dim) and _rows(dt) and pos.dtype == torch.int64
+    assert ring.shape[::2] == xbc.shape and weight.shape == ring.shape[1:]
+    _require_cuda(xbc, dt, state, ring, pos)
+    y = torch.empty((rows, heads * vdim), dtype=torch.float32, device=xbc.device)
+    _lib.call("b200_ssd_decode", _ptr(xbc), xbc.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(weight),
+              _ptr(bias), _ptr(ring), ring.shape[1], _ptr(state), _ptr(pos), _ptr(active), _ptr(y), rows, heads, groups, dim, vdim,
+              _f32(xbc), int(overlap), _stream())
+    return y
+
+
+def gated_group_norm(y, z, weight, out, heads: int, true_vdim: int, groups: int, eps: float, overlap: int = 0):
+    """out = f / rms(f) * weight with f = y * silu(z), the root mean square over each of `groups` equal parts of the channels;
+    heads of weight.numel() / heads columns, the first true_vdim of each in use."""
+    assert _rows(y) and _rows(z) and _rows(out) and y.shape == z.shape == out.shape and weight.numel() == y.shape[1]
+    assert z.dtype == out.dtype and weight.dtype == torch.float32
+    _require_cuda(y, z, weight, out)
+    _lib.call("b200_gated_group_norm", _ptr(y), y.stride(0), _ptr(z), z.stride(0), _ptr(weight), _ptr(out), out.stride(0), y.shape[0],
+              heads, y.shape[1] // heads, true_vdim, groups, float(eps), _f32(y), _f32(z), int(overlap), _stream())
+    return out
+
+
+# ----------------------------------------------------------------------------------------------- gated linear attention
+def _check_gla(qkv, gate, out, norm, bias, state):
+    _, heads, dim, vdim = state.shape
+    assert _rows(qkv) and qkv.shape[1] >= heads * (2 * dim + vdim) and norm.numel() == vdim and bias.numel() == heads * dim
+    assert _rows(gate) and _rows(out) and gate.shape == out.shape == (qkv.shape[0], heads * vdim)
+    for t in (norm, bias, state):
+        assert t.dtype == torch.float32 and t.is_contiguous()
+    _require_cuda(qkv, gate, out, norm, bias, state)
+    return heads, dim, vdim
+
+
+def gla_prefill(qkv, z, bias, norm, gate, state, out, batch, true_vdim: int, q_scale: float, tau: float, eps: float,
+                serial: bool = False, segments=None):
+    """Gated linear attention of a packed batch: qkv rows [q | k | v | ...], z fp32 [tokens, heads*dim]; state in place."""
+    heads, dim, vdim = _check_gla(qkv, gate, out, norm, bias, state)
+    tokens = qkv.shape[0]
+    assert z.dtype == torch.float32 and _rows(z) and z.shape == (tokens, heads * dim)
+    chunked = qkv.dtype == torch.bfloat16 and dim <= 128 and not serial
+    segment, count = (batch.max_len, 1) if not chunked else segments or hgrn2_segments(
+        batch.max_len, batch.count * heads * -(-vdim // 128), sm_count(qkv.device))
+    ws = None
+    if count > 1:
+        ws = torch.empty(_lib.load().b200_hgrn2_workspace_bytes(batch.count, count, heads, dim, vdim) // 4, dtype=torch.float32,
+                         device=qkv.device)
+    scratch = None if chunked and vdim <= 128 else torch.empty((tokens, heads * vdim), dtype=torch.float32, device=qkv.device)
+    _lib.call("b200_gla_prefill", _ptr(qkv), qkv.stride(0), _ptr(z), z.stride(0), _ptr(bias), _ptr(norm), _ptr(gate), gate.stride(0),
+              _ptr(state), _ptr(batch.cu), _ptr(batch.slots), _ptr(batch.start), _ptr(scratch), _ptr(out), out.stride(0), batch.count,
+              tokens, heads, dim, vdim, true_vdim, float(q_scale), 1.0 / float(tau), float(eps), _f32(qkv), int(serial), segment, count,
+              _ptr(ws), _stream())
+    return out
+
+
+def gla_decode(qkv, low, w_low, bias, norm, gate, state, out, pos, active, true_vdim: int, q_scale: float, tau: float, eps: float,
+               overlap: int = 0):
+    """One token per slot; low [B, rank] (columns of the same matrix as qkv), w_low [heads*dim, rank]."""
+    heads, dim, vdim = _check_gla(qkv, gate, out, norm, bias, state)
+    assert low.stride(0) == qkv.stride(0) and w_low.shape == (heads * dim, low.shape[1]) and w_low.is_contiguous()
+    _lib.call("b200_gla_decode", _ptr(qkv), qkv.stride(0), _ptr(low), _ptr(w_low), low.shape[1], _ptr(bias), _ptr(norm), _ptr(gate),
+              gate.stride(0), _ptr(state), _ptr(pos), _ptr(active), _ptr(out), out.stride(0), qkv.shape[0], heads, dim, vdim, true_vdim,
+              float(q_scale), 1.0 / float(tau), float(eps), _f32(qkv), int(overlap), _stream())
+    return out

@@ -110,6 +110,6 @@ def _qwen_engine(cfg, weights, batch, max_context, device, **options):
     return Engine(cfg, weights, batch, max_context, device, **options)
 
 
-register(Family("Tofilorn", _hybrid_config, _hybrid_load, _hybrid_random, _hybrid_engine,
-                (torch.bfloat16, torch.float32), part="hybrid"))
+for _name in ("Tofilorn", "Dugilorn"):
+    register(Family(_name, _hybrid_config, _hybrid_load, _hybrid_random, _hybrid_engine, (torch.bfloat16, torch.float32), part="hybrid"))
 register(Family("Qwen3.5", _qwen_config, None, _qwen_random, _qwen_engine, (torch.bfloat16,)))

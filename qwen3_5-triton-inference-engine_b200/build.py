@@ -25,7 +25,7 @@ LIB = HERE / "libb200attn.so"
 # Sources one model family needs, linked into a library of their own (b200attn/_lib.py loads it when the whole library
 # has not been built): what a first run on a machine without built files compiles.
 PARTS = {
-    "hybrid": (HERE / "libb200hybrid.so", ["paged_kv", "tensor_maps", "layer_glue", "skinny_gemm", "streams", "linear_rnn", "linear_rnn_chunk",
+    "hybrid": (HERE / "libb200hybrid.so", ["paged_kv", "tensor_maps", "layer_glue", "skinny_gemm", "streams", "linear_rnn", "linear_rnn_chunk", "ssd",
                                            "latent", "latent_decode", "latent_prefill_umma", "row_attention", "window"]),
 }
 
