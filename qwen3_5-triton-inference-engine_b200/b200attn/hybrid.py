@@ -202,7 +202,7 @@ def random_tensors(weights: HybridWeights, seed: int, device="cpu", std: float =
             noise = torch.rand(shape, generator=gen, device=device) * 0.9
         elif leaf == "mix":
             noise = noise + torch.eye(shape[0], device=device)
-        elif leaf == "in":
+        elif leaf == "in" and len(shape) == 1:
             noise = noise + 1.0 / shape[0]
         elif leaf == "out":
             noise = noise + 1.0

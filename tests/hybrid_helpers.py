@@ -32,6 +32,28 @@ def stack(width, vocab, streams, layers, eps=1e-5):
             "layers": [{**layer, "mlp": None if ff is None else {"kind": "dense", "ff": ff}} for layer, ff in layers]}
 
 
+def window(heads, kv_heads, dim, vdim, size, dims=None, base=1000.0, scale=None):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": size},
+            "rot": {"base": base, "dims": dim if dims is None else dims}, "scale": scale or dim ** -0.5}
+
+
+def state_space(heads, vdim, state, groups, conv, norm_groups):
+    return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups}
+
+
+def parallel(left, right, left_scale=1.0, right_scale=1.0):
+    return {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": left_scale, "right_scale": right_scale}}
+
+
+def gla(heads, dim, vdim, tau):
+    return {"type": "gla", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}}
+
+
+def dugilorn(width, vocab, cap, layers, eps=1e-5):
+    return {"architecture": "Dugilorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "logit_softcap": cap,
+            "layers": [{**layer, "mlp": None if ff is None else {"kind": "dense", "ff": ff}} for layer, ff in layers]}
+
+
 YARN = {"factor": 8.0, "original": 64, "fast": 16.0, "slow": 0.5}
 
 CONFIGS = {
@@ -56,6 +78,27 @@ CONFIGS = {
         (latent(17, 192, 64, 256, 640, 192, 45), None),
         (hgrn2(2, 200, 72), 192),
         (latent(40, 16, 16, 16, 128, 64, 300, kv_from=None), 64)]),
+    # Dugilorn.  Sizes odd in their own way: partly rotated heads, norm parts that cut through heads, one to five taps, a
+    # window of one, layers without a feed-forward
+    "odd": dugilorn(136, 331, 12.0, [
+        (parallel(window(6, 3, 20, 24, 37, dims=12), state_space(6, 20, 24, 3, 3, 5), 0.7, 1.3), 200),
+        (gla(3, 24, 40, 8.0), None),
+        (parallel(window(5, 1, 40, 72, 1, base=50.0), state_space(4, 16, 16, 4, 1, 1), -0.9, 0.8), None),
+        (gla(2, 8, 12, 1.0), 40),
+        (parallel(window(4, 4, 16, 8, 70, scale=0.4), state_space(2, 136, 40, 1, 5, 2), 1.0, 0.5), 72)], eps=1e-4),
+    # values that often coincide
+    "plain": dugilorn(64, 64, 30.0, [(parallel(window(1, 1, 64, 64, 2), state_space(1, 64, 64, 1, 4, 1)), 64),
+                                     (gla(1, 64, 64, 16.0), 64)]),
+    # the sizes of a real layer, few of them
+    "real": dugilorn(512, 512, 50.0, [
+        (parallel(window(8, 2, 128, 128, 150, base=1e5), state_space(8, 64, 128, 2, 4, 2), 0.8, 0.6), 1024),
+        (gla(4, 128, 128, 16.0), 512),
+        (parallel(window(8, 4, 64, 192, 129, dims=32), state_space(8, 32, 64, 1, 4, 8), 0.5, 1.2), None)], eps=1e-6),
+    # more heads than a tile, keys, values, states and recurrent heads beyond the tensor-core forms
+    "broad": dugilorn(192, 260, 20.0, [
+        (parallel(window(34, 2, 72, 136, 45), state_space(3, 144, 200, 1, 9, 3), 0.9, 0.9), 64),
+        (gla(2, 200, 136, 4.0), None),
+        (parallel(window(2, 1, 264, 320, 300), state_space(4, 8, 8, 2, 2, 2), 1.1, 0.7), 64)]),
 }
 
 
@@ -81,13 +124,19 @@ def checkpoint(config, seed=0):
             x = x * 1.5
         elif leaf == "mix":
             x = 0.6 * torch.eye(shape[0]) + 0.3 * x
-        elif leaf == "in":
+        elif leaf == "dt_bias":
+            x = 1.2 * x - 1.5
+        elif leaf == "D":
+            x = 1.0 + 0.3 * x
+        elif leaf == "conv":
+            x = 0.6 * x
+        elif leaf == "in" and len(shape) == 1:
             x = (1.0 + 0.5 * x) / shape[0] ** 0.5
         elif leaf == "out":
             x = 1.0 + 0.3 * x
         elif len(shape) == 2:
             x = x / shape[1] ** 0.5
-            if leaf == "uq":
+            if leaf in ("uq", "q"):
                 x = x * 1.7                       # attention that is not flat
         out[name] = x.to(torch.bfloat16)
     return out

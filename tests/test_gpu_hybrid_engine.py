@@ -87,14 +87,14 @@ def test_whole_prompt_layer_by_layer(name, dt):
 @pytest.mark.parametrize("name", H.CONFIGS)
 def test_token_by_token_from_the_first(name, dt):
     toks, want, _ = wanted(name, 170, 1)
-    n = 60 if name == "wide" else 100
+    n = 60 if name in ("wide", "broad") else 100
     got = run_portions(engine(name, dt), 2, toks[:n], [1])
     check(name, got, want[:n], dt)
 
 
 @pytest.mark.parametrize("sizes", [[2], [3, 2], [16], [17, 1, 30], [64, 2, 63, 1], [150, 1]])
 @pytest.mark.parametrize("dt", DTYPES)
-@pytest.mark.parametrize("name", ["ragged", "large"])
+@pytest.mark.parametrize("name", ["ragged", "large", "odd", "real"])
 def test_portions(name, dt, sizes):
     toks, want, _ = wanted(name, 170, 1)
     got = run_portions(engine(name, dt), 0, toks, sizes)
@@ -131,10 +131,11 @@ def test_unequal_batch_and_used_slots(name, dt):
 
 
 @pytest.mark.parametrize("dt", DTYPES)
-def test_decoding_some_slots_leaves_the_others_alone(dt):
-    toks, want, _ = wanted("ragged", 170, 1)
-    other, other_want, _ = wanted("ragged", 60, 5)
-    eng = engine("ragged", dt)
+@pytest.mark.parametrize("name", ["ragged", "odd"])
+def test_decoding_some_slots_leaves_the_others_alone(name, dt):
+    toks, want, _ = wanted(name, 170, 1)
+    other, other_want, _ = wanted(name, 60, 5)
+    eng = engine(name, dt)
     a = [eng.extend([0], [0], [toks[:30]], [[29]])]
     b = [eng.extend([2], [0], [other[:20]], [[19]])]
     for i in range(30, 60):                                # slot 2 pauses every other step, in between both decode
@@ -145,16 +146,17 @@ def test_decoding_some_slots_leaves_the_others_alone(dt):
             both = eng.extend([2, 0], [j, i], [[other[j]], [toks[i]]], [[0], [0]])
             b.append(both[:1])
             a.append(both[1:])
-    check("ragged", torch.cat(a), want[29:60], dt)
-    check("ragged", torch.cat(b), other_want[19:35], dt)
+    check(name, torch.cat(a), want[29:60], dt)
+    check(name, torch.cat(b), other_want[19:35], dt)
 
 
-def test_long_decoding_stays_exact():
+@pytest.mark.parametrize("name", ["ragged", "odd"])
+def test_long_decoding_stays_exact(name):
     """Several windows' worth of decoded tokens: windows slide over decoded keys, pages fill, states run on."""
-    toks, want, _ = wanted("ragged", 400, 3)
-    eng = engine("ragged", "f32", context=400)
+    toks, want, _ = wanted(name, 400, 3)
+    eng = engine(name, "f32", context=400)
     got = torch.cat((eng.extend([0], [0], [toks[:20]], [list(range(20))]), run_from(eng, 0, toks, 20)))
-    check("ragged", got, want, "f32", limit=3e-5)
+    check(name, got, want, "f32", limit=3e-5)
 
 
 def run_from(eng, slot, toks, at):
@@ -163,10 +165,11 @@ def run_from(eng, slot, toks, at):
 
 @pytest.mark.parametrize("dt", DTYPES)
 @pytest.mark.parametrize("chunk", [None, 7, 64])
-def test_prefill_in_chunks_and_graph_decode(dt, chunk):
+@pytest.mark.parametrize("name", ["ragged", "odd"])
+def test_prefill_in_chunks_and_graph_decode(name, dt, chunk):
     """`prefill` (whole or cut) + `step`, eager and as a graph replay, teacher-forced on the restatement's greedy choice:
     where its margin is beyond rounding the engine's token is the same."""
-    config = H.CONFIGS["ragged"]
+    config = H.CONFIGS[name]
     w = H.oracle_weights(H.checkpoint(config))
     prompts = [H.tokens(config, n, 40 + n) for n in (3, 50, 130)]
     refs = []
@@ -178,7 +181,7 @@ def test_prefill_in_chunks_and_graph_decode(dt, chunk):
         refs.append((seq, logits))
     runs = []
     for graph in (False, True):
-        eng = engine("ragged", dt, on_demand_pages=False, page_seed=3, prefill_chunk=chunk)
+        eng = engine(name, dt, on_demand_pages=False, page_seed=3, prefill_chunk=chunk)
         ids = [eng.prefill(prompts).tolist()]
         for k in range(8):
             eng.tok.copy_(torch.tensor([refs[b][0][len(prompts[b]) + k] for b in range(3)]))
@@ -196,13 +199,14 @@ def test_prefill_in_chunks_and_graph_decode(dt, chunk):
 
 
 @pytest.mark.parametrize("graph", [False, True])
-def test_continuous_batching(graph):
+@pytest.mark.parametrize("name", ["ragged", "odd"])
+def test_continuous_batching(name, graph):
     """Requests of different lengths through few slots and a pool too small for all: every page comes back, and each
     request's greedy tokens are the restatement's (fp32; a near-tie may fall either way, checked by its margin)."""
     from b200attn.serving import ContinuousBatcher
-    config = H.CONFIGS["ragged"]
+    config = H.CONFIGS[name]
     w = H.oracle_weights(H.checkpoint(config))
-    eng = engine("ragged", "f32", batch=3, context=96, num_pages=12, prefill_chunk=20)
+    eng = engine(name, "f32", batch=3, context=96, num_pages=12, prefill_chunk=20)
     cb = ContinuousBatcher(eng, check_invariants=True)
     prompts = [H.tokens(config, n, 70 + n) for n in (5, 40, 17, 48, 33, 9)]
     budgets = [12, 20, 30, 8, 25, 28]
@@ -234,10 +238,11 @@ def test_shared_latent_reads_the_rows_of_its_source(dt):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-def test_command_line(tmp_path, dtype):
+@pytest.mark.parametrize("name", ["ragged", "odd"])
+def test_command_line(tmp_path, name, dtype):
     """generate and trace on a model folder: the trace of a prompt plus what was generated gives the same tokens."""
     from b200attn import checkpoint
-    config = H.CONFIGS["ragged"]
+    config = H.CONFIGS[name]
     (tmp_path / "config.json").write_text(json.dumps(config))
     checkpoint.write_safetensors(tmp_path / "model.safetensors", H.checkpoint(config))
     prompts = [H.tokens(config, n, 5 + n) for n in (4, 60)]
@@ -260,4 +265,4 @@ def test_command_line(tmp_path, dtype):
         got = torch.stack([torch.frombuffer(bytearray((tmp_path / f"{2 * i + k}.f32").read_bytes()), dtype=torch.float32)
                            for k in range(2)])
         assert got.shape == (2, config["vocab"])
-        check("ragged", got, want, "f32" if dtype == "float32" else "bf16")
+        check(name, got, want, "f32" if dtype == "float32" else "bf16")
