@@ -168,7 +168,7 @@ def causal_conv(x, taps, bias):
     out = torch.zeros_like(x)
     for j in range(taps.shape[1]):
         moved = torch.zeros_like(x)
-        moved[j:] = x[: x.shape[0] - j]
+        moved[j:] = x[: max(x.shape[0] - j, 0)]
         out = out + moved * taps[:, taps.shape[1] - 1 - j]
     return out + bias
 
