@@ -487,8 +487,10 @@ def main():
     ap.add_argument("--model-steps", type=int, default=512)
     ap.add_argument("--hybrid", action="store_true",
                     help="instead of the default workload: the kernels of the hybrid stacks (latent attention, HGRN2, minGRU, "
-                         "hyper-connections) and whole-model prefill / decode, beside the Qwen3.5 engine at equal size")
+                         "hyper-connections; windowed attention, state space, gated linear attention) and whole-model prefill / "
+                         "decode, beside the Qwen3.5 engine at equal size")
     ap.add_argument("--hybrid-part", default="all", choices=["all", "kernels", "models"])
+    ap.add_argument("--hybrid-design", default="all", choices=["all", "Tofilorn", "Dugilorn"])
     ap.add_argument("--workload", default="decode", choices=["decode", "chain", "prefill", "gdn", "gdn_decode", "gemm", "model_prefill"],
                     help="with --kernel-only: which kernel family to run (profiler captures of the other families)")
     args = ap.parse_args()
@@ -517,8 +519,13 @@ def main():
 
     if args.hybrid:
         with ClockSampler(local_rank) as clocks:
-            rows = run_hybrid_kernel_rows(ops, device, args.sweep_steps) if args.hybrid_part != "models" else []
-            models = run_hybrid_models(device, args.sweep_steps) if args.hybrid_part != "kernels" else []
+            rows = []
+            if args.hybrid_part != "models":
+                if args.hybrid_design != "Dugilorn":
+                    rows += run_hybrid_kernel_rows(ops, device, args.sweep_steps)
+                if args.hybrid_design != "Tofilorn":
+                    rows += run_core_kernel_rows(ops, device, args.sweep_steps)
+            models = run_hybrid_models(device, args.sweep_steps, args.hybrid_design) if args.hybrid_part != "kernels" else []
         emit({"workload": "hybrid", "data": "synthetic", "dtype": "bf16", "hbm_peak_gbs": hbm_peak(), "tensor_peak_tflops": tensor_peak(),
               "clocks": clocks.summary(), "kernels": rows, "models": models})
         return
@@ -1068,17 +1075,33 @@ def hybrid_config(width: int, layers: int, heads: int, vocab: int) -> dict:
             "layers": [{**order[i % 4], "mlp": {"kind": "dense", "ff": 7 * width // 2}} for i in range(layers)]}
 
 
-def run_hybrid_models(device, steps):
-    """Whole models of random weights: the hybrid stack and the Qwen3.5 stack of the same width, depth, feed-forward and
+def dugilorn_config(width: int, layers: int, vocab: int) -> dict:
+    """Three layers of windowed attention beside a state-space mixer and one of gated linear attention in turn; a layer's mixers
+    have about the weights of a Gated-DeltaNet layer of the Qwen3.5 stack of the same width, and its feed-forward."""
+    heads, ssm = width // 128, width // 32
+    parallel = {"type": "parallel",
+                "mixer": {"left": {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "mask": {"size": HYBRID_WINDOW},
+                                   "rot": {"base": 1e6, "dims": 128}, "scale": 128 ** -0.5},
+                          "right": {"heads": ssm, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1},
+                          "left_scale": 0.7, "right_scale": 0.7}}
+    gla = {"type": "gla", "mixer": {"heads": 2 * heads, "dim": 128, "vdim": 128, "tau": 16.0}}
+    return {"architecture": "Dugilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "layers": [{**(gla if i % 4 == 3 else parallel), "mlp": {"kind": "dense", "ff": 7 * width // 2}} for i in range(layers)]}
+
+
+def run_hybrid_models(device, steps, design="all"):
+    """Whole models of random weights: the hybrid stacks and the Qwen3.5 stack of the same width, depth, feed-forward and
     vocabulary.  Decode is one CUDA-graph replay per step after a prefill of the stated prompts; prefill is timed from the
     first host instruction to the last kernel (median of five)."""
     from b200attn import models
     vocab, rows = 65536, []
     for width, layers, heads in ((1024, 24, 16), (2048, 12, 32)):
-        stacks = {"Tofilorn": hybrid_config(width, layers, heads, vocab),
+        stacks = {"Tofilorn": hybrid_config(width, layers, heads, vocab), "Dugilorn": dugilorn_config(width, layers, vocab),
                   "Qwen3.5": {"architecture": "Qwen3.5", "hidden": width, "num_layers": layers, "num_q_heads": heads // 2,
                               "num_kv_heads": heads // 8, "gdn_heads": heads, "intermediate": 7 * width // 2, "vocab": vocab}}
         for name, config in stacks.items():
+            if name in ("Tofilorn", "Dugilorn") and design not in ("all", name):
+                continue
             model = models.random_model(config, seed=4, device=device)
             for batch, prompt in ((1, 2048), (32, 128), (32, 2048), (8, 4096)):
                 gen = torch.Generator().manual_seed(4)
@@ -1130,17 +1153,12 @@ class _Rows:
         self.slot_of = self.slots.repeat_interleave(length)
 
 
-def run_hybrid_kernel_rows(ops, device, steps):
-    """Every kernel of the hybrid stacks at a real layer's sizes beside the like kernel of the Qwen3.5 stack: algorithmic bytes
-    (or FLOPs) over device time.  Inputs rotate over enough copies that no call finds its own in L2."""
-    from b200attn import hybrid_ops as hops
-    from b200attn.mixers import Rotation
-    hbm, tensor = hbm_peak()[0], tensor_peak()[0]
-    bf, f32 = torch.bfloat16, torch.float32
-    rows = []
+def _kernel_rows(device, steps):
+    """(rows, random tensor, timer that appends a row, copies of an input so that no call finds its own in L2)"""
+    hbm, tensor, rows = hbm_peak()[0], tensor_peak()[0], []
 
-    def rnd(*shape, dtype=bf):
-        return torch.randn(*shape, dtype=f32, device=device).mul_(0.5).to(dtype)
+    def rnd(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, dtype=torch.float32, device=device).mul_(0.5).to(dtype)
 
     def row(op, like, shape, fn, sets, nbytes=None, flops=None):
         ms = time_steps(fn, max(steps, sets), 3)
@@ -1155,6 +1173,18 @@ def run_hybrid_kernel_rows(ops, device, steps):
 
     def copies(nbytes):
         return max(1, min(48, cdiv(3 * L2_BYTES, nbytes)))
+
+    return rows, rnd, row, copies
+
+
+def run_hybrid_kernel_rows(ops, device, steps):
+    """Every kernel of the hybrid stacks at a real layer's sizes beside the like kernel of the Qwen3.5 stack: algorithmic bytes
+    (or FLOPs) over device time.  Inputs rotate over enough copies that no call finds its own in L2."""
+    from b200attn import hybrid_ops as hops
+    from b200attn.mixers import Rotation
+    hbm = hbm_peak()[0]
+    bf, f32 = torch.bfloat16, torch.float32
+    rows, rnd, row, copies = _kernel_rows(device, steps)
 
     # ---- decode attention
     for batch, heads, ctx in ((1, 16, 4096), (32, 16, 4096), (32, 32, 4096), (256, 16, 2048), (32, 16, 640)):
@@ -1271,6 +1301,169 @@ def run_hybrid_kernel_rows(ops, device, steps):
         n2 = copies(nb)
         rs = [rnd(tokens, width) for _ in range(n2)]
         wn = torch.zeros(width, dtype=bf, device=device)
+        row("add_rmsnorm", None, f"{tokens} rows, width {width}", lambda i: ops.add_rmsnorm(y, wn, 1e-6, residual=rs[i % n2]), n2, nb)
+        del xs, rs
+    return rows
+
+
+def run_core_kernel_rows(ops, device, steps):
+    """The kernels of the Dugilorn layers at a real layer's sizes beside the like kernels of the Qwen3.5 stack (rows whose `like`
+    is None), counted as in run_hybrid_kernel_rows."""
+    from b200attn import hybrid_ops as hops
+    from b200attn.mixers import Rotation
+    bf, f32 = torch.bfloat16, torch.float32
+    rows, rnd, row, copies = _kernel_rows(device, steps)
+    sms = torch.cuda.get_device_properties(device).multi_processor_count
+    # ---- decode attention
+    for batch, heads, kv, dim, ctx in ((1, 16, 4, 128, 2048), (32, 16, 4, 128, 2048), (32, 8, 2, 128, 4096), (32, 16, 4, 128, 640),
+                                       (32, 8, 2, 96, 2048), (256, 16, 4, 128, 2048)):
+        vdim = 2 * dim if dim == 96 else dim
+        pitch, pages = cdiv(dim + vdim, 64) * 64, ctx // 16
+        nbytes = batch * (ctx * kv * (dim + vdim) * 2 + heads * (dim + vdim) * 2)
+        n = copies(nbytes)
+        caches = [rnd(batch * pages, kv, 16, pitch) for _ in range(n)]
+        tables = [torch.randperm(batch * pages, device=device).view(batch, pages).to(torch.int32) for _ in range(n)]
+        x, gate = rnd(batch, (heads + kv) * dim + kv * vdim), rnd(batch, heads * vdim)
+        pos = torch.full((batch,), ctx - 1, dtype=torch.int64, device=device)
+        splits = hops.window_decode_splits(batch, heads, kv, ctx, sms)
+        ws = hops.latent_decode_workspace(batch, heads, vdim, splits, device)
+        shape = f"B={batch} H={heads}/{kv} {dim}+{vdim} ctx={ctx} splits={splits}"
+        row("window_decode", "fused_decode_attention", shape,
+            lambda i: hops.window_decode(x, caches[i % n], tables[i % n], pos, None, ws, dim, HYBRID_WINDOW, 0.07), n, nbytes)
+        out = torch.empty(batch, heads * vdim, dtype=bf, device=device)
+        row("window_merge", "paged_decode_combine", shape, lambda i: hops.window_merge(ws, gate, out), 1,
+            batch * heads * (splits * (vdim * 4 + 8) + vdim * 4))
+        angles, bias = Rotation(dim, 1e6).table(ctx, device), torch.zeros(x.shape[1], device=device)
+        row("window_prep", "add_rmsnorm", shape,
+            lambda i: hops.window_prep(x, bias, pos, None, None, tables[0], angles, caches[0], heads, dim, vdim), 1, x.numel() * 4)
+        del caches
+    for batch in (1, 32, 256):
+        w = Workload([2048] * batch, device, max_sets=32)
+        fd = fused_step(ops, w, ops.fused_decode_workspace(device))
+        row("fused_decode_attention", None, f"B={batch} ctx=2048", fd, w.sets, w.bytes)
+        del w, fd
+    # ---- prefill attention
+    for batch, length, heads, kv in ((8, 4096, 16, 4), (32, 128, 16, 4), (1, 2048, 16, 4)):
+        dim = vdim = 128
+        pitch, total = dim + vdim, batch * length
+        b = _Rows(batch, length, device)
+        x, ctx = rnd(total, (heads + kv) * dim + (kv + heads) * vdim), rnd(total, kv, pitch)
+        out = torch.empty(total, heads * vdim, dtype=bf, device=device)
+        gate = x[:, (heads + kv) * dim + kv * vdim:]
+        for window in (HYBRID_WINDOW, 1024):
+            pairs = sum(min(i + 1, window) for i in range(length)) * batch
+            row("window_prefill", "gqa_attention_varlen_causal", f"{batch}x{length} H={heads}/{kv} window={window}",
+                lambda i: hops.window_prefill(x, ctx, gate, out, b.cu, b.cu, b.start, b.start, length, heads, dim, dim, vdim, window, 0.07), 1,
+                total * (heads * (dim + 2 * vdim) + kv * pitch) * 2, 2 * pairs * heads * (dim + vdim))
+        cu, max_len = ops.build_cu_seqlens([length] * batch, device=device)
+        qq, kk, vv = rnd(total, HQ, D), rnd(total, HKV, D), rnd(total, HKV, D)
+        row("gqa_attention_varlen_causal", None, f"{batch}x{length}", lambda i: ops.gqa_attention_varlen_causal(qq, kk, vv, cu, max_len), 1,
+            total * (2 * HQ + 2 * HKV) * D * 2, 4 * HQ * D * batch * length * (length + 1) // 2)
+        angles, bias = Rotation(dim, 1e6).table(length, device), torch.zeros((heads + 2 * kv) * dim, device=device)
+        table = torch.arange(batch * cdiv(length, 16), dtype=torch.int32, device=device).view(batch, -1)
+        cache = hops.allocate_window_cache(table.numel(), kv, pitch, bf, device=device)
+        at = torch.arange(total, dtype=torch.int32, device=device)
+        row("window_prep", "add_rmsnorm", f"{batch}x{length} H={heads}/{kv}",
+            lambda i: hops.window_prep(x, bias, b.pos, b.slot_of, None, table, angles, cache, heads, dim, vdim, ctx=ctx, ctx_row=at), 1,
+            total * ((heads + 2 * kv) * dim * 2 + heads * dim * 2 + kv * pitch * 4))
+        row("window_gather", "add_rmsnorm", f"{batch}x{length}",
+            lambda i: hops.window_gather(cache, ctx, table, b.slots, b.cu, b.start, length), 1, total * kv * pitch * 4)
+        del x, ctx, out, qq, kk, vv, cache
+    # ---- recurrences, prefill
+    from b200attn.glue_ops import depthwise_causal_conv4_prefill
+    conv = getattr(depthwise_causal_conv4_prefill, "_init_fn", depthwise_causal_conv4_prefill)
+    ones = torch.ones(8192, device=device)
+    for batch, length in ((32, 128), (1, 2048), (32, 1024)):
+        total = batch * length
+        b = _Rows(batch, length, device)
+        for heads, groups, vdim, state_rows in ((32, 1, 64, 128), (64, 8, 64, 128), (16, 1, 128, 64)):
+            inner, channels = heads * vdim, heads * vdim + 2 * groups * state_rows
+            state = torch.zeros(batch, heads, state_rows, vdim, device=device)
+            nbytes = total * (channels * 2 + heads * 2 + inner * 2) + state.numel() * 4
+            n = copies(nbytes)
+            xbc, dt = [rnd(total, channels) for _ in range(n)], rnd(total, heads)
+            shape = f"{batch}x{length} H={heads} groups={groups} {state_rows}x{vdim}"
+            row("ssd_prefill", "gdn_chunked_prefill", shape,
+                lambda i: hops.ssd_prefill(xbc[i % n], dt, ones[:heads], -ones[:heads], ones[:heads], state, groups, b), n, nbytes)
+            if vdim == 64:
+                ring, w4 = torch.zeros(batch, 4, channels, device=device), rnd(4, channels, dtype=f32)
+                row("conv_prefill", "depthwise_causal_conv4_prefill", f"{batch}x{length} channels={channels}",
+                    lambda i: hops.conv_prefill(xbc[i % n], w4, ones[:channels], ring, b), n, total * channels * 4)
+                out, z = torch.empty(total, inner, dtype=bf, device=device), [rnd(total, inner) for _ in range(n)]
+                row("gated_group_norm", "gdn_gated_rmsnorm", f"{batch}x{length} groups={groups} of {inner // groups}",
+                    lambda i: hops.gated_group_norm(z[i % n], z[(i + 1) % n], ones[:inner], out, heads, vdim, groups, 1e-6), n, total * inner * 6)
+                del out, z
+            del xbc
+        heads = 16
+        state = torch.zeros(batch, heads, 128, 128, device=device)
+        nbytes = total * heads * 128 * (2 * 5 + 4) + state.numel() * 4
+        n = copies(nbytes)
+        x, z = [rnd(total, 4 * heads * 128) for _ in range(n)], [rnd(total, heads * 128, dtype=f32) for _ in range(n)]
+        out = torch.empty(total, heads * 128, dtype=bf, device=device)
+        row("gla_prefill", "gdn_chunked_prefill", f"{batch}x{length} H={heads} 128x128",
+            lambda i: hops.gla_prefill(x[i % n], z[i % n], ones[: heads * 128], ones[:128], x[i % n][:, 3 * heads * 128:], state, out, b, 128, 0.09,
+                                       16.0, 1e-6), n, nbytes)
+        gq = torch.nn.functional.normalize(torch.randn(total, heads, 128, device=device), dim=-1).to(bf)
+        beta, g = torch.rand(total, heads, device=device), -torch.rand(total, heads, device=device)
+        cu, _ = ops.build_cu_seqlens([length] * batch, device=device)
+        row("gdn_chunked_prefill", None, f"{batch}x{length} H={heads} 128x128", lambda i: ops.gdn_chunked_prefill_packed(gq, gq, gq, beta, g, cu), 1,
+            total * heads * (4 * 128 * 2 + 8) + batch * heads * 128 * 128 * 4)
+        del x, z, out
+        nb = total * 6144 * 2 * 2
+        n = copies(nb)
+        cx, w4, seq_start = [rnd(total, 6144) for _ in range(n)], rnd(6144, 4), (b.slot_of * length).to(torch.int32)
+        row("depthwise_causal_conv4_prefill", None, f"{batch}x{length} channels=6144", lambda i: conv(cx[i % n], w4, seq_start), n, nb)
+        del cx
+        gx = [rnd(total, heads, 128) for _ in range(copies(total * heads * 128 * 6))]
+        n = len(gx)
+        row("gdn_gated_rmsnorm", None, f"{batch}x{length} H={heads}",
+            lambda i: ops.gdn_gated_rmsnorm_fused(gx[i % n], gx[(i + 1) % n].view(total, -1), ones[:128]), n, total * heads * 128 * 6)
+        del gx
+        ff = 3584
+        n = copies(total * ff * 6)
+        gu, act = [rnd(total, 2 * ff) for _ in range(n)], torch.empty(total, ff, dtype=bf, device=device)
+        row("gated_act", "swiglu", f"{batch}x{length} width={ff}", lambda i: hops.gated_act(gu[i % n], ff, act, hops.ACT_GELU_TANH), n, total * ff * 6)
+        row("swiglu", None, f"{batch}x{length} width={ff}", lambda i: ops.swiglu_fused(gu[i % n], ff), n, total * ff * 6)
+        del gu, act
+    # ---- recurrences, decode
+    for batch in (1, 32, 256):
+        pos = torch.ones(batch, dtype=torch.int64, device=device)
+        for heads, groups, vdim, state_rows in ((32, 1, 64, 128), (64, 8, 64, 128)):
+            inner, channels = heads * vdim, heads * vdim + 2 * groups * state_rows
+            nbytes = batch * (heads * vdim * state_rows * 8 + channels * (2 + 16) + inner * 4)
+            n = copies(nbytes)
+            states = [torch.zeros(batch, heads, state_rows, vdim, device=device) for _ in range(n)]
+            xbc, dt, ring, w4 = rnd(batch, channels), rnd(batch, heads), torch.zeros(batch, 4, channels, device=device), rnd(4, channels, dtype=f32)
+            row("ssd_decode", "gdn_decode_fused", f"B={batch} H={heads} groups={groups} {state_rows}x{vdim}",
+                lambda i: hops.ssd_decode(xbc, dt, ones[:heads], -ones[:heads], ones[:heads], w4, ones[:channels], ring, states[i % n], groups, pos,
+                                          None), n, nbytes)
+            del states
+        y, z, out = rnd(batch, 2048, dtype=f32), rnd(batch, 2048), torch.empty(batch, 2048, dtype=bf, device=device)
+        row("gated_group_norm", "gdn_gated_rmsnorm", f"B={batch} 2048", lambda i: hops.gated_group_norm(y, z, ones[:2048], out, 32, 64, 1, 1e-6), 1,
+            batch * 2048 * 8)
+        heads = 16
+        nbytes = batch * heads * (2 * 128 * 128 * 4 + 5 * 128 * 2)
+        n = copies(nbytes)
+        states = [torch.zeros(batch, heads, 128, 128, device=device) for _ in range(n)]
+        x, w_low, out = rnd(batch, 4 * heads * 128 + 16), rnd(heads * 128, 16), torch.empty(batch, heads * 128, dtype=bf, device=device)
+        row("gla_decode", "gdn_decode_fused", f"B={batch} H={heads} 128x128",
+            lambda i: hops.gla_decode(x, x[:, 4 * heads * 128:], w_low, ones[: heads * 128], ones[:128], x[:, 3 * heads * 128: 4 * heads * 128],
+                                      states[i % n], out, pos, None, 128, 0.09, 16.0, 1e-6), n, nbytes)
+        del states
+        gu, act = rnd(batch, 7168), torch.empty(batch, 3584, dtype=bf, device=device)
+        row("gated_act", "swiglu", f"B={batch} width=3584", lambda i: hops.gated_act(gu, 3584, act, hops.ACT_GELU_TANH), 1, batch * 3584 * 6)
+        row("swiglu", None, f"B={batch} width=3584", lambda i: ops.swiglu_fused(gu, 3584), 1, batch * 3584 * 6)
+    rows += [{**r, "like": None} for r in run_gdn_decode_rows(ops, device, hbm_peak()[0], steps, (1, 32, 256))]
+    # ---- residual and norm
+    for tokens, width in ((32, 1024), (4096, 1024), (32768, 1024), (4096, 2048)):
+        nbytes = tokens * width * (2 * 4 + 2 + 2)
+        n = copies(nbytes)
+        xs, y = [rnd(tokens, 1, width, dtype=f32) for _ in range(n)], rnd(tokens, width)
+        row("hyper_connect (one stream, weights)", "add_rmsnorm", f"{tokens} rows, width {width}",
+            lambda i: hops.hyper_connect(xs[i % n], ones[:4], width, 1e-6, bf, y=y, gains=ones[:width]), n, nbytes)
+        nb = tokens * width * 8
+        n2 = copies(nb)
+        rs, wn = [rnd(tokens, width) for _ in range(n2)], torch.zeros(width, dtype=bf, device=device)
         row("add_rmsnorm", None, f"{tokens} rows, width {width}", lambda i: ops.add_rmsnorm(y, wn, 1e-6, residual=rs[i % n2]), n2, nb)
         del xs, rs
     return rows
