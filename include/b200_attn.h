@@ -358,6 +358,9 @@ int b200_gdn_decode_fused(const void* fused, int64_t fused_stride, void* conv_st
  * Replaces triton_kernels/gemm_2d.py for the decode-step projections of the hidden state. */
 int b200_skinny_gemm(const void* x, int64_t x_stride, const void* weight, void* y, int64_t y_stride, int32_t m,
                      int32_t n, int32_t k, int32_t overlap, b200_stream_t stream);
+/* The same for columns of a wider weight matrix: rows w_stride elements apart (one part of a product split along K). */
+int b200_skinny_gemm_part(const void* x, int64_t x_stride, const void* weight, int64_t w_stride, void* y, int64_t y_stride,
+                          int32_t m, int32_t n, int32_t k, int32_t overlap, b200_stream_t stream);
 /* The gate/up projection of the MLP with its activation folded into the epilogue (one launch instead of two):
  *   weight = [gate rows | up rows] [2*intermediate, K];  y[:, j] = silu(bf16(x . gate_j)) * bf16(x . up_j)
  * (triton_kernels/gemm_2d.py on the fused gate/up weight followed by triton_kernels/swiglu.py).  y is
@@ -448,9 +451,10 @@ int b200_swiglu_pair(const void* gate, int64_t gate_stride, const void* up, int6
  * b200_hyper_connect: S residual streams (fp32 [rows, S, width]) between two sublayers:
  *     x_t <- sum_s mix[s,t] x_s + out[t] * y;   h = (sum_s in[s] x_s) / sqrt(mean(.^2) + eps) * gain
  *   weights = [mix S*S | out S | in S | gain] fp32; gains fp32 [width] or NULL: h is multiplied by it as well.  ids != NULL: the streams are first set to table[ids[row]] (y NULL).
+ *   y comes as y_parts matrices [rows, width], one behind the other, that are summed (a product split along K).
  *   y == NULL, ids == NULL: streams are only read. */
 int b200_hyper_connect(const void* ids, int32_t ids_are_int64, const void* table, float* streams, const void* y,
-                       const float* weights, const float* gains, void* h, int32_t rows, int32_t num_streams, int32_t width,
+                       int32_t y_parts, const float* weights, const float* gains, void* h, int32_t rows, int32_t num_streams, int32_t width,
                        int32_t true_width, float eps, int32_t f32, int32_t overlap, b200_stream_t stream);
 /* b200_gated_act: out[r,c] = act(x[r,c]) * x[r, up + c], c < width, over strided rows (8-element groups).
  * b200_softcap: logits[r,c] <- cap * tanh(logits[r,c] / cap) in place for c < vocab, -inf for vocab <= c < width. */

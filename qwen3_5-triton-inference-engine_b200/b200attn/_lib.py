@@ -46,6 +46,7 @@ SIGNATURES: dict[str, list] = {
     "b200_gdn_chunked_prefill_packed": [P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I32, I32, I32,
                                         P, P, P, I64, I64, I32, I32, I32, P],
     "b200_skinny_gemm": [P, I64, P, P, I64, I32, I32, I32, I32, P],
+    "b200_skinny_gemm_part": [P, I64, P, I64, P, I64, I32, I32, I32, I32, P],
     "b200_skinny_gemm_swiglu": [P, I64, P, P, I64, I32, I32, I32, I32, P],
     "b200_argmax_rows": [P, I64, P, P, I32, I32, I32, P],
     "b200_lm_head_argmax": [P, I64, P, P, P, I32, I32, I32, I32, P],
@@ -63,7 +64,7 @@ SIGNATURES: dict[str, list] = {
     "b200_swiglu_pair": [P, I64, P, I64, P, I32, I32, P],
     "b200_gdn_chunked_prefill_fused": [P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I64, I64, P, I32, I32,
                                        P, P, I64, I64, I32, I32, I32, P],
-    "b200_hyper_connect": [P, I32, P, P, P, P, P, P, I32, I32, I32, I32, c_float, I32, I32, P],
+    "b200_hyper_connect": [P, I32, P, P, P, I32, P, P, P, I32, I32, I32, I32, c_float, I32, I32, P],
     "b200_swiglu_f32": [P, I64, P, I32, I32, P],
     "b200_mingru_prefill": [P, I64, P, P, P, P, P, P, P, I32, I32, I32, I32, I32, P],
     "b200_mingru_decode": [P, I64, P, P, P, P, P, I32, I32, I32, I32, P],

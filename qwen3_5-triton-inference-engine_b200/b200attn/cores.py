@@ -8,7 +8,8 @@ which reads the same normed input (mixers side by side, a mixer and a feed-forwa
     load(get, width_p, dtype, device)    -> (input rows [in_size, width_p], output columns [width_p, out_size])
     allocate(engine)                     cache or state, indexed by page or by slot
     prefill(x, out, batch, engine, state)          packed tokens; x and out are column ranges of the unit's matrices
-    decode(x, out, engine, state, own_next)        one token per slot, no host value that changes from step to step
+    decode(x, out, engine, state, first, last)     one token per slot, no host value that changes from step to step; first and
+                                                   last: overlap flags of its first and its last kernel
 """
 from __future__ import annotations
 
@@ -27,6 +28,11 @@ def _by_head(w, heads: int, size: int, size_p: int, *rest: int):
 
 def _out_by_head(w, heads: int, size: int, size_p: int, width_p: int):
     return padded(w.view(w.shape[0], heads, size), width_p, heads, size_p).flatten(1, 2)
+
+
+def one_kernel(first: int, last: int) -> int:
+    """Overlap flags of a kernel that is both: starts as the first, triggers as the last."""
+    return (first & ops.OVERLAP_START) | (last & ops.OVERLAP_TRIGGER)
 
 
 class Core:
@@ -84,13 +90,13 @@ class WindowAttention(Core):
         hops.window_prefill(x, ctx, x[:, self.qkv:], out, batch.cu, span.cu, batch.start, span.first, batch.max_len, self.heads, self.dim_p,
                             self.dim, self.vdim_p, self.window, self.score_scale, self.scale)
 
-    def decode(self, x, out, engine, state, own_next: bool) -> None:
+    def decode(self, x, out, engine, state, first: int, last: int) -> None:
         then = engine.then(True)
         hops.window_prep(x, self.bias, engine.pos, None, engine.active, engine.block_table, state["angles"], state["cache"], self.heads,
-                         self.dim_p, self.vdim_p, overlap=then)
+                         self.dim_p, self.vdim_p, overlap=first)
         hops.window_decode(x, state["cache"], engine.block_table, engine.pos, engine.active, state["workspace"], self.dim_p, self.window,
                            self.score_scale, overlap=then)
-        hops.window_merge(state["workspace"], x[:, self.qkv:], out, self.scale, overlap=engine.then(own_next))
+        hops.window_merge(state["workspace"], x[:, self.qkv:], out, self.scale, overlap=last)
 
 
 # --------------------------------------------------------------------------------------------------------- state space
@@ -144,11 +150,11 @@ class StateSpace(Core):
         y = hops.ssd_prefill(xbc, x[:, self.dt_at:], self.dt_bias, self.a_log, self.skip, state["state"], self.groups, batch)
         hops.gated_group_norm(y, x[:, : self.out_size], self.norm, out, self.heads, self.vdim, self.norm_groups, self.eps)
 
-    def decode(self, x, out, engine, state, own_next: bool) -> None:
+    def decode(self, x, out, engine, state, first: int, last: int) -> None:
         y = hops.ssd_decode(x[:, self.out_size: self.dt_at], x[:, self.dt_at:], self.dt_bias, self.a_log, self.skip, self.conv,
-                            self.conv_bias, state["ring"], state["state"], self.groups, engine.pos, engine.active, overlap=engine.then(True))
+                            self.conv_bias, state["ring"], state["state"], self.groups, engine.pos, engine.active, overlap=first)
         hops.gated_group_norm(y, x[:, : self.out_size], self.norm, out, self.heads, self.vdim, self.norm_groups, self.eps,
-                              overlap=engine.then(own_next))
+                              overlap=last)
 
 
 # ----------------------------------------------------------------------------------------------- gated linear attention
@@ -199,10 +205,10 @@ class GatedLinear(Core):
         z = F.linear(low, self.w_low) if x.dtype == torch.float32 else torch.mm(low, self.w_low.t(), out_dtype=torch.float32)
         hops.gla_prefill(qkv, z, self.bias, self.norm, gate, state["state"], out, batch, self.vdim, self.dim ** -0.5, self.tau, self.eps)
 
-    def decode(self, x, out, engine, state, own_next: bool) -> None:
+    def decode(self, x, out, engine, state, first: int, last: int) -> None:
         qkv, gate, low = self._split(x)
         hops.gla_decode(qkv, low, self.w_low, self.bias, self.norm, gate, state["state"], out, engine.pos, engine.active, self.vdim,
-                        self.dim ** -0.5, self.tau, self.eps, overlap=engine.then(own_next))
+                        self.dim ** -0.5, self.tau, self.eps, overlap=one_kernel(first, last))
 
 
 # -------------------------------------------------------------------------------------------------------- feed-forward
@@ -227,8 +233,8 @@ class GatedMLP(Core):
     def prefill(self, x, out, batch, engine, state) -> None:
         hops.gated_act(x, self.out_size, out, self.act)
 
-    def decode(self, x, out, engine, state, own_next: bool) -> None:
-        hops.gated_act(x, self.out_size, out, self.act, overlap=engine.then(own_next))
+    def decode(self, x, out, engine, state, first: int, last: int) -> None:
+        hops.gated_act(x, self.out_size, out, self.act, overlap=one_kernel(first, last))
 
 
 # ---------------------------------------------------------------------------------------------------- layers from cores
@@ -276,13 +282,17 @@ class FusedUnit:
         rows, cols = zip(*(core.load(lambda n, pre=pre: get(pre + n), width_p, dtype, device) for pre, core in self.parts))
         self.ins = [r.shape[0] for r in rows]
         self.outs = [c.shape[1] for c in cols]
+        # the product out, in parts along K that the weight-streaming kernel splits over pairs of CTAs
         used = sum(self.outs)
-        size = round_up(used, 128)               # a size the weight-streaming product takes, if there is one nearby
-        if not ops.skinny_gemm_supports(1, width_p, size):
-            size = next((s for s in range(size, size + 1024, 128) if ops.skinny_gemm_supports(1, width_p, s)), size)
+        parts = -(-used // ops.SKINNY_GEMM_PAIR_MAX_K)
+        part = next((n for n in range(round_up(-(-used // parts), 128), ops.SKINNY_GEMM_PAIR_MAX_K + 1, 128)
+                     if ops.skinny_gemm_supports(1, width_p, n)), round_up(-(-used // parts), 128))
+        size = part * parts
         self.pad = size - used
         self.w_in = torch.cat(rows).to(device, dtype)
         self.w_out = padded(torch.cat(cols, dim=1), width_p, size).to(device, dtype)
+        self.part = part
+        self.w_parts = list(self.w_out.split(part, dim=1))
 
     def keys(self):
         """Where the cores' caches and states live in the engine's table."""
@@ -306,10 +316,33 @@ class FusedUnit:
     def starts_own(self, engine) -> bool:
         return engine.streams_weight(self.w_in)
 
+    def out_parts(self, engine):
+        """(weight, first and last column) of the product's parts in a decode step, or None: one library product."""
+        if not all(engine.streams_weight(w) for w in self.w_parts):
+            return None
+        return [(w, n * self.part, (n + 1) * self.part) for n, w in enumerate(self.w_parts)]
+
     def decode(self, h, engine, states, nxt: bool):
-        fused = engine.proj(h, self.w_in, True)
+        """Several cores: the first runs on the current stream, the others beside it on a second one."""
+        own, side = engine.then(True), len(self.parts) > 1
+        outs = self.out_parts(engine)
+        own_out = outs is not None
+        fused = engine.proj(h, self.w_in, not side)
         act = engine.zero_scratch(sum(self.outs), self.pad)      # padding columns stay zero
-        last = self.keys()[-1]
-        for key, (_, core), x, out in self._ranges(fused, act):
-            core.decode(x, out, engine, states[key], engine.streams_weight(self.w_out) if key == last else True)
-        return engine.proj(act, self.w_out, nxt)
+        ranges = list(self._ranges(fused, act))
+        plain = own & ~ops.OVERLAP_START                          # behind a kernel of another stream
+        if side:
+            with torch.cuda.stream(engine.fork()):
+                for n, (key, (_, core), x, out) in enumerate(ranges[1:]):
+                    core.decode(x, out, engine, states[key], own if n else plain, own if n + 2 < len(ranges) else own & ~ops.OVERLAP_TRIGGER)
+        key, (_, core), x, out = ranges[0]
+        core.decode(x, out, engine, states[key], plain if side else own, engine.then(own_out and not side))
+        if side:
+            engine.join()
+        if not own_out:
+            return F.linear(act, self.w_out)
+        y = torch.empty((len(outs), act.shape[0], self.w_out.shape[0]), dtype=act.dtype, device=act.device)
+        for n, (weight, lo, hi) in enumerate(outs):
+            flags = engine.then(nxt or n + 1 < len(outs))
+            ops.skinny_gemm_part(act[:, lo:hi], weight, y[n], overlap=flags & ~ops.OVERLAP_START if side and n == 0 else flags)
+        return y

@@ -274,7 +274,7 @@ class HybridEngine(SlotEngine):
         # 32-bit means 32-bit: no TF32 products, no 16-bit partial sums
         torch.backends.cuda.matmul.allow_tf32 = False
         torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
-        self._tables, self._workspaces, self._scratch = {}, {}, {}
+        self._tables, self._workspaces, self._scratch, self._side = {}, {}, {}, None
         self.states: dict = {}               # caches and states of the units, by the unit's own keys (a mixer's: its layer)
         for unit in weights.units:
             self.states |= unit.allocate(self)
@@ -312,6 +312,16 @@ class HybridEngine(SlotEngine):
     def then(self, own_next: bool) -> int:
         """Overlap flags of a decode-step kernel whose successor is (not) one of this package's."""
         return ops.OVERLAP_START | ops.OVERLAP_TRIGGER if own_next else ops.OVERLAP_START
+
+    def fork(self):
+        """A second stream that has waited for the current one (`join` waits for it in turn)."""
+        if self._side is None:
+            self._side = torch.cuda.Stream(device=self.device)
+        self._side.wait_stream(torch.cuda.current_stream(self.device))
+        return self._side
+
+    def join(self) -> None:
+        torch.cuda.current_stream(self.device).wait_stream(self._side)
 
     def proj(self, x, weight, own_next: bool):
         """Decode-step projection: the weight-streaming kernel where it takes the shape, cuBLAS otherwise."""

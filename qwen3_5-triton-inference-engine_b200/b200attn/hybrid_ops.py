@@ -25,14 +25,16 @@ def hyper_connect(streams, weights, true_width: int, eps: float, dtype, y=None, 
     assert weights.numel() == s * s + 2 * s + 1
     assert gains is None or (gains.dtype == torch.float32 and gains.numel() == width and gains.is_contiguous())
     h = torch.empty((rows, width), dtype=dtype, device=streams.device)
-    if y is not None:
-        assert y.shape == (rows, width) and y.is_contiguous() and y.dtype == dtype
+    parts = 1
+    if y is not None:                       # [rows, width], or [parts, rows, width] to be summed
+        parts = y.shape[0] if y.ndim == 3 else 1
+        assert y.shape[-2:] == (rows, width) and y.is_contiguous() and y.dtype == dtype
     if ids is not None:
         assert ids.numel() == rows and ids.is_contiguous() and ids.dtype in (torch.int32, torch.int64)
         assert table.dtype == dtype and table.shape[1] == width and table.is_contiguous()
     _require_cuda(streams, weights)
     _lib.call("b200_hyper_connect", _ptr(ids), int(ids is not None and ids.dtype == torch.int64), _ptr(table), _ptr(streams),
-              _ptr(y), _ptr(weights), _ptr(gains), _ptr(h), rows, s, width, true_width, float(eps), _f32(h), int(overlap),
+              _ptr(y), parts, _ptr(weights), _ptr(gains), _ptr(h), rows, s, width, true_width, float(eps), _f32(h), int(overlap),
               _stream())
     return h
 

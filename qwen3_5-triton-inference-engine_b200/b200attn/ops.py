@@ -888,6 +888,16 @@ def skinny_gemm(x, weight, overlap: int = 0, swiglu: bool = False):
     return y
 
 
+def skinny_gemm_part(x, weight, out, overlap: int = 0):
+    """out = x @ weight^T where weight is a column range of a wider matrix: one part of a product split along K."""
+    assert x.shape[1] == weight.shape[1] and x.stride(1) == weight.stride(1) == 1 and out.shape == (x.shape[0], weight.shape[0])
+    assert x.dtype == weight.dtype == out.dtype == torch.bfloat16 and out.stride(1) == 1
+    _require_cuda(x, weight, out)
+    _lib.call("b200_skinny_gemm_part", _ptr(x), x.stride(0), _ptr(weight), weight.stride(0), _ptr(out), out.stride(0), *x.shape[:1],
+              weight.shape[0], x.shape[1], int(overlap), _stream())
+    return out
+
+
 # eager callers reach the implementations directly; the registered operators stay available as `<name>.op` and under
 # torch.ops.wy_lib (see _direct.py)
 from ._direct import rebind as _rebind  # noqa: E402

@@ -26,7 +26,7 @@ LIB = HERE / "libb200attn.so"
 # has not been built): what a first run on a machine without built files compiles.
 PARTS = {
     "hybrid": (HERE / "libb200hybrid.so", ["paged_kv", "tensor_maps", "layer_glue", "skinny_gemm", "streams", "linear_rnn", "linear_rnn_chunk", "ssd",
-                                           "latent", "latent_decode", "latent_prefill_umma", "row_attention", "window"]),
+                                           "latent", "latent_decode", "latent_prefill_umma", "row_attention", "window", "window_pair_umma"]),
 }
 
 NVCC_FLAGS = [

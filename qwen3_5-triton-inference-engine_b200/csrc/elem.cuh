@@ -37,10 +37,51 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&f)[8]) {
   *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
 }
 
+// 8 raw elements as they come
+template <typename E>
+struct Raw8 {
+  uint4 v[sizeof(E) / 2];
+  __device__ __forceinline__ void load(const E* p) {
+#pragma unroll
+    for (int i = 0; i < static_cast<int>(sizeof(E) / 2); ++i) v[i] = reinterpret_cast<const uint4*>(p)[i];
+  }
+  __device__ __forceinline__ void get(float (&f)[8]) const { load8(reinterpret_cast<const E*>(&v[0]), f); }
+};
+
 __device__ __forceinline__ float rcp_fast(float x) {  // 1 / x, one hardware instruction (about an ulp; 1 / inf = 0)
   float y;
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// packed fp32 pairs
+struct F2 {
+  uint64_t v;
+};
+__device__ __forceinline__ F2 f2(float lo, float hi) {
+  F2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 unf2(F2 a) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a.v));
+  return r;
+}
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+  F2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+  return r;
+}
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+  F2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
+  return r;
+}
+__device__ __forceinline__ F2 add2(F2 a, F2 b) {
+  F2 r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
+  return r;
 }
 
 // Logistic function in fp32: exact library exponential and division for fp32 activations, the hardware exponential and

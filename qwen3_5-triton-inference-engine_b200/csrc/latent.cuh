@@ -69,6 +69,9 @@ struct RowPrefillOperands {
   float scale, out_scale;
 };
 int row_prefill_launch(const RowPrefillOperands& a, const char* name, cudaStream_t st);
+// ... and its form for pairs of heads that share keys and values (window_pair_umma.cu)
+bool row_prefill_pairs(const RowPrefillOperands& a);
+int row_prefill_pair_launch(const RowPrefillOperands& a, const char* name, cudaStream_t st);
 
 struct LatentAbsorbParams {
   const void *q, *w;     // [batch, heads, dim + rot], [heads, dim, rank]

@@ -260,35 +260,39 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     }
     named_barrier(9, LP_SOFTMAX_THREADS);
     if (ok) {
-      const int vecs = p.vdim / 8;
-      for (int i = tid; i < LP_TILE * vecs; i += LP_SOFTMAX_THREADS) {
-        const int r = i / vecs, c = i % vecs;
-        if (q0 + r >= len) continue;
-        const int64_t row_at = q_row0 + q0 + r;
-        uint4 o = *reinterpret_cast<const uint4*>(smem + r * out_pitch + c * 16);
+      const int vecs = p.vdim / 8, col = h * p.vdim;
+      constexpr int U = 8;                             // rows' parts per thread whose gates are requested together
+      for (int i0 = tid; i0 < LP_TILE * vecs; i0 += U * LP_SOFTMAX_THREADS) {
+        uint4 z[U];
         if (p.gate) {
-          float f[8], z[8];
-          load8(reinterpret_cast<const __nv_bfloat16*>(&o), f);
-          load8(p.gate + row_at * p.gate_stride + h * p.vdim + c * 8, z);
 #pragma unroll
-          for (int k = 0; k < 8; ++k) f[k] *= sigmoid_f<__nv_bfloat16>(z[k]) * p.out_scale;
-          store8(reinterpret_cast<__nv_bfloat16*>(&o), f);
+          for (int u = 0; u < U; ++u) {
+            const int i = i0 + u * LP_SOFTMAX_THREADS, r = i / vecs;
+            if (r < LP_TILE && q0 + r < len)
+              z[u] = *reinterpret_cast<const uint4*>(p.gate + static_cast<int64_t>(q_row0 + q0 + r) * p.gate_stride + col + (i - r * vecs) * 8);
+          }
         }
-        *reinterpret_cast<uint4*>(p.out + row_at * p.out_stride + h * p.vdim + c * 8) = o;
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int i = i0 + u * LP_SOFTMAX_THREADS, r = i / vecs, c = i - r * vecs;
+          if (r >= LP_TILE || q0 + r >= len) continue;
+          uint4 o = *reinterpret_cast<const uint4*>(smem + r * out_pitch + c * 16);
+          if (p.gate) {
+            float f[8], g8[8];
+            load8(reinterpret_cast<const __nv_bfloat16*>(&o), f);
+            load8(reinterpret_cast<const __nv_bfloat16*>(&z[u]), g8);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) f[k] *= sigmoid_f<__nv_bfloat16>(g8[k]) * p.out_scale;
+            store8(reinterpret_cast<__nv_bfloat16*>(&o), f);
+          }
+          *reinterpret_cast<uint4*>(p.out + static_cast<int64_t>(q_row0 + q0 + r) * p.out_stride + col + c * 8) = o;
+        }
       }
     }
   }
   tc_fence_before_sync();
   __syncthreads();
   if (warp == 0) tmem_dealloc(tmem, LP_TMEM_COLS);
-}
-
-// A strided matrix of `heads` parts, `blocks` column blocks of 64 each, as the 4-D tensor {64, rows, blocks, heads}
-static bool head_map(CUtensorMap* map, const void* base, uint64_t rows, int64_t row_stride, int blocks, int64_t head_stride, int heads) {
-  const uint64_t dims[4] = {64, rows, static_cast<uint64_t>(blocks), static_cast<uint64_t>(heads)};
-  const uint64_t st[3] = {static_cast<uint64_t>(row_stride) * 2, 128, static_cast<uint64_t>(head_stride) * 2};
-  const uint32_t box[4] = {64, LP_TILE, static_cast<uint32_t>(blocks), 1};
-  return encode_map_bf16_sw128(map, base, 4, dims, st, box);
 }
 
 int row_prefill_launch(const RowPrefillOperands& a, const char* name, cudaStream_t st) {
@@ -306,10 +310,11 @@ int row_prefill_launch(const RowPrefillOperands& a, const char* name, cudaStream
   const int head_width = a.dim + a.rot;
   B200_REQUIRE(a.q_stride >= static_cast<int64_t>(a.heads - 1) * head_width + (dim_blocks + rot_blocks) * 64,
                "%s: rows of q end inside the last head's column blocks", name);
+  if (row_prefill_pairs(a)) return row_prefill_pair_launch(a, name, st);
   CUtensorMap map_q, map_k, map_r = {}, map_v;
-  if (!head_map(&map_q, a.q, a.tokens, a.q_stride, dim_blocks + rot_blocks, head_width, a.heads) ||
-      !head_map(&map_k, a.k, a.keys, a.k_stride, dim_blocks, a.k_head, kv_heads) ||
-      !head_map(&map_v, a.v, a.keys, a.v_stride, a.vdim / 64, a.v_head, kv_heads))
+  if (!encode_head_map(&map_q, a.q, a.tokens, a.q_stride, dim_blocks + rot_blocks, head_width, a.heads, LP_TILE) ||
+      !encode_head_map(&map_k, a.k, a.keys, a.k_stride, dim_blocks, a.k_head, kv_heads, LP_TILE) ||
+      !encode_head_map(&map_v, a.v, a.keys, a.v_stride, a.vdim / 64, a.v_head, kv_heads, LP_TILE))
     return fail(ERR_RUNTIME, "%s: cannot encode a tensor map", name);
   if (rot_blocks > 0) {
     const uint64_t dims[3] = {64, static_cast<uint64_t>(a.keys), static_cast<uint64_t>(rot_blocks)};

@@ -168,31 +168,6 @@ __global__ void __launch_bounds__(128) mingru_decode_kernel(const E* zxg, int64_
 }
 
 // ------------------------------------------------------------------------------------------ outer-product recurrences
-// packed fp32 pairs
-struct F2 {
-  uint64_t v;
-};
-__device__ __forceinline__ F2 f2(float lo, float hi) {
-  F2 r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r.v) : "f"(lo), "f"(hi));
-  return r;
-}
-__device__ __forceinline__ float2 unf2(F2 a) {
-  float2 r;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(a.v));
-  return r;
-}
-__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
-  F2 r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r.v) : "l"(a.v), "l"(b.v));
-  return r;
-}
-__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
-  F2 r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r.v) : "l"(a.v), "l"(b.v), "l"(c.v));
-  return r;
-}
-
 constexpr int OR_TB = 16;        // tokens staged at a time
 constexpr int OR_WARPS = 4;
 constexpr int OR_THREADS = OR_WARPS * 32;

@@ -574,12 +574,12 @@ skinny_gemm_pairk_kernel(const __grid_constant__ WideKParams p, const __grid_con
 }
 
 // Shared by all host threads: searched and filled under a mutex, the map is copied out.
-static bool cache_weight_map(const void* base, int64_t n, int64_t k, int box_rows, CUtensorMap* out) {
+static bool cache_weight_map(const void* base, int64_t n, int64_t k, int64_t stride, int box_rows, CUtensorMap* out) {
   static std::mutex mu;
   std::lock_guard<std::mutex> lock(mu);
   struct Entry {
     const void* base;
-    int64_t n, k;
+    int64_t n, k, stride;
     int dev, box_rows;
     CUtensorMap map;
   };
@@ -589,18 +589,19 @@ static bool cache_weight_map(const void* base, int64_t n, int64_t k, int box_row
   int dev = 0;
   cudaGetDevice(&dev);
   for (int i = 0; i < used; ++i)
-    if (entries[i].base == base && entries[i].n == n && entries[i].k == k && entries[i].dev == dev &&
+    if (entries[i].base == base && entries[i].n == n && entries[i].k == k && entries[i].stride == stride && entries[i].dev == dev &&
         entries[i].box_rows == box_rows) {
       *out = entries[i].map;
       return true;
     }
   Entry& e = entries[next];
   e.base = nullptr;  // not a valid entry while it is being rewritten
-  if (!encode_tile_map(&e.map, base, static_cast<uint64_t>(n), static_cast<uint64_t>(k), static_cast<uint64_t>(k) * 2, box_rows, 2))
+  if (!encode_tile_map(&e.map, base, static_cast<uint64_t>(n), static_cast<uint64_t>(k), static_cast<uint64_t>(stride) * 2, box_rows, 2))
     return false;
   e.base = base;
   e.n = n;
   e.k = k;
+  e.stride = stride;
   e.dev = dev;
   e.box_rows = box_rows;
   next = (next + 1) % N;
@@ -614,9 +615,9 @@ static bool cache_weight_map(const void* base, int64_t n, int64_t k, int box_row
 using namespace b200;
 
 template <bool SWIGLU, bool ARGMAX = false>
-static int launch_skinny(SkinnyGemmParams p, const void* weight, int w_rows, cudaStream_t stream, const char* what) {
+static int launch_skinny(SkinnyGemmParams p, const void* weight, int64_t w_stride, int w_rows, cudaStream_t stream, const char* what) {
   CUtensorMap map;
-  if (!cache_weight_map(weight, w_rows, p.k, SWIGLU ? 8 : 16, &map)) return fail(ERR_RUNTIME, "%s: cannot encode the weight tensor map", what);
+  if (!cache_weight_map(weight, w_rows, p.k, w_stride, SWIGLU ? 8 : 16, &map)) return fail(ERR_RUNTIME, "%s: cannot encode the weight tensor map", what);
   constexpr int smem_max =
       SG_WARPS * SG_RING_BYTES + SG_MAX_M * SG_ROWS * 2 + SG_PART_BYTES + SG_MAX_M * (SG_MAX_K * 2 + 16) + 1024;
   static_assert(smem_max <= 227 * 1024, "weight rings + X staging must fit the 227 KiB a CTA may use");
@@ -653,10 +654,10 @@ static bool widek_chunks(int k, int* chunk_k, int* n_chunks) {
   return true;
 }
 
-static int launch_widek(WideKParams p, const void* weight, cudaStream_t stream) {
+static int launch_widek(WideKParams p, const void* weight, int64_t w_stride, cudaStream_t stream) {
   const char* what = "skinny_gemm";
   CUtensorMap map;
-  if (!cache_weight_map(weight, p.n, p.k, 16, &map)) return fail(ERR_RUNTIME, "%s: cannot encode the weight tensor map", what);
+  if (!cache_weight_map(weight, p.n, p.k, w_stride, 16, &map)) return fail(ERR_RUNTIME, "%s: cannot encode the weight tensor map", what);
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -679,10 +680,10 @@ static int launch_widek(WideKParams p, const void* weight, cudaStream_t stream) 
   return check_launch(what);
 }
 
-static int launch_pairk(WideKParams p, const void* weight, cudaStream_t stream) {
+static int launch_pairk(WideKParams p, const void* weight, int64_t w_stride, cudaStream_t stream) {
   const char* what = "skinny_gemm";
   CUtensorMap map;
-  if (!cache_weight_map(weight, p.n, p.k, 16, &map)) return fail(ERR_RUNTIME, "%s: cannot encode the weight tensor map", what);
+  if (!cache_weight_map(weight, p.n, p.k, w_stride, 16, &map)) return fail(ERR_RUNTIME, "%s: cannot encode the weight tensor map", what);
   static bool configured[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -713,8 +714,9 @@ static int check_skinny_shape(const char* what, int m, int n, int k) {
   return OK;
 }
 
-extern "C" int b200_skinny_gemm(const void* x, int64_t x_stride, const void* weight, void* y, int64_t y_stride,
-                                int32_t m, int32_t n, int32_t k, int32_t overlap, b200_stream_t stream) {
+extern "C" int b200_skinny_gemm_part(const void* x, int64_t x_stride, const void* weight, int64_t w_stride, void* y,
+                                     int64_t y_stride, int32_t m, int32_t n, int32_t k, int32_t overlap, b200_stream_t stream) {
+  B200_REQUIRE(w_stride >= k && w_stride % 8 == 0, "skinny_gemm: weight rows must be whole 16-byte groups apart");
   B200_REQUIRE(aligned16(x) && aligned16(weight) && aligned16(y) && x_stride % 8 == 0 && y_stride % 8 == 0,
                "skinny_gemm: pointers must be 16-byte aligned, row strides multiples of 8 elements");
   if (k > SG_MAX_K) {  // long rows: K split over the warps of a CTA, X staged in chunks
@@ -730,8 +732,8 @@ extern "C" int b200_skinny_gemm(const void* x, int64_t x_stride, const void* wei
     wp.n = n;
     wp.k = k;
     wp.overlap = overlap;
-    if (k <= PK_MAX_K && k % (2 * SG_TILE_K) == 0) return launch_pairk(wp, weight, reinterpret_cast<cudaStream_t>(stream));
-    return launch_widek(wp, weight, reinterpret_cast<cudaStream_t>(stream));
+    if (k <= PK_MAX_K && k % (2 * SG_TILE_K) == 0) return launch_pairk(wp, weight, w_stride, reinterpret_cast<cudaStream_t>(stream));
+    return launch_widek(wp, weight, w_stride, reinterpret_cast<cudaStream_t>(stream));
   }
   int rc = check_skinny_shape("skinny_gemm", m, n, k);
   if (rc != OK) return rc;
@@ -744,7 +746,12 @@ extern "C" int b200_skinny_gemm(const void* x, int64_t x_stride, const void* wei
   p.n = n;
   p.k = k;
   p.overlap = overlap;
-  return launch_skinny<false>(p, weight, n, reinterpret_cast<cudaStream_t>(stream), "skinny_gemm");
+  return launch_skinny<false>(p, weight, w_stride, n, reinterpret_cast<cudaStream_t>(stream), "skinny_gemm");
+}
+
+extern "C" int b200_skinny_gemm(const void* x, int64_t x_stride, const void* weight, void* y, int64_t y_stride, int32_t m,
+                                int32_t n, int32_t k, int32_t overlap, b200_stream_t stream) {
+  return b200_skinny_gemm_part(x, x_stride, weight, k, y, y_stride, m, n, k, overlap, stream);
 }
 
 extern "C" int b200_skinny_gemm_swiglu(const void* x, int64_t x_stride, const void* weight, void* y, int64_t y_stride,
@@ -764,7 +771,7 @@ extern "C" int b200_skinny_gemm_swiglu(const void* x, int64_t x_stride, const vo
   p.k = k;
   p.overlap = overlap;
   p.up_row0 = intermediate;
-  return launch_skinny<true>(p, weight, 2 * intermediate, reinterpret_cast<cudaStream_t>(stream), "skinny_gemm_swiglu");
+  return launch_skinny<true>(p, weight, k, 2 * intermediate, reinterpret_cast<cudaStream_t>(stream), "skinny_gemm_swiglu");
 }
 
 extern "C" int b200_lm_head_argmax(const void* x, int64_t x_stride, const void* weight, int64_t* ids, void* workspace,
@@ -785,5 +792,5 @@ extern "C" int b200_lm_head_argmax(const void* x, int64_t x_stride, const void* 
   p.ids = ids;
   p.keys = static_cast<unsigned long long*>(workspace);  // the layout of b200_argmax_rows: 1024 keys, then counters
   p.counter = reinterpret_cast<int*>(p.keys + 1024);
-  return launch_skinny<false, true>(p, weight, n, reinterpret_cast<cudaStream_t>(stream), "lm_head_argmax");
+  return launch_skinny<false, true>(p, weight, k, n, reinterpret_cast<cudaStream_t>(stream), "lm_head_argmax");
 }

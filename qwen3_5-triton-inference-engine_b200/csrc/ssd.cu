@@ -23,7 +23,6 @@
 namespace b200 {
 
 // ------------------------------------------------------------------------------------------------------ convolution
-constexpr int CV_RUN = 16;        // tokens per thread
 constexpr int CV_THREADS = 64;    // 8 channels each
 
 struct ConvParams {
@@ -37,14 +36,22 @@ struct ConvParams {
   int channels;
 };
 
-template <typename E, int T>
+// A thread takes RUN tokens of 8 channels, BATCH of them requested at a time.
+template <typename E, int T, int RUN, int BATCH>
 __global__ void __launch_bounds__(CV_THREADS) conv_prefill_kernel(const __grid_constant__ ConvParams p) {
-  const int seq = blockIdx.z, t0 = blockIdx.y * CV_RUN, c = (blockIdx.x * CV_THREADS + threadIdx.x) * 8;
+  const int seq = blockIdx.z, t0 = blockIdx.y * RUN, c = (blockIdx.x * CV_THREADS + threadIdx.x) * 8;
+  pdl_trigger();                  // the launch behind (conv_state_kernel) waits for this one
   const int row0 = p.cu[seq], len = p.cu[seq + 1] - row0;
   if (t0 >= len || c >= p.channels) return;
   const int start = p.start[seq];
   const E* x = static_cast<const E*>(p.x) + static_cast<int64_t>(row0) * p.stride + c;
   const float* ring = p.ring + static_cast<int64_t>(p.slots[seq]) * T * p.channels + c;
+  Raw8<E> raw[BATCH];
+  auto request = [&](int i0) {
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) raw[i].load(x + static_cast<int64_t>(min(t0 + i0 + i, len - 1)) * p.stride);
+  };
+  request(0);
   float w[T][8], b[8], h[T][8];   // h[j]: the input j tokens back
 #pragma unroll
   for (int j = 0; j < T; ++j) load8(p.w + static_cast<int64_t>(j) * p.channels + c, w[j]);
@@ -59,24 +66,28 @@ __global__ void __launch_bounds__(CV_THREADS) conv_prefill_kernel(const __grid_c
       for (int k = 0; k < 8; ++k) h[j - 1][k] = 0.f;
   }
   E* out = static_cast<E*>(p.out) + static_cast<int64_t>(row0) * p.out_stride + c;
-#pragma unroll(T <= 4 ? CV_RUN : 1)
-  for (int i = 0; i < CV_RUN; ++i) {
-    const int t = t0 + i;
-    if (t >= len) break;
+#pragma unroll 1
+  for (int i0 = 0; i0 < RUN; i0 += BATCH) {
+    if (i0 > 0) request(i0);
 #pragma unroll
-    for (int j = T - 1; j > 0; --j)
+    for (int i = 0; i < BATCH; ++i) {
+      const int t = t0 + i0 + i;
+      if (t >= len) break;
 #pragma unroll
-      for (int k = 0; k < 8; ++k) h[j][k] = h[j - 1][k];
-    load8(x + t * p.stride, h[0]);
-    float y[8];
+      for (int j = T - 1; j > 0; --j)
 #pragma unroll
-    for (int k = 0; k < 8; ++k) {
-      float acc = b[k];
+        for (int k = 0; k < 8; ++k) h[j][k] = h[j - 1][k];
+      raw[i].get(h[0]);
+      float y[8];
 #pragma unroll
-      for (int j = 0; j < T; ++j) acc = fmaf(w[j][k], h[j][k], acc);
-      y[k] = silu_f<E>(acc);
+      for (int k = 0; k < 8; ++k) {
+        float acc = b[k];
+#pragma unroll
+        for (int j = 0; j < T; ++j) acc = fmaf(w[j][k], h[j][k], acc);
+        y[k] = silu_f<E>(acc);
+      }
+      store8(out + t * p.out_stride, y);
     }
-    store8(out + t * p.out_stride, y);
   }
 }
 
@@ -84,6 +95,7 @@ __global__ void __launch_bounds__(CV_THREADS) conv_prefill_kernel(const __grid_c
 template <typename E, int T>
 __global__ void __launch_bounds__(CV_THREADS) conv_state_kernel(const __grid_constant__ ConvParams p) {
   const int seq = blockIdx.z, c = (blockIdx.x * CV_THREADS + threadIdx.x) * 8;
+  pdl_wait();
   const int row0 = p.cu[seq], len = p.cu[seq + 1] - row0, t = len - 1 - static_cast<int>(blockIdx.y);
   if (t < 0 || c >= p.channels) return;
   float f[8];
@@ -91,12 +103,24 @@ __global__ void __launch_bounds__(CV_THREADS) conv_state_kernel(const __grid_con
   store8(p.ring + (static_cast<int64_t>(p.slots[seq]) * T + (p.start[seq] + t) % T) * p.channels + c, f);
 }
 
+template <typename E, int T, int RUN, int BATCH>
+static int launch_conv_run(const ConvParams& p, int batch, int max_len, cudaStream_t st) {
+  const unsigned cols = (p.channels / 8 + CV_THREADS - 1) / CV_THREADS;
+  B200_REQUIRE(max_len <= 65535 * RUN, "conv_prefill: sequences of at most %d tokens", 65535 * RUN);
+  conv_prefill_kernel<E, T, RUN, BATCH><<<dim3(cols, (max_len + RUN - 1) / RUN, batch), CV_THREADS, 0, st>>>(p);
+  if (launch_pdl(true, conv_state_kernel<E, T>, dim3(cols, T, batch), dim3(CV_THREADS), 0, st, p) != cudaSuccess)
+    return fail(ERR_LAUNCH, "conv_prefill: %s", cudaGetErrorString(cudaGetLastError()));
+  return check_launch("conv_prefill");
+}
+
 template <typename E, int T>
 static int launch_conv(const ConvParams& p, int batch, int max_len, cudaStream_t st) {
-  const unsigned cols = (p.channels / 8 + CV_THREADS - 1) / CV_THREADS;
-  conv_prefill_kernel<E, T><<<dim3(cols, (max_len + CV_RUN - 1) / CV_RUN, batch), CV_THREADS, 0, st>>>(p);
-  conv_state_kernel<E, T><<<dim3(cols, T, batch), CV_THREADS, 0, st>>>(p);
-  return check_launch("conv_prefill");
+  if constexpr (T == 4) {         // short runs when long ones leave SMs without enough requests in flight
+    const int64_t warps = static_cast<int64_t>(p.channels / 256 + 1) * (max_len / 16 + 1) * batch;
+    return warps < 16 * sm_count() ? launch_conv_run<E, T, 4, 4>(p, batch, max_len, st) : launch_conv_run<E, T, 16, 8>(p, batch, max_len, st);
+  } else {
+    return launch_conv_run<E, T, 16, 1>(p, batch, max_len, st);
+  }
 }
 
 // ------------------------------------------------------------------------------------------------------ gated norm
@@ -484,7 +508,7 @@ extern "C" int b200_conv_prefill(const void* x, int64_t stride, const float* wei
                                  int64_t out_stride, int32_t batch, int32_t max_len, int32_t channels, int32_t taps, int32_t f32,
                                  b200_stream_t stream) {
   if (batch <= 0 || max_len <= 0) return OK;
-  B200_REQUIRE(channels > 0 && channels % 8 == 0 && stride % 8 == 0 && out_stride % 8 == 0 && batch <= 65535 && max_len <= 65535 * CV_RUN,
+  B200_REQUIRE(channels > 0 && channels % 8 == 0 && stride % 8 == 0 && out_stride % 8 == 0 && batch <= 65535,
                "conv_prefill: channels and strides must be multiples of 8");
   B200_REQUIRE(taps == 4 || taps == 8 || taps == 16, "conv_prefill: 4, 8 or 16 taps (pad with zero weights), got %d", taps);
   B200_REQUIRE(aligned16(x) && aligned16(weight) && aligned16(bias) && aligned16(ring) && aligned16(out), "conv_prefill: unaligned tensor");

@@ -21,7 +21,9 @@ struct HyperParams {
   int ids_are_int64;
   const void* table;      // [vocab, width] E
   float* streams;         // [rows, S, width]
-  const void* y;          // [rows, width] E or NULL
+  const void* y;          // [parts][rows, width] E, summed, or NULL
+  int parts;
+  int64_t part_stride;
   const float* weights;   // [mix S*S | out S | in S | gain]
   const float* gains;     // [width] or NULL
   void* h;                // [rows, width] E
@@ -66,7 +68,11 @@ __global__ void __launch_bounds__(512) hyper_connect_kernel(const __grid_constan
       for (int i = 0; i < MAXS; ++i)
         if (i < s) old[i] = load4(x + i * width + c);
       if (p.y) {
-        const float4 y = load4(static_cast<const E*>(p.y) + static_cast<int64_t>(row) * width + c);
+        float4 y = load4(static_cast<const E*>(p.y) + static_cast<int64_t>(row) * width + c);
+        for (int i = 1; i < p.parts; ++i) {
+          const float4 more = load4(static_cast<const E*>(p.y) + i * p.part_stride + static_cast<int64_t>(row) * width + c);
+          y.x += more.x, y.y += more.y, y.z += more.z, y.w += more.w;
+        }
 #pragma unroll
         for (int t = 0; t < MAXS; ++t)
           if (t < s) {
@@ -186,7 +192,7 @@ __global__ void __launch_bounds__(256) swiglu_f32_kernel(const float* gate_up, i
 using namespace b200;
 
 extern "C" int b200_hyper_connect(const void* ids, int32_t ids_are_int64, const void* table, float* streams, const void* y,
-                                  const float* weights, const float* gains, void* h, int32_t rows, int32_t num_streams, int32_t width,
+                                  int32_t y_parts, const float* weights, const float* gains, void* h, int32_t rows, int32_t num_streams, int32_t width,
                                   int32_t true_width, float eps, int32_t f32, int32_t overlap, b200_stream_t stream) {
   if (rows <= 0) return OK;
   B200_REQUIRE(num_streams >= 1 && num_streams <= HC_MAX_STREAMS, "hyper_connect: 1 to %d streams (got %d)",
@@ -196,8 +202,9 @@ extern "C" int b200_hyper_connect(const void* ids, int32_t ids_are_int64, const 
                HC_MAX_WIDTH, width, true_width);
   B200_REQUIRE(streams && weights && h && aligned16(streams) && aligned16(h) && aligned16(y) && aligned16(gains),
                "hyper_connect: NULL or unaligned tensor");
+  B200_REQUIRE(!y || y_parts >= 1, "hyper_connect: y comes in at least one part");
   B200_REQUIRE(!ids || (table && aligned16(table) && !y), "hyper_connect: the embedding form takes a table, no y");
-  HyperParams p = {ids, ids_are_int64, table, streams, y, weights, gains, h, num_streams, width, true_width, overlap, eps};
+  HyperParams p = {ids, ids_are_int64, table, streams, y, y_parts, static_cast<int64_t>(rows) * width, weights, gains, h, num_streams, width, true_width, overlap, eps};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const cudaError_t e = f32 ? launch_hyper_e<float>(p, rows, st) : launch_hyper_e<__nv_bfloat16>(p, rows, st);
   if (e != cudaSuccess) return fail(ERR_LAUNCH, "hyper_connect: %s", cudaGetErrorString(e));

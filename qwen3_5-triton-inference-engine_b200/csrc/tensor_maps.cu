@@ -45,4 +45,12 @@ bool encode_tile_map(CUtensorMap* map, const void* base, uint64_t rows, uint64_t
   return encode_map_bf16_sw128(map, base, 3, dims, strides, box);
 }
 
+bool encode_head_map(CUtensorMap* map, const void* base, int64_t rows, int64_t row_stride, int blocks, int64_t head_stride, int heads,
+                     int box_rows) {
+  const uint64_t dims[4] = {64, static_cast<uint64_t>(rows), static_cast<uint64_t>(blocks), static_cast<uint64_t>(heads)};
+  const uint64_t strides[3] = {static_cast<uint64_t>(row_stride) * 2, 128, static_cast<uint64_t>(head_stride) * 2};
+  const uint32_t box[4] = {64, static_cast<uint32_t>(box_rows), static_cast<uint32_t>(blocks), 1};
+  return encode_map_bf16_sw128(map, base, 4, dims, strides, box);
+}
+
 }  // namespace b200

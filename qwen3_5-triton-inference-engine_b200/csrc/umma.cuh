@@ -160,6 +160,11 @@ __device__ __forceinline__ void tma_load_5d(void* dst_smem, const CUtensorMap* m
 bool encode_map_bf16_sw128(CUtensorMap* map, const void* base, int rank, const uint64_t* dims,
                            const uint64_t* strides_bytes, const uint32_t* box);
 
+// Rows x `heads` parts of 64 * blocks columns (parts may overlap), as the 4-D tensor {64, rows, blocks, heads}; one load brings
+// box_rows rows of a part.
+bool encode_head_map(CUtensorMap* map, const void* base, int64_t rows, int64_t row_stride, int blocks, int64_t head_stride, int heads,
+                     int box_rows);
+
 // Byte offset of element (row, col) inside a swizzled tile of `rows` rows (see the file comment).
 __device__ __forceinline__ uint32_t sw128_offset(int row, int col, int rows) {
   const int block = col >> 6, chunk = (col & 63) >> 3;

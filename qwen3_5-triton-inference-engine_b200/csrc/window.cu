@@ -4,6 +4,8 @@
 //   b200_window_prefill   packed portions: tcgen05 (latent_prefill_umma.cu), or CUDA cores for fp32 and wide heads (here)
 //   b200_window_decode    one token per slot over the pages (latent_decode.cu, row_attention.cu)
 //   b200_window_merge     merge of the key ranges, gate (row_attention.cu)
+#include <type_traits>
+
 #include "latent.cuh"
 
 namespace b200 {
@@ -30,75 +32,100 @@ __device__ __forceinline__ void load_w(const E* p, float (&f)[W]) {
   if constexpr (W == 8) load8(p, f);
   else f[0] = load1(p);
 }
+template <typename E>
+struct Raw1 {
+  E v;
+  __device__ __forceinline__ void load(const E* p) { v = *p; }
+  __device__ __forceinline__ void get(float (&f)[1]) const { f[0] = load1(&v); }
+};
+template <typename E, int W>
+using RawW = std::conditional_t<W == 8, Raw8<E>, Raw1<E>>;
 template <typename E, int W>
 __device__ __forceinline__ void store_w(E* p, const float (&f)[W]) {
   if constexpr (W == 8) store8(p, f);
   else store1(p, f[0]);
 }
 
-// One CTA per row.  An item is W consecutive elements that stay as they are, or W rotated pairs; W = 8 when the halves and
-// what lies behind them start on groups of 8.
-template <typename E, int W>
-__global__ void __launch_bounds__(256) window_prep_kernel(const __grid_constant__ WindowPrepParams p) {
-  const int row = blockIdx.x;
+// One CTA per ROWS rows.  An item is W consecutive elements that stay as they are, or W rotated pairs; W = 8 when the halves
+// and what lies behind them start on groups of 8.  An item's biases are loaded once for all rows, and its elements of all rows
+// before the first is used.
+template <typename E, int W, int ROWS>
+__global__ void __launch_bounds__(256) window_prep_kernel(const __grid_constant__ WindowPrepParams p, int rows) {
+  __shared__ int64_t row_pos[ROWS], row_at[ROWS], row_ctx[ROWS];   // position; row of key/value head 0 in the cache (-1: none) and in ctx
+  const int row0 = blockIdx.x * ROWS, count = min(ROWS, rows - row0);
   if (p.overlap & OVERLAP_TRIGGER) pdl_trigger();
   pdl_wait();
-  E* x = static_cast<E*>(p.x) + row * p.stride;
-  const int slot = p.slot ? p.slot[row] : row;
-  const int64_t pos = p.pos_is_int64 ? static_cast<const int64_t*>(p.pos)[row] : static_cast<int64_t>(static_cast<const int32_t*>(p.pos)[row]);
-  const bool write = !(p.active && p.active[slot] == 0);
-  int64_t at = 0;           // row of key/value head 0 in the cache
-  if (write) at = static_cast<int64_t>(p.table[slot * p.table_stride + pos / PAGE]) * p.kv_heads * PAGE + pos % PAGE;
+  E* const x0 = static_cast<E*>(p.x) + row0 * p.stride;
   E* const cache = static_cast<E*>(p.cache);
-  E* const ctx = p.ctx ? static_cast<E*>(p.ctx) + static_cast<int64_t>(p.ctx_row[row]) * p.kv_heads * p.pitch : nullptr;
+  E* const ctx = static_cast<E*>(p.ctx);
   const int n = p.pairs, ri = n / W, qi = ri + (p.dim - 2 * n) / W, vi = p.vdim / W;
-  const int q_items = p.heads * qi, k_items = p.kv_heads * qi, total = q_items + k_items + p.kv_heads * vi;
-  for (int i = threadIdx.x; i < total; i += blockDim.x) {
-    if (i < q_items + k_items) {
+  const int qk_items = (p.heads + p.kv_heads) * qi, total = qk_items + p.kv_heads * vi;
+  bool first = true;
+  for (int i = threadIdx.x; i < total || first; i += blockDim.x) {
+    // source column, column in a cache row, key/value head (negative: a query), rotated or not
+    int src = 0, dst = 0, g = 0;
+    bool rotated = false;
+    if (i < qk_items) {
       const int h = i / qi, j = i - h * qi;
-      const bool is_k = h >= p.heads, rotated = j < ri;
-      const int off = rotated ? j * W : 2 * n + (j - ri) * W;
-      E* src = x + h * p.dim + off;
-      float u[W], v[W], b[W];
-      load_w<E, W>(src, u);
-      load_w<float, W>(p.bias + h * p.dim + off, b);
+      rotated = j < ri;
+      dst = rotated ? j * W : 2 * n + (j - ri) * W;
+      src = h * p.dim + dst;
+      g = h - p.heads;
+    } else if (i < total) {
+      const int e = i - qk_items;
+      g = e / vi;
+      const int c = (e - g * vi) * W;
+      src = (p.heads + p.kv_heads) * p.dim + g * p.vdim + c;
+      dst = p.dim + c;
+    }
+    float bu[W], bv[W];
+    RawW<E, W> ru[ROWS], rv[ROWS];
 #pragma unroll
-      for (int k = 0; k < W; ++k) u[k] += b[k];
-      if (rotated) {
-        load_w<E, W>(src + n, v);
-        load_w<float, W>(p.bias + h * p.dim + off + n, b);
-        const float2* a = p.angles + pos * n + off;
+    for (int r = 0; r < ROWS; ++r) {
+      const E* from = x0 + min(r, count - 1) * p.stride + src;
+      ru[r].load(from);
+      if (rotated) rv[r].load(from + n);
+    }
+    load_w<float, W>(p.bias + src, bu);
+    if (rotated) load_w<float, W>(p.bias + src + n, bv);
+    if (first) {                 // where the rows go, looked up while their elements are on the way
+      first = false;
+      if (threadIdx.x < count) {
+        const int row = row0 + threadIdx.x, slot = p.slot ? p.slot[row] : row;
+        const int64_t pos = p.pos_is_int64 ? static_cast<const int64_t*>(p.pos)[row] : static_cast<int64_t>(static_cast<const int32_t*>(p.pos)[row]);
+        row_pos[threadIdx.x] = pos;
+        row_at[threadIdx.x] = p.active && p.active[slot] == 0
+                                  ? -1 : static_cast<int64_t>(p.table[slot * p.table_stride + pos / PAGE]) * p.kv_heads * PAGE + pos % PAGE;
+        row_ctx[threadIdx.x] = p.ctx ? static_cast<int64_t>(p.ctx_row[row]) * p.kv_heads : 0;
+      }
+      __syncthreads();
+      if (i >= total) break;
+    }
 #pragma unroll
-        for (int k = 0; k < W; ++k) {
-          v[k] += b[k];
+    for (int r = 0; r < ROWS; ++r) {
+      if (r >= count) break;
+      const float2* a = p.angles + row_pos[r] * n + dst;
+      float u[W], v[W];
+      ru[r].get(u);
+      if (rotated) rv[r].get(v);
+#pragma unroll
+      for (int k = 0; k < W; ++k) {
+        u[k] += bu[k];
+        if (rotated) {
+          v[k] += bv[k];
           rotate_pair(u[k], v[k], a[k]);
         }
       }
-      if (!is_k) {
-        store_w<E, W>(src, u);
-        if (rotated) store_w<E, W>(src + n, v);
+      auto put = [&](E* to) {
+        store_w<E, W>(to, u);
+        if (rotated) store_w<E, W>(to + n, v);
+      };
+      if (g < 0) {
+        put(x0 + r * p.stride + src);
       } else {
-        const int g = h - p.heads;
-        if (write) {
-          E* dst = cache + (at + g * PAGE) * p.pitch + off;
-          store_w<E, W>(dst, u);
-          if (rotated) store_w<E, W>(dst + n, v);
-        }
-        if (ctx) {
-          E* dst = ctx + g * p.pitch + off;
-          store_w<E, W>(dst, u);
-          if (rotated) store_w<E, W>(dst + n, v);
-        }
+        if (row_at[r] >= 0) put(cache + (row_at[r] + g * PAGE) * p.pitch + dst);
+        if (ctx) put(ctx + (row_ctx[r] + g) * p.pitch + dst);
       }
-    } else {
-      const int e = i - q_items - k_items, g = e / vi, c = (e - g * vi) * W, src = (p.heads + p.kv_heads) * p.dim + g * p.vdim + c;
-      float u[W], b[W];
-      load_w<E, W>(x + src, u);
-      load_w<float, W>(p.bias + src, b);
-#pragma unroll
-      for (int k = 0; k < W; ++k) u[k] += b[k];
-      if (write) store_w<E, W>(cache + (at + g * PAGE) * p.pitch + p.dim + c, u);
-      if (ctx) store_w<E, W>(ctx + g * p.pitch + p.dim + c, u);
     }
   }
 }
@@ -166,10 +193,11 @@ extern "C" int b200_window_prep(void* x, int64_t stride, const float* bias, cons
   const bool early = (overlap & OVERLAP_START) != 0;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   cudaError_t e;
-  if (f32) e = w == 8 ? launch_pdl(early, window_prep_kernel<float, 8>, dim3(rows), block, 0, st, p)
-                      : launch_pdl(early, window_prep_kernel<float, 1>, dim3(rows), block, 0, st, p);
-  else e = w == 8 ? launch_pdl(early, window_prep_kernel<__nv_bfloat16, 8>, dim3(rows), block, 0, st, p)
-                  : launch_pdl(early, window_prep_kernel<__nv_bfloat16, 1>, dim3(rows), block, 0, st, p);
+  if (f32) e = w == 8 ? launch_pdl(early, window_prep_kernel<float, 8, 1>, dim3(rows), block, 0, st, p, rows)
+                      : launch_pdl(early, window_prep_kernel<float, 1, 1>, dim3(rows), block, 0, st, p, rows);
+  else if (w == 8 && rows >= GLUE_WIDE_ROWS) e = launch_pdl(early, window_prep_kernel<__nv_bfloat16, 8, 4>, dim3((rows + 3) / 4), block, 0, st, p, rows);
+  else e = w == 8 ? launch_pdl(early, window_prep_kernel<__nv_bfloat16, 8, 1>, dim3(rows), block, 0, st, p, rows)
+                  : launch_pdl(early, window_prep_kernel<__nv_bfloat16, 1, 1>, dim3(rows), block, 0, st, p, rows);
   if (e != cudaSuccess) return fail(ERR_LAUNCH, "window_prep: %s", cudaGetErrorString(e));
   return check_launch("window_prep");
 }
