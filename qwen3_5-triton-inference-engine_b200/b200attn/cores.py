@@ -314,7 +314,10 @@ class FusedUnit:
         return engine.linear(act, self.w_out)
 
     def starts_own(self, engine) -> bool:
-        return engine.streams_weight(self.w_in)
+        """Whether the product in runs on the weight-streaming kernel: its form for inputs of up to 1280 takes any number of
+        outputs, the split one meets after every 16 outputs and is for few."""
+        n, k = self.w_in.shape
+        return engine.streams_weight(self.w_in) and (k <= ops.SKINNY_GEMM_MAX_K or n <= 8192)
 
     def out_parts(self, engine):
         """(weight, first and last column) of the product's parts in a decode step, or None: one library product."""
@@ -327,7 +330,7 @@ class FusedUnit:
         own, side = engine.then(True), len(self.parts) > 1
         outs = self.out_parts(engine)
         own_out = outs is not None
-        fused = engine.proj(h, self.w_in, not side)
+        fused = engine.proj(h, self.w_in, not side) if self.starts_own(engine) else F.linear(h, self.w_in)
         act = engine.zero_scratch(sum(self.outs), self.pad)      # padding columns stay zero
         ranges = list(self._ranges(fused, act))
         plain = own & ~ops.OVERLAP_START                          # behind a kernel of another stream
