@@ -104,16 +104,24 @@ __global__ void __launch_bounds__(256) window_prep_kernel(const __grid_constant_
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
       if (r >= count) break;
-      const float2* a = p.angles + row_pos[r] * n + dst;
       float u[W], v[W];
       ru[r].get(u);
-      if (rotated) rv[r].get(v);
 #pragma unroll
-      for (int k = 0; k < W; ++k) {
-        u[k] += bu[k];
-        if (rotated) {
+      for (int k = 0; k < W; ++k) u[k] += bu[k];
+      if (rotated) {
+        const float2* at = p.angles + row_pos[r] * n + dst;
+        float a[2 * W];                      // (cos, sin) of the W pairs
+        if constexpr (W == 8) {
+#pragma unroll
+          for (int k = 0; k < W / 2; ++k) reinterpret_cast<float4*>(a)[k] = reinterpret_cast<const float4*>(at)[k];
+        } else {
+          a[0] = at->x, a[1] = at->y;
+        }
+        rv[r].get(v);
+#pragma unroll
+        for (int k = 0; k < W; ++k) {
           v[k] += bv[k];
-          rotate_pair(u[k], v[k], a[k]);
+          rotate_pair(u[k], v[k], make_float2(a[2 * k], a[2 * k + 1]));
         }
       }
       auto put = [&](E* to) {
@@ -183,7 +191,7 @@ extern "C" int b200_window_prep(void* x, int64_t stride, const float* bias, cons
   B200_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dim > 0 && dim % 32 == 0 && vdim > 0 && vdim % 64 == 0 &&
                    pitch % 64 == 0 && pitch >= dim + vdim && rot_pairs >= 0 && 2 * rot_pairs <= dim && stride % 8 == 0,
                "window_prep: keys must be a multiple of 32, values and rows of 64, rotated pairs inside the keys");
-  B200_REQUIRE(aligned16(x) && aligned16(bias) && aligned16(cache) && aligned16(ctx) && (!ctx || ctx_row), "window_prep: unaligned tensor");
+  B200_REQUIRE(aligned16(x) && aligned16(bias) && aligned16(cache) && aligned16(ctx) && aligned16(angles) && (!ctx || ctx_row), "window_prep: unaligned tensor");
   const WindowPrepParams p = {x, stride, bias, pos, pos_is_int64, slot, active, block_table, table_stride,
                               reinterpret_cast<const float2*>(angles), cache, ctx, ctx_row, heads, kv_heads, dim, rot_pairs, vdim,
                               pitch, overlap};
