@@ -31,8 +31,8 @@ struct HyperParams {
   float eps;
 };
 
-// V: float4 groups a thread may own
-template <typename E, int MAXS, int V>
+// V: float4 groups a thread may own.  EXTRA: norm weights or several parts of y
+template <typename E, int MAXS, int V, bool EXTRA>
 __global__ void __launch_bounds__(512) hyper_connect_kernel(const __grid_constant__ HyperParams p) {
   __shared__ float wt[HC_MAX_STREAMS * HC_MAX_STREAMS + 2 * HC_MAX_STREAMS + 1];
   __shared__ float red[32];
@@ -43,13 +43,15 @@ __global__ void __launch_bounds__(512) hyper_connect_kernel(const __grid_constan
   __syncthreads();
   const float *mix = wt, *out = wt + s * s, *in = out + s;
   float* x = p.streams + static_cast<int64_t>(row) * s * width;
-  float4 u[V];
+  float4 u[V], g[V];
   float sq[1] = {0.f};
 #pragma unroll
   for (int v = 0; v < V; ++v) {
     const int c = (tid + v * blockDim.x) * 4;
     u[v] = make_float4(0.f, 0.f, 0.f, 0.f);
+    g[v] = make_float4(1.f, 1.f, 1.f, 1.f);
     if (c >= width) continue;
+    if (EXTRA && p.gains) g[v] = load4(p.gains + c);
     if (p.ids) {
       const int64_t id = p.ids_are_int64 ? static_cast<const int64_t*>(p.ids)[row]
                                          : static_cast<int64_t>(static_cast<const int32_t*>(p.ids)[row]);
@@ -69,10 +71,11 @@ __global__ void __launch_bounds__(512) hyper_connect_kernel(const __grid_constan
         if (i < s) old[i] = load4(x + i * width + c);
       if (p.y) {
         float4 y = load4(static_cast<const E*>(p.y) + static_cast<int64_t>(row) * width + c);
-        for (int i = 1; i < p.parts; ++i) {
-          const float4 more = load4(static_cast<const E*>(p.y) + i * p.part_stride + static_cast<int64_t>(row) * width + c);
-          y.x += more.x, y.y += more.y, y.z += more.z, y.w += more.w;
-        }
+        if (EXTRA && p.parts > 1)
+          for (int i = 1; i < p.parts; ++i) {
+            const float4 more = load4(static_cast<const E*>(p.y) + i * p.part_stride + static_cast<int64_t>(row) * width + c);
+            y.x += more.x, y.y += more.y, y.z += more.z, y.w += more.w;
+          }
 #pragma unroll
         for (int t = 0; t < MAXS; ++t)
           if (t < s) {
@@ -109,19 +112,23 @@ __global__ void __launch_bounds__(512) hyper_connect_kernel(const __grid_constan
   for (int v = 0; v < V; ++v) {
     const int c = (tid + v * blockDim.x) * 4;
     if (c >= width) continue;
-    const float4 g = p.gains ? load4(p.gains + c) : make_float4(1.f, 1.f, 1.f, 1.f);
-    store4(h + c, make_float4(u[v].x * scale * g.x, u[v].y * scale * g.y, u[v].z * scale * g.z, u[v].w * scale * g.w));
+    store4(h + c, make_float4(u[v].x * scale * g[v].x, u[v].y * scale * g[v].y, u[v].z * scale * g[v].z, u[v].w * scale * g[v].w));
   }
+}
+
+template <typename E, int MAXS, bool EXTRA>
+static cudaError_t launch_hyper_form(const HyperParams& p, int rows, cudaStream_t st) {
+  const int quads = p.width / 4;
+  const bool early = (p.overlap & OVERLAP_START) != 0;
+  int threads = (quads + 31) / 32 * 32;
+  if (threads <= 512) return launch_pdl(early, hyper_connect_kernel<E, MAXS, 1, EXTRA>, dim3(rows), dim3(threads), 0, st, p);
+  threads = ((quads + 3) / 4 + 31) / 32 * 32;
+  return launch_pdl(early, hyper_connect_kernel<E, MAXS, 4, EXTRA>, dim3(rows), dim3(threads), 0, st, p);
 }
 
 template <typename E, int MAXS>
 static cudaError_t launch_hyper(const HyperParams& p, int rows, cudaStream_t st) {
-  const int quads = p.width / 4;
-  const bool early = (p.overlap & OVERLAP_START) != 0;
-  int threads = (quads + 31) / 32 * 32;
-  if (threads <= 512) return launch_pdl(early, hyper_connect_kernel<E, MAXS, 1>, dim3(rows), dim3(threads), 0, st, p);
-  threads = ((quads + 3) / 4 + 31) / 32 * 32;
-  return launch_pdl(early, hyper_connect_kernel<E, MAXS, 4>, dim3(rows), dim3(threads), 0, st, p);
+  return p.gains || p.parts > 1 ? launch_hyper_form<E, MAXS, true>(p, rows, st) : launch_hyper_form<E, MAXS, false>(p, rows, st);
 }
 
 template <typename E>

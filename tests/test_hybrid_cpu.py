@@ -18,9 +18,10 @@ ROOT = Path(__file__).resolve().parent.parent
 def test_registry_chooses_by_architecture():
     from b200attn import models
 
-    assert {"Tofilorn", "Qwen3.5"} <= set(models.families())
-    fam = models.family(H.CONFIGS["ragged"])
-    assert fam.name == "Tofilorn" and torch.float32 in fam.dtypes and fam.part == "hybrid"
+    assert {"Tofilorn", "Dugilorn", "Qwen3.5"} <= set(models.families())
+    for name, config in (("Tofilorn", "ragged"), ("Dugilorn", "odd")):
+        fam = models.family(H.CONFIGS[config])
+        assert fam.name == name and torch.float32 in fam.dtypes and fam.part == "hybrid"
     assert models.family({"architecture": "Qwen3.5"}).config({"architecture": "Qwen3.5", "hidden": 512}).hidden == 512
     with pytest.raises(ValueError, match="unknown architecture"):
         models.family({"architecture": "nobody"})
@@ -105,6 +106,82 @@ def test_padding_keeps_heads_apart():
     assert torch.equal(w.joints[1][: s * s].view(s, s), tensors["l0.hc1.mix"].float())     # [from, to]
 
 
+def _core_weights(config, seed=0, rank=None):
+    from b200attn.hybrid import HybridConfig, HybridWeights
+    tensors = H.checkpoint(config, seed)
+    if rank is not None:
+        for name in [n for n in tensors if n.endswith(".a1")]:
+            tensors[name] = torch.randn(rank, config["width"]).to(torch.bfloat16)
+            tensors[name[:-1] + "2"] = torch.randn(tensors[name[:-1] + "2"].shape[0], rank).to(torch.bfloat16)
+    return tensors, HybridWeights(HybridConfig.from_config(config)).load(tensors, torch.float32, "cpu")
+
+
+def _unit_restated(unit, core_index, h):
+    """What a core's columns of the input product hold."""
+    x = h @ unit.w_in.T
+    return x.split(unit.ins, dim=1)[core_index]
+
+
+def test_cores_share_products_without_mixing():
+    """Columns of the stacked products against the restatement's own projections, head by head; padding is zero."""
+    config = H.CONFIGS["odd"]
+    tensors, w = _core_weights(config)
+    t = {k: v.float() for k, v in tensors.items()}
+    h = torch.zeros(3, w.width_p)
+    h[:, :136] = torch.randn(3, 136, generator=torch.Generator().manual_seed(1))
+    unit = w.units[0]
+    attn, ssm, mlp = (core for _, core in unit.parts)
+    x = _unit_restated(unit, 0, h)
+    q, k, v, g = x.split([6 * attn.dim_p, 3 * attn.dim_p, 3 * attn.vdim_p, 6 * attn.vdim_p], dim=1)
+    for cols, name, heads, size in ((q, "q", 6, 20), (k, "k", 3, 20), (v, "v", 3, 24), (g, "g", 6, 24)):
+        cols = cols.reshape(3, heads, -1)
+        want = (h[:, :136] @ t[f"l0.mix.left.{name}"].T).view(3, heads, size)
+        assert torch.allclose(cols[..., :size], want, atol=1e-4) and not cols[..., size:].any()
+    x = _unit_restated(unit, 1, h)
+    raw = h[:, :136] @ t["l0.mix.right.in"].T
+    z, xs, b, c, dt = raw.split([120, 120, 72, 72, 6], dim=1)
+    zp, xp, bp, cp, dp = x.split([6 * 32, 6 * 32, 3 * 32, 3 * 32, 8], dim=1)
+    for got, want, heads, size in ((zp, z, 6, 20), (xp, xs, 6, 20), (bp, b, 3, 24), (cp, c, 3, 24)):
+        got = got.reshape(3, heads, -1)
+        assert torch.allclose(got[..., :size], want.reshape(3, heads, size), atol=1e-4) and not got[..., size:].any()
+    assert torch.allclose(dp[:, :6], dt, atol=1e-4) and not dp[:, 6:].any()
+    assert ssm.conv.shape == (4, ssm.channels) and not ssm.conv[3].any()             # three taps, the current token's first
+    assert torch.equal(ssm.conv[0, :20], t["l0.mix.right.conv"][:20, 2]) and torch.equal(ssm.conv[2, 32:52], t["l0.mix.right.conv"][20:40, 0])
+    assert torch.allclose(ssm.norm.view(6, 32)[:, :20].reshape(-1), 1.3 * t["l0.mix.right.norm"]) and not ssm.norm.view(6, 32)[:, 20:].any()
+    assert attn.scale == 0.7 and mlp.out_size == 256
+    # the product out: the parts' columns side by side, the rest zero
+    a, s, m, rest = unit.w_out.split([*unit.outs, unit.pad], dim=1)
+    assert torch.equal(a[:136].reshape(136, 6, 64)[..., :24].reshape(136, -1), t["l0.mix.left.o"])
+    assert torch.equal(s[:136].reshape(136, 6, 32)[..., :20].reshape(136, -1), t["l0.mix.right.o"])
+    assert torch.equal(m[:136, :200], t["l0.mlp.down"]) and not rest.any() and not unit.w_out[136:].any()
+    assert all(torch.equal(p, unit.w_out[:, n * unit.part: (n + 1) * unit.part]) for n, p in enumerate(unit.w_parts))
+    # norms: one weight vector per joint
+    assert len(w.joints) == len(w.gains) == len(w.units) + 1 == 6 and torch.equal(w.gains[1][:136], t["l1.norm1"])
+    assert torch.equal(w.gains[5][:136], t["final.norm"]) and not w.gains[5][136:].any()
+    assert [u.layer for u in w.units] == [0, 1, 2, 3, 4] and [len(u.parts) for u in w.units] == [3, 1, 2, 2, 3]
+
+
+@pytest.mark.parametrize("rank", [5, 16, 32])
+def test_decay_rank_comes_from_the_checkpoint(rank):
+    tensors, w = _core_weights(H.CONFIGS["odd"], rank=rank)
+    core = w.units[1].parts[0][1]
+    assert core.rank == rank and core.w_low.shape == (3 * core.dim_p, -(-rank // 8) * 8)
+    assert torch.equal(core.w_low.view(3, core.dim_p, -1)[:, :24, :rank].reshape(72, rank), tensors["l1.mix.a2"].float())
+    assert w.units[1].w_in.shape[0] == core.in_size == core.low_at + core.rank_p
+
+
+def test_product_out_is_split_into_parts_the_kernel_takes():
+    from b200attn import ops
+    config = H.dugilorn(256, 64, 30.0, [(H.parallel(H.window(16, 4, 64, 128, 64), H.state_space(32, 64, 16, 1, 4, 1)), 1500), (H.gla(2, 16, 16, 4.0), None)])
+    _, w = _core_weights(config)
+    unit = w.units[0]
+    assert sum(unit.outs) == 2048 + 2048 + 1536 and len(unit.w_parts) == 2 and unit.part <= ops.SKINNY_GEMM_PAIR_MAX_K
+    assert ops.skinny_gemm_supports(32, 256, unit.part) and len(w.units[1].w_parts) == 1
+    with pytest.raises(ValueError, match="cannot share its norm"):
+        from b200attn.hybrid import HybridConfig, HybridWeights
+        HybridWeights(HybridConfig.from_config(H.dugilorn(64, 64, 1.0, [(H.mingru(32), 64)])))
+
+
 def test_chunking_and_splits():
     from b200attn import hybrid_ops as hops
 
@@ -116,6 +193,12 @@ def test_chunking_and_splits():
             seg, segs = hops.hgrn2_segments(n, groups, 148)
             assert (segs - 1) * seg < n <= segs * seg and (segs == 1 or (seg % 16 == 0 and seg >= 128))
             assert segs == 1 or segs * groups <= 2 * 148
+            seg, segs = hops.ssd_segments(n, groups, 148)
+            assert (segs - 1) * seg < n <= segs * seg and (segs == 1 or (seg % 32 == 0 and segs * groups <= 2 * 148))
+    assert [hops.conv_taps(n) for n in (1, 4, 5, 8, 9, 16)] == [4, 4, 8, 8, 16, 16]
+    for batch, heads, kv, span in [(1, 1, 1, 16), (1, 32, 2, 4096), (32, 16, 4, 2048), (256, 64, 8, 512)]:
+        s = hops.window_decode_splits(batch, heads, kv, span, 148)
+        assert 1 <= s <= hops.LATENT_MAX_SPLITS and (s == 1 or span // s >= 16)
     for batch, heads, span in [(1, 1, 16), (1, 16, 4096), (32, 16, 4096), (256, 128, 512), (1, 1, 1)]:
         s = hops.latent_decode_splits(batch, heads, span, 148)
         assert 1 <= s <= hops.LATENT_MAX_SPLITS and (s == 1 or span // s >= 16)
@@ -129,6 +212,11 @@ def test_packed_batch_rows():
     assert b.cu.tolist() == [0, 3, 4] and b.slots.tolist() == [4, 1] and b.start.tolist() == [10, 0]
     span = b.context(4)       # query 10 sees 7..10
     assert span.first.tolist() == [7, 0] and span.cu.tolist() == [0, 6, 7] and (span.keys, span.max_keys) == (7, 6)
+    assert span.rows.tolist() == [3, 4, 5, 6] and span.max_old == 3      # behind the three keys of earlier passes
+    b = PackedBatch([0, 1, 2], [0, 5, 2], [[1, 2], [3], [4, 5, 6]], "cpu")
+    span = b.context(3)
+    assert span.first.tolist() == [0, 3, 0] and span.cu.tolist() == [0, 2, 5, 10] and span.rows.tolist() == [0, 1, 4, 7, 8, 9]
+    assert span.max_old == 2 and b.context(1).max_old == 0
 
 
 def test_oracle_special_cases():
@@ -149,6 +237,25 @@ def test_oracle_special_cases():
     x = torch.randn(1, 5, 4, generator=g, dtype=torch.float64)
     w = {"in": torch.ones(1).double(), "out": torch.ones(1).double(), "mix": torch.ones(1, 1).double()}
     assert torch.allclose(R.hyper_connect(x, w, "", lambda u: 2 * u), 3 * x)
+    x = torch.randn(6, 3, generator=g, dtype=torch.float64)
+    assert torch.allclose(R.causal_conv(x, torch.tensor([[2.0]] * 3).double(), torch.zeros(3).double()), 2 * x)
+    shift = R.causal_conv(x, torch.tensor([[1.0, 0.0]] * 3).double(), torch.ones(3).double())
+    assert torch.allclose(shift[1:], x[:-1] + 1) and torch.allclose(shift[0], torch.ones(3).double())
+    B, C, xs = (torch.randn(5, 2, n, generator=g, dtype=torch.float64) for n in (3, 3, 4))
+    dt, D = torch.rand(5, 2, generator=g).double(), torch.tensor([0.5, -1.0]).double()
+    gone = R.state_space_recurrence(xs, B, C, dt, torch.full((2,), 40.0).double(), D)            # every step forgets all
+    assert torch.allclose(gone, (dt * (B * C).sum(-1))[..., None] * xs + D[:, None] * xs)
+    kept = R.state_space_recurrence(xs, B, C, dt, torch.full((2,), -60.0).double(), 0 * D)       # nothing is forgotten
+    assert torch.allclose(kept[4, 0], sum(dt[s, 0] * (B[s, 0] @ C[4, 0]) * xs[s, 0] for s in range(5)))
+    keep = torch.zeros(5, 2, 3).double()
+    assert torch.allclose(R.decayed_outer_recurrence(C, B, xs, keep), (B * C).sum(-1, keepdim=True) * xs)
+    assert torch.allclose(R.decayed_outer_recurrence(C, B, xs, keep + 1)[4, 1], sum((B[s, 1] @ C[4, 1]) * xs[s, 1] for s in range(5)))
+    y = torch.randn(2, 12, generator=g, dtype=torch.float64)
+    assert torch.allclose(R.grouped_rms(y, 3, 0.0)[:, 4:8], R.rms(y[:, 4:8], 0.0)) and torch.allclose(R.gelu_tanh(torch.tensor(0.0)), torch.tensor(0.0))
+    z = torch.randn(7, 2, 8, generator=g, dtype=torch.float64)
+    rot = R.rotate_halves(z, {"base": 100.0, "dims": 6}, torch.arange(7))
+    assert torch.equal(rot[0], z[0]) and torch.equal(rot[..., 6:], z[..., 6:]) and torch.allclose(rot.norm(dim=-1), z.norm(dim=-1))
+    assert torch.allclose(rot[2, 0, 0], z[2, 0, 0] * math.cos(2.0) - z[2, 0, 3] * math.sin(2.0))
     assert math.isclose(float(R.silu(torch.tensor(1.0))), 1 / (1 + math.exp(-1)), rel_tol=1e-6)
 
 
