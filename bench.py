@@ -1316,8 +1316,8 @@ def run_core_kernel_rows(ops, device, steps):
     sms = torch.cuda.get_device_properties(device).multi_processor_count
     # ---- decode attention
     for batch, heads, kv, dim, ctx in ((1, 16, 4, 128, 2048), (32, 16, 4, 128, 2048), (32, 8, 2, 128, 4096), (32, 16, 4, 128, 640),
-                                       (32, 8, 2, 96, 2048), (256, 16, 4, 128, 2048)):
-        vdim = 2 * dim if dim == 96 else dim
+                                       (32, 12, 3, 64, 2048), (256, 16, 4, 128, 2048)):
+        vdim = 3 * dim if dim == 64 else dim         # 64 + 192: keys and values of different sizes
         pitch, pages = cdiv(dim + vdim, 64) * 64, ctx // 16
         nbytes = batch * (ctx * kv * (dim + vdim) * 2 + heads * (dim + vdim) * 2)
         n = copies(nbytes)

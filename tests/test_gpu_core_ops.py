@@ -157,7 +157,7 @@ def pages(slots, context, seed=3):
     return perm.view(slots, per).to(torch.int32).to(DEV), slots * per + 2
 
 
-SIZES = [(4, 2, 32, 64, 32), (6, 3, 20, 24, 12), (5, 1, 72, 136, 72), (2, 2, 96, 192, 48), (17, 1, 128, 128, 64), (2, 1, 256, 256, 256),
+SIZES = [(4, 2, 32, 64, 32), (6, 3, 20, 24, 12), (5, 1, 72, 136, 72), (2, 2, 160, 192, 48), (17, 1, 128, 128, 64), (2, 1, 256, 256, 256),
          (2, 1, 264, 264, 40), (3, 3, 64, 64, 2)]
 
 
